@@ -9,7 +9,9 @@ Two shared objects are produced under ``dgpp_b200/lib``:
   tokenizer, chat template, grammars, sampler oracle, HTTP server), a pybind11 module
   compiled by g++.
 
-Objects are cached under ``build/`` and rebuilt when a source or header is newer.
+Objects are cached under ``build/`` and rebuilt when a source or header is newer.  ``ensure(family)`` builds what one model
+family needs and no more: the host runtime and, where the full kernel library is not there, a library of that family's
+translation units (``libdgpp_kernels_<family>.so``).
 """
 from __future__ import annotations
 
@@ -33,6 +35,10 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC", "-Xcompiler", "-Wall",
     "-Xcompiler", "-Wno-unused-function", "-I", str(CSRC),
 ]
+# Translation units of the kernel library that a family's runner calls.
+KERNEL_SETS = {
+    "sitirax": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "window_attn", "linear_state", "graph_exec"],
+}
 # Translation units that must not contract a*b+c into fma (sampler parity with the host oracle).
 NO_FMA = {"sample.cu"}
 
@@ -70,15 +76,17 @@ def rt_sources() -> list[Path]:
     return sorted((CSRC / "rt").glob("*.cpp"))
 
 
-def build_kernels(verbose: bool = False, force: bool = False, ptxas_info: bool = False) -> Path:
+def build_kernels(verbose: bool = False, force: bool = False, ptxas_info: bool = False, family: str = "") -> Path:
     LIB.mkdir(exist_ok=True)
     odir = BUILD / "kernels"
     odir.mkdir(parents=True, exist_ok=True)
     hdr = _newest_header()
-    out = LIB / "libdgpp_kernels.so"
+    out = LIB / (f"libdgpp_kernels_{family}.so" if family else "libdgpp_kernels.so")
     jobs = []
     objs = []
     for src in kernel_sources():
+        if family and src.stem not in KERNEL_SETS[family]:
+            continue
         obj = odir / (src.stem + ".o")
         objs.append(obj)
         if force or _needs(obj, src, hdr):
@@ -142,6 +150,28 @@ def build_rt(verbose: bool = False, force: bool = False) -> Path:
 def build_all(verbose: bool = False, force: bool = False) -> None:
     build_rt(verbose=verbose, force=force)
     build_kernels(verbose=verbose, force=force)
+
+
+def _stale(out: Path, sources: list[Path]) -> bool:
+    return not out.exists() or max([_newest_header()] + [p.stat().st_mtime for p in sources]) > out.stat().st_mtime
+
+
+def ensure(family: str) -> Path:
+    """Builds what is missing to run `family` from a checkout and returns the kernel library to load.  Concurrent callers wait
+    for one another."""
+    import fcntl
+
+    BUILD.mkdir(exist_ok=True)
+    with open(BUILD / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        with cf.ThreadPoolExecutor(max_workers=1) as ex:
+            host = ex.submit(build_rt) if _stale(rt_module_path(), rt_sources()) else None
+            kernels = LIB / "libdgpp_kernels.so"
+            if _stale(kernels, kernel_sources()):
+                kernels = build_kernels(family=family if family in KERNEL_SETS else "")
+            if host is not None:
+                host.result()
+    return kernels
 
 
 if __name__ == "__main__":

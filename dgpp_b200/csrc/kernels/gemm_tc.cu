@@ -133,7 +133,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA,   // bf16 weights, or pa
   if (p.ag) my = (min(p.comm.rank * p.tiles_per_rank, static_cast<int>(gridDim.y)) + static_cast<int>(blockIdx.y)) % static_cast<int>(gridDim.y);
   const int m0 = my * BN;
   const int split = blockIdx.z, splits = gridDim.z;
-  const int num_kb_total = p.K / kBK;
+  const int num_kb_total = (p.K + kBK - 1) / kBK;    // bf16 weights: the columns beyond K of the last block read as zero
   const int kb_begin = split * p.kb_per_split;
   const int kb_end = min(num_kb_total, kb_begin + p.kb_per_split);
   const int nkb = max(0, kb_end - kb_begin);
@@ -566,7 +566,8 @@ static int gemm_tc_impl(int wmode, int a_f16, int bn, const void* x, int64_t x_s
                         int T, int N, int K, int splits, void* ws, void* counters, void* comm_push, cudaStream_t st,
                         void* comm_ag = nullptr) {
   DGPP_REQUIRE(T >= 1 && N >= 1, "gemm_tc: empty problem");
-  DGPP_REQUIRE(K % 64 == 0, "gemm_tc: K %d must be a multiple of 64", K);
+  DGPP_REQUIRE(K % 64 == 0 || (wmode == 0 && K % 8 == 0 && !comm_ag),
+               "gemm_tc: K %d must be a multiple of 64 (bf16 weights: of 8)", K);
   const bool nibble_src = wmode == 1 || wmode == 3 || wmode == 6;
   const bool byte_src = wmode == 2 || wmode == 4 || wmode == 5 || wmode == 7;
   if (nibble_src) DGPP_REQUIRE(K % 256 == 0, "gemm_tc: 4-bit weights need K %% 256 == 0 (K=%d)", K);
@@ -620,7 +621,7 @@ static int gemm_tc_impl(int wmode, int a_f16, int bn, const void* x, int64_t x_s
   }
   p.status = device_status_ptr();
   p.T = T; p.N = N; p.K = K; p.ldc = ldc;
-  const int num_kb = K / 64;
+  const int num_kb = dgpp_ceil_div(K, 64);
   const int align = nibble_src ? 4 : (byte_src ? 2 : 1);
   int per = dgpp_ceil_div(num_kb, splits);
   per = dgpp_ceil_div(per, align) * align;

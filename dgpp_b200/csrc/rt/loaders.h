@@ -288,7 +288,7 @@ inline std::string resolve_model(const std::string& spec, const std::string& cac
 }
 
 // ------------------------------------------------------------------------------------------- architecture detect
-enum class Family { Unknown, QwenHybrid, QwenFlashNext, Glm4, GlmFlash, GlmDsa, DeepSeekV4, DeepSeekV41, MiMo, MiniMax, Flint, Dory, DenseGqa };
+enum class Family { Unknown, QwenHybrid, QwenFlashNext, Glm4, GlmFlash, GlmDsa, DeepSeekV4, DeepSeekV41, MiMo, MiniMax, Flint, Dory, Sitirax, DenseGqa };
 
 inline const char* family_name(Family f) {
   switch (f) {
@@ -303,6 +303,7 @@ inline const char* family_name(Family f) {
     case Family::MiniMax: return "minimax";
     case Family::Flint: return "flint";
     case Family::Dory: return "dory";
+    case Family::Sitirax: return "sitirax";
     case Family::DenseGqa: return "dense_gqa";
     default: return "unknown";
   }
@@ -315,6 +316,7 @@ inline Family detect_family(const json::Value& config) {
   std::string arch;
   if (const json::Value* a = config.find("architectures"))
     if (a->is_array() && a->size() > 0 && a->at(0).is_string()) arch = a->at(0).as_string();
+  if (arch.empty()) arch = config.get_string("architecture");
   std::string type = config.get_string("model_type");
   if (const json::Value* tc = config.find("text_config"))
     if (tc->is_object() && type.empty()) { cfg = tc; type = tc->get_string("model_type"); }
@@ -332,6 +334,7 @@ inline Family detect_family(const json::Value& config) {
   if (has("minimax")) return Family::MiniMax;
   if (has("flint")) return Family::Flint;
   if (has("dory")) return Family::Dory;
+  if (has("sitirax")) return Family::Sitirax;
   if (has("qwen3") || has("qwen2") || has("llama") || has("mistral")) return Family::DenseGqa;
   throw std::runtime_error("detect_family: unsupported architecture '" + arch + "' / model_type '" + type + "'");
 }

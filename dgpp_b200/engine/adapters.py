@@ -203,7 +203,89 @@ class ReferenceEngine(EmbedSplice, rt.SchedulerEngine):
         return out
 
 
-class KernelEngine(EmbedSplice, rt.SchedulerEngine):
+class SlotSampling:
+    """Per-request sampling parameters and token grammars bound to engine slots, shared by the engines behind the scheduler.
+    The engine provides `filled` (tokens per slot) and `_sampling_geometry()` -> (vocabulary, slots, device)."""
+
+    def _sampling_init(self, slots: int) -> None:
+        self.by_id = {}
+        self.emitted = {}                              # request id -> tokens the sampler picked for it so far
+        self.slot_req = [None] * slots
+        self.slot_cfg = [None] * slots
+        self.last_logprobs = [None] * slots
+        self.sampler = None
+
+    def configure(self, request_id: str, params=None, grammar=None, prompt_ids=None) -> None:
+        """Registers sampling parameters (``SamplingParams``), a token grammar (``rt.JsonGrammar``) and the prompt ids
+        (for the penalties' token counts) of a request before it is submitted to the scheduler."""
+        self.by_id[request_id] = (params, grammar, prompt_ids)
+
+    def forget(self, request_id: str) -> None:
+        """Drops what configure() / set_embeds() registered for a request.  The owner of the request calls it when
+        the request retires (or is rejected / cancelled while still queued); until then the entries stay, because a
+        request shed back to the queue is opened again under the same id and must get the same sampling parameters,
+        its grammar in the state its generated tokens left it in, and its image rows."""
+        self.by_id.pop(request_id, None)
+        self.emitted.pop(request_id, None)
+
+    def _sampling_open(self, slot, request_id) -> None:
+        cfg = self.by_id.get(request_id)
+        self.slot_cfg[slot] = None
+        self.slot_req[slot] = request_id
+        self.last_logprobs[slot] = None
+        if cfg is None or (cfg[0] is None and cfg[1] is None):
+            return
+        params, grammar, prompt_ids = cfg
+        from ..sampling.device import DeviceSampler, SamplingParams
+        if self.sampler is None:
+            vocab, slots, dev = self._sampling_geometry()
+            self.sampler = DeviceSampler(vocab, slots, slots, dev)
+        self.sampler.reset_slot(slot)
+        params = params or SamplingParams()
+        if params.repetition_penalty != 1.0 or params.presence_penalty or params.frequency_penalty:
+            # token counts of the prompt and, for a re-admitted request, of what it had generated before it was shed
+            seen = list(prompt_ids or []) + self.emitted.get(request_id, [])
+            if seen:
+                self.sampler.count(slot, seen)
+        # (the grammar object itself has consumed every token picked so far, so it resumes where the request stopped)
+        self.slot_cfg[slot] = (params, grammar)
+
+    def _pick_rows(self, logits, rows, params, slots, masks):
+        return self.sampler.sample(logits, params, [s if self.slot_cfg[s] else -1 for s in slots],
+                                   [self.filled[s] for s in slots], masks=masks)
+
+    def _sample_rows(self, logits, slots):
+        """Device sampler over the rows of `slots` (rows of plain greedy slots keep the engine's own pick)."""
+        import numpy as np
+        from ..sampling.device import SamplingParams
+        rows = len(slots)
+        vocab, _, dev = self._sampling_geometry()
+        params, masks = [], None
+        for s in slots:
+            cfg = self.slot_cfg[s]
+            params.append(cfg[0] if cfg else SamplingParams())
+        if any(self.slot_cfg[s] and self.slot_cfg[s][1] is not None for s in slots):
+            words = (vocab + 31) // 32
+            m = np.full((rows, words), 0xFFFFFFFF, dtype=np.uint32)
+            for r, s in enumerate(slots):
+                cfg = self.slot_cfg[s]
+                if cfg and cfg[1] is not None:
+                    gm = cfg[1].mask()
+                    m[r, :] = 0
+                    m[r, :min(words, gm.shape[0])] = gm[:words]
+            masks = torch.from_numpy(m.view(np.int32)).to(dev)
+        picked = self._pick_rows(logits, rows, params, slots, masks)
+        for r, s in enumerate(slots):
+            cfg = self.slot_cfg[s]
+            if cfg:
+                self.last_logprobs[s] = (picked[r].logprob, picked[r].top)
+                if cfg[1] is not None:
+                    cfg[1].accept(picked[r].token)
+                self.emitted.setdefault(self.slot_req[s], []).append(picked[r].token)
+        return [p.token for p in picked]
+
+
+class KernelEngine(EmbedSplice, SlotSampling, rt.SchedulerEngine):
     """The CUDA engine behind the scheduler: chunked prefill and graph-replayed decode for arbitrary slot sets."""
 
     def __init__(self, engine, spec_drafts: int = 0):
@@ -238,12 +320,7 @@ class KernelEngine(EmbedSplice, rt.SchedulerEngine):
             self.s_req = torch.zeros(hb, dtype=torch.int32, device=dev)
         self.poll_status = True                        # read the device status block after every step (see _poll_device)
         self.step_deadline_s = 120.0                   # host-side bound on one prefill chunk / decode pass
-        self.by_id = {}
-        self.emitted = {}                              # request id -> tokens the sampler picked for it so far
-        self.slot_req = [None] * b
-        self.slot_cfg = [None] * b
-        self.last_logprobs = [None] * b
-        self.sampler = None
+        self._sampling_init(b)
         from ..utils.step_timing import StepTimer
         self.timer = StepTimer()                 # DGPP_STEP_TIMING=1 turns the event slots on
 
@@ -314,81 +391,27 @@ class KernelEngine(EmbedSplice, rt.SchedulerEngine):
         self.filled[slot] += tokens
 
     # ------------------------------------------------------------------ sampling / constraints
-    def configure(self, request_id: str, params=None, grammar=None, prompt_ids=None) -> None:
-        """Registers sampling parameters (``SamplingParams``), a token grammar (``rt.JsonGrammar``) and the prompt ids
-        (for the penalties' token counts) of a request before it is submitted to the scheduler."""
-        self.by_id[request_id] = (params, grammar, prompt_ids)
+    def _sampling_geometry(self):
+        return self.e.model.cfg.vocab, self.e.max_batch, self.e.dev
 
     def forget(self, request_id: str) -> None:
-        """Drops what configure() / set_embeds() registered for a request.  The owner of the request calls it when
-        the request retires (or is rejected / cancelled while still queued); until then the entries stay, because a
-        request shed back to the queue is opened again under the same id and must get the same sampling parameters,
-        its grammar in the state its generated tokens left it in, and its image rows."""
-        self.by_id.pop(request_id, None)
-        self.emitted.pop(request_id, None)
+        SlotSampling.forget(self, request_id)
         self._splice_forget(request_id)
 
     def open(self, slot, request_id):
         self._splice_open(slot, request_id)
-        cfg = self.by_id.get(request_id)
-        self.slot_cfg[slot] = None
-        self.slot_req[slot] = request_id
-        self.last_logprobs[slot] = None
-        if cfg is None or (cfg[0] is None and cfg[1] is None):
-            return
-        params, grammar, prompt_ids = cfg
-        from ..sampling.device import DeviceSampler, SamplingParams
-        if self.sampler is None:
-            self.sampler = DeviceSampler(self.e.model.cfg.vocab, self.e.max_batch, self.e.max_batch, self.e.dev)
-        self.sampler.reset_slot(slot)
-        params = params or SamplingParams()
-        if params.repetition_penalty != 1.0 or params.presence_penalty or params.frequency_penalty:
-            # token counts of the prompt and, for a re-admitted request, of what it had generated before it was shed
-            seen = list(prompt_ids or []) + self.emitted.get(request_id, [])
-            if seen:
-                self.sampler.count(slot, seen)
-        # (the grammar object itself has consumed every token picked so far, so it resumes where the request stopped)
-        self.slot_cfg[slot] = (params, grammar)
+        self._sampling_open(slot, request_id)
 
-    def _sample_rows(self, logits, slots):
-        """Device sampler over the rows of `slots` (rows of plain greedy slots keep the engine's own pick)."""
-        import numpy as np
-        from ..sampling.device import SamplingParams
-        rows = len(slots)
-        params, masks = [], None
-        for s in slots:
-            cfg = self.slot_cfg[s]
-            params.append(cfg[0] if cfg else SamplingParams())
-        if any(self.slot_cfg[s] and self.slot_cfg[s][1] is not None for s in slots):
-            words = (self.e.model.cfg.vocab + 31) // 32
-            m = np.full((rows, words), 0xFFFFFFFF, dtype=np.uint32)
-            for r, s in enumerate(slots):
-                cfg = self.slot_cfg[s]
-                if cfg and cfg[1] is not None:
-                    gm = cfg[1].mask()
-                    m[r, :] = 0
-                    m[r, :min(words, gm.shape[0])] = gm[:words]
-            masks = torch.from_numpy(m.view(np.int32)).to(self.e.dev)
+    def _pick_rows(self, logits, rows, params, slots, masks):
+        counted, at = [s if self.slot_cfg[s] else -1 for s in slots], [self.filled[s] for s in slots]
         if self.e.model.tp_size > 1:
             # vocabulary-sharded head: every rank builds the candidate table of its slice (a few KB per row), the tables
             # are all-gathered and folded identically on every rank: no logits gather, the same token everywhere
             vl = self.e.runner.vocab_local
             base = self.e.model.tp_rank * vl
             width = max(0, min(vl, self.e.model.cfg.vocab - base))
-            picked = self.sampler.sample_sharded(logits[:rows, :width], base, params,
-                                                 [s if self.slot_cfg[s] else -1 for s in slots],
-                                                 [self.filled[s] for s in slots], masks=masks)
-        else:
-            picked = self.sampler.sample(logits, params, [s if self.slot_cfg[s] else -1 for s in slots],
-                                         [self.filled[s] for s in slots], masks=masks)
-        for r, s in enumerate(slots):
-            cfg = self.slot_cfg[s]
-            if cfg:
-                self.last_logprobs[s] = (picked[r].logprob, picked[r].top)
-                if cfg[1] is not None:
-                    cfg[1].accept(picked[r].token)
-                self.emitted.setdefault(self.slot_req[s], []).append(picked[r].token)
-        return [p.token for p in picked]
+            return self.sampler.sample_sharded(logits[:rows, :width], base, params, counted, at, masks=masks)
+        return self.sampler.sample(logits, params, counted, at, masks=masks)
 
     def _poll_device(self) -> None:
         """Every bounded device wait (pipeline barriers, accumulators, peer flags, grid barriers) reports its expiry
@@ -744,21 +767,35 @@ class HybridEngine(rt.SchedulerEngine):
         self.pending[slot] = None
 
 
-class RunnerEngine(rt.SchedulerEngine):
+class RunnerEngine(SlotSampling, rt.SchedulerEngine):
     """Any family runner with `prefill(slot, tokens, chunk)`, `decode(slots, tokens)`, `reset(slot)` and `lengths` behind
-    the scheduler (greedy decoding).  The runner's state (recurrent memories, caches laid out per slot) is not
-    addressable by block, so this engine never resumes from the prefix cache: it hands the scheduler a private block
-    table for admission arithmetic only and reports no usable prefix.  (reference counterparts: the per-family
-    SessionModel adapters of src/engine/session_model.hpp.)"""
+    the scheduler.  The runner's state (recurrent memories, caches laid out per slot) is not addressable by block, so this
+    engine never resumes from the prefix cache and reports no usable prefix.  A runner with a shared pool (`pooled`) is asked
+    for its own blocks; for the others a private block table does the admission arithmetic.  A runner with mixed passes
+    (`mixed_runs`, `step`) takes several readers, or a reader's piece and a decode step, in one pass.  Requests decode greedily
+    unless they were configured with sampling parameters or a grammar; those rows go through the device sampler.
+    (reference counterparts: the per-family SessionModel adapters of src/engine/session_model.hpp.)"""
 
     def __init__(self, runner, max_context: int, block_tokens: int = 64, prefill_chunk: int = 256):
         super().__init__()
-        self.r, self.bt, self.maxctx, self.prefill_chunk = runner, block_tokens, max_context, prefill_chunk
+        self.r, self.maxctx, self.prefill_chunk = runner, max_context, prefill_chunk
         n = len(runner.lengths)
-        self.per_slot = (max_context + block_tokens - 1) // block_tokens + 1
-        self.table = rt.PagedBlockTable(n * self.per_slot + 1)
+        self.pool = runner.kv if getattr(runner, "pooled", False) else None
+        self.mixed = getattr(runner, "mixed_runs", False)
+        self.bt = self.pool.page if self.pool is not None else block_tokens
+        self.per_slot = (max_context + self.bt - 1) // self.bt + 1
+        self.table = self.pool.alloc if self.pool is not None else rt.PagedBlockTable(n * self.per_slot + 1)
         self.blocks: List[List[int]] = [[] for _ in range(n)]
         self.pending: List[Optional[int]] = [None] * n
+        self.step_deadline_s = 120.0
+        self._sampling_init(n)
+
+    @property
+    def filled(self):
+        return self.r.lengths
+
+    def _sampling_geometry(self):
+        return self.r.c.vocab, len(self.r.lengths), torch.device(self.r.dev)
 
     # ---- geometry
     def max_concurrent(self):
@@ -776,8 +813,10 @@ class RunnerEngine(rt.SchedulerEngine):
     def max_context(self):
         return self.maxctx
 
-    # ---- blocks (accounting only)
+    # ---- blocks (the runner's own, or accounting only)
     def reserve(self, slot, tokens):
+        if self.pool is not None:
+            return self.pool.reserve(slot, tokens)
         need = (tokens + self.bt - 1) // self.bt
         if need > self.per_slot or need - len(self.blocks[slot]) > self.table.free_count():
             return False
@@ -786,7 +825,7 @@ class RunnerEngine(rt.SchedulerEngine):
         return True
 
     def slot_blocks(self, slot):
-        return list(self.blocks[slot])
+        return list(self.pool.req_blocks[slot] if self.pool is not None else self.blocks[slot])
 
     def retain_block(self, b):
         self.table.retain(b)
@@ -803,38 +842,86 @@ class RunnerEngine(rt.SchedulerEngine):
     def attach_prefix(self, slot, blocks):
         raise AssertionError("attach_prefix on an engine that reports no usable prefix")
 
+    def open(self, slot, request_id):
+        self._sampling_open(slot, request_id)
+
     # ---- execution
-    def prefill(self, slot, tokens, pos, last):
-        tokens = list(tokens)
+    def _poll_device(self) -> None:
+        """See KernelEngine._poll_device: a non-zero device status after a pass fails the engine."""
+        if torch.device(getattr(self.r, "dev", "cpu")).type != "cuda":
+            return
+        import ctypes as C
+        from ..ops import _lib
+        from ..ops import core as _ops
+        if not _ops.stream_wait(self.step_deadline_s):
+            raise EngineFailure(f"the device did not finish a step within {self.step_deadline_s:.0f} s")
+        buf = (C.c_int * 4)()
+        _lib.call("dgpp_status_read", C.cast(buf, C.c_void_p))
+        if buf[0] != 0:
+            raise EngineFailure(f"device status code={buf[0]} count={buf[1]} detail={buf[2]}")
+
+    def _pick(self, logits, slots):
+        """Next tokens of `slots` from their logits rows: greedy, or the device sampler where a request asks for it."""
+        toks = torch.argmax(logits[:len(slots)], dim=-1).tolist()
+        if any(self.slot_cfg[s] for s in slots):
+            sampled = self._sample_rows(logits[:len(slots)].contiguous(), slots)
+            toks = [sampled[i] if self.slot_cfg[s] else t for i, (s, t) in enumerate(zip(slots, toks))]
+        for s, t in zip(slots, toks):
+            self.pending[s] = int(t)
+        return [int(t) for t in toks]
+
+    def _start(self, slot, pos):
         if pos == 0 and self.r.lengths[slot] != 0:
             self.r.reset(slot)
         assert self.r.lengths[slot] == pos, (self.r.lengths[slot], pos)
+
+    def _mixed(self, entries):
+        """entries [(slot, tokens, wants a token)] in one pass -> {slot: picked token}."""
+        logits = self.r.step([(s, t, [len(t) - 1] if w else []) for s, t, w in entries])
+        slots = [s for s, _, w in entries if w]
+        picked = self._pick(logits, slots) if slots else []
+        self._poll_device()
+        return dict(zip(slots, picked))
+
+    def prefill(self, slot, tokens, pos, last):
+        tokens = list(tokens)
+        self._start(slot, pos)
+        if self.mixed:
+            return self._mixed([(slot, tokens, last)]).get(slot, -1)
         logits = self.r.prefill(slot, tokens, chunk=self.prefill_chunk)
         if last:
-            self.pending[slot] = int(torch.argmax(logits[-1]).item())
-            return self.pending[slot]
+            return self._pick(logits[-1:], [slot])[0]
         return -1
+
+    def prefill_group(self, pieces):
+        pieces = [(s, list(t), p, bool(w)) for s, t, p, w in pieces]
+        if not self.mixed:
+            return [self.prefill(s, t, p, w) for s, t, p, w in pieces]
+        for s, _, p, _ in pieces:
+            self._start(s, p)
+        got = self._mixed([(s, t, w) for s, t, _, w in pieces])
+        return [got.get(s, -1) for s, _, _, _ in pieces]
+
+    def mixed_step(self, piece, slots):
+        """One pass for a reader's piece and one decode step of `slots`; None when the runner has no such pass."""
+        if not self.mixed:
+            return None
+        s0, toks, pos, last = piece[0], list(piece[1]), piece[2], bool(piece[3])
+        slots = list(slots)
+        self._start(s0, pos)
+        got = self._mixed([(s0, toks, last)] + [(s, [self.pending[s]], True) for s in slots])
+        return got.get(s0, -1), [[got[s]] for s in slots]
 
     def step_batch(self, slots):
         slots = list(slots)
-        logits = self.r.decode(slots, [self.pending[s] for s in slots])
-        toks = torch.argmax(logits[:len(slots)], dim=-1).tolist()
-        if torch.device(getattr(self.r, "dev", "cpu")).type == "cuda":
-            import ctypes as C
-            from ..ops import _lib
-            buf = (C.c_int * 4)()
-            _lib.call("dgpp_status_read", C.cast(buf, C.c_void_p))
-            if buf[0] != 0:
-                raise EngineFailure(f"device status code={buf[0]} count={buf[1]} detail={buf[2]}")
-        out = []
-        for s, t in zip(slots, toks):
-            self.pending[s] = int(t)
-            out.append([int(t)])
-        return out
+        toks = self._pick(self.r.decode(slots, [self.pending[s] for s in slots]), slots)
+        self._poll_device()
+        return [[t] for t in toks]
 
     def close(self, slot):
         for b in self.blocks[slot]:
             self.table.release(b)
         self.blocks[slot] = []
         self.pending[slot] = None
+        self.slot_cfg[slot] = None
         self.r.reset(slot)

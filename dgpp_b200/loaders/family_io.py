@@ -3,7 +3,8 @@ under its path in the model object (`layers.3.qkv.payload`, `layers.3.moe.expert
 `config.json` that names the family (`model_type` = "dgpp-<family>") and carries the configuration and the format of
 every quantised matrix.  `save_family` writes one; `load_family` rebuilds the model on a device.  Quantised payloads
 and scales travel byte for byte.  The fixture writer of the per-family load / bind / forward checks, and the hand-off
-format between a conversion script and the server for these families.
+format between a conversion script and the server for these families.  The Sitirax family has a published layout of its
+own (`"architecture": "Sitirax"` in config.json, bf16 tensors named layer by layer); it is read and written as published.
 (reference counterparts: src/models/*/loader.cpp + binding.cpp per family, tools' fixture writers; there every family
  binds its publisher's tensor names, which this build does for the dense family only.)
 """
@@ -70,6 +71,26 @@ def _walk(obj: Any, prefix: str = "") -> Iterator[Tuple[str, Any, Callable[[Any]
             yield from _walk(v, path + ".")
 
 
+def load_sitirax(ck, device="cuda", dtype: torch.dtype = torch.bfloat16) -> Any:
+    """A published Sitirax checkpoint -> the packed model (`dtype`: bf16, or fp32 to run everything in 32 bits)."""
+    from ..models.sitirax import SitiraxConfig, SitiraxModel, tensor_shapes
+
+    cfg = SitiraxConfig.from_dict(ck.config)
+    want = set(tensor_shapes(cfg))
+    missing, stray = sorted(want - set(ck.names())), sorted(set(ck.names()) - want)
+    if missing or stray:
+        raise ValueError(f"{ck.dir}: missing tensors {missing[:4]}, tensors the configuration does not use {stray[:4]}")
+    return SitiraxModel.from_tensors(cfg, ck.tensor, device, dtype)
+
+
+def save_sitirax(cfg: Any, tensors: Dict[str, torch.Tensor], out_dir: str) -> None:
+    """Writes config.json and the bf16 tensors of a Sitirax model in its published layout."""
+    os.makedirs(out_dir, exist_ok=True)
+    with open(os.path.join(out_dir, "config.json"), "w") as f:
+        json.dump(cfg.to_dict(), f, indent=1)
+    write_safetensors(os.path.join(out_dir, "model.safetensors"), tensors, {"format": "pt"})
+
+
 def _family_of(model: Any) -> str:
     for name, (_, cls) in _registry().items():
         if type(model) is cls:
@@ -117,11 +138,15 @@ def save_family(model: Any, out_dir: str) -> None:
     write_safetensors(os.path.join(out_dir, "model.safetensors"), tensors, {"format": "pt"})
 
 
-def load_family(spec: str, device="cuda") -> Any:
-    """Rebuilds the model a `save_family` directory holds.  The object tree comes from the family's own constructor
+def load_family(spec: str, device="cuda", dtype: torch.dtype = torch.bfloat16) -> Any:
+    """Rebuilds the model a `save_family` directory (or a published Sitirax checkpoint) holds.  The object tree comes from the family's own constructor
     (every member then takes the stored bytes), so the configuration alone decides which tensors must exist: a missing
     or mis-shaped one is an error that names it."""
     ck = open_checkpoint(spec)
+    if ck.family == "sitirax":
+        return load_sitirax(ck, device, dtype)
+    if dtype != torch.bfloat16:
+        raise ValueError(f"{spec}: the {ck.family} family runs in bf16")
     mt = ck.config.get("model_type", "")
     if not mt.startswith("dgpp-") or mt[5:] not in _registry():
         raise ValueError(f"{spec}: model_type {mt!r} is not a native family checkpoint")
@@ -171,8 +196,15 @@ def _restack(obj: Any, device) -> None:
             _restack(v, device)
 
 
-def runner_for(model: Any, max_rows: int, slots: int, max_seq_len: int, device="cuda") -> Any:
-    """The kernel runner of a family model (what `engine.adapters.RunnerEngine` drives)."""
+def runner_for(model: Any, max_rows: int, slots: int, max_seq_len: int, device="cuda", pool_tokens: int = 0) -> Any:
+    """The kernel runner of a family model (what `engine.adapters.RunnerEngine` drives).  pool_tokens: cache positions shared
+    by all slots (families with a shared pool; 0: every slot at full length)."""
+    from ..models.sitirax import SitiraxModel, SitiraxRunner
+
+    if isinstance(model, SitiraxModel):
+        return SitiraxRunner(model, max_rows, slots, max_seq_len, device, pool_tokens)
+    if pool_tokens:
+        raise ValueError(f"{type(model).__name__} lays its caches out per slot: no shared pool")
     from ..models.dory import DoryRunner
     from ..models.flash_next import FlashNextRunner
     from ..models.glm_flash import GlmFlashRunner
@@ -184,10 +216,22 @@ def runner_for(model: Any, max_rows: int, slots: int, max_seq_len: int, device="
     return cls(model, max_rows, slots, max_seq_len, device)
 
 
+def _tiny_sitirax(vocab: int):
+    from ..models.sitirax import DeltaSpec, LightningSpec, ParallelSpec, SitiraxConfig, WindowSpec
+
+    return SitiraxConfig.uniform(4, 512, vocab, ParallelSpec(WindowSpec(8, 2, 64, 128, 0.125, 256),
+                                                             LightningSpec(4, 64, 64, (0.8, 0.95, 0.99, 0.999)), 0.7, 0.9),
+                                 DeltaSpec(4, 2, 64, 128, 4), 1024, logit_scale=0.25)
+
+
 def tiny_model(family: str, device="cpu", seed: int = 0, vocab: int = 4096) -> Any:
     """A small random-init model of `family` (the shapes the server's `--model <family>-tiny` choices use)."""
     from ..models.moe import MoEConfig
 
+    if family == "sitirax":
+        from ..models.sitirax import SitiraxModel, random_tensors
+        cfg = _tiny_sitirax(vocab)
+        return SitiraxModel.from_tensors(cfg, random_tensors(cfg, seed).__getitem__, device)
     cfg_cls, model_cls = _registry()[family]
     moe = MoEConfig(hidden=512, experts=16, top_k=2, moe_ffn=512, shared_ffn=512)
     if family == "glm_flash":
@@ -212,15 +256,21 @@ def main(argv=None) -> int:
     import argparse
 
     ap = argparse.ArgumentParser(description=main.__doc__)
-    ap.add_argument("--family", required=True, choices=sorted(_registry()))
+    ap.add_argument("--family", required=True, choices=sorted(_registry()) + ["sitirax"])
     ap.add_argument("--out", required=True)
     ap.add_argument("--seed", type=int, default=0)
     ap.add_argument("--vocab", type=int, default=4096)
     ap.add_argument("--check", action="store_true", help="load the directory back and compare the oracle logits of a short prompt")
     a = ap.parse_args(argv)
     model = tiny_model(a.family, "cpu", a.seed, a.vocab)
-    save_family(model, a.out)
-    report = {"family": a.family, "out": a.out, "tensors": sum(1 for _ in _walk(model))}
+    if a.family == "sitirax":
+        from ..models.sitirax import random_tensors
+        tensors = random_tensors(model.cfg, a.seed)
+        save_sitirax(model.cfg, tensors, a.out)
+        report = {"family": a.family, "out": a.out, "tensors": len(tensors)}
+    else:
+        save_family(model, a.out)
+        report = {"family": a.family, "out": a.out, "tensors": sum(1 for _ in _walk(model))}
     if a.check:
         back = load_family(a.out, "cpu")
         t = torch.arange(3, 19) % a.vocab

@@ -2,12 +2,15 @@
 one CUDA graph per batch width (static id / position / request tensors; recurrent state saved around warm-up and
 capture so that only replays move the model), paged KV reservation, full-attention rows on the tensor-core kernels.
 A subclass provides `forward(tokens, positions, row_req, chunk_slot, all_logits, pos0)` and, if it keeps state besides
-the KV cache, `_state_tensors()` and `_reset_state(slot)`.
+the KV cache, `_state_tensors()` and `_reset_state(slot)`.  A subclass whose layers take runs of consecutive tokens of
+several requests in one pass sets `mixed_runs` and provides `forward_runs`; `step` then carries prompt portions and
+single decoded tokens of any requests together.
 (reference counterparts: src/engine/graph_engine.hpp capture / replay, src/engine/paged_blocks.hpp.)
 """
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 from typing import List, Optional
 
 import torch
@@ -15,7 +18,33 @@ import torch
 from ..ops import core as ops
 
 
+@dataclass
+class RowRuns:
+    """The rows of one pass as runs of consecutive tokens, one run per request."""
+    start: torch.Tensor          # int32 [runs + 1] first row of every run
+    row_run0: torch.Tensor       # int32 [rows] first row of the row's run
+    lens: List[int]              # tokens per run
+    slots: List[int]
+    pos0: List[int]              # position of every run's first token
+
+
 class RowRunner:
+    mixed_runs = False           # True: `forward_runs` exists and `step` may be used
+    pooled = False               # True: `kv` is the pool that admission has to ask (its blocks are this runner's memory)
+
+    def _init_pool(self, slots: int, device, kv_shapes, kv_dtype, page: int, max_seq_len: int, max_rows: int,
+                   pool_tokens: int = 0) -> None:
+        """Rows over one shared pool of `pool_tokens` cache positions (default: every slot at full length); kv_shapes lists
+        (kv heads, key width, value width) per attention layer."""
+        from ..engine.kv_cache import PagedKV
+
+        self._init_rows(slots, device, max_rows=max_rows)
+        per = (max_seq_len + page - 1) // page
+        blocks = (pool_tokens + page - 1) // page if pool_tokens else slots * per
+        self.kv = PagedKV(len(kv_shapes), 0, 0, max(blocks, 1), slots, max(min(per, blocks), 1), page, False, device,
+                          shapes=kv_shapes, dtype=kv_dtype)
+        self.pooled = True
+
     def _init_rows(self, slots: int, device, kv_layers: int = 0, kv_heads: int = 0, q_heads: int = 0, head_dim: int = 0,
                    page: int = 64, max_seq_len: int = 0, max_rows: int = 0) -> None:
         from ..engine.kv_cache import PagedKV
@@ -83,9 +112,70 @@ class RowRunner:
         self.lengths[slot] = 0
         self._reset_state(slot)
 
+    def forward_runs(self, tokens, positions, row_req, runs: RowRuns, logit_rows: torch.Tensor):
+        """One pass over runs of several requests -> fp32 logits of the rows named by logit_rows (int64)."""
+        raise NotImplementedError
+
+    @torch.no_grad()
+    def step(self, entries) -> torch.Tensor:
+        """One mixed pass: entries = [(slot, tokens, want)], the next tokens of each (distinct) request and the places among
+        them whose logits are wanted.  Every request advances by its tokens; returns fp32 logits [wanted, V] in the order
+        of the entries and of their `want`.  Passes beyond `max_rows` rows are cut (the state carries over)."""
+        assert self.mixed_runs and entries and len({s for s, _, _ in entries}) == len(entries)
+        for slot, tokens, _ in entries:
+            assert len(tokens) >= 1
+            if not self.kv.reserve(slot, self.lengths[slot] + len(tokens)):
+                raise RuntimeError("KV pool exhausted")
+        if all(len(t) == 1 for _, t, _ in entries):
+            logits = self.decode([s for s, _, _ in entries], [t[0] for _, t, _ in entries])
+            rows = [i for i, (_, _, want) in enumerate(entries) for _ in want]
+            return logits if rows == list(range(len(entries))) else logits[torch.tensor(rows, dtype=torch.long, device=self.dev)]
+        parts, order = [], {}                       # logits per pass; (entry, place) -> row of their concatenation
+        done, found = [0] * len(entries), 0
+        while any(d < len(t) for d, (_, t, _) in zip(done, entries)):
+            room, piece = self.max_rows, []
+            for i, (slot, tokens, _) in enumerate(entries):
+                n = min(len(tokens) - done[i], room)
+                if n > 0:
+                    piece.append((i, slot, tokens[done[i]:done[i] + n]))
+                    room -= n
+            toks, pos, req, run0, start, rows = [], [], [], [], [0], []
+            for i, slot, part in piece:
+                p0 = self.lengths[slot]
+                wanted = set(entries[i][2])
+                for k in range(len(part)):
+                    if done[i] + k in wanted:
+                        order[(i, done[i] + k)] = found
+                        found += 1
+                        rows.append(start[-1] + k)
+                toks += part
+                pos += range(p0, p0 + len(part))
+                req += [slot] * len(part)
+                run0 += [start[-1]] * len(part)
+                start.append(start[-1] + len(part))
+            n = len(toks)
+            flat = torch.tensor(toks + pos + req + run0 + start, dtype=torch.int32).to(self.dev)
+            runs = RowRuns(flat[4 * n:], flat[3 * n:4 * n], [len(p) for _, _, p in piece], [s for _, s, _ in piece],
+                           [self.lengths[s] for _, s, _ in piece])
+            out = self.forward_runs(flat[:n], flat[n:2 * n], flat[2 * n:3 * n], runs,
+                                    torch.tensor(rows, dtype=torch.long, device=self.dev))
+            if rows:
+                parts.append(out)
+            for i, slot, part in piece:
+                self.lengths[slot] += len(part)
+                done[i] += len(part)
+                self._note_tokens(slot, part)
+        idx = [order[(i, k)] for i, (_, _, want) in enumerate(entries) for k in want]
+        if not idx:
+            return torch.empty(0, 0, dtype=torch.float32, device=self.dev)
+        logits = parts[0] if len(parts) == 1 else torch.cat(parts)
+        return logits if idx == list(range(logits.shape[0])) else logits[torch.tensor(idx, dtype=torch.long, device=self.dev)]
+
     @torch.no_grad()
     def prefill(self, slot: int, tokens: List[int], chunk: int = 64) -> torch.Tensor:
         """Appends `tokens` to request `slot`; returns the logits of the last token [1, V]."""
+        if self.mixed_runs:
+            return self.step([(slot, list(tokens), [len(tokens) - 1])])
         start = self.lengths[slot]
         if self.kv is not None:
             assert self.kv.reserve(slot, start + len(tokens)), "KV pool exhausted"

@@ -69,6 +69,13 @@ def lib_path() -> Path:
     return _LIB_PATH
 
 
+def use(path) -> None:
+    """Loads another build of the kernel library (a family's subset, see ``build.ensure``); before the first call only."""
+    global _LIB_PATH
+    assert _LIB is None or Path(path) == _LIB_PATH, "the kernel library is loaded already"
+    _LIB_PATH = Path(path)
+
+
 def available() -> bool:
     return _LIB_PATH.exists()
 

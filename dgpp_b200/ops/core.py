@@ -426,8 +426,25 @@ def pick_splits_fp4(rows: int, n: int, k: int, bn: int, sms: int = 148) -> int:
 
 def linear(x: torch.Tensor, w: QuantLinear, out: Optional[torch.Tensor] = None,
            resid: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Dispatch a linear layer to the tensor-core kernel (all row counts)."""
+    """Dispatch a linear layer to the tensor-core kernel (all row counts); fp32 weights run in true fp32."""
+    if w.fmt == "fp32":
+        assert resid is None
+        return gemm_f32(x, w, out=out)
     return gemm_tc(x, w, out=out, resid=resid)
+
+
+_lib.declare("dgpp_gemm_f32", [P, L, P, F, P, L, I, I, I, P])
+
+
+def gemm_f32(x: torch.Tensor, w: QuantLinear, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[T, N] = alpha * x[T, K] @ w[N, K]^T, everything fp32 (no reduced-precision tensor mode)."""
+    _chk(x, torch.float32, "x")
+    rows, k = x.shape
+    assert k == w.k and w.fmt == "fp32"
+    if out is None:
+        out = torch.empty(rows, w.n, dtype=torch.float32, device=x.device)
+    call("dgpp_gemm_f32", ptr(x), x.stride(0), ptr(w.payload), float(w.alpha), ptr(out), out.stride(0), rows, w.n, k, stream_ptr())
+    return out
 
 
 def rope_kv_write(qkv, positions, row_req, block_table, inv_freq, cache, hq: int, hkv: int, d: int,

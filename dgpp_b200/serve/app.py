@@ -540,9 +540,13 @@ def main(argv=None) -> int:
     ap.add_argument("--host", default="127.0.0.1")
     ap.add_argument("--port", type=int, default=8000)
     ap.add_argument("--model", default="tiny", choices=["tiny", "fake", "hybrid-tiny", "hybrid", "glm-flash-tiny", "dory-tiny", "flash-next-tiny",
-                                                           "minimax-tiny", "mimo-tiny"])
+                                                           "minimax-tiny", "mimo-tiny", "sitirax-tiny"])
     ap.add_argument("--family-dir", default="",
                     help="a native family checkpoint (dgpp_b200.loaders.family_io.save_family) served through the runner adapter")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                    help="--family-dir: float32 runs everything in 32 bits (families that support it)")
+    ap.add_argument("--pool-tokens", type=int, default=0,
+                    help="cache positions shared by all requests (families with a shared pool; 0: every slot at full length)")
     ap.add_argument("--slots", type=int, default=8)
     ap.add_argument("--max-context", type=int, default=4096, help="hybrid models: tokens per request (prompt + output)")
     ap.add_argument("--prefill-chunk", type=int, default=0, help="hybrid models: rows per prefill pass (0: 256 tiny, 2048 full)")
@@ -599,15 +603,20 @@ def main(argv=None) -> int:
         # ids above the byte vocabulary get a printable piece each, so that streamed chunks carry text for every token
         tok = rt.Tokenizer.byte_level([], [("<|im_start|>", 256, True), ("<|im_end|>", 257, True)] +
                                       [(f"<{i}>", i, False) for i in range(258, hc.vocab)], rt.SplitPattern.Qwen2)
-    elif args.family_dir or args.model in ("glm-flash-tiny", "dory-tiny", "flash-next-tiny", "minimax-tiny", "mimo-tiny"):
+    elif args.family_dir or args.model in ("glm-flash-tiny", "dory-tiny", "flash-next-tiny", "minimax-tiny", "mimo-tiny", "sitirax-tiny"):
         # the smaller families behind the generic runner adapter (a native family checkpoint, or random-init smoke
-        # models; greedy, needs a GPU)
+        # models; needs a GPU)
         from ..engine.adapters import RunnerEngine
         from ..models.moe import MoEConfig
 
         if args.family_dir:
             from ..loaders.family_io import load_family, runner_for
-            runner = runner_for(load_family(args.family_dir, "cuda"), 256, args.slots, args.max_context, "cuda")
+            import torch
+            model = load_family(args.family_dir, "cuda", getattr(torch, args.dtype))
+            runner = runner_for(model, 256, args.slots, args.max_context, "cuda", args.pool_tokens)
+        elif args.model == "sitirax-tiny":
+            from ..loaders.family_io import runner_for, tiny_model
+            runner = runner_for(tiny_model("sitirax", "cuda"), 256, args.slots, args.max_context, "cuda", args.pool_tokens)
         elif args.model == "glm-flash-tiny":
             from ..models.glm_flash import GlmFlashConfig, GlmFlashModel, GlmFlashRunner
             fc = GlmFlashConfig(layers=4, hidden=512, vocab=4096, mla_every=2, k_heads=2, v_heads=4, heads=8, q_lora=256,
@@ -636,6 +645,8 @@ def main(argv=None) -> int:
         sched_config = rt.SchedulerConfig()
         sched_config.prefix_cache = False          # the adapter never resumes from cached blocks
         sched_config.prefill_chunk = 256
+        if eng.mixed:
+            sched_config.prefill_group_max = 4     # readers share a pass
     else:
         import torch
 
