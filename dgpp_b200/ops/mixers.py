@@ -143,3 +143,7 @@ def linear_state(g: StateHeads, proj, state, ring, row_slot, positions, low=None
          None if runs is None else ptr(runs.start), None if runs is None else ptr(runs.row_run0), ptr(prep), ptr(o), ptr(out),
          0 if out is None else out.stride(0), ptr(g.norm_w), rows, rows if runs is None else len(runs.lens), g.hk, g.hv, g.DK, g.DV,
          g.vdim, float(g.dim ** -0.5), float(g.eps), int(g.delta), int(runs is None), _f32(proj), stream_ptr())
+
+
+def window_prefill_usable(g: WindowHeads, proj) -> bool:
+    return False

@@ -62,7 +62,7 @@ def tensors(cfg, seed=0, rank_a=10, rank_g=12):
         elif name.endswith(".conv"):
             t = 0.7 * r
         elif name == "embed":
-            t = r
+            t = 0.15 * r                     # small: the layers, not the tied embedding, decide the logits
         else:
             t = r * s[1] ** -0.5 * 1.3
         out[name] = t.to(torch.bfloat16)
