@@ -125,7 +125,6 @@ def kernels(dev, heads: int = 32, kv: int = 8, dim: int = 128, window: int = 102
         req = torch.arange(n, dtype=torch.int32, device=dev) if not seq else torch.zeros(n, dtype=torch.int32, device=dev)
         x, y = rnd(n, cols).to(BF), torch.empty(n, heads * dim, dtype=BF, device=dev)
         runs = RowRuns(i32([0, n]), i32([0] * n), [n], [0], [ctx])
-        tiles = mx.prefill_tiles(runs, dev) if seq and mx.window_prefill_usable(g, x) else None
         scratch = (torch.empty(n * heads * 2 * 2, device=dev), torch.empty(n * heads * 2 * dim, device=dev))
 
         def w_step(c):
@@ -133,10 +132,7 @@ def kernels(dev, heads: int = 32, kv: int = 8, dim: int = 128, window: int = 102
             if not seq:
                 return mx.window_attn(*a, y, fused=True)
             mx.qk_norm_append(*a)
-            if tiles is not None:
-                mx.window_prefill(*a, y, tiles)
-            else:
-                mx.window_attn(*a, y)
+            mx.window_prefill(g, x, c.layers[0], c.block_table, req, pos, runs, y)
 
         def s_step(c):
             ops.rope_kv_write(x, pos, req, c.block_table, inv, c.layers[0], heads, kv, dim)

@@ -37,7 +37,7 @@ NVCC_FLAGS = [
 ]
 # Translation units of the kernel library that a family's runner calls.
 KERNEL_SETS = {
-    "sitirax": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "window_attn", "linear_state", "graph_exec"],
+    "sitirax": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "window_attn", "window_attn_tc", "linear_state", "graph_exec"],
 }
 # Translation units that must not contract a*b+c into fma (sampler parity with the host oracle).
 NO_FMA = {"sample.cu"}

@@ -63,9 +63,30 @@ struct LinGeom {
   static constexpr int kPer = DK / kParts;                      // state rows per thread
 };
 
-__device__ __forceinline__ float conv_tap(const LinearArgs& a, int C, int slot, int pos, int j, int ch) {
-  const int p = pos - j;
-  return p >= 0 ? a.ring[(static_cast<size_t>(slot) * a.taps + p % a.taps) * C + ch] : 0.f;
+// Convolution of one channel at position pos: w[taps - 1] x + sum_j w[taps - 1 - j] past(j).  The loads of four taps are in
+// flight together.  `rows_back` inputs before this one are rows of the pass (x - j * stride), older ones sit in the ring.
+template <typename T>
+__device__ __forceinline__ float conv_channel(const LinearArgs& a, const T* x, int64_t stride, float xv, int rows_back, int C, int slot,
+                                              int pos, int base, int ch) {
+  float acc = a.conv_w[static_cast<size_t>(a.taps - 1) * C + ch] * xv;
+  const float* ring = a.ring + static_cast<size_t>(slot) * a.taps * C + ch;
+  for (int j0 = 1; j0 < a.taps; j0 += 4) {
+    float past[4], w[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int j = j0 + e;
+      past[e] = 0.f;
+      w[e] = 0.f;
+      if (j < a.taps && j <= pos) {
+        w[e] = a.conv_w[static_cast<size_t>(a.taps - 1 - j) * C + ch];
+        if (j <= rows_back) past[e] = ld_elem(x - j * stride);
+        else past[e] = ring[static_cast<size_t>(base - j + (base < j ? a.taps : 0)) * C];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc = fmaf(w[e], past[e], acc);
+  }
+  return acc;
 }
 
 __device__ __forceinline__ float4 fma4(float4 s, float a, float4 acc) {
@@ -96,16 +117,16 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
 #pragma unroll
   for (int i = 0; i < PER; ++i) s[i] = pos > 0 ? sp[static_cast<size_t>(part + PARTS * i) * G::kCols4] : make_float4(0.f, 0.f, 0.f, 0.f);
   // ---- inputs of this head
+  const int base = a.conv_w != nullptr ? pos % a.taps : 0;       // this token's ring entry
   const T* x = static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.c_off;
+#pragma unroll 2
   for (int c = tid; c < 2 * DK + DV; c += NT) {
     const int ch = c < DK ? hk * DK + c : (c < 2 * DK ? (a.hk + hk) * DK + c - DK : 2 * a.hk * DK + h * DV + c - 2 * DK);
     const float xv = ld_elem(x + ch);
     float acc = xv;
     if (a.conv_w != nullptr) {
-      acc = 0.f;
-      for (int j = a.taps - 1; j > 0; --j) acc = fmaf(a.conv_w[static_cast<size_t>(a.taps - 1 - j) * C + ch], conv_tap(a, C, slot, pos, j, ch), acc);
-      acc = fmaf(a.conv_w[static_cast<size_t>(a.taps - 1) * C + ch], xv, acc);
-      if (c >= 2 * DK || h % ratio == 0) a.ring[(static_cast<size_t>(slot) * a.taps + pos % a.taps) * C + ch] = xv;
+      acc = conv_channel(a, x + ch, a.stride, xv, 0, C, slot, pos, base, ch);
+      if (c >= 2 * DK || h % ratio == 0) a.ring[(static_cast<size_t>(slot) * a.taps + base) * C + ch] = xv;
     }
     acc = silu_f32(acc);
     if (c < DK) qs[c] = acc;
@@ -194,55 +215,52 @@ __device__ __forceinline__ PrepView prep_view(const LinearArgs& a) {
   return p;
 }
 
-// grid (hk + hv, rows): blocks x < hk prepare a key head, the others a value head
+// One warp per (row, unit): units < hk prepare a key head, the others a value head.
 template <typename T, int DK, int DV, bool DELTA>
-__global__ void __launch_bounds__(128) lin_prep_kernel(LinearArgs a) {
-  __shared__ float qs[DK], ks[DK], scratch[4];
+__global__ void __launch_bounds__(256) lin_prep_kernel(LinearArgs a) {
   pdl_wait();
-  const int row = blockIdx.y, tid = threadIdx.x;
-  const int slot = a.row_slot[row], pos = a.positions[row], run0 = a.row_run0[row];
+  const int lane = threadIdx.x & 31, units = a.hk + a.hv;
+  const int warp = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (warp >= a.rows * units) return;
+  const int row = warp / units, unit = warp % units;
+  const int slot = a.row_slot[row], pos = a.positions[row], back = row - a.row_run0[row];
   const int C = 2 * a.hk * DK + a.hv * DV;
+  const int base = a.conv_w != nullptr ? pos % a.taps : 0;
   const PrepView pv = prep_view<DK, DV, DELTA>(a);
   auto input = [&](int ch) {
-    const T* x = static_cast<const T*>(a.proj) + a.c_off + ch;
-    const float xv = ld_elem(x + static_cast<size_t>(row) * a.stride);
-    if (a.conv_w == nullptr) return silu_f32(xv);
-    float acc = 0.f;
-    for (int j = a.taps - 1; j > 0; --j) {
-      const float past = row - j >= run0 ? ld_elem(x + static_cast<size_t>(row - j) * a.stride) : conv_tap(a, C, slot, pos, j, ch);
-      acc = fmaf(a.conv_w[static_cast<size_t>(a.taps - 1 - j) * C + ch], past, acc);
-    }
-    return silu_f32(fmaf(a.conv_w[static_cast<size_t>(a.taps - 1) * C + ch], xv, acc));
+    const T* x = static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.c_off + ch;
+    const float xv = ld_elem(x);
+    return silu_f32(a.conv_w == nullptr ? xv : conv_channel(a, x, a.stride, xv, back, C, slot, pos, base, ch));
   };
-  if (static_cast<int>(blockIdx.x) < a.hk) {
-    const int h = blockIdx.x;
-    float q2 = 0.f, k2 = 0.f, qk = 0.f;
-    for (int c = tid; c < DK; c += 128) {
-      const float q = input(h * DK + c), k = input((a.hk + h) * DK + c);
-      qs[c] = q;
-      ks[c] = k;
-      q2 = fmaf(q, q, q2); k2 = fmaf(k, k, k2); qk = fmaf(q, k, qk);
+  if (unit < a.hk) {
+    float q[DK / 32], k[DK / 32], q2 = 0.f, k2 = 0.f, qk = 0.f;
+#pragma unroll
+    for (int i = 0; i < DK / 32; ++i) {
+      q[i] = input(unit * DK + 32 * i + lane);
+      k[i] = input((a.hk + unit) * DK + 32 * i + lane);
+      q2 = fmaf(q[i], q[i], q2); k2 = fmaf(k[i], k[i], k2); qk = fmaf(q[i], k[i], qk);
     }
-    q2 = block_sum_f32(q2, scratch);
-    k2 = block_sum_f32(k2, scratch);
-    qk = block_sum_f32(qk, scratch);
+    q2 = warp_sum_f32(q2); k2 = warp_sum_f32(k2); qk = warp_sum_f32(qk);
     const float rq = DELTA ? a.q_scale / sqrtf(q2 + 1e-6f) : 1.f, rk = DELTA ? 1.f / sqrtf(k2 + 1e-6f) : 1.f;
-    const size_t o = (static_cast<size_t>(row) * a.hk + h) * DK;
-    for (int c = tid; c < DK; c += 128) {
-      pv.q[o + c] = qs[c] * rq;
-      pv.k[o + c] = ks[c] * rk;
+    const size_t o = (static_cast<size_t>(row) * a.hk + unit) * DK + lane;
+#pragma unroll
+    for (int i = 0; i < DK / 32; ++i) {
+      pv.q[o + 32 * i] = q[i] * rq;
+      pv.k[o + 32 * i] = k[i] * rk;
     }
-    if (tid == 0) pv.qk[static_cast<size_t>(row) * a.hk + h] = qk * rq * rk;
+    if (lane == 0) pv.qk[static_cast<size_t>(row) * a.hk + unit] = qk * rq * rk;
     return;
   }
-  const int h = static_cast<int>(blockIdx.x) - a.hk;
+  const int h = unit - a.hk;
   const size_t rh = static_cast<size_t>(row) * a.hv + h;
-  for (int c = tid; c < DV; c += 128) pv.v[rh * DV + c] = input(2 * a.hk * DK + h * DV + c);
+#pragma unroll
+  for (int i = 0; i < DV / 32; ++i) pv.v[rh * DV + 32 * i + lane] = input(2 * a.hk * DK + h * DV + 32 * i + lane);
   if (DELTA) {
     const float ea = -expf(a.A_log[h]);
-    const float* ar = a.low + static_cast<size_t>(row) * a.low_stride + h * DK;
-    for (int c = tid; c < DK; c += 128) pv.g[rh * DK + c] = expf(ea * softplus_f32(ar[c] + a.dt_bias[h * DK + c]));
-    if (tid == 0) pv.b[rh] = sigmoid_f32(ld_elem(static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.b_off + h));
+    const float* ar = a.low + static_cast<size_t>(row) * a.low_stride + h * DK + lane;
+#pragma unroll
+    for (int i = 0; i < DK / 32; ++i) pv.g[rh * DK + 32 * i + lane] = expf(ea * softplus_f32(ar[32 * i] + a.dt_bias[h * DK + 32 * i + lane]));
+    if (lane == 0) pv.b[rh] = sigmoid_f32(ld_elem(static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.b_off + h));
   }
 }
 
@@ -259,54 +277,97 @@ __global__ void __launch_bounds__(256) lin_tail_kernel(LinearArgs a, int C) {
         ld_elem(static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.c_off + ch);
 }
 
-constexpr int kScanCols = 32, kScanParts = 8, kScanThreads = kScanCols * kScanParts, kScanTokens = 16;
+// Token-sequential pass.  A CTA owns 32 columns of one head's state; a thread 4 columns and the rows 4 part + 4 PARTS i + e.
+// Per token the threads of a column group reduce 4 read-outs (and, delta, 4 recalls S^T k) with a halving exchange: every
+// step sends the half of the values the partner keeps, so 8 values over 16 lanes take 8 shuffles instead of 32.
+// Tokens are staged 16 at a time; places behind the run's end hold k = q = v = 0, decay 1, strength 0 and change nothing.
+constexpr int kScanCols = 32, kScanTokens = 16;
 
 template <int DK, bool DELTA>
-struct ScanStage {                                  // floats of one staging buffer
-  static constexpr int kK = 0, kQ = kScanTokens * DK, kG = 2 * kScanTokens * DK;
+struct ScanGeom {
+  static constexpr int kParts = DK >= 64 ? 16 : 8;
+  static constexpr int kThreads = kParts * (kScanCols / 4);
+  static constexpr int kNI = DK / (4 * kParts);
+  static constexpr int kK = 0, kQ = kScanTokens * DK, kG = 2 * kScanTokens * DK;       // floats of one staging buffer
   static constexpr int kV = kG + (DELTA ? kScanTokens * DK : 0);
   static constexpr int kTotal = kV + kScanTokens * kScanCols;
 };
 
-// grid (DV / 32, hv, runs).  Thread (column, part): state rows 4 * part + 32 * i + e of its column.
+// Sums NV values over PARTS lanes; lane `part` ends with the total of value (part / (PARTS / NV)).
+template <int NV, int PARTS>
+__device__ __forceinline__ float halving_sum(float (&v)[NV], int part) {
+  int half = NV / 2;
+#pragma unroll
+  for (int o = PARTS / 2; o > 0; o >>= 1) {
+    if (half >= 1) {
+      const bool up = (part & o) != 0;
+#pragma unroll
+      for (int i = 0; i < NV / 2; ++i) {
+        if (i < half) {
+          const float give = up ? v[i] : v[i + half], keep = up ? v[i + half] : v[i];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+      }
+      half >>= 1;
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+    }
+  }
+  return v[0];
+}
+
+// grid (DV / 32, hv, runs)
 template <int DK, int DV, bool DELTA>
-__global__ void __launch_bounds__(kScanThreads) lin_scan_kernel(LinearArgs a) {
-  using St = ScanStage<DK, DELTA>;
-  constexpr int NI = DK / 32;
-  extern __shared__ __align__(16) float sc_smem[];  // [2][St::kTotal]
+__global__ void __launch_bounds__(ScanGeom<DK, DELTA>::kThreads) lin_scan_kernel(LinearArgs a) {
+  using G = ScanGeom<DK, DELTA>;
+  constexpr int NI = G::kNI, PARTS = G::kParts, NT = G::kThreads;
+  constexpr int SHARE_M = PARTS / (DELTA ? 8 : 4);          // lanes that hold one total
+  extern __shared__ __align__(16) float sc_smem[];          // [2][G::kTotal]
   __shared__ float qk_s[2][kScanTokens], b_s[2][kScanTokens];
   pdl_wait();
-  const int tid = threadIdx.x, col = tid / kScanParts, part = tid % kScanParts;
-  const int h = blockIdx.y, j0 = blockIdx.x * kScanCols;
+  const int tid = threadIdx.x, cg = tid / PARTS, part = tid % PARTS, lane0 = (tid & 31) - part;
+  const int h = blockIdx.y, j0 = blockIdx.x * kScanCols + 4 * cg;
   const int first = a.run_start[blockIdx.z], last = a.run_start[blockIdx.z + 1];
   const int slot = a.row_slot[first];
   const int hk = h / (a.hv / a.hk);
   const PrepView pv = prep_view<DK, DV, DELTA>(a);
   const float dh = DELTA ? 1.f : a.decay[h];
-  float* sp = a.state + (static_cast<size_t>(slot) * a.hv + h) * DK * DV + j0 + col;
+  float* sp = a.state + (static_cast<size_t>(slot) * a.hv + h) * DK * DV + j0;
   const bool fresh = a.positions[first] == 0;
-  float s[NI][4];
+  float s[NI][4][4];                                        // [i][row e][column]
 #pragma unroll
   for (int i = 0; i < NI; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) s[i][e] = fresh ? 0.f : sp[static_cast<size_t>(32 * i + 4 * part + e) * DV];
+    for (int e = 0; e < 4; ++e) {
+      const float4 v = fresh ? make_float4(0.f, 0.f, 0.f, 0.f)
+                             : *reinterpret_cast<const float4*>(sp + static_cast<size_t>(4 * PARTS * i + 4 * part + e) * DV);
+      s[i][e][0] = v.x; s[i][e][1] = v.y; s[i][e][2] = v.z; s[i][e][3] = v.w;
+    }
   auto stage = [&](int buf, int t0) {
-    float* b = sc_smem + buf * St::kTotal;
+    float* b = sc_smem + buf * G::kTotal;
     const int n = min(kScanTokens, last - t0);
-    for (int i = tid; i < n * (DK / 4); i += kScanThreads) {
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), one = make_float4(1.f, 1.f, 1.f, 1.f);
+    for (int i = tid; i < kScanTokens * (DK / 4); i += NT) {
       const int tt = i / (DK / 4), c = (i % (DK / 4)) * 4;
-      const size_t o = (static_cast<size_t>(t0 + tt) * a.hk + hk) * DK + c;
-      cp_async_16(b + St::kK + tt * DK + c, pv.k + o);
-      cp_async_16(b + St::kQ + tt * DK + c, pv.q + o);
-      if (DELTA) cp_async_16(b + St::kG + tt * DK + c, pv.g + (static_cast<size_t>(t0 + tt) * a.hv + h) * DK + c);
+      if (tt < n) {
+        const size_t o = (static_cast<size_t>(t0 + tt) * a.hk + hk) * DK + c;
+        cp_async_16(b + G::kK + tt * DK + c, pv.k + o);
+        cp_async_16(b + G::kQ + tt * DK + c, pv.q + o);
+        if (DELTA) cp_async_16(b + G::kG + tt * DK + c, pv.g + (static_cast<size_t>(t0 + tt) * a.hv + h) * DK + c);
+      } else {
+        *reinterpret_cast<float4*>(b + G::kK + tt * DK + c) = zero;
+        *reinterpret_cast<float4*>(b + G::kQ + tt * DK + c) = zero;
+        if (DELTA) *reinterpret_cast<float4*>(b + G::kG + tt * DK + c) = one;
+      }
     }
-    for (int i = tid; i < n * (kScanCols / 4); i += kScanThreads) {
+    for (int i = tid; i < kScanTokens * (kScanCols / 4); i += NT) {
       const int tt = i / (kScanCols / 4), c = (i % (kScanCols / 4)) * 4;
-      cp_async_16(b + St::kV + tt * kScanCols + c, pv.v + (static_cast<size_t>(t0 + tt) * a.hv + h) * DV + j0 + c);
+      if (tt < n) cp_async_16(b + G::kV + tt * kScanCols + c, pv.v + (static_cast<size_t>(t0 + tt) * a.hv + h) * DV + blockIdx.x * kScanCols + c);
+      else *reinterpret_cast<float4*>(b + G::kV + tt * kScanCols + c) = zero;
     }
-    if (tid < n) {
-      qk_s[buf][tid] = pv.qk[static_cast<size_t>(t0 + tid) * a.hk + hk];
-      if (DELTA) b_s[buf][tid] = pv.b[static_cast<size_t>(t0 + tid) * a.hv + h];
+    if (tid < kScanTokens) {
+      qk_s[buf][tid] = tid < n ? pv.qk[static_cast<size_t>(t0 + tid) * a.hk + hk] : 0.f;
+      if (DELTA) b_s[buf][tid] = tid < n ? pv.b[static_cast<size_t>(t0 + tid) * a.hv + h] : 0.f;
     }
     cp_async_group_commit();
   };
@@ -320,45 +381,69 @@ __global__ void __launch_bounds__(kScanThreads) lin_scan_kernel(LinearArgs a) {
       cp_async_group_wait<0>();
     }
     __syncthreads();
-    const float* b = sc_smem + buf * St::kTotal;
+    const float* b = sc_smem + buf * G::kTotal;
     const int n = min(kScanTokens, last - t0);
-    for (int tt = 0; tt < n; ++tt) {
-      float no = 0.f, mo = 0.f;
-      float4 kv[NI];
+#pragma unroll 4
+    for (int tt = 0; tt < kScanTokens; ++tt) {
+      float val[DELTA ? 8 : 4];
+#pragma unroll
+      for (int c = 0; c < (DELTA ? 8 : 4); ++c) val[c] = 0.f;
+      float kf[NI][4];
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
-        const int c = 32 * i + 4 * part;
-        kv[i] = *reinterpret_cast<const float4*>(b + St::kK + tt * DK + c);
-        const float4 qv = *reinterpret_cast<const float4*>(b + St::kQ + tt * DK + c);
-        float4 gv = make_float4(dh, dh, dh, dh);
-        if (DELTA) gv = *reinterpret_cast<const float4*>(b + St::kG + tt * DK + c);
-        s[i][0] *= gv.x; s[i][1] *= gv.y; s[i][2] *= gv.z; s[i][3] *= gv.w;
-        no = fmaf(s[i][0], qv.x, no); no = fmaf(s[i][1], qv.y, no); no = fmaf(s[i][2], qv.z, no); no = fmaf(s[i][3], qv.w, no);
+        const int r = 4 * PARTS * i + 4 * part;
+        const float4 k4 = *reinterpret_cast<const float4*>(b + G::kK + tt * DK + r);
+        const float4 q4 = *reinterpret_cast<const float4*>(b + G::kQ + tt * DK + r);
+        const float d1 = tt < n ? dh : 1.f;
+        float gf[4] = {d1, d1, d1, d1};
         if (DELTA) {
-          mo = fmaf(s[i][0], kv[i].x, mo); mo = fmaf(s[i][1], kv[i].y, mo);
-          mo = fmaf(s[i][2], kv[i].z, mo); mo = fmaf(s[i][3], kv[i].w, mo);
+          const float4 g4 = *reinterpret_cast<const float4*>(b + G::kG + tt * DK + r);
+          gf[0] = g4.x; gf[1] = g4.y; gf[2] = g4.z; gf[3] = g4.w;
         }
+        const float qf[4] = {q4.x, q4.y, q4.z, q4.w};
+        kf[i][0] = k4.x; kf[i][1] = k4.y; kf[i][2] = k4.z; kf[i][3] = k4.w;
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            s[i][e][c] *= gf[e];
+            if (DELTA) {
+              val[c] = fmaf(s[i][e][c], kf[i][e], val[c]);
+              val[(DELTA ? 4 : 0) + c] = fmaf(s[i][e][c], qf[e], val[(DELTA ? 4 : 0) + c]);
+            } else {
+              val[c] = fmaf(s[i][e][c], qf[e], val[c]);
+            }
+          }
+      }
+      const float4 v4 = *reinterpret_cast<const float4*>(b + G::kV + tt * kScanCols + 4 * cg);
+      float u[4] = {v4.x, v4.y, v4.z, v4.w};
+      const float total = halving_sum<DELTA ? 8 : 4, PARTS>(val, part);
+      if (DELTA) {
+        const float bt = b_s[buf][tt];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) u[c] = bt * (u[c] - __shfl_sync(0xffffffffu, total, lane0 + c * SHARE_M));
       }
 #pragma unroll
-      for (int o = kScanParts / 2; o > 0; o >>= 1) {
-        if (DELTA) mo += __shfl_xor_sync(0xffffffffu, mo, o);
-        no += __shfl_xor_sync(0xffffffffu, no, o);
-      }
-      const float vv = b[St::kV + tt * kScanCols + col];
-      const float u = DELTA ? b_s[buf][tt] * (vv - mo) : vv;
+      for (int i = 0; i < NI; ++i)
 #pragma unroll
-      for (int i = 0; i < NI; ++i) {
-        s[i][0] = fmaf(kv[i].x, u, s[i][0]); s[i][1] = fmaf(kv[i].y, u, s[i][1]);
-        s[i][2] = fmaf(kv[i].z, u, s[i][2]); s[i][3] = fmaf(kv[i].w, u, s[i][3]);
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) s[i][e][c] = fmaf(kf[i][e], u[c], s[i][e][c]);
+      // the lanes that hold the read-out totals add (q . k) u and store their column
+      const int which = part / SHARE_M - (DELTA ? 4 : 0);
+      if (which >= 0 && part % SHARE_M == 0 && tt < n) {
+        const float uc = which == 0 ? u[0] : (which == 1 ? u[1] : (which == 2 ? u[2] : u[3]));
+        a.o[(static_cast<size_t>(t0 + tt) * a.hv + h) * DV + j0 + which] = fmaf(qk_s[buf][tt], uc, total);
       }
-      if (part == 0) a.o[(static_cast<size_t>(t0 + tt) * a.hv + h) * DV + j0 + col] = fmaf(qk_s[buf][tt], u, no);
     }
-    __syncthreads();                                // this buffer's readers are done before it is staged again
+    __syncthreads();                                        // this buffer's readers are done before it is staged again
   }
 #pragma unroll
   for (int i = 0; i < NI; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) sp[static_cast<size_t>(32 * i + 4 * part + e) * DV] = s[i][e];
+    for (int e = 0; e < 4; ++e)
+      *reinterpret_cast<float4*>(sp + static_cast<size_t>(4 * PARTS * i + 4 * part + e) * DV) =
+          make_float4(s[i][e][0], s[i][e][1], s[i][e][2], s[i][e][3]);
 }
 
 template <typename T, int DK, int DV, bool DELTA>
@@ -371,15 +456,15 @@ static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
     DGPP_CUDA_OK(cudaGetLastError());
     return 0;
   }
-  constexpr size_t smem = 2 * ScanStage<DK, DELTA>::kTotal * sizeof(float);
+  constexpr size_t smem = 2 * ScanGeom<DK, DELTA>::kTotal * sizeof(float);
   static bool attr = false;
   if (!attr) {
     DGPP_CUDA_OK(cudaFuncSetAttribute(lin_scan_kernel<DK, DV, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     attr = true;
   }
-  lin_prep_kernel<T, DK, DV, DELTA><<<dim3(a.hk + a.hv, a.rows), 128, 0, st>>>(a);
+  lin_prep_kernel<T, DK, DV, DELTA><<<dgpp_ceil_div(a.rows * (a.hk + a.hv), 8), 256, 0, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
-  lin_scan_kernel<DK, DV, DELTA><<<dim3(DV / kScanCols, a.hv, a.runs), kScanThreads, smem, st>>>(a);
+  lin_scan_kernel<DK, DV, DELTA><<<dim3(DV / kScanCols, a.hv, a.runs), ScanGeom<DK, DELTA>::kThreads, smem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   if (a.conv_w != nullptr) {
     const int C = 2 * a.hk * DK + a.hv * DV;

@@ -52,25 +52,31 @@ resid_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, const 
   }
 }
 
-// grid (groups, rows).  o [rows, groups * gp] fp32, gate [rows, gate_stride] (TG), w [gp] shared by the groups.
+// o [rows, groups * gp] fp32, gate [rows, gate_stride] (TG), w [gp] shared by the groups.  A group is handled by `team` threads
+// (a warp, or the whole CTA for wide groups).
 template <typename T, typename TG>
 __global__ void __launch_bounds__(kStreamThreads)
 gated_group_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int64_t gate_stride, const float* __restrict__ w,
-                        T* __restrict__ out, int64_t out_stride, int groups, int gp, int n, float eps, float scale) {
+                        T* __restrict__ out, int64_t out_stride, int rows, int groups, int gp, int n, float eps, float scale, int team) {
   __shared__ float scratch[kStreamThreads / 32];
   pdl_wait();
-  const int g = blockIdx.x;
-  const size_t row = blockIdx.y;
+  const size_t unit = (static_cast<size_t>(blockIdx.x) * kStreamThreads + threadIdx.x) / team;
+  const bool live = unit < static_cast<size_t>(rows) * groups;
+  const int me = threadIdx.x % team;
+  const size_t row = live ? unit / groups : 0;
+  const int g = live ? static_cast<int>(unit % groups) : 0;
   const float* op = o + (row * groups + g) * static_cast<size_t>(gp);
   const TG* gt = gate + row * gate_stride + static_cast<size_t>(g) * gp;
   T* dst = out + row * out_stride + static_cast<size_t>(g) * gp;
   float ss = 0.f;
-  for (int i = threadIdx.x * 4; i < gp; i += blockDim.x * 4) {
+  for (int i = me * 4; i < gp; i += team * 4) {
     const float4 v = ld_elem4(op + i);
     ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
   }
-  const float r = scale / sqrtf(block_sum_f32(ss, scratch) / static_cast<float>(n) + eps);
-  for (int i = threadIdx.x * 4; i < gp; i += blockDim.x * 4) {
+  ss = team == 32 ? warp_sum_f32(ss) : block_sum_f32(ss, scratch);
+  if (!live) return;
+  const float r = scale / sqrtf(ss / static_cast<float>(n) + eps);
+  for (int i = me * 4; i < gp; i += team * 4) {
     const float4 v = ld_elem4(op + i), a = ld_elem4(gt + i), ww = ld_elem4(w + i);
     st_elem4(dst + i, make_float4(v.x * r * ww.x * sigmoid_f32(a.x), v.y * r * ww.y * sigmoid_f32(a.y),
                                   v.z * r * ww.z * sigmoid_f32(a.z), v.w * r * ww.w * sigmoid_f32(a.w)));
@@ -124,14 +130,15 @@ DGPP_API int dgpp_gated_group_norm(const void* o, const void* gate, int64_t gate
                                    int rows, int groups, int gp, int n, float eps, float scale, int f32, int gate_f32, cudaStream_t st) {
   DGPP_REQUIRE(gp % 8 == 0 && gate_stride % 8 == 0 && out_stride % 8 == 0 && n >= 1 && n <= gp, "gated_group_norm: %d of %d columns", n, gp);
   if (rows == 0) return 0;
-  DGPP_REQUIRE(rows <= 65535, "gated_group_norm: %d rows", rows);
-  int threads = (gp / 4 + 31) / 32 * 32;
-  threads = threads > kStreamThreads ? kStreamThreads : threads;
-  const dim3 grid(groups, rows);
+  const int team = gp <= 512 ? 32 : kStreamThreads;
+  const int64_t blocks = dgpp_ceil_div64(static_cast<int64_t>(rows) * groups * team, kStreamThreads);
   const float *op = static_cast<const float*>(o), *wp = static_cast<const float*>(w);
-  if (f32) gated_group_norm_kernel<float, float><<<grid, threads, 0, st>>>(op, static_cast<const float*>(gate), gate_stride, wp, static_cast<float*>(out), out_stride, groups, gp, n, eps, scale);
-  else if (gate_f32) gated_group_norm_kernel<bf16, float><<<grid, threads, 0, st>>>(op, static_cast<const float*>(gate), gate_stride, wp, static_cast<bf16*>(out), out_stride, groups, gp, n, eps, scale);
-  else gated_group_norm_kernel<bf16, bf16><<<grid, threads, 0, st>>>(op, static_cast<const bf16*>(gate), gate_stride, wp, static_cast<bf16*>(out), out_stride, groups, gp, n, eps, scale);
+#define DGPP_GGN(TT, TG) gated_group_norm_kernel<TT, TG><<<static_cast<unsigned>(blocks), kStreamThreads, 0, st>>>( \
+      op, static_cast<const TG*>(gate), gate_stride, wp, static_cast<TT*>(out), out_stride, rows, groups, gp, n, eps, scale, team)
+  if (f32) DGPP_GGN(float, float);
+  else if (gate_f32) DGPP_GGN(bf16, float);
+  else DGPP_GGN(bf16, bf16);
+#undef DGPP_GGN
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;
 }

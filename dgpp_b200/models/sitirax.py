@@ -461,6 +461,7 @@ class SitiraxRunner(RowRunner):
         self.gu = e(R * big(P.gate_up.n for P in model.layers if P.gate_up is not None), T)
         self.act = e(R * big(P.down.k for P in model.layers if P.down is not None), T)
         self.prep = e(big(P.state.prep_floats(R) for P in model.layers), torch.float32)
+        self.tc_prefill = True                     # prompt rows' window attention on the tensor cores where the kernel takes them
         self.max_splits = 32
         self.scratch = (e(slots * big(g.hq for g in heads) * self.max_splits * 2, torch.float32),
                         e(slots * big(g.hq * g.DV for g in heads) * self.max_splits, torch.float32))
@@ -492,7 +493,10 @@ class SitiraxRunner(RowRunner):
             mx.linear_state(s, proj, *self.states[i], row_req, positions, o=o)
         else:
             mx.qk_norm_append(g, proj, P.q_norm, P.k_norm, cache, bt, row_req, positions)
-            mx.window_attn(g, proj, P.q_norm, P.k_norm, cache, bt, row_req, positions, mixed, m.left_scale)
+            if self.tc_prefill and mx.window_prefill_usable(g, proj, cache.page):
+                mx.window_prefill(g, proj, cache, bt, row_req, positions, runs, mixed, m.left_scale)
+            else:
+                mx.window_attn(g, proj, P.q_norm, P.k_norm, cache, bt, row_req, positions, mixed, m.left_scale)
             mx.linear_state(s, proj, *self.states[i], row_req, positions, runs=runs, prep=self.prep, o=o)
         mx.gated_group_norm(o, proj[:, P.gate_off:], P.right_norm, mixed[:, n_left:], 1, s.hv * s.vdim, self.c.eps, m.right_scale)
 

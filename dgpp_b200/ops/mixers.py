@@ -145,5 +145,20 @@ def linear_state(g: StateHeads, proj, state, ring, row_slot, positions, low=None
          g.vdim, float(g.dim ** -0.5), float(g.eps), int(g.delta), int(runs is None), _f32(proj), stream_ptr())
 
 
-def window_prefill_usable(g: WindowHeads, proj) -> bool:
-    return False
+_lib.declare("dgpp_window_attn_tc", [P, L, I, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, I, I, F, F, P])
+
+
+def window_prefill_usable(g: WindowHeads, proj, page: int = 64) -> bool:
+    """Whether the tensor-core kernel takes these rows (bf16, pages of 64 tokens, at most 128 query heads per key head)."""
+    return proj.dtype == torch.bfloat16 and page == 64 and g.hq // g.hkv <= 128
+
+
+def window_prefill(g: WindowHeads, proj, cache, block_table, row_req, positions, runs, out, out_scale: float = 1.0) -> torch.Tensor:
+    """`window_attn` for runs of prompt rows on the tensor cores (tcgen05); `qk_norm_append` comes before it."""
+    assert cache.k.dtype == proj.dtype == out.dtype == torch.bfloat16
+    per = 128 // (g.hq // g.hkv)
+    tiles = sum(-(-n // per) for n in runs.lens)
+    call("dgpp_window_attn_tc", ptr(proj), proj.stride(0), g.q_off, ptr(cache.k), ptr(cache.v), ptr(block_table), ptr(row_req),
+         ptr(positions), ptr(runs.start), ptr(out), out.stride(0), len(runs.lens), tiles, g.hq, g.hkv, g.D, g.DV, cache.page,
+         block_table.shape[1], cache.k.shape[0], g.window, float(g.scale), float(out_scale), stream_ptr())
+    return out

@@ -141,8 +141,8 @@ class WindowRig:
             starts.append(starts[-1] + q.shape[0])
         runs = type("Runs", (), dict(start=i32(starts), lens=[q.shape[0] for _, q, _, _ in batch], slots=[r for r, _, _, _ in batch],
                                      pos0=[self.lengths[r] for r, _, _, _ in batch]))
-        if not fused and tc and self.mx.window_prefill_usable(self.g, x):
-            self.mx.window_prefill(self.g, x, *args, out, self.mx.prefill_tiles(runs, self.dev), 0.7)
+        if not fused and tc and self.mx.window_prefill_usable(self.g, x, self.kv.page):
+            self.mx.window_prefill(self.g, x, *args[2:], runs, out, 0.7)
         else:
             self.mx.window_attn(self.g, x, *args, out, 0.7, fused=fused, splits=splits, scratch=scratch, row_list=row_list)
         res, o = [], 0
@@ -176,9 +176,10 @@ SHAPES = [(6, 2, 64, 64, 40, 0.2), (5, 1, 24, 72, 17, 0.4), (4, 4, 128, 128, 100
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("page", [64, 16])              # pages of 64 tokens: bf16 prompt rows take the tensor-core kernel
 @pytest.mark.parametrize("shape", SHAPES)
-def test_window_attention_prompt_portions_and_decoding(dev, dtype, shape):
-    rig = WindowRig(dev, dtype, *shape)
+def test_window_attention_prompt_portions_and_decoding(dev, dtype, shape, page):
+    rig = WindowRig(dev, dtype, *shape, page=page)
     n = 150
     q, k, v = rig.random(n, 3)
     want = rig.want(q, k, v)
@@ -217,11 +218,12 @@ def test_a_key_that_stands_out_is_seen_just_inside_the_window_only(dev, dtype, w
             rig.release(0)
 
 
+@pytest.mark.parametrize("page", [64, 16])
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_window_attention_in_unequal_batches_with_reused_pages(dev, dtype):
+def test_window_attention_in_unequal_batches_with_reused_pages(dev, dtype, page):
     """Portions of several requests in one pass, single tokens beside them, requests that end and others that take over their
     pages: each request gets what it gets alone."""
-    rig = WindowRig(dev, dtype, 6, 3, 40, 64, 37, 0.3, max_tokens=192, page=16)
+    rig = WindowRig(dev, dtype, 6, 3, 40, 64, 37, 0.3, max_tokens=192, page=page)
     data = [rig.random(160, 10 + i) for i in range(4)]
     want = [rig.want(*d) for d in data]
     part = lambda i, a, b: tuple(t[a:b] for t in data[i])
