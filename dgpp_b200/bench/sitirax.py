@@ -73,7 +73,7 @@ def kernels(dev, heads: int = 32, kv: int = 8, dim: int = 128, window: int = 102
 
     big = max(rows, batch)
     buf = {"conv": torch.empty(big, C, dtype=BF, device=dev), "o": torch.empty(big, K, dtype=BF, device=dev),
-           "prep": torch.empty(max(delta.prep_floats(big), light.prep_floats(big)), device=dev)}
+           "prep": torch.empty(max(delta.prep_floats(big, 1), light.prep_floats(big, 1)), device=dev)}
     o32, gated = torch.empty(big, K, device=dev), torch.empty(big, K, dtype=BF, device=dev)
     for n, seq in ((batch, False), (rows, True)):
         pos = torch.full((n,), 5, dtype=torch.int32, device=dev) if not seq else torch.arange(5, 5 + n, dtype=torch.int32, device=dev)

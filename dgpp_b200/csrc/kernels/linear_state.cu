@@ -10,13 +10,14 @@
 //
 //   lin_decode   runs of one token: convolution, norms, gates, state update and read-out of a (row, head) in one CTA with
 //                the whole S in registers; the delta rule's output norm and gate are fused in as well
-//   lin_prep     token-parallel part of longer runs -> fp32 scratch (unit q / k, their dot product, v, decays, strengths)
-//   lin_scan     token-sequential part: one CTA per (32 state columns, head, run), S in registers, the next tokens' operands
-//                streaming in with cp.async while the current ones are consumed
+//   lin_prep     token-parallel part of longer runs -> fp32 scratch (unit q / k, v, decays, strengths)
+//   lin_block    16-token blocks in parallel: the block's decay products and token-pair matrices
+//   lin_scan     block-sequential part: one CTA per (32 state columns, head, run), S in registers, the next block's operands
+//                streaming in with cp.async while the current one is consumed
 //   lin_tail     the newest inputs of the convolution go to the request's ring after every reader is done
 //
-// o_t is taken as (g S)^T q + (k . q) u, the read-out after the write, so both reductions over the key channels run
-// together.  A request's first token (position 0) starts from S = 0 and from zeros before it: a slot needs no clearing
+// The decode kernel takes o_t as (g S)^T q + (k . q) u, the read-out after the write, so both reductions over the key channels
+// run together.  A request's first token (position 0) starts from S = 0 and from zeros before it: a slot needs no clearing
 // between requests.  The convolution's history is a ring of `taps` inputs per channel, entry p % taps for position p: a
 // token never overwrites an entry that its own window reads, so decode CTAs of heads that share key heads do not race.
 #include <math.h>
@@ -50,7 +51,7 @@ struct LinearArgs {
   void* out;                // [rows, out_stride] (T): normed and gated read-outs (delta decode)
   int64_t out_stride;
   const float* norm_w;      // [DV]
-  int rows, runs, hk, hv, taps, vdim;
+  int rows, runs, blocks, hk, hv, taps, vdim;
   float q_scale, eps;
 };
 
@@ -68,7 +69,17 @@ struct LinGeom {
 template <typename T>
 __device__ __forceinline__ float conv_channel(const LinearArgs& a, const T* x, int64_t stride, float xv, int rows_back, int C, int slot,
                                               int pos, int base, int ch) {
-  float acc = a.conv_w[static_cast<size_t>(a.taps - 1) * C + ch] * xv;
+  const float* w0 = a.conv_w + static_cast<size_t>(a.taps - 1) * C + ch;
+  float acc = *w0 * xv;
+  if (rows_back >= a.taps - 1) {                 // the usual place in a prompt: every past input is a row of the pass
+#pragma unroll 3
+    for (int j = 1; j < a.taps; ++j) {
+      w0 -= C;
+      x -= stride;
+      acc = fmaf(*w0, ld_elem(x), acc);
+    }
+    return acc;
+  }
   const float* ring = a.ring + static_cast<size_t>(slot) * a.taps * C + ch;
   for (int j0 = 1; j0 < a.taps; j0 += 4) {
     float past[4], w[4];
@@ -197,21 +208,27 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
   }
 }
 
-// Scratch layout of lin_prep (fp32): q [rows, hk, DK] | k [rows, hk, DK] | v [rows, hv, DV] | decay [rows, hv, DK] (delta)
-// | q . k [rows, hk] | strength [rows, hv] (delta)
+// Scratch of a pass over runs (fp32): per row q, k [hk, DK], v [hv, DV], decays [hv, DK] (delta; lin_block replaces them by
+// K * gamma), Q * gamma and the suffix-weighted keys [hv, DK]; per block gamma_16 [hv, DK], P and (delta) T B [hv, 16, 16]; the
+// strengths [rows, hv] (delta) at the end.
 struct PrepView {
-  float *q, *k, *v, *g, *qk, *b;
+  float *q, *k, *v, *g, *kt, *qt, *kh, *gam, *pm, *tb, *b;
 };
 template <int DK, int DV, bool DELTA>
 __device__ __forceinline__ PrepView prep_view(const LinearArgs& a) {
   PrepView p;
-  const size_t R = a.rows;
+  const size_t R = a.rows, B = a.blocks;
   p.q = a.prep;
   p.k = p.q + R * a.hk * DK;
   p.v = p.k + R * a.hk * DK;
   p.g = p.v + R * a.hv * DV;
-  p.qk = p.g + (DELTA ? R * a.hv * DK : 0);
-  p.b = p.qk + R * a.hk;
+  p.kt = p.g;
+  p.qt = p.g + (DELTA ? R * a.hv * DK : 0);
+  p.kh = p.qt + R * a.hv * DK;
+  p.gam = p.kh + R * a.hv * DK;
+  p.pm = p.gam + B * a.hv * DK;
+  p.tb = p.pm + B * a.hv * 256;
+  p.b = p.tb + (DELTA ? B * a.hv * 256 : 0);
   return p;
 }
 
@@ -233,14 +250,14 @@ __global__ void __launch_bounds__(256) lin_prep_kernel(LinearArgs a) {
     return silu_f32(a.conv_w == nullptr ? xv : conv_channel(a, x, a.stride, xv, back, C, slot, pos, base, ch));
   };
   if (unit < a.hk) {
-    float q[DK / 32], k[DK / 32], q2 = 0.f, k2 = 0.f, qk = 0.f;
+    float q[DK / 32], k[DK / 32], q2 = 0.f, k2 = 0.f;
 #pragma unroll
     for (int i = 0; i < DK / 32; ++i) {
       q[i] = input(unit * DK + 32 * i + lane);
       k[i] = input((a.hk + unit) * DK + 32 * i + lane);
-      q2 = fmaf(q[i], q[i], q2); k2 = fmaf(k[i], k[i], k2); qk = fmaf(q[i], k[i], qk);
+      q2 = fmaf(q[i], q[i], q2); k2 = fmaf(k[i], k[i], k2);
     }
-    q2 = warp_sum_f32(q2); k2 = warp_sum_f32(k2); qk = warp_sum_f32(qk);
+    q2 = warp_sum_f32(q2); k2 = warp_sum_f32(k2);
     const float rq = DELTA ? a.q_scale / sqrtf(q2 + 1e-6f) : 1.f, rk = DELTA ? 1.f / sqrtf(k2 + 1e-6f) : 1.f;
     const size_t o = (static_cast<size_t>(row) * a.hk + unit) * DK + lane;
 #pragma unroll
@@ -248,7 +265,6 @@ __global__ void __launch_bounds__(256) lin_prep_kernel(LinearArgs a) {
       pv.q[o + 32 * i] = q[i] * rq;
       pv.k[o + 32 * i] = k[i] * rk;
     }
-    if (lane == 0) pv.qk[static_cast<size_t>(row) * a.hk + unit] = qk * rq * rk;
     return;
   }
   const int h = unit - a.hk;
@@ -277,25 +293,21 @@ __global__ void __launch_bounds__(256) lin_tail_kernel(LinearArgs a, int C) {
         ld_elem(static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.c_off + ch);
 }
 
-// Token-sequential pass.  A CTA owns 32 columns of one head's state; a thread 4 columns and the rows 4 part + 4 PARTS i + e.
-// Per token the threads of a column group reduce 4 read-outs (and, delta, 4 recalls S^T k) with a halving exchange: every
-// step sends the half of the values the partner keeps, so 8 values over 16 lanes take 8 shuffles instead of 32.
-// Tokens are staged 16 at a time; places behind the run's end hold k = q = v = 0, decay 1, strength 0 and change nothing.
-constexpr int kScanCols = 32, kScanTokens = 16;
+// Block form of the recurrences, 16 tokens at a time.  With gamma_t = g_1 .. g_t (per key channel, products of decays, never a
+// quotient) and S the state before the block:
+//     delta      W = V - (K * gamma) S,   U = T B W,   T = (I + A)^-1,   A_ts = b_t sum_c k_t k_s (g_(s+1) .. g_t)   (s < t)
+//     lightning  U = V
+//     O = (Q * gamma) S + P U,            P_ts = sum_c q_t k_s (g_(s+1) .. g_t)                                      (s <= t)
+//     S <- gamma_16 * S + (K * g_(t+1) .. g_16)^T U
+// lin_block (parallel over blocks and heads) makes K * gamma, Q * gamma, the suffix-weighted keys, gamma_16, T B and P.
+// Places behind a run's end hold k = q = v = 0, decay 1 and strength 0: they change nothing.
+constexpr int kBlk = 16;
 
-template <int DK, bool DELTA>
-struct ScanGeom {
-  static constexpr int kParts = DK >= 64 ? 16 : 8;
-  static constexpr int kThreads = kParts * (kScanCols / 4);
-  static constexpr int kNI = DK / (4 * kParts);
-  static constexpr int kK = 0, kQ = kScanTokens * DK, kG = 2 * kScanTokens * DK;       // floats of one staging buffer
-  static constexpr int kV = kG + (DELTA ? kScanTokens * DK : 0);
-  static constexpr int kTotal = kV + kScanTokens * kScanCols;
-};
-
-// Sums NV values over PARTS lanes; lane `part` ends with the total of value (part / (PARTS / NV)).
+// Sums NV values over PARTS lanes with a halving exchange: every step sends the half of the values the partner keeps.  Lane
+// `part` ends with the totals of values [part * n, part * n + n), n = max(NV / PARTS, 1) (NV < PARTS: PARTS / NV lanes share
+// value part * NV / PARTS), in v[0 .. n - 1].
 template <int NV, int PARTS>
-__device__ __forceinline__ float halving_sum(float (&v)[NV], int part) {
+__device__ __forceinline__ void halving_sum(float (&v)[NV], int part) {
   int half = NV / 2;
 #pragma unroll
   for (int o = PARTS / 2; o > 0; o >>= 1) {
@@ -313,25 +325,144 @@ __device__ __forceinline__ float halving_sum(float (&v)[NV], int part) {
       v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
     }
   }
-  return v[0];
 }
 
+// The run and the first row of block `blk` (blocks are dealt run by run).
+__device__ __forceinline__ bool find_block(const LinearArgs& a, int blk, int& row0, int& n) {
+  for (int r = 0; r < a.runs; ++r) {
+    const int s = a.run_start[r], len = a.run_start[r + 1] - s, nb = (len + kBlk - 1) / kBlk;
+    if (blk < nb) {
+      row0 = s + blk * kBlk;
+      n = min(kBlk, len - blk * kBlk);
+      return true;
+    }
+    blk -= nb;
+  }
+  return false;
+}
+
+// grid (hv, blocks), 256 threads
+template <int DK, int DV, bool DELTA>
+__global__ void __launch_bounds__(256) lin_block_kernel(LinearArgs a) {
+  extern __shared__ __align__(16) float bl_smem[];
+  float* ks = bl_smem;                                    // [16][DK]
+  float* qs = ks + kBlk * DK;
+  float* gs = qs + kBlk * DK;                             // (delta)
+  __shared__ float A[kBlk][kBlk + 1], b_s[kBlk];
+  pdl_wait();
+  const int h = blockIdx.x, blk = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  int row0 = 0, n = 0;
+  if (!find_block(a, blk, row0, n)) return;
+  const int hk = h / (a.hv / a.hk);
+  const PrepView pv = prep_view<DK, DV, DELTA>(a);
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int i = tid; i < kBlk * (DK / 4); i += 256) {
+    const int t = i / (DK / 4), c = (i % (DK / 4)) * 4;
+    const size_t o = (static_cast<size_t>(row0 + t) * a.hk + hk) * DK + c, og = (static_cast<size_t>(row0 + t) * a.hv + h) * DK + c;
+    *reinterpret_cast<float4*>(ks + t * DK + c) = t < n ? *reinterpret_cast<const float4*>(pv.k + o) : zero;
+    *reinterpret_cast<float4*>(qs + t * DK + c) = t < n ? *reinterpret_cast<const float4*>(pv.q + o) : zero;
+    if (DELTA) *reinterpret_cast<float4*>(gs + t * DK + c) = t < n ? *reinterpret_cast<const float4*>(pv.g + og) : make_float4(1.f, 1.f, 1.f, 1.f);
+  }
+  if (tid < kBlk) b_s[tid] = DELTA && tid < n ? pv.b[static_cast<size_t>(row0 + tid) * a.hv + h] : 0.f;
+  const float dh = DELTA ? 1.f : a.decay[h];
+  __syncthreads();
+  const size_t bh = static_cast<size_t>(blk) * a.hv + h;
+  // ---- products of decays up to and behind every token: two passes over a channel, by different threads where there are enough
+  for (int i = tid; i < 2 * DK; i += 256) {
+    const int c = i % DK;
+    float w = 1.f;
+    if (i < DK) {
+      for (int t = 0; t < n; ++t) {
+        w *= DELTA ? gs[t * DK + c] : dh;
+        const size_t o = (static_cast<size_t>(row0 + t) * a.hv + h) * DK + c;
+        if (DELTA) pv.kt[o] = ks[t * DK + c] * w;
+        pv.qt[o] = qs[t * DK + c] * w;
+      }
+      pv.gam[bh * DK + c] = w;
+    } else {
+      for (int t = n - 1; t >= 0; --t) {
+        pv.kh[(static_cast<size_t>(row0 + t) * a.hv + h) * DK + c] = ks[t * DK + c] * w;
+        w *= DELTA ? gs[t * DK + c] : dh;
+      }
+    }
+  }
+  // ---- token pairs: a warp takes the writers s = warp and 15 - warp and walks the readers t >= s
+#pragma unroll 1
+  for (int which = 0; which < 2; ++which) {
+    const int s = which ? kBlk - 1 - warp : warp;
+    float run[DK / 32], val[2 * kBlk];
+#pragma unroll
+    for (int i = 0; i < DK / 32; ++i) run[i] = ks[s * DK + 32 * i + lane];
+#pragma unroll
+    for (int t = 0; t < kBlk; ++t) {
+      val[t] = 0.f;
+      val[kBlk + t] = 0.f;
+      if (t >= s) {
+#pragma unroll
+        for (int i = 0; i < DK / 32; ++i) {
+          const int c = t * DK + 32 * i + lane;
+          if (t > s) run[i] *= DELTA ? gs[c] : dh;
+          if (DELTA) val[t] = fmaf(run[i], ks[c], val[t]);
+          val[kBlk + t] = fmaf(run[i], qs[c], val[kBlk + t]);
+        }
+      }
+    }
+    halving_sum<2 * kBlk, 32>(val, lane);
+    const int t = lane & (kBlk - 1);
+    if (lane < kBlk) A[t][s] = DELTA && t > s ? b_s[t] * val[0] : 0.f;
+    else pv.pm[bh * kBlk * kBlk + t * kBlk + s] = t >= s ? val[0] : 0.f;
+  }
+  if (!DELTA) return;
+  __syncthreads();
+  // ---- T B: column j of (I + A)^-1 by forward substitution, one lane per column
+  if (tid < kBlk) {
+    float col[kBlk];
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) {
+      float acc = i == tid ? 1.f : 0.f;
+#pragma unroll
+      for (int j = 0; j < i; ++j) acc = fmaf(-A[i][j], col[j], acc);
+      col[i] = acc;
+      pv.tb[bh * kBlk * kBlk + i * kBlk + tid] = acc * b_s[tid];
+    }
+  }
+}
+
+constexpr int kScanCols = 32;
+
+template <int DK, bool DELTA>
+struct ScanGeom {
+  static constexpr int kParts = DK >= 128 ? 32 : DK / 4;    // threads that share a column
+  static constexpr int kThreads = kParts * (kScanCols / 4);
+  static constexpr int kNI = DK / (4 * kParts);
+  // floats of one staging buffer
+  static constexpr int kQ = 0, kH = kBlk * DK, kK = 2 * kBlk * DK;
+  static constexpr int kV = kK + (DELTA ? kBlk * DK : 0);
+  static constexpr int kP = kV + kBlk * kScanCols, kT = kP + kBlk * kBlk;
+  static constexpr int kG = kT + (DELTA ? kBlk * kBlk : 0);
+  static constexpr int kTotal = kG + DK;
+};
+
+// Block-sequential pass.  A CTA owns 32 columns of one head's state in registers: a thread 4 columns and the rows
+// 4 part + 4 PARTS i + e; the PARTS lanes of a column group sit in one warp, so a group works through a block on its own and
+// the CTA only meets at the staging buffers (the next block streams in with cp.async meanwhile).
 // grid (DV / 32, hv, runs)
 template <int DK, int DV, bool DELTA>
 __global__ void __launch_bounds__(ScanGeom<DK, DELTA>::kThreads) lin_scan_kernel(LinearArgs a) {
   using G = ScanGeom<DK, DELTA>;
   constexpr int NI = G::kNI, PARTS = G::kParts, NT = G::kThreads;
-  constexpr int SHARE_M = PARTS / (DELTA ? 8 : 4);          // lanes that hold one total
-  extern __shared__ __align__(16) float sc_smem[];          // [2][G::kTotal]
-  __shared__ float qk_s[2][kScanTokens], b_s[2][kScanTokens];
+  constexpr int NV = 4 * kBlk, CNT = NV / PARTS;            // values of a group's block; totals per lane (2, 4 or 8)
+  extern __shared__ __align__(16) float sc_smem[];          // [2][G::kTotal], then W and U of every group [8][2][64]
   pdl_wait();
-  const int tid = threadIdx.x, cg = tid / PARTS, part = tid % PARTS, lane0 = (tid & 31) - part;
-  const int h = blockIdx.y, j0 = blockIdx.x * kScanCols + 4 * cg;
+  const int tid = threadIdx.x, cg = tid / PARTS, part = tid % PARTS;
+  const int h = blockIdx.y, jb = blockIdx.x * kScanCols, j0 = jb + 4 * cg;
   const int first = a.run_start[blockIdx.z], last = a.run_start[blockIdx.z + 1];
+  int blk = 0;
+  for (int r = 0; r < static_cast<int>(blockIdx.z); ++r) blk += (a.run_start[r + 1] - a.run_start[r] + kBlk - 1) / kBlk;
   const int slot = a.row_slot[first];
-  const int hk = h / (a.hv / a.hk);
   const PrepView pv = prep_view<DK, DV, DELTA>(a);
-  const float dh = DELTA ? 1.f : a.decay[h];
+  float* ws = sc_smem + 2 * G::kTotal + cg * 2 * NV;        // [16][4] W
+  float* us = ws + NV;                                      // [16][4] U
   float* sp = a.state + (static_cast<size_t>(slot) * a.hv + h) * DK * DV + j0;
   const bool fresh = a.positions[first] == 0;
   float s[NI][4][4];                                        // [i][row e][column]
@@ -343,97 +474,128 @@ __global__ void __launch_bounds__(ScanGeom<DK, DELTA>::kThreads) lin_scan_kernel
                              : *reinterpret_cast<const float4*>(sp + static_cast<size_t>(4 * PARTS * i + 4 * part + e) * DV);
       s[i][e][0] = v.x; s[i][e][1] = v.y; s[i][e][2] = v.z; s[i][e][3] = v.w;
     }
-  auto stage = [&](int buf, int t0) {
-    float* b = sc_smem + buf * G::kTotal;
-    const int n = min(kScanTokens, last - t0);
-    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), one = make_float4(1.f, 1.f, 1.f, 1.f);
-    for (int i = tid; i < kScanTokens * (DK / 4); i += NT) {
-      const int tt = i / (DK / 4), c = (i % (DK / 4)) * 4;
-      if (tt < n) {
-        const size_t o = (static_cast<size_t>(t0 + tt) * a.hk + hk) * DK + c;
-        cp_async_16(b + G::kK + tt * DK + c, pv.k + o);
-        cp_async_16(b + G::kQ + tt * DK + c, pv.q + o);
-        if (DELTA) cp_async_16(b + G::kG + tt * DK + c, pv.g + (static_cast<size_t>(t0 + tt) * a.hv + h) * DK + c);
+  auto stage = [&](int buf, int t0, int b) {
+    float* d = sc_smem + buf * G::kTotal;
+    const int n = min(kBlk, last - t0);
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = tid; i < kBlk * (DK / 4); i += NT) {
+      const int t = i / (DK / 4), c = (i % (DK / 4)) * 4;
+      const size_t o = (static_cast<size_t>(t0 + t) * a.hv + h) * DK + c;
+      if (t < n) {
+        cp_async_16(d + G::kQ + t * DK + c, pv.qt + o);
+        cp_async_16(d + G::kH + t * DK + c, pv.kh + o);
+        if (DELTA) cp_async_16(d + G::kK + t * DK + c, pv.kt + o);
       } else {
-        *reinterpret_cast<float4*>(b + G::kK + tt * DK + c) = zero;
-        *reinterpret_cast<float4*>(b + G::kQ + tt * DK + c) = zero;
-        if (DELTA) *reinterpret_cast<float4*>(b + G::kG + tt * DK + c) = one;
+        *reinterpret_cast<float4*>(d + G::kQ + t * DK + c) = zero;
+        *reinterpret_cast<float4*>(d + G::kH + t * DK + c) = zero;
+        if (DELTA) *reinterpret_cast<float4*>(d + G::kK + t * DK + c) = zero;
       }
     }
-    for (int i = tid; i < kScanTokens * (kScanCols / 4); i += NT) {
-      const int tt = i / (kScanCols / 4), c = (i % (kScanCols / 4)) * 4;
-      if (tt < n) cp_async_16(b + G::kV + tt * kScanCols + c, pv.v + (static_cast<size_t>(t0 + tt) * a.hv + h) * DV + blockIdx.x * kScanCols + c);
-      else *reinterpret_cast<float4*>(b + G::kV + tt * kScanCols + c) = zero;
+    for (int i = tid; i < kBlk * (kScanCols / 4); i += NT) {
+      const int t = i / (kScanCols / 4), c = (i % (kScanCols / 4)) * 4;
+      if (t < n) cp_async_16(d + G::kV + t * kScanCols + c, pv.v + (static_cast<size_t>(t0 + t) * a.hv + h) * DV + jb + c);
+      else *reinterpret_cast<float4*>(d + G::kV + t * kScanCols + c) = zero;
     }
-    if (tid < kScanTokens) {
-      qk_s[buf][tid] = tid < n ? pv.qk[static_cast<size_t>(t0 + tid) * a.hk + hk] : 0.f;
-      if (DELTA) b_s[buf][tid] = tid < n ? pv.b[static_cast<size_t>(t0 + tid) * a.hv + h] : 0.f;
+    const size_t bh = static_cast<size_t>(b) * a.hv + h;
+    for (int i = tid * 4; i < kBlk * kBlk; i += NT * 4) {
+      cp_async_16(d + G::kP + i, pv.pm + bh * kBlk * kBlk + i);
+      if (DELTA) cp_async_16(d + G::kT + i, pv.tb + bh * kBlk * kBlk + i);
     }
+    for (int i = tid * 4; i < DK; i += NT * 4) cp_async_16(d + G::kG + i, pv.gam + bh * DK + i);
     cp_async_group_commit();
   };
-  stage(0, first);
+  // partial products of 16 staged rows with this thread's part of the state, summed over the group
+  auto rows_times_state = [&](const float* m, float (&val)[NV]) {
+#pragma unroll
+    for (int t = 0; t < kBlk; ++t) {
+#pragma unroll
+      for (int c = 0; c < 4; ++c) val[4 * t + c] = 0.f;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const float4 m4 = *reinterpret_cast<const float4*>(m + t * DK + 4 * PARTS * i + 4 * part);
+        const float mf[4] = {m4.x, m4.y, m4.z, m4.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) val[4 * t + c] = fmaf(mf[e], s[i][e][c], val[4 * t + c]);
+      }
+    }
+    halving_sum<NV, PARTS>(val, part);
+  };
+  // rows of a 16 x 16 matrix (row-major) times a group's [16][4] block `x` (row stride xs): this lane's CNT entries
+  auto pairs_times = [&](const float* m, const float* x, int xs, float (&out)[CNT]) {
+#pragma unroll
+    for (int i = 0; i < CNT; ++i) {
+      const int t = (part * CNT + i) / 4, c = (part * CNT + i) % 4;
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < kBlk; j += 4) {
+        const float4 m4 = *reinterpret_cast<const float4*>(m + t * kBlk + j);
+        acc = fmaf(m4.x, x[j * xs + c], acc);
+        acc = fmaf(m4.y, x[(j + 1) * xs + c], acc);
+        acc = fmaf(m4.z, x[(j + 2) * xs + c], acc);
+        acc = fmaf(m4.w, x[(j + 3) * xs + c], acc);
+      }
+      out[i] = acc;
+    }
+  };
+  stage(0, first, blk);
   int buf = 0;
-  for (int t0 = first; t0 < last; t0 += kScanTokens, buf ^= 1) {
-    if (t0 + kScanTokens < last) {
-      stage(buf ^ 1, t0 + kScanTokens);
+  for (int t0 = first; t0 < last; t0 += kBlk, buf ^= 1, ++blk) {
+    if (t0 + kBlk < last) {
+      stage(buf ^ 1, t0 + kBlk, blk + 1);
       cp_async_group_wait<1>();
     } else {
       cp_async_group_wait<0>();
     }
     __syncthreads();
-    const float* b = sc_smem + buf * G::kTotal;
-    const int n = min(kScanTokens, last - t0);
-#pragma unroll 4
-    for (int tt = 0; tt < kScanTokens; ++tt) {
-      float val[DELTA ? 8 : 4];
+    const float* d = sc_smem + buf * G::kTotal;
+    const float* vb = d + G::kV + 4 * cg;                   // [16] rows of 32 columns, this group's 4
+    const int n = min(kBlk, last - t0);
+    float val[NV], x[CNT];
+    if (DELTA) {
+      rows_times_state(d + G::kK, val);
 #pragma unroll
-      for (int c = 0; c < (DELTA ? 8 : 4); ++c) val[c] = 0.f;
-      float kf[NI][4];
+      for (int i = 0; i < CNT; ++i) {
+        const int idx = part * CNT + i;
+        ws[idx] = vb[(idx / 4) * kScanCols + idx % 4] - val[i];
+      }
+      __syncwarp();
+      pairs_times(d + G::kT, ws, 4, x);
+#pragma unroll
+      for (int i = 0; i < CNT; ++i) us[part * CNT + i] = x[i];
+    }
+    rows_times_state(d + G::kQ, val);
+    __syncwarp();
+    const float* u = DELTA ? us : vb;
+    constexpr int ustride = DELTA ? 4 : kScanCols;
+    pairs_times(d + G::kP, u, ustride, x);
+#pragma unroll
+    for (int i = 0; i < CNT; ++i) {
+      const int idx = part * CNT + i;
+      if (idx / 4 < n) a.o[(static_cast<size_t>(t0 + idx / 4) * a.hv + h) * DV + j0 + idx % 4] = val[i] + x[i];
+    }
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const float4 g4 = *reinterpret_cast<const float4*>(d + G::kG + 4 * PARTS * i + 4 * part);
+      const float gf[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) s[i][e][c] *= gf[e];
+    }
+#pragma unroll
+    for (int t = 0; t < kBlk; ++t) {
+      const float4 u4 = *reinterpret_cast<const float4*>(u + t * ustride);
+      const float uf[4] = {u4.x, u4.y, u4.z, u4.w};
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
-        const int r = 4 * PARTS * i + 4 * part;
-        const float4 k4 = *reinterpret_cast<const float4*>(b + G::kK + tt * DK + r);
-        const float4 q4 = *reinterpret_cast<const float4*>(b + G::kQ + tt * DK + r);
-        const float d1 = tt < n ? dh : 1.f;
-        float gf[4] = {d1, d1, d1, d1};
-        if (DELTA) {
-          const float4 g4 = *reinterpret_cast<const float4*>(b + G::kG + tt * DK + r);
-          gf[0] = g4.x; gf[1] = g4.y; gf[2] = g4.z; gf[3] = g4.w;
-        }
-        const float qf[4] = {q4.x, q4.y, q4.z, q4.w};
-        kf[i][0] = k4.x; kf[i][1] = k4.y; kf[i][2] = k4.z; kf[i][3] = k4.w;
+        const float4 k4 = *reinterpret_cast<const float4*>(d + G::kH + t * DK + 4 * PARTS * i + 4 * part);
+        const float kf[4] = {k4.x, k4.y, k4.z, k4.w};
 #pragma unroll
         for (int e = 0; e < 4; ++e)
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            s[i][e][c] *= gf[e];
-            if (DELTA) {
-              val[c] = fmaf(s[i][e][c], kf[i][e], val[c]);
-              val[(DELTA ? 4 : 0) + c] = fmaf(s[i][e][c], qf[e], val[(DELTA ? 4 : 0) + c]);
-            } else {
-              val[c] = fmaf(s[i][e][c], qf[e], val[c]);
-            }
-          }
-      }
-      const float4 v4 = *reinterpret_cast<const float4*>(b + G::kV + tt * kScanCols + 4 * cg);
-      float u[4] = {v4.x, v4.y, v4.z, v4.w};
-      const float total = halving_sum<DELTA ? 8 : 4, PARTS>(val, part);
-      if (DELTA) {
-        const float bt = b_s[buf][tt];
-#pragma unroll
-        for (int c = 0; c < 4; ++c) u[c] = bt * (u[c] - __shfl_sync(0xffffffffu, total, lane0 + c * SHARE_M));
-      }
-#pragma unroll
-      for (int i = 0; i < NI; ++i)
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-#pragma unroll
-          for (int c = 0; c < 4; ++c) s[i][e][c] = fmaf(kf[i][e], u[c], s[i][e][c]);
-      // the lanes that hold the read-out totals add (q . k) u and store their column
-      const int which = part / SHARE_M - (DELTA ? 4 : 0);
-      if (which >= 0 && part % SHARE_M == 0 && tt < n) {
-        const float uc = which == 0 ? u[0] : (which == 1 ? u[1] : (which == 2 ? u[2] : u[3]));
-        a.o[(static_cast<size_t>(t0 + tt) * a.hv + h) * DV + j0 + which] = fmaf(qk_s[buf][tt], uc, total);
+          for (int c = 0; c < 4; ++c) s[i][e][c] = fmaf(kf[e], uf[c], s[i][e][c]);
       }
     }
     __syncthreads();                                        // this buffer's readers are done before it is staged again
@@ -456,13 +618,17 @@ static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
     DGPP_CUDA_OK(cudaGetLastError());
     return 0;
   }
-  constexpr size_t smem = 2 * ScanGeom<DK, DELTA>::kTotal * sizeof(float);
+  constexpr size_t smem = (2 * ScanGeom<DK, DELTA>::kTotal + 8 * 2 * 4 * kBlk) * sizeof(float);
+  constexpr size_t bsmem = (DELTA ? 3 : 2) * static_cast<size_t>(kBlk) * DK * sizeof(float);
   static bool attr = false;
   if (!attr) {
+    DGPP_CUDA_OK(cudaFuncSetAttribute(lin_block_kernel<DK, DV, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bsmem)));
     DGPP_CUDA_OK(cudaFuncSetAttribute(lin_scan_kernel<DK, DV, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     attr = true;
   }
   lin_prep_kernel<T, DK, DV, DELTA><<<dgpp_ceil_div(a.rows * (a.hk + a.hv), 8), 256, 0, st>>>(a);
+  DGPP_CUDA_OK(cudaGetLastError());
+  lin_block_kernel<DK, DV, DELTA><<<dim3(a.hv, a.blocks), 256, bsmem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   lin_scan_kernel<DK, DV, DELTA><<<dim3(DV / kScanCols, a.hv, a.runs), ScanGeom<DK, DELTA>::kThreads, smem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
@@ -491,15 +657,16 @@ static int launch_lin_dims(const LinearArgs& a, int DK, int DV, int decode, cuda
 using namespace dgpp;
 
 // decode = 1: every row is a run of its own; norm and gate are applied (delta) and `out` is written, or the raw read-outs go
-// to `o` (lightning).  decode = 0: the runs named by run_start / row_run0; `o` receives the raw read-outs, prep is scratch
-// of rows * (2 hk DK + hv DV + hv DK + hk + hv) floats.  delta = 0: lightning (decay [hv]; hk = hv, no low / A_log / dt_bias).
+// to `o` (lightning).  decode = 0: the runs named by run_start / row_run0, cut into `blocks` = sum of ceil(length / 16) blocks;
+// `o` receives the raw read-outs, prep is scratch of rows * (2 hk DK + hv (DV + 3 DK + 1)) + blocks * hv (DK + 512) floats.  delta = 0: lightning (decay [hv]; hk = hv, no low / A_log / dt_bias).
 DGPP_API int dgpp_linear_state(const void* proj, int64_t stride, int c_off, int b_off, const void* low, int64_t low_stride,
                                const void* conv_w, void* ring, int taps, const void* A_log, const void* dt_bias, const void* decay,
                                void* state, const void* row_slot, const void* positions, const void* run_start, const void* row_run0,
-                               void* prep, void* o, void* out, int64_t out_stride, const void* norm_w, int rows, int runs, int hk,
+                               void* prep, void* o, void* out, int64_t out_stride, const void* norm_w, int rows, int runs, int blocks, int hk,
                                int hv, int DK, int DV, int vdim, float q_scale, float eps, int delta, int decode, int f32,
                                cudaStream_t st) {
   DGPP_REQUIRE(hk > 0 && hv % hk == 0, "linear_state: %d value heads over %d key heads", hv, hk);
+  DGPP_REQUIRE(decode || (blocks >= 1 && blocks <= 65535), "linear_state: %d blocks", blocks);
   DGPP_REQUIRE(rows >= 0 && rows <= 65535 && runs <= 65535, "linear_state: %d rows in %d runs", rows, runs);
   DGPP_REQUIRE(conv_w == nullptr || (taps >= 1 && ring), "linear_state: a convolution of %d taps needs its ring", taps);
   DGPP_REQUIRE(!delta || (low && A_log && dt_bias), "linear_state: the delta rule needs its decay inputs");
@@ -518,7 +685,7 @@ DGPP_API int dgpp_linear_state(const void* proj, int64_t stride, int c_off, int 
   a.run_start = static_cast<const int32_t*>(run_start); a.row_run0 = static_cast<const int32_t*>(row_run0);
   a.prep = static_cast<float*>(prep); a.o = static_cast<float*>(o);
   a.out = out; a.out_stride = out_stride; a.norm_w = static_cast<const float*>(norm_w);
-  a.rows = rows; a.runs = runs; a.hk = hk; a.hv = hv; a.vdim = vdim; a.q_scale = q_scale; a.eps = eps;
+  a.rows = rows; a.runs = runs; a.blocks = blocks; a.hk = hk; a.hv = hv; a.vdim = vdim; a.q_scale = q_scale; a.eps = eps;
   if (f32) return delta ? launch_lin_dims<float, true>(a, DK, DV, decode, st) : launch_lin_dims<float, false>(a, DK, DV, decode, st);
   return delta ? launch_lin_dims<bf16, true>(a, DK, DV, decode, st) : launch_lin_dims<bf16, false>(a, DK, DV, decode, st);
 }

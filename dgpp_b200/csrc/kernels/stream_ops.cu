@@ -83,8 +83,9 @@ gated_group_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate
   }
 }
 
+// 0.5 z (1 + tanh(u)) = z / (1 + exp(-2 u)),  u = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_tanh_f32(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
 // gate_up [rows, 2 * inter] (gate columns, then up columns) -> out [rows, inter]

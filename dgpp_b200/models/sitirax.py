@@ -460,7 +460,7 @@ class SitiraxRunner(RowRunner):
         self.o = e(R * big(P.state.hv * P.state.DV for P in model.layers), torch.float32)
         self.gu = e(R * big(P.gate_up.n for P in model.layers if P.gate_up is not None), T)
         self.act = e(R * big(P.down.k for P in model.layers if P.down is not None), T)
-        self.prep = e(big(P.state.prep_floats(R) for P in model.layers), torch.float32)
+        self.prep = e(big(P.state.prep_floats(R, slots) for P in model.layers), torch.float32)
         self.tc_prefill = True                     # prompt rows' window attention on the tensor cores where the kernel takes them
         self.max_splits = 32
         self.scratch = (e(slots * big(g.hq for g in heads) * self.max_splits * 2, torch.float32),

@@ -16,7 +16,7 @@ _lib.declare("dgpp_gated_group_norm", [P, P, L, P, P, L, I, I, I, I, F, F, I, I,
 _lib.declare("dgpp_geglu", [P, P, I, I, I, P])
 _lib.declare("dgpp_qk_norm_append", [P, L, I, I, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P])
 _lib.declare("dgpp_window_attn", [P, L, I, I, I, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, I, I, I, F, F, F, I, P])
-_lib.declare("dgpp_linear_state", [P, L, I, I, P, L, P, P, I, P, P, P, P, P, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, F, F,
+_lib.declare("dgpp_linear_state", [P, L, I, I, P, L, P, P, I, P, P, P, P, P, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, F, F,
                                    I, I, I, P])
 
 
@@ -128,8 +128,10 @@ class StateHeads:
         ring = torch.zeros(slots, self.taps, self.channels, dtype=torch.float32, device=device) if self.taps else None
         return state, ring
 
-    def prep_floats(self, rows: int) -> int:
-        return rows * (self.channels + self.hv * self.DK + self.hk + self.hv)
+    def prep_floats(self, rows: int, runs: int) -> int:
+        """Scratch of a pass over `rows` rows in at most `runs` runs."""
+        blocks = rows // 16 + runs
+        return rows * (self.channels + self.hv * (3 * self.DK + 1)) + blocks * self.hv * (self.DK + 512)
 
 
 def linear_state(g: StateHeads, proj, state, ring, row_slot, positions, low=None, runs=None, prep=None, o=None, out=None) -> None:
@@ -137,11 +139,12 @@ def linear_state(g: StateHeads, proj, state, ring, row_slot, positions, low=None
     gated read-outs to `out`, lightning its raw read-outs to `o` (fp32).  runs given: runs of consecutive rows, raw read-outs
     to `o`, `prep` is fp32 scratch (`StateHeads.prep_floats`)."""
     rows = proj.shape[0]
-    assert state.dtype == torch.float32 and (prep is None or prep.numel() >= g.prep_floats(rows))
+    blocks = 0 if runs is None else sum(-(-n // 16) for n in runs.lens)
+    assert state.dtype == torch.float32 and (runs is None or prep.numel() >= g.prep_floats(rows, len(runs.lens)))
     call("dgpp_linear_state", ptr(proj), proj.stride(0), g.c_off, g.b_off, ptr(low), 0 if low is None else low.stride(0),
          ptr(g.conv_w), ptr(ring), g.taps, ptr(g.A_log), ptr(g.dt_bias), ptr(g.decay), ptr(state), ptr(row_slot), ptr(positions),
          None if runs is None else ptr(runs.start), None if runs is None else ptr(runs.row_run0), ptr(prep), ptr(o), ptr(out),
-         0 if out is None else out.stride(0), ptr(g.norm_w), rows, rows if runs is None else len(runs.lens), g.hk, g.hv, g.DK, g.DV,
+         0 if out is None else out.stride(0), ptr(g.norm_w), rows, rows if runs is None else len(runs.lens), blocks, g.hk, g.hv, g.DK, g.DV,
          g.vdim, float(g.dim ** -0.5), float(g.eps), int(g.delta), int(runs is None), _f32(proj), stream_ptr())
 
 

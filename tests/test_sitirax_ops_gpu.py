@@ -324,7 +324,7 @@ class StateRig:
             self.mx.linear_state(self.g, x, self.state, self.ring, i32(slot), i32(pos), low=low, o=o, out=out)
         else:
             runs = type("Runs", (), dict(start=i32(starts), row_run0=i32([starts[i] for i, n in enumerate(lens) for _ in range(n)]), lens=lens))
-            prep = torch.empty(self.g.prep_floats(rows), device=self.dev)
+            prep = torch.empty(self.g.prep_floats(rows, len(lens)), device=self.dev)
             self.mx.linear_state(self.g, x, self.state, self.ring, i32(slot), i32(pos), low=low, runs=runs, prep=prep, o=o)
             if self.delta:
                 self.mx.gated_group_norm(o, low[:, self.hv * self.K:], self.g.norm_w, out, self.hv, self.vdim, self.eps)
