@@ -148,3 +148,12 @@ def test_runner_engine_with_a_shared_pool(mixed_pass):
         assert got[rid] == want
     assert r.kv.free_blocks() == 8 and r.lengths == [0, 0, 0]
     assert any(k == "runs" and len(set(q)) > 1 for k, _, _, q in r.passes)
+
+
+def test_fixture_writer(tmp_path, capsys):
+    from dgpp_b200.loaders.family_io import main
+
+    assert main(["--family", "sitirax", "--out", str(tmp_path / "ck"), "--vocab", "300", "--check"]) == 0
+    report = json.loads(capsys.readouterr().out)
+    assert report["round_trip_equal"] and report["tensors"] == len(sc.tensor_shapes(SitiraxConfig.from_dict(
+        json.load(open(tmp_path / "ck" / "config.json")))))
