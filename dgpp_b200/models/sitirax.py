@@ -128,14 +128,13 @@ class SitiraxConfig:
                 if e["mlp"].get("kind") != "dense":
                     raise ValueError(f"layer {i}: unknown feed-forward kind {e['mlp'].get('kind')!r}")
                 ff = int(e["mlp"]["ff"])
-            src = int(e.get("weights_of", i))
-            if src != i:
-                if not 0 <= src < i:
-                    raise ValueError(f"layer {i}: weights_of names layer {src}, which does not come before it")
-                src = layers[src].source
-                if layers[src].mixer != spec or layers[src].ff != ff:
-                    raise ValueError(f"layer {i} shares the weights of layer {src} but is described differently")
-            layers.append(LayerSpec(spec, ff, src))
+            layers.append(LayerSpec(spec, ff, int(e.get("weights_of", i))))
+        for i, L in enumerate(layers):
+            src = L.source
+            if not 0 <= src < len(layers) or layers[src].source != src:
+                raise ValueError(f"layer {i}: weights_of names no layer with weights of its own")
+            if (layers[src].mixer, layers[src].ff) != (L.mixer, L.ff):
+                raise ValueError(f"layer {i} shares the weights of layer {src} but is described differently")
         return SitiraxConfig(int(d["width"]), int(d["vocab"]), layers, float(d["norm"]["eps"]), float(d["logit_scale"]))
 
     def to_dict(self) -> dict:
@@ -223,7 +222,7 @@ def random_tensors(cfg: SitiraxConfig, seed: int = 0, rank_a: int = 0, rank_g: i
         elif name.endswith(".conv"):
             t = 0.6 * rnd(*s)
         elif name == "embed":
-            t = rnd(*s) * (std * 4 if std else 1.0)
+            t = rnd(*s) * (std * 4 if std else 0.25)
         else:
             t = rnd(*s) * (std or s[1] ** -0.5)
         out[name] = t.to(BF)
@@ -347,19 +346,17 @@ class SitiraxModel:
                                               norm_w=vec(_pad_vec(t(p + "norm"), 1, m.vdim, V))),
                           gate_off=off[4], w_low=lin(low))
 
-        layers: List[Packed] = []
-        for i, L in enumerate(cfg.plan):
-            if L.source != i:
-                layers.append(layers[L.source])
-                continue
-            p = f"l{i}."
+        own: Dict[int, Packed] = {}
+        for i in sorted({L.source for L in cfg.plan}):
+            L, p = cfg.plan[i], f"l{i}."
             w = parallel(p + "mix.", L.mixer) if isinstance(L.mixer, ParallelSpec) else delta(p + "mix.", L.mixer)
             if L.ff is not None:
                 fp = up8(L.ff)
                 w.norm2 = hvec(p + "norm2")
                 w.gate_up = lin(hid(torch.cat([_pad_rows(t(p + "mlp.gate"), 1, L.ff, fp), _pad_rows(t(p + "mlp.up"), 1, L.ff, fp)])))
                 w.down = lin(hout(_pad_cols(t(p + "mlp.down"), 1, L.ff, fp)))
-            layers.append(w)
+            own[i] = w
+        layers = [own[L.source] for L in cfg.plan]
         embed = hid(t("embed")).to(dtype).contiguous()
         return SitiraxModel(cfg, embed, layers, hvec("final.norm"), dtype)
 

@@ -31,6 +31,9 @@ CONFIGS = {
         layer(parallel(8, 2, 64, 32, 48, 0.2, 2, 32, 64, (0.7, 0.99)), 256), layer(delta(4, 2, 64, 32, 4)),
         layer(delta(2, 2, 32, 128, 3), 128), layer(parallel(8, 2, 64, 32, 48, 0.2, 2, 32, 64, (0.7, 0.99)), 256, of=0),
         layer(delta(4, 2, 64, 32, 4), of=1)]),
+    # weights of a layer further on
+    "ahead": config(64, 80, [layer(delta(2, 1, 32, 32, 3), of=2), layer(parallel(2, 1, 32, 32, 20, 0.3, 2, 16, 32, (0.9, 0.6)), 64),
+                             layer(delta(2, 1, 32, 32, 3)), layer(delta(2, 1, 32, 32, 3), of=2)]),
     # sizes that fit no tile: width, ranks, head widths and counts; one kv head; a window of one page and a bit; decay one
     "odd": config(100, 131, [
         layer(delta(3, 1, 20, 40, 2), 52), layer(parallel(5, 1, 24, 72, 70, 0.31, 3, 40, 20, (0.5, 1.0, 0.9), 1.2, 0.4)),

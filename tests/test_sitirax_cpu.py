@@ -40,7 +40,8 @@ def test_refused_configurations():
     broken(lambda L: L[0]["mixer"]["right"]["decay"].pop())
     broken(lambda L: L[0]["mixer"]["left"].update(kv_heads=3))
     broken(lambda L: L[3]["mixer"].update(left_scale=0.5))          # shares weights but differs from its source
-    broken(lambda L: L[1].update(weights_of=4))
+    broken(lambda L: L[1].update(weights_of=4))                     # 4 takes them from 1
+    broken(lambda L: L[1].update(weights_of=9))
     broken(lambda L: L[1]["mixer"].update(bias=True))
 
 
