@@ -75,6 +75,10 @@ struct GemmParams {
   // this rank's own tiles, and its producer warp waits (bounded) for the owner's flag before the first load.
   int ag;
   CommState comm;
+  // Grouped form (bf16 experts): token tile t multiplies the matrix named by groups[t] out of a stack [experts * N, K]; tiles
+  // with a negative entry do nothing.  group_x: every tile has its own BN activation rows, else all tiles read the rows from 0.
+  const int32_t* groups;
+  int group_x;
 };
 
 template <int BN>
@@ -132,6 +136,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA,   // bf16 weights, or pa
   int my = blockIdx.y;
   if (p.ag) my = (min(p.comm.rank * p.tiles_per_rank, static_cast<int>(gridDim.y)) + static_cast<int>(blockIdx.y)) % static_cast<int>(gridDim.y);
   const int m0 = my * BN;
+  int a_row = n0, b_row = m0;                        // first weight row and first activation row of this CTA
+  if (!kQuant && p.groups != nullptr) {
+    pdl_wait();
+    const int e = p.groups[my];
+    if (e < 0) return;
+    a_row = e * p.N + n0;
+    b_row = p.group_x ? m0 : 0;
+  }
   const int split = blockIdx.z, splits = gridDim.z;
   const int num_kb_total = (p.K + kBK - 1) / kBK;    // bf16 weights: the columns beyond K of the last block read as zero
   const int kb_begin = split * p.kb_per_split;
@@ -202,8 +214,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA,   // bf16 weights, or pa
           ag_waited = true;
         }
         if (p.ag) tma_load_3d(sB + sb * L::kStageB, &tmB, kb * kBK, m0, ag_z, &b_full[sb]);
-        else tma_load_2d(sB + sb * L::kStageB, &tmB, kb * kBK, m0, &b_full[sb]);
-        if (!kQuant) tma_load_2d(sA + sb * L::kStageA, &tmA, kb * kBK, n0, &b_full[sb]);
+        else tma_load_2d(sB + sb * L::kStageB, &tmB, kb * kBK, b_row, &b_full[sb]);
+        if (!kQuant) tma_load_2d(sA + sb * L::kStageA, &tmA, kb * kBK, a_row, &b_full[sb]);
         if (*abort_flag) break;
       }
     }
@@ -564,7 +576,7 @@ using namespace dgpp;
 static int gemm_tc_impl(int wmode, int a_f16, int bn, const void* x, int64_t x_stride, const void* w,
                         const void* w_scale, float alpha, void* out, void* out32, const void* resid, int ldc,
                         int T, int N, int K, int splits, void* ws, void* counters, void* comm_push, cudaStream_t st,
-                        void* comm_ag = nullptr) {
+                        void* comm_ag = nullptr, const int32_t* groups = nullptr, int experts = 1, int x_rows = 0, int group_x = 1) {
   DGPP_REQUIRE(T >= 1 && N >= 1, "gemm_tc: empty problem");
   DGPP_REQUIRE(K % 64 == 0 || (wmode == 0 && K % 8 == 0 && !comm_ag),
                "gemm_tc: K %d must be a multiple of 64 (bf16 weights: of 8)", K);
@@ -578,6 +590,8 @@ static int gemm_tc_impl(int wmode, int a_f16, int bn, const void* x, int64_t x_s
   GemmParams p;
   p.push = 0;
   p.ag = 0;
+  p.groups = groups;
+  p.group_x = group_x;
   p.tiles_per_rank = 1;
   if (comm_ag) {
     const DgppComm* c = static_cast<const DgppComm*>(comm_ag);
@@ -636,10 +650,10 @@ static int gemm_tc_impl(int wmode, int a_f16, int bn, const void* x, int64_t x_s
     if (make_tmap_3d(&tB, c->st.peers[c->st.rank], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, T, 2 * c->st.world,
                      static_cast<uint64_t>(K) * 2, c->st.slot_bytes, 64, bn, CU_TENSOR_MAP_SWIZZLE_128B))
       return -1;
-  } else if (make_tmap_2d(&tB, x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, T, x_stride * 2, 64, bn, CU_TENSOR_MAP_SWIZZLE_128B))
+  } else if (make_tmap_2d(&tB, x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, groups ? x_rows : T, x_stride * 2, 64, bn, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
   if (wmode == 0) {
-    if (make_tmap_2d(&tA, w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, N, static_cast<uint64_t>(K) * 2, 64, kBM,
+    if (make_tmap_2d(&tA, w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, static_cast<uint64_t>(N) * experts, static_cast<uint64_t>(K) * 2, 64, kBM,
                      CU_TENSOR_MAP_SWIZZLE_128B))
       return -1;
   } else if (byte_src) {
@@ -696,4 +710,15 @@ DGPP_API int dgpp_gemm_tc_push(int wmode, int a_f16, int bn, const void* x, int6
                                const void* w_scale, float alpha, int T, int N, int K, void* comm_push, cudaStream_t st) {
   return gemm_tc_impl(wmode, a_f16, bn, x, x_stride, w, w_scale, alpha, nullptr, nullptr, nullptr, N, T, N, K, 1, nullptr,
                       nullptr, comm_push, st);
+}
+
+// Grouped linear over a stack of bf16 matrices w [experts * N, K]: token tile t (rows t * bn .. of `out`) is multiplied by matrix
+// groups[t] (negative: skipped).  group_x = 1: x holds the tiles' own rows [tiles * bn, K]; 0: every tile reads rows 0 .. x_rows - 1
+// of x (x_rows <= bn).
+DGPP_API int dgpp_gemm_tc_grouped(int bn, const void* x, int64_t x_stride, int x_rows, int group_x, const void* w, int experts,
+                                  const void* groups, void* out, int ldc, int tiles, int N, int K, cudaStream_t st) {
+  DGPP_REQUIRE(groups != nullptr && experts >= 1 && tiles >= 1 && tiles <= 65535, "gemm_tc_grouped: %d tiles over %d matrices", tiles, experts);
+  DGPP_REQUIRE(group_x ? x_rows == tiles * bn : (x_rows >= 1 && x_rows <= bn), "gemm_tc_grouped: %d rows in %d tiles of %d", x_rows, tiles, bn);
+  return gemm_tc_impl(0, 0, bn, x, x_stride, w, nullptr, 1.f, out, nullptr, nullptr, ldc, tiles * bn, N, K, 1, nullptr, nullptr, nullptr, st,
+                      nullptr, static_cast<const int32_t*>(groups), experts, x_rows, group_x);
 }

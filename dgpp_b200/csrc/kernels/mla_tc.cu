@@ -13,6 +13,8 @@
 // The tile is single buffered (147 KB at dc + dr = 576): the PV product of tile i must retire before tile i + 1 lands.
 // S^T, P and O^T are double buffered, so the fold of tile i overlaps the load of tile i + 1.
 // Warps: 0 = TMA producer (walks the block table), 1 = MMA issuer / TMEM owner, 2..5 = softmax and accumulation.
+// TERMS = 2 is the form for models whose scores and weights are 32-bit: queries (fp32 here) and probabilities enter the tensor
+// cores as two bf16 terms each (value + residual), side by side in the 32 columns, so a CTA takes 16 heads; outputs are fp32.
 // Every wait is bounded (status code + clean exit).  Split partials use the layout of mla.cu and its combine kernel.
 // (reference counterparts: src/kernels/dsa.cu:2502 attn_flash_kernel, latent decode kernels of the same file.)
 #include <cuda.h>
@@ -21,6 +23,7 @@
 
 #include "common/common.h"
 #include "common/dtypes.cuh"
+#include "common/elem.cuh"
 #include "common/ptx.cuh"
 #include "kernels/gemm_common.cuh"
 
@@ -32,27 +35,29 @@ constexpr int kMtNQ = 32;      // head columns per CTA
 constexpr int kMtBlk = kMtTile * 128;   // 16 KB: one 64-element column block of the latent tile
 
 struct MlaTcParams {
-  const bf16* q;               // [rows, heads, dc + dr] absorbed query, rotary part rotated
+  const void* q;               // [rows, heads, dc + dr] absorbed query, rotary part rotated (bf16; TERMS = 2: fp32)
   const bf16* cache;           // [blocks, page, dc + dr] (the sparse form gathers rows itself)
   const int32_t* sel;          // sparse form: [rows, sel_stride] selected token positions, ascending, -1 padded
   int sel_stride;
   const int32_t* block_table;  // [requests, max_blocks]
-  const int32_t* row_req;      // [rows]
-  const int32_t* positions;    // [rows] position of the row's own token (already in the cache)
+  const int32_t* row_req;      // per row of the pass
+  const int32_t* positions;    // per row of the pass: position of the row's own token (already in the cache)
+  const int32_t* row_list;     // optional: the pass row of every row here (q, partials and outputs are indexed from 0)
   float* part_ml;              // [rows, heads, splits, 2]   (max in natural-log units, sum)
   float* part_acc;             // [rows, heads, splits, dc]
-  bf16* out;                   // [rows, heads, dc]
+  void* out;                   // [rows, heads, dc] (bf16; TERMS = 2: fp32)
   DeviceStatus* status;
-  int rows, heads, page, max_blocks, splits;
+  int rows, heads, page, max_blocks, splits, window;   // window: positions a row sees, its own included (0: all)
   float scale;
 };
 
 // SPARSE: the tokens of a tile come from the row's selection list instead of consecutive positions; the four softmax
 // warps (idle while a tile loads: it is single buffered) gather them, thread = token: 72 16-byte chunks of the token's
 // latent row into the swizzled column blocks, then a proxy fence and one arrival per warp on the tile barrier.
-template <int DC, int DR, bool SPARSE>
+template <int DC, int DR, bool SPARSE, int TERMS = 1>
 __global__ void __launch_bounds__(kMtThreads, 1)
 mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
+  constexpr int NH = kMtNQ / TERMS;      // heads per CTA
   constexpr int D = DC + DR;
   constexpr int KB = D / 64;     // column blocks of the tile and of Q
   constexpr int MB = DC / 128;   // 128-dim output blocks
@@ -79,8 +84,10 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int split = blockIdx.x, row = blockIdx.y, hg = blockIdx.z;
-  const int req = p.row_req[row];
-  int len = p.positions[row] + 1;
+  const int prow = p.row_list != nullptr ? p.row_list[row] : row;
+  const int req = p.row_req[prow];
+  int len = p.positions[prow] + 1;
+  const int first = p.window > 0 ? max(0, len - p.window) : 0;
   const int32_t* sel = nullptr;
   if (SPARSE) {
     // listed tokens at or before the row's own position (lists are ascending, so they form a prefix of the list)
@@ -92,12 +99,12 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
     }
     len = n;
   }
-  const int total_tiles = (len + kMtTile - 1) / kMtTile;
-  const int per = (total_tiles + p.splits - 1) / p.splits;
-  const int tile_begin = split * per;
-  const int ntiles = max(0, min(total_tiles, tile_begin + per) - tile_begin);
+  const int tile0 = first / kMtTile, tile_end = (len + kMtTile - 1) / kMtTile;
+  const int per = (tile_end - tile0 + p.splits - 1) / p.splits;
+  const int tile_begin = tile0 + split * per;
+  const int ntiles = max(0, min(tile_end, tile_begin + per) - tile_begin);
   const int32_t* bt = p.block_table + static_cast<size_t>(req) * p.max_blocks;
-  const int nheads = min(kMtNQ, p.heads - hg * kMtNQ);
+  const int nheads = min(NH, p.heads - hg * NH);
 
   if (threadIdx.x == 0) {
     mbar_init(c_full, SPARSE ? 4 : 1); mbar_init(c_empty, 1);
@@ -115,12 +122,26 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
   if (warp >= 2) {
     const int t = threadIdx.x - 64;
     constexpr int kChunks = D / 8;   // 16-byte chunks per head
-    for (int i = t; i < kMtNQ * kChunks; i += 128) {
+    for (int i = t; i < NH * kChunks; i += 128) {
       const int h = i / kChunks, c = i % kChunks;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (h < nheads)
-        v = *reinterpret_cast<const uint4*>(p.q + (static_cast<size_t>(row) * p.heads + hg * kMtNQ + h) * D + c * 8);
-      *reinterpret_cast<uint4*>(sQ + (c >> 3) * kQBlk + h * 128 + (((c & 7) ^ (h & 7)) << 4)) = v;
+      const size_t at = (static_cast<size_t>(row) * p.heads + hg * NH + h) * D + c * 8;
+      Pack16 v, lo;
+      v.u = lo.u = make_uint4(0u, 0u, 0u, 0u);
+      if (h < nheads) {
+        if constexpr (TERMS == 1) {
+          v.u = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(p.q) + at);
+        } else {
+          const float* f = static_cast<const float*>(p.q) + at;
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            v.h[j] = f32_to_bf16(f[j]);
+            lo.h[j] = f32_to_bf16(f[j] - bf16_to_f32(v.h[j]));
+          }
+        }
+      }
+      unsigned char* dst = sQ + (c >> 3) * kQBlk + h * 128 + (((c & 7) ^ (h & 7)) << 4);
+      *reinterpret_cast<uint4*>(dst) = v.u;
+      if constexpr (TERMS == 2) *reinterpret_cast<uint4*>(dst + NH * 128) = lo.u;      // NH is a multiple of 8: same swizzle
     }
     if (t < kMtNQ) { mrun[kMtNQ + t] = -INFINITY; mrun[t] = -INFINITY; }
     fence_proxy_async_smem();
@@ -194,10 +215,10 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const int wslot = warp - 2;
     const float sm = p.scale * 1.4426950408889634f;  // scores in log2 units
-    float l_thr[kMtNQ];
-    float o_acc[MB][kMtNQ];
+    float l_thr[NH];
+    float o_acc[MB][NH];
 #pragma unroll
-    for (int c = 0; c < kMtNQ; ++c) {
+    for (int c = 0; c < NH; ++c) {
       l_thr[c] = 0.f;
 #pragma unroll
       for (int mb = 0; mb < MB; ++mb) o_acc[mb][c] = 0.f;
@@ -214,7 +235,7 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
           tmem_ld_x16(tmem_o + (bp * MB + mb) * kMtNQ + half * 16 + lane_addr, oc);
           tmem_ld_wait();
 #pragma unroll
-          for (int c = 0; c < 16; ++c) o_acc[mb][half * 16 + c] += __uint_as_float(oc[c]);
+          for (int c = 0; c < 16; ++c) o_acc[mb][TERMS == 2 ? c : half * 16 + c] += __uint_as_float(oc[c]);
         }
       }
       return true;
@@ -223,7 +244,7 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
     for (int i = 0; i < ntiles; ++i) {
       const int b = i & 1;
       const int t = (tile_begin + i) * kMtTile + idx;
-      const bool valid = t < len;
+      const bool valid = t < len && t >= first;
       if (SPARSE) {
         if (wait_bar(c_empty, (i & 1) ^ 1)) {
           // a warp gathers its 32 tokens one after the other: lanes take the 72 chunks of a token's row in turns, so the
@@ -266,18 +287,22 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
       bool okw = ok && wait_bar(&s_full[b], (i >> 1) & 1);
       if (!okw && ok) { report(p.status, kTimeoutAccum, 54); *abort_flag = 1; }
       tc_fence_after();
-      float s[kMtNQ];
+      float s[NH];
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         uint32_t raw[16];
         tmem_ld_x16(tmem_s + b * kMtNQ + half * 16 + lane_addr, raw);
         tmem_ld_wait();
 #pragma unroll
-        for (int c = 0; c < 16; ++c) s[half * 16 + c] = valid ? __uint_as_float(raw[c]) * sm : -INFINITY;
+        for (int c = 0; c < 16; ++c) {
+          const float v = valid ? __uint_as_float(raw[c]) * sm : -INFINITY;
+          if constexpr (TERMS == 2) s[c] = half == 0 || !valid ? v : s[c] + v;
+          else s[half * 16 + c] = v;
+        }
       }
       float* rp = red + (b * 4 + wslot) * kMtNQ;
 #pragma unroll
-      for (int c = 0; c < kMtNQ; ++c) {
+      for (int c = 0; c < NH; ++c) {
         float mx = s[c];
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -292,7 +317,7 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
       unsigned char* pbuf = sP + b * 2 * kQBlk + (idx >> 6) * kQBlk;
       const uint32_t pbyte = (idx & 63) * 2;
 #pragma unroll
-      for (int c = 0; c < kMtNQ; ++c) {
+      for (int c = 0; c < NH; ++c) {
         const float mt = fmaxf(fmaxf(r0[c], r0[kMtNQ + c]), fmaxf(r0[2 * kMtNQ + c], r0[3 * kMtNQ + c]));
         const float mo = m_prev[c];
         const float mn = fmaxf(mo, mt);
@@ -301,7 +326,10 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
         l_thr[c] = l_thr[c] * cr + pv;
         if (idx == c) { mrun[b * kMtNQ + c] = mn; corr[b * kMtNQ + c] = cr; }
         // P[head c][token idx]: row c of the 64-token block, 2 bytes at the token's column (128-byte swizzle)
-        *reinterpret_cast<bf16*>(pbuf + c * 128 + ((((pbyte >> 4) ^ (c & 7)) << 4) | (pbyte & 15))) = f32_to_bf16(pv);
+        const bf16 ph = f32_to_bf16(pv);
+        unsigned char* pd = pbuf + c * 128 + ((((pbyte >> 4) ^ (c & 7)) << 4) | (pbyte & 15));
+        *reinterpret_cast<bf16*>(pd) = ph;
+        if constexpr (TERMS == 2) *reinterpret_cast<bf16*>(pd + NH * 128) = f32_to_bf16(pv - bf16_to_f32(ph));
       }
       fence_proxy_async_smem();
       tc_fence_before();
@@ -315,7 +343,7 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
       }
       const float* cb = corr + b * kMtNQ;
 #pragma unroll
-      for (int c = 0; c < kMtNQ; ++c) {
+      for (int c = 0; c < NH; ++c) {
         const float cr = cb[c];
 #pragma unroll
         for (int mb = 0; mb < MB; ++mb) o_acc[mb][c] *= cr;
@@ -329,7 +357,7 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
     }
     // total probability mass per head: sum the per-thread partials
 #pragma unroll
-    for (int c = 0; c < kMtNQ; ++c) {
+    for (int c = 0; c < NH; ++c) {
       float l = l_thr[c];
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
@@ -339,14 +367,18 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
     if (done) {
       const float* m_fin = mrun + ((ntiles > 0 ? (ntiles - 1) & 1 : 0)) * kMtNQ;
 #pragma unroll
-      for (int c = 0; c < kMtNQ; ++c) {
+      for (int c = 0; c < NH; ++c) {
         if (c < nheads) {
           const float l = lred[c] + lred[kMtNQ + c] + lred[2 * kMtNQ + c] + lred[3 * kMtNQ + c];
-          const size_t rh = static_cast<size_t>(row) * p.heads + hg * kMtNQ + c;
+          const size_t rh = static_cast<size_t>(row) * p.heads + hg * NH + c;
           if (p.splits == 1) {
             const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
-            for (int mb = 0; mb < MB; ++mb) p.out[rh * DC + mb * 128 + idx] = f32_to_bf16(o_acc[mb][c] * inv);
+            for (int mb = 0; mb < MB; ++mb) {
+              const float v = o_acc[mb][c] * inv;
+              if constexpr (TERMS == 2) static_cast<float*>(p.out)[rh * DC + mb * 128 + idx] = v;
+              else static_cast<bf16*>(p.out)[rh * DC + mb * 128 + idx] = f32_to_bf16(v);
+            }
           } else {
             const size_t pi = rh * p.splits + split;
 #pragma unroll
@@ -366,8 +398,9 @@ mla_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, MlaTcParams p) {
   if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
+template <typename T>
 __global__ void mla_tc_combine_kernel(const float* __restrict__ part_ml, const float* __restrict__ part_acc,
-                                      bf16* __restrict__ out, int splits, int dc) {
+                                      T* __restrict__ out, int splits, int dc) {
   pdl_wait();
   const size_t rh = blockIdx.x;
   float mm = -INFINITY;
@@ -380,8 +413,13 @@ __global__ void mla_tc_combine_kernel(const float* __restrict__ part_ml, const f
       ll += part_ml[(rh * splits + s) * 2 + 1] * c;
       acc += part_acc[(rh * splits + s) * dc + d] * c;
     }
-    out[rh * dc + d] = f32_to_bf16(ll > 0.f ? acc / ll : 0.f);
+    st_elem(out + rh * dc + d, ll > 0.f ? acc / ll : 0.f);
   }
+}
+
+template <int KB>
+constexpr size_t mla_tc_smem() {
+  return 1024 + KB * kMtBlk + KB * kMtNQ * 128 + 4 * kMtNQ * 128 + (2 * 4 + 2 + 2 + 4) * kMtNQ * 4 + 2 * 4 * 4 + 8 * 8 + 64;
 }
 
 }  // namespace dgpp
@@ -401,7 +439,9 @@ DGPP_API int dgpp_mla_decode_tc(const void* q, const void* cache, const void* bl
   DGPP_REQUIRE(out != nullptr && heads >= 1, "mla_decode_tc: bad arguments");
   if (rows == 0) return 0;
   MlaTcParams p;
-  p.q = static_cast<const bf16*>(q);
+  p.row_list = nullptr;
+  p.window = 0;
+  p.q = q;
   p.cache = static_cast<const bf16*>(cache);
   p.sel = static_cast<const int32_t*>(sel);
   p.sel_stride = sel_stride;
@@ -410,7 +450,7 @@ DGPP_API int dgpp_mla_decode_tc(const void* q, const void* cache, const void* bl
   p.positions = static_cast<const int32_t*>(positions);
   p.part_ml = static_cast<float*>(part_ml);
   p.part_acc = static_cast<float*>(part_acc);
-  p.out = static_cast<bf16*>(out);
+  p.out = out;
   p.status = device_status_ptr();
   p.rows = rows; p.heads = heads; p.page = page; p.max_blocks = max_blocks; p.splits = splits; p.scale = scale;
   const int D = dc + dr;
@@ -418,9 +458,7 @@ DGPP_API int dgpp_mla_decode_tc(const void* q, const void* cache, const void* bl
   if (make_tmap_2d(&tC, cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, static_cast<uint64_t>(num_blocks) * page,
                    static_cast<uint64_t>(D) * 2, 64, page, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
-  constexpr int KB = 576 / 64;
-  constexpr size_t smem = 1024 + KB * kMtBlk + KB * kMtNQ * 128 + 4 * kMtNQ * 128 + (2 * 4 + 2 + 2 + 4) * kMtNQ * 4 + 2 * 4 * 4 +
-                          8 * 8 + 64;
+  constexpr size_t smem = mla_tc_smem<576 / 64>();
   static_assert(smem <= 227 * 1024, "mla_decode_tc: shared memory over the per-CTA limit");
   static bool attr = false;
   if (!attr) {
@@ -435,8 +473,60 @@ DGPP_API int dgpp_mla_decode_tc(const void* q, const void* cache, const void* bl
   else mla_decode_tc_kernel<512, 64, false><<<grid, kMtThreads, smem, st>>>(tC, p);
   DGPP_CUDA_OK(cudaGetLastError());
   if (splits > 1) {
-    mla_tc_combine_kernel<<<rows * heads, 256, 0, st>>>(p.part_ml, p.part_acc, p.out, splits, dc);
+    mla_tc_combine_kernel<bf16><<<rows * heads, 256, 0, st>>>(p.part_ml, p.part_acc, static_cast<bf16*>(out), splits, dc);
     DGPP_CUDA_OK(cudaGetLastError());
   }
   return 0;
+}
+
+template <int DC>
+static int launch_latent_tc(const MlaTcParams& p, const CUtensorMap& tC, cudaStream_t st) {
+  constexpr size_t smem = mla_tc_smem<(DC + 64) / 64>();
+  static_assert(smem <= 227 * 1024, "latent_decode_tc: shared memory over the per-CTA limit");
+  auto kern = mla_decode_tc_kernel<DC, 64, false, 2>;
+  static bool attr = false;
+  if (!attr) {
+    DGPP_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    attr = true;
+  }
+  kern<<<dim3(p.splits, p.rows, dgpp_ceil_div(p.heads, kMtNQ / 2)), kMtThreads, smem, st>>>(tC, p);
+  DGPP_CUDA_OK(cudaGetLastError());
+  if (p.splits > 1) {
+    mla_tc_combine_kernel<float><<<p.rows * p.heads, 128, 0, st>>>(p.part_ml, p.part_acc, static_cast<float*>(p.out), p.splits, DC);
+    DGPP_CUDA_OK(cudaGetLastError());
+  }
+  return 0;
+}
+
+// Windowed form with 32-bit queries, scores, weights and outputs (two bf16 terms in the tensor cores): every row sees the last
+// `window` positions of its request, its own included (0: all of them).  q [rows, heads, dc + 64] fp32, out [rows, heads, dc] fp32,
+// cache [num_blocks, page, dc + 64] bf16; dc 128, 256, 384 or 512.  row_list: the pass rows that rows 0 .. rows - 1 stand for.
+DGPP_API int dgpp_latent_decode_tc(const void* q, const void* cache, const void* block_table, const void* row_req, const void* positions,
+                                   const void* row_list, void* part_ml, void* part_acc, void* out, int rows, int heads, int dc, int page,
+                                   int max_blocks, int num_blocks, int splits, int window, float scale, cudaStream_t st) {
+  DGPP_REQUIRE(page == 16 || page == 32 || page == 64 || page == 128, "latent_decode_tc: page %d unsupported", page);
+  DGPP_REQUIRE(splits >= 1 && (splits == 1 || (part_ml && part_acc)), "latent_decode_tc: scratch required for splits");
+  DGPP_REQUIRE(out != nullptr && heads >= 1 && window >= 0 && rows >= 0 && rows <= 65535, "latent_decode_tc: bad arguments");
+  if (rows == 0) return 0;
+  MlaTcParams p;
+  p.q = q; p.cache = static_cast<const bf16*>(cache); p.sel = nullptr; p.sel_stride = 0;
+  p.block_table = static_cast<const int32_t*>(block_table);
+  p.row_req = static_cast<const int32_t*>(row_req);
+  p.positions = static_cast<const int32_t*>(positions);
+  p.row_list = static_cast<const int32_t*>(row_list);
+  p.part_ml = static_cast<float*>(part_ml); p.part_acc = static_cast<float*>(part_acc);
+  p.out = out;
+  p.status = device_status_ptr();
+  p.rows = rows; p.heads = heads; p.page = page; p.max_blocks = max_blocks; p.splits = splits; p.window = window; p.scale = scale;
+  const int D = dc + 64;
+  CUtensorMap tC;
+  if (make_tmap_2d(&tC, cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, static_cast<uint64_t>(num_blocks) * page,
+                   static_cast<uint64_t>(D) * 2, 64, page, CU_TENSOR_MAP_SWIZZLE_128B))
+    return -1;
+  if (dc == 128) return launch_latent_tc<128>(p, tC, st);
+  if (dc == 256) return launch_latent_tc<256>(p, tC, st);
+  if (dc == 384) return launch_latent_tc<384>(p, tC, st);
+  if (dc == 512) return launch_latent_tc<512>(p, tC, st);
+  dgpp_set_error("latent_decode_tc: latent width %d (128, 256, 384 or 512)", dc);
+  return -1;
 }

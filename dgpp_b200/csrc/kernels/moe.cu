@@ -32,7 +32,8 @@ struct RouterArgs {
   const float* bias;     // [E] selection correction, may be null
   int32_t* ids;          // [T, k] ascending
   float* weights;        // [T, k]
-  float* logits_out;     // [T, E] optional (tests, auditing)
+  float* logits_out;     // [T, logits_stride]
+  int64_t logits_stride;
   int T, H, E, k, n_group, topk_group;
   int softmax, norm_topk;
   float scaling;
@@ -77,7 +78,7 @@ __global__ void __launch_bounds__(kRouterThreads) moe_router_logits_kernel(Route
     float v = acc[r];
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    if (lane == 0 && r < nt) a.logits_out[static_cast<size_t>(t0 + r) * a.E + e] = v;
+    if (lane == 0 && r < nt) a.logits_out[(t0 + r) * a.logits_stride + e] = v;
   }
 }
 
@@ -90,7 +91,7 @@ __global__ void __launch_bounds__(kRouterThreads) moe_router_select_kernel(Route
   __shared__ int pick_id[kMoeMaxTopK];
   pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
-  for (int e = tid; e < a.E; e += kRouterThreads) score[e] = a.logits_out[static_cast<size_t>(t) * a.E + e];
+  for (int e = tid; e < a.E; e += kRouterThreads) score[e] = a.logits_out[t * a.logits_stride + e];
   __syncthreads();
   if (a.softmax) {
     // softmax over all experts: max, then the sum of exp, each by a fixed tree (thread-strided partials, xor-shuffle
@@ -333,12 +334,30 @@ DGPP_API int dgpp_moe_route(const void* x, int64_t x_stride, const void* gate, c
   a.ids = static_cast<int32_t*>(ids);
   a.weights = static_cast<float*>(weights);
   a.logits_out = static_cast<float*>(logits_out);
+  a.logits_stride = E;
   a.T = T; a.H = H; a.E = E; a.k = k; a.n_group = n_group; a.topk_group = topk_group;
   a.softmax = softmax; a.norm_topk = norm_topk; a.scaling = scaling;
   DGPP_REQUIRE(logits_out != nullptr, "moe_route: a [T, E] fp32 logits buffer is required");
   dim3 grid(dgpp_ceil_div(E, kRouterThreads / 32), dgpp_ceil_div(T, kRouterRowsPerCta));
   moe_router_logits_kernel<<<grid, kRouterThreads, 0, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
+  moe_router_select_kernel<<<T, kRouterThreads, 0, st>>>(a);
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// Selection alone, over logits [T, E] (row stride logits_stride) that another kernel made; no correction, no groups.
+DGPP_API int dgpp_moe_select(const void* logits, int64_t logits_stride, void* ids, void* weights, int T, int E, int k, int softmax, int norm_topk,
+                             float scaling, cudaStream_t st) {
+  DGPP_REQUIRE(E >= 1 && E <= kMoeMaxExperts && k >= 1 && k <= kMoeMaxTopK && k <= E, "moe_select: E %d / k %d unsupported", E, k);
+  if (T == 0) return 0;
+  RouterArgs a = {};
+  a.ids = static_cast<int32_t*>(ids);
+  a.weights = static_cast<float*>(weights);
+  a.logits_out = static_cast<float*>(const_cast<void*>(logits));
+  a.logits_stride = logits_stride;
+  a.T = T; a.E = E; a.k = k; a.n_group = 1; a.topk_group = 1;
+  a.softmax = softmax; a.norm_topk = norm_topk; a.scaling = scaling;
   moe_router_select_kernel<<<T, kRouterThreads, 0, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;

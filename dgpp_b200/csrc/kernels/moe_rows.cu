@@ -1,0 +1,152 @@
+// Mixture of experts over plain 16-bit or 32-bit rows (expert matrices without block scales): the launches between the router
+// logits and the grouped linears.
+//
+//   moe_route_small    up to 16 tokens, one CTA: picks every token's experts from its logits (sigmoid or softmax scores, ties to
+//                      the lower id), lists the experts in use as tiles of 16 rows over the SAME activation rows, and writes the
+//                      row of every (token, choice) pair and every tile row's weight (0: the token did not choose the expert)
+//   moe_scatter_rows   any number of tokens, after the counting sort of moe_prefill.cu: copies a pair's activation row to its place
+//                      in the sorted tiles and writes the row's weight there
+// The weights ride along per tile row, so the activation kernel can scale what an expert sees.
+#include <math.h>
+
+#include "common/common.h"
+#include "common/dtypes.cuh"
+#include "common/elem.cuh"
+#include "common/ptx.cuh"
+
+namespace dgpp {
+
+constexpr int kSmallTokens = 16, kSmallExperts = 512, kSmallTop = 16, kSmallThreads = kSmallTokens * 32;
+
+struct RouteSmall {
+  const float* logits;     // [T, stride]
+  int64_t stride;
+  int32_t* pair_row;       // [T * top]
+  int32_t* tiles;          // [max_tiles]
+  float* row_w;            // [max_tiles * 16]
+  int T, E, top, max_tiles, softmax;
+};
+
+__global__ void __launch_bounds__(kSmallThreads) moe_route_small_kernel(RouteSmall a) {
+  __shared__ int slot[kSmallExperts];
+  __shared__ int ids[kSmallTokens][kSmallTop];
+  __shared__ float wts[kSmallTokens][kSmallTop];
+  __shared__ int warp_cnt[kSmallTokens];
+  pdl_wait();
+  const int tid = threadIdx.x, t = tid >> 5, lane = tid & 31;
+  for (int e = tid; e < kSmallExperts; e += kSmallThreads) slot[e] = 0;
+  for (int i = tid; i < a.max_tiles * kSmallTokens; i += kSmallThreads) a.row_w[i] = 0.f;
+  __syncthreads();
+  if (t < a.T) {
+    float z[kSmallExperts / 32];
+    float mx = -INFINITY;
+#pragma unroll
+    for (int i = 0; i < kSmallExperts / 32; ++i) {
+      const int e = lane + 32 * i;
+      z[i] = e < a.E ? a.logits[t * a.stride + e] : -INFINITY;
+      mx = fmaxf(mx, z[i]);
+    }
+    float norm = 1.f;
+    if (a.softmax) {
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < kSmallExperts / 32; ++i) sum += expf(z[i] - mx);
+      norm = warp_sum_f32(sum);
+    }
+    // both scores grow with the logit; equal scores of different logits go to the larger logit
+    for (int r = 0; r < a.top; ++r) {
+      float bv = -INFINITY;
+      int be = 0x7fffffff;
+#pragma unroll
+      for (int i = 0; i < kSmallExperts / 32; ++i) {
+        const int e = lane + 32 * i;
+        if (e < a.E && (z[i] > bv || (z[i] == bv && e < be))) { bv = z[i]; be = e; }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+        const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+        if (ov > bv || (ov == bv && oe < be)) { bv = ov; be = oe; }
+      }
+      if (be >= a.E) be = 0;                           // only with logits that are not numbers
+#pragma unroll
+      for (int i = 0; i < kSmallExperts / 32; ++i)
+        if (lane + 32 * i == be) z[i] = -INFINITY;
+      if (lane == 0) {
+        int j = r;                                     // ascending ids: the order of the sum
+        while (j > 0 && ids[t][j - 1] > be) { ids[t][j] = ids[t][j - 1]; wts[t][j] = wts[t][j - 1]; --j; }
+        ids[t][j] = be;
+        wts[t][j] = a.softmax ? expf(bv - mx) / norm : sigmoid_f32(bv);
+        slot[be] = 1;
+      }
+    }
+  }
+  __syncthreads();
+  // experts in use, ascending (one thread per expert)
+  const bool on = slot[tid] != 0;
+  const unsigned bal = __ballot_sync(0xffffffffu, on);
+  if (lane == 0) warp_cnt[t] = __popc(bal);
+  __syncthreads();
+  int at = __popc(bal & ((1u << lane) - 1u)), total = 0;
+  for (int w = 0; w < kSmallTokens; ++w) {
+    if (w < t) at += warp_cnt[w];
+    total += warp_cnt[w];
+  }
+  slot[tid] = at;
+  if (on && at < a.max_tiles) a.tiles[at] = tid;
+  for (int i = total + tid; i < a.max_tiles; i += kSmallThreads) a.tiles[i] = -1;
+  __syncthreads();
+  if (t < a.T && lane < a.top) {
+    const int row = min(slot[ids[t][lane]], a.max_tiles - 1) * kSmallTokens + t;
+    a.pair_row[t * a.top + lane] = row;
+    a.row_w[row] = wts[t][lane];
+  }
+}
+
+// grid (T * top), 128 threads
+template <typename T>
+__global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const T* __restrict__ x, const int32_t* __restrict__ pair_row,
+                                                               const float* __restrict__ weights, T* __restrict__ xs, float* __restrict__ row_w,
+                                                               int cols, int top) {
+  pdl_wait();
+  const size_t p = blockIdx.x;
+  const int row = pair_row[p];
+  if (row < 0) return;
+  const uint4* src = reinterpret_cast<const uint4*>(x + (p / top) * cols);
+  uint4* dst = reinterpret_cast<uint4*>(xs + static_cast<size_t>(row) * cols);
+  const int n = cols * static_cast<int>(sizeof(T)) / 16;
+  for (int i = threadIdx.x; i < n; i += 128) dst[i] = src[i];
+  if (threadIdx.x == 0) row_w[row] = weights[p];
+}
+
+}  // namespace dgpp
+
+using namespace dgpp;
+
+// logits [T, E] fp32 with row stride `stride`, T <= 16.  max_tiles >= min(E, T * top).
+DGPP_API int dgpp_moe_route_small(const void* logits, int64_t stride, void* pair_row, void* tiles, void* row_w, int T, int E, int top, int max_tiles,
+                                  int softmax, cudaStream_t st) {
+  DGPP_REQUIRE(E >= 1 && E <= kSmallExperts && top >= 1 && top <= kSmallTop && top <= E, "moe_route_small: %d of %d experts", top, E);
+  DGPP_REQUIRE(T <= kSmallTokens && max_tiles >= (E < T * top ? E : T * top), "moe_route_small: %d tokens in %d tiles", T, max_tiles);
+  if (T == 0) return 0;
+  const RouteSmall a = {static_cast<const float*>(logits), stride, static_cast<int32_t*>(pair_row), static_cast<int32_t*>(tiles),
+                        static_cast<float*>(row_w), T, E, top, max_tiles, softmax};
+  moe_route_small_kernel<<<1, kSmallThreads, 0, st>>>(a);
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// x [T, cols] -> xs [tiles * bn, cols], row_w [tiles * bn]: pair (t, j) goes to row pair_row[t * top + j] (negative: nowhere).
+DGPP_API int dgpp_moe_scatter_rows(const void* x, const void* pair_row, const void* weights, void* xs, void* row_w, int T, int cols, int top,
+                                   int f32, cudaStream_t st) {
+  DGPP_REQUIRE(cols % 8 == 0, "moe_scatter_rows: %d columns (a multiple of 8)", cols);
+  if (T == 0) return 0;
+  const int32_t* pr = static_cast<const int32_t*>(pair_row);
+  const float* w = static_cast<const float*>(weights);
+  if (f32) moe_scatter_rows_kernel<float><<<T * top, 128, 0, st>>>(static_cast<const float*>(x), pr, w, static_cast<float*>(xs), static_cast<float*>(row_w), cols, top);
+  else moe_scatter_rows_kernel<bf16><<<T * top, 128, 0, st>>>(static_cast<const bf16*>(x), pr, w, static_cast<bf16*>(xs), static_cast<float*>(row_w), cols, top);
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}

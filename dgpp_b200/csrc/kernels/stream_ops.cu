@@ -3,6 +3,13 @@
 //   resid_norm        x += delta (fp32, optional); out = x / sqrt(mean(x^2) + eps) * w           (out in T)
 //   gated_group_norm  per group of columns: out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) * scale
 //   geglu             out = gelu_tanh(gate) * up
+//   stream_norm       x += post(delta); out = pre(x); post and pre each nothing, an RMS norm or a layer norm (weight, no bias);
+//                     delta is a row of fp32 or the weighed rows of a mixture of experts plus its gated shared expert
+//   gated_part_norm   a = y * silu(z); every one of `parts` runs of columns by its own root mean square, times w
+//   clamped_glu       g = min(s gate, limit), u = clamp(s up, -limit, limit); out = g * sigmoid(alpha g) * (u + 1); s: a factor per
+//                     row (the input weight of a routed expert; the product with the weights is linear) or one
+//   token_gate        out = gelu_tanh(gate) * table[ids[r]][columns of one layer]
+//   softcap           x = cap * tanh(x / cap)
 // Rows may carry zero columns behind their `n` true ones (the padding of the tensor-core GEMM): means divide by the true
 // count and the padded columns stay zero.  Norms, gates and the sum are fp32; one rounding to T at the end.
 #include <math.h>
@@ -101,6 +108,197 @@ geglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter) {
                                               gelu_tanh_f32(g.z) * u.z, gelu_tanh_f32(g.w) * u.w));
 }
 
+enum NormKind { kNormNone = 0, kNormRms = 1, kNormLayer = 2 };
+
+// The rows of a mixture of experts that make up a delta: sum over j of y[pair_row[r * top + j]] (fp32, ascending j) and, with a
+// shared expert, sigmoid(gate[r]) * shared[r].
+template <typename T>
+struct MoeRows {
+  const T* y;
+  const int32_t* pair_row;
+  const T* shared;
+  const float* gate;
+  int64_t gate_stride;
+  int top;
+};
+
+// Norm of a row held in registers; columns at or beyond n are zero and stay zero (their weights are zero).
+template <int NT, int NV>
+__device__ __forceinline__ void norm_row(float4 (&v)[NV], int kind, const float* __restrict__ w, int cols, int n, float eps, float* scratch) {
+  if (kind == kNormNone) return;
+  float mean = 0.f;
+  if (kind == kNormLayer) {
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) sum += (v[j].x + v[j].y) + (v[j].z + v[j].w);
+    mean = block_sum_f32(sum, scratch) / static_cast<float>(n);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    float* f = reinterpret_cast<float*>(&v[j]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (kind == kNormLayer) f[e] = (threadIdx.x + NT * j) * 4 + e < n ? f[e] - mean : 0.f;
+      ss = fmaf(f[e], f[e], ss);
+    }
+  }
+  const float r = 1.f / sqrtf(block_sum_f32(ss, scratch) / static_cast<float>(n) + eps);
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + NT * j) * 4;
+    if (i < cols) {
+      const float4 g = ld_elem4(w + i);
+      v[j].x *= r * g.x; v[j].y *= r * g.y; v[j].z *= r * g.z; v[j].w *= r * g.w;
+    }
+  }
+}
+
+template <typename T, int NT, int NV>
+__global__ void __launch_bounds__(NT)
+stream_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, MoeRows<T> moe, int post, const float* __restrict__ wp, int pre,
+                   const float* __restrict__ wn, T* __restrict__ out, int cols, int n, float eps) {
+  __shared__ float scratch[NT / 32];
+  pdl_wait();
+  const size_t row = blockIdx.x, base = row * cols;
+  float4 v[NV];
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  const bool add = delta != nullptr || moe.y != nullptr;
+  const float sg = moe.shared != nullptr ? sigmoid_f32(moe.gate[row * moe.gate_stride]) : 0.f;
+  if (add) {
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int i = (threadIdx.x + NT * j) * 4;
+      v[j] = zero;
+      if (i >= cols) continue;
+      if (delta != nullptr) { v[j] = ld_elem4(delta + base + i); continue; }
+      for (int k = 0; k < moe.top; ++k) {
+        const float4 a = ld_elem4(moe.y + static_cast<size_t>(moe.pair_row[row * moe.top + k]) * cols + i);
+        v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
+      }
+      if (moe.shared != nullptr) {
+        const float4 a = ld_elem4(moe.shared + base + i);
+        v[j].x = fmaf(sg, a.x, v[j].x); v[j].y = fmaf(sg, a.y, v[j].y); v[j].z = fmaf(sg, a.z, v[j].z); v[j].w = fmaf(sg, a.w, v[j].w);
+      }
+    }
+    norm_row<NT, NV>(v, post, wp, cols, n, eps, scratch);
+  }
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + NT * j) * 4;
+    const float4 a = i < cols ? ld_elem4(x + base + i) : zero;
+    if (!add) { v[j] = a; continue; }
+    v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
+    if (i < cols) st_elem4(x + base + i, v[j]);
+  }
+  norm_row<NT, NV>(v, pre, wn, cols, n, eps, scratch);
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + NT * j) * 4;
+    if (i < cols) st_elem4(out + base + i, v[j]);
+  }
+}
+
+template <typename T>
+static int launch_stream_norm(float* x, const float* delta, const MoeRows<T>& moe, int post, const float* wp, int pre, const float* wn,
+                              T* out, int rows, int cols, int n, float eps, cudaStream_t st) {
+#define DGPP_SN(NT, NV) stream_norm_kernel<T, NT, NV><<<rows, NT, 0, st>>>(x, delta, moe, post, wp, pre, wn, out, cols, n, eps)
+  if (cols <= 1024) DGPP_SN(256, 1);
+  else if (cols <= 2048) DGPP_SN(256, 2);
+  else if (cols <= 4096) DGPP_SN(256, 4);
+  else if (cols <= 8192) DGPP_SN(512, 4);
+  else DGPP_SN(1024, 4);
+#undef DGPP_SN
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// grid (parts, rows); y [rows, parts * gp] fp32.  The last part's CTA also clears the columns up to `pad`.
+template <typename T, int V>
+__global__ void __launch_bounds__(kStreamThreads)
+gated_part_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, int64_t z_stride, const float* __restrict__ w,
+                       T* __restrict__ out, int64_t out_stride, int gp, int pad, float eps) {
+  extern __shared__ __align__(16) float pn_smem[];         // [gp]
+  __shared__ float scratch[kStreamThreads / 32];
+  pdl_wait();
+  const int part = blockIdx.x, n = static_cast<int>(gridDim.x) * gp;
+  const size_t row = blockIdx.y;
+  const float* yp = y + row * n + static_cast<size_t>(part) * gp;
+  const T* zp = z + row * z_stride + static_cast<size_t>(part) * gp;
+  T* dst = out + row * out_stride + static_cast<size_t>(part) * gp;
+  const float* wp = w + static_cast<size_t>(part) * gp;
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < gp; i += kStreamThreads * V) {
+    float a[V];
+    if (V == 4) {
+      const float4 u = ld_elem4(yp + i), g = ld_elem4(zp + i);
+      a[0] = u.x * silu_f32(g.x); a[1 % V] = u.y * silu_f32(g.y); a[2 % V] = u.z * silu_f32(g.z); a[3 % V] = u.w * silu_f32(g.w);
+    } else {
+      a[0] = yp[i] * silu_f32(ld_elem(zp + i));
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      ss = fmaf(a[e], a[e], ss);
+      pn_smem[i + e] = a[e];
+    }
+  }
+  const float r = 1.f / sqrtf(block_sum_f32(ss, scratch) / static_cast<float>(gp) + eps);
+  for (int i = threadIdx.x * V; i < gp; i += kStreamThreads * V) {      // a thread reads back what it wrote
+    if (V == 4) {
+      const float4 a = *reinterpret_cast<const float4*>(pn_smem + i), g = ld_elem4(wp + i);
+      st_elem4(dst + i, make_float4(a.x * r * g.x, a.y * r * g.y, a.z * r * g.z, a.w * r * g.w));
+    } else {
+      st_elem(dst + i, pn_smem[i] * r * wp[i]);
+    }
+  }
+  if (part == static_cast<int>(gridDim.x) - 1)
+    for (int i = n + threadIdx.x; i < pad; i += kStreamThreads) st_elem(out + row * out_stride + i, 0.f);
+}
+
+// gate_up [rows, stride] (TI): gate columns, then up columns, `inter` each.  tiles: rows come in tiles of `bn`, and those whose
+// entry is negative are skipped.
+template <typename TI, typename T>
+__global__ void __launch_bounds__(kStreamThreads)
+clamped_glu_kernel(const TI* __restrict__ gate_up, int64_t stride, const float* __restrict__ row_w, const int32_t* __restrict__ tiles, int bn,
+                   T* __restrict__ out, int inter, float limit, float alpha) {
+  pdl_wait();
+  const size_t row = blockIdx.y;
+  if (tiles != nullptr && tiles[row / bn] < 0) return;
+  const int i = (blockIdx.x * kStreamThreads + threadIdx.x) * 4;
+  if (i >= inter) return;
+  const float s = row_w != nullptr ? row_w[row] : 1.f;
+  const float4 g4 = ld_elem4(gate_up + row * stride + i), u4 = ld_elem4(gate_up + row * stride + inter + i);
+  const float gi[4] = {g4.x, g4.y, g4.z, g4.w}, ui[4] = {u4.x, u4.y, u4.z, u4.w};
+  float o[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float g = fminf(gi[e] * s, limit), u = fminf(fmaxf(ui[e] * s, -limit), limit);
+    o[e] = g * sigmoid_f32(alpha * g) * (u + 1.f);
+  }
+  st_elem4(out + row * inter + i, make_float4(o[0], o[1], o[2], o[3]));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kStreamThreads)
+token_gate_kernel(const float* __restrict__ gate, const int32_t* __restrict__ ids, const T* __restrict__ table, int64_t table_stride, int col,
+                  T* __restrict__ out, int dim, int vocab) {
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  int id = ids[row];
+  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  const T* e = table + static_cast<size_t>(id) * table_stride + col;
+  for (int i = threadIdx.x * 4; i < dim; i += kStreamThreads * 4) {
+    const float4 g = ld_elem4(gate + row * dim + i), t = ld_elem4(e + i);
+    st_elem4(out + row * dim + i, make_float4(gelu_tanh_f32(g.x) * t.x, gelu_tanh_f32(g.y) * t.y, gelu_tanh_f32(g.z) * t.z, gelu_tanh_f32(g.w) * t.w));
+  }
+}
+
+__global__ void __launch_bounds__(kStreamThreads) softcap_kernel(float* __restrict__ x, int64_t n, float cap) {
+  pdl_wait();
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * kStreamThreads + threadIdx.x; i < n; i += static_cast<int64_t>(gridDim.x) * kStreamThreads)
+    x[i] = cap * tanhf(x[i] / cap);
+}
+
 }  // namespace dgpp
 
 using namespace dgpp;
@@ -151,6 +349,91 @@ DGPP_API int dgpp_geglu(const void* gate_up, void* out, int rows, int inter, int
   const dim3 grid(dgpp_ceil_div(inter / 4, kStreamThreads), rows);
   if (f32) geglu_kernel<float><<<grid, kStreamThreads, 0, st>>>(static_cast<const float*>(gate_up), static_cast<float*>(out), inter);
   else geglu_kernel<bf16><<<grid, kStreamThreads, 0, st>>>(static_cast<const bf16*>(gate_up), static_cast<bf16*>(out), inter);
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// post / pre: 0 nothing, 1 RMS norm, 2 layer norm, each with its weights.  The delta is `delta` (fp32 [rows, cols]), or the
+// expert rows y[pair_row[r * top + j]] plus sigmoid(gate) * shared (y, shared: activations), or absent.
+DGPP_API int dgpp_stream_norm(void* x, const void* delta, const void* y, const void* pair_row, int top, const void* shared, const void* gate,
+                              int64_t gate_stride, int post, const void* post_w, int pre, const void* pre_w, void* out, int rows, int cols,
+                              int n, float eps, int f32, cudaStream_t st) {
+  DGPP_REQUIRE(cols % 8 == 0 && cols <= 16384 && n >= 1 && n <= cols, "stream_norm: %d of %d columns (at most 16384)", n, cols);
+  DGPP_REQUIRE(post >= 0 && post <= 2 && pre >= 0 && pre <= 2 && (!post || post_w) && (!pre || pre_w), "stream_norm: norms %d / %d", post, pre);
+  DGPP_REQUIRE(!(delta && y) && (!y || (pair_row && top >= 1)) && (!shared || (y && gate)), "stream_norm: one delta only");
+  if (rows == 0) return 0;
+  float* xp = static_cast<float*>(x);
+  const float *dp = static_cast<const float*>(delta), *wp = static_cast<const float*>(post_w), *wn = static_cast<const float*>(pre_w);
+  const int32_t* pr = static_cast<const int32_t*>(pair_row);
+  const float* gp = static_cast<const float*>(gate);
+  if (f32) {
+    const MoeRows<float> m = {static_cast<const float*>(y), pr, static_cast<const float*>(shared), gp, gate_stride, top};
+    return launch_stream_norm<float>(xp, dp, m, post, wp, pre, wn, static_cast<float*>(out), rows, cols, n, eps, st);
+  }
+  const MoeRows<bf16> m = {static_cast<const bf16*>(y), pr, static_cast<const bf16*>(shared), gp, gate_stride, top};
+  return launch_stream_norm<bf16>(xp, dp, m, post, wp, pre, wn, static_cast<bf16*>(out), rows, cols, n, eps, st);
+}
+
+DGPP_API int dgpp_gated_part_norm(const void* y, const void* z, int64_t z_stride, const void* w, void* out, int64_t out_stride, int rows,
+                                  int parts, int gp, int pad, float eps, int f32, cudaStream_t st) {
+  DGPP_REQUIRE(parts >= 1 && gp >= 1 && parts <= 65535 && rows <= 65535, "gated_part_norm: %d parts of %d columns", parts, gp);
+  const size_t smem = static_cast<size_t>(gp) * sizeof(float);
+  DGPP_REQUIRE(smem <= 200 * 1024, "gated_part_norm: parts of %d columns (at most 51200)", gp);
+  if (rows == 0) return 0;
+  static bool attr = false;
+  if (!attr) {
+    DGPP_CUDA_OK(cudaFuncSetAttribute(gated_part_norm_kernel<bf16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(gated_part_norm_kernel<bf16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(gated_part_norm_kernel<float, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(gated_part_norm_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    attr = true;
+  }
+  const bool wide = gp % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0;
+  const float *yp = static_cast<const float*>(y), *wp = static_cast<const float*>(w);
+#define DGPP_GPN(TT, V) gated_part_norm_kernel<TT, V><<<dim3(parts, rows), kStreamThreads, smem, st>>>( \
+      yp, static_cast<const TT*>(z), z_stride, wp, static_cast<TT*>(out), out_stride, gp, pad, eps)
+  if (f32) { if (wide) DGPP_GPN(float, 4); else DGPP_GPN(float, 1); }
+  else { if (wide) DGPP_GPN(bf16, 4); else DGPP_GPN(bf16, 1); }
+#undef DGPP_GPN
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// in_f32: gate_up is fp32 although the output is bf16.
+DGPP_API int dgpp_clamped_glu(const void* gate_up, int64_t stride, const void* row_w, const void* tiles, int bn, void* out, int rows, int inter,
+                              float limit, float alpha, int f32, int in_f32, cudaStream_t st) {
+  DGPP_REQUIRE(inter % 8 == 0 && stride % 4 == 0 && bn >= 1, "clamped_glu: width %d (a multiple of 8)", inter);
+  if (rows == 0) return 0;
+  DGPP_REQUIRE(rows <= 65535, "clamped_glu: %d rows", rows);
+  const dim3 grid(dgpp_ceil_div(inter / 4, kStreamThreads), rows);
+  const float* rw = static_cast<const float*>(row_w);
+  const int32_t* tl = static_cast<const int32_t*>(tiles);
+#define DGPP_CG(TI, TT) clamped_glu_kernel<TI, TT><<<grid, kStreamThreads, 0, st>>>(static_cast<const TI*>(gate_up), stride, rw, tl, bn, \
+                                                                                   static_cast<TT*>(out), inter, limit, alpha)
+  if (f32) DGPP_CG(float, float);
+  else if (in_f32) DGPP_CG(float, bf16);
+  else DGPP_CG(bf16, bf16);
+#undef DGPP_CG
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// gate [rows, dim] fp32; table [vocab, table_stride] in the activations' type, `col`: the layer's first column.
+DGPP_API int dgpp_token_gate(const void* gate, const void* ids, const void* table, int64_t table_stride, int col, void* out, int rows, int dim,
+                             int vocab, int f32, cudaStream_t st) {
+  DGPP_REQUIRE(dim % 8 == 0 && table_stride % 8 == 0 && col % 8 == 0, "token_gate: %d columns from %d", dim, col);
+  if (rows == 0) return 0;
+  if (f32) token_gate_kernel<float><<<rows, kStreamThreads, 0, st>>>(static_cast<const float*>(gate), static_cast<const int32_t*>(ids), static_cast<const float*>(table), table_stride, col, static_cast<float*>(out), dim, vocab);
+  else token_gate_kernel<bf16><<<rows, kStreamThreads, 0, st>>>(static_cast<const float*>(gate), static_cast<const int32_t*>(ids), static_cast<const bf16*>(table), table_stride, col, static_cast<bf16*>(out), dim, vocab);
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+DGPP_API int dgpp_softcap(void* x, int64_t n, float cap, cudaStream_t st) {
+  DGPP_REQUIRE(cap > 0.f, "softcap: %f", static_cast<double>(cap));
+  if (n == 0) return 0;
+  const int64_t blocks = dgpp_ceil_div64(n, kStreamThreads);
+  softcap_kernel<<<static_cast<unsigned>(blocks > 1184 ? 1184 : blocks), kStreamThreads, 0, st>>>(static_cast<float*>(x), n, cap);
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;
 }

@@ -13,6 +13,11 @@
 // then the exponents are taken against the older maximum, for the weights and for their sum alike, so the quotient is the
 // softmax either way.
 // Warps: 0 = TMA producer (one page of keys and values per stage), 1 = MMA issuer / TMEM owner, 2..5 = softmax.
+//
+// FLAT is the form for latent attention, whose keys and values are expanded from the cached latents before the launch: every head
+// is its own kv head; key columns 0 .. DN - 1 and the values come from the expanded rows [flat rows, hq * DN + hq * DV], the other
+// key columns (the rotated part that all heads share) from the gathered cache rows.  A run's page g starts at flat row
+// flat_base[run] + 64 g.  An output gate per (row, head) may multiply the result.
 // Every wait is bounded; on expiry the kernel records a status code and unwinds.
 #include <cuda.h>
 #include <math.h>
@@ -20,6 +25,7 @@
 
 #include "common/common.h"
 #include "common/dtypes.cuh"
+#include "common/elem.cuh"
 #include "common/ptx.cuh"
 #include "kernels/gemm_common.cuh"
 
@@ -34,11 +40,15 @@ struct WindowTcParams {
   const int32_t* block_table;
   const int32_t* row_req;
   const int32_t* positions;
-  const int32_t* run_start; // [runs + 1]
+  const int32_t* run_start; // [runs + 1], or [runs] with run_len
+  const int32_t* run_len;   // optional [runs]: the runs are not back to back
+  const int32_t* flat_base; // [runs] (FLAT)
+  const bf16* gate;         // optional [rows, stride]: sigmoid(gate[row, head]) multiplies the output
   bf16* out;
   int64_t out_stride;
   DeviceStatus* status;
   int runs, hq, hkv, D, DV, max_blocks, window, stages;
+  int DN, rot_col;          // FLAT: key columns from the expanded rows; first rotated column of a gathered cache row
   float scale, out_scale;
 };
 
@@ -91,6 +101,7 @@ __device__ __forceinline__ float wt_probs(uint32_t taddr, unsigned char* sP, int
 }
 
 // grid (tiles of all runs, hkv)
+template <bool FLAT>
 __global__ void __launch_bounds__(kWtThreads, 1)
 window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, WindowTcParams p) {
   extern __shared__ __align__(1024) unsigned char smem_dyn[];
@@ -129,10 +140,15 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   }
   pdl_wait();
   // the run this tile lies in (tiles are dealt run by run)
-  int tile = blockIdx.x, row0 = 0, ntok = 0;
+  int tile = blockIdx.x, row0 = 0, ntok = 0, flat0 = 0;
   for (int r = 0; r < p.runs; ++r) {
-    const int a = p.run_start[r], n = p.run_start[r + 1] - a, t = (n + per - 1) / per;
-    if (tile < t) { row0 = a + tile * per; ntok = min(per, n - tile * per); break; }
+    const int a = p.run_start[r], n = p.run_len != nullptr ? p.run_len[r] : p.run_start[r + 1] - a, t = (n + per - 1) / per;
+    if (tile < t) {
+      row0 = a + tile * per;
+      ntok = min(per, n - tile * per);
+      if (FLAT) flat0 = p.flat_base[r];
+      break;
+    }
     tile -= t;
   }
   const int first_pos = p.positions[row0], last_pos = first_pos + ntok - 1;
@@ -164,9 +180,16 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         const int s = i % p.stages;
         if (!wait_bar(&kv_empty[s], ((i / p.stages) & 1) ^ 1)) { report(p.status, kTimeoutStageEmpty, 71); *abort_flag = 1; break; }
         mbar_expect_tx(&kv_full[s], (natom + vatom) * kblk);
-        const int y = (bt[page0 + i] * p.hkv + kvh) * kWtKeys;
-        for (int a = 0; a < natom; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmK, a * 64, y, &kv_full[s]);
-        for (int a = 0; a < vatom; ++a) tma_load_2d(sV + (s * vatom + a) * kblk, &tmV, a * 64, y, &kv_full[s]);
+        if (FLAT) {                              // tmK: expanded rows, tmV: gathered cache rows
+          const int y = flat0 + (page0 + i) * kWtKeys, nn = p.DN / 64;
+          for (int a = 0; a < nn; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmK, kvh * p.DN + a * 64, y, &kv_full[s]);
+          for (int a = nn; a < natom; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmV, p.rot_col + (a - nn) * 64, y, &kv_full[s]);
+          for (int a = 0; a < vatom; ++a) tma_load_2d(sV + (s * vatom + a) * kblk, &tmK, p.hq * p.DN + kvh * p.DV + a * 64, y, &kv_full[s]);
+        } else {
+          const int y = (bt[page0 + i] * p.hkv + kvh) * kWtKeys;
+          for (int a = 0; a < natom; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmK, a * 64, y, &kv_full[s]);
+          for (int a = 0; a < vatom; ++a) tma_load_2d(sV + (s * vatom + a) * kblk, &tmV, a * 64, y, &kv_full[s]);
+        }
         if (*abort_flag) break;
       }
     }
@@ -272,7 +295,8 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         *abort_flag = 1;
       } else {
         tc_fence_after();
-        const float f = l_run > 0.f ? p.out_scale / l_run : 0.f;
+        float f = l_run > 0.f ? p.out_scale / l_run : 0.f;
+        if (FLAT && p.gate != nullptr && live) f *= sigmoid_f32(bf16_to_f32(p.gate[static_cast<size_t>(row0 + tok) * p.stride + kvh * group + r % group]));
         bf16* dst = p.out + static_cast<size_t>(row0 + (live ? tok : 0)) * p.out_stride + static_cast<size_t>(kvh * group + r % group) * p.DV;
         for (int c0 = 0; c0 < p.DV; c0 += 16) {
           uint32_t raw[16];
@@ -297,20 +321,44 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 
 using namespace dgpp;
 
-// Runs of consecutive rows (run_start [runs + 1]); `tiles` = sum over the runs of ceil(length / (128 / group)).  The cache
-// (pages of 64 tokens) holds the runs' own positions already.
-DGPP_API int dgpp_window_attn_tc(const void* proj, int64_t stride, int q_off, const void* k_cache, const void* v_cache,
-                                 const void* block_table, const void* row_req, const void* positions, const void* run_start, void* out,
-                                 int64_t out_stride, int runs, int tiles, int hq, int hkv, int D, int DV, int page, int max_blocks,
-                                 int num_blocks, int window, float scale, float out_scale, cudaStream_t st) {
+static int wt_check(const void* proj, int64_t stride, int q_off, const void* out, int64_t out_stride, int runs, int hq, int hkv, int D, int DV,
+                    int page, int window) {
   DGPP_REQUIRE(hkv > 0 && hq % hkv == 0 && hq / hkv <= kWtRows, "window_attn_tc: %d query heads over %d key heads", hq, hkv);
   DGPP_REQUIRE(D % 64 == 0 && D >= 64 && D <= 256 && DV % 64 == 0 && DV >= 64 && DV <= 256, "window_attn_tc: head widths %d / %d", D, DV);
   DGPP_REQUIRE(page == kWtKeys, "window_attn_tc: page %d (64)", page);
   DGPP_REQUIRE(stride % 8 == 0 && q_off % 8 == 0 && out_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0 &&
                    (reinterpret_cast<uintptr_t>(out) & 15) == 0, "window_attn_tc: rows must be 16-byte aligned");
   DGPP_REQUIRE(window >= 1 && runs >= 1, "window_attn_tc: window %d, %d runs", window, runs);
+  return 0;
+}
+
+template <bool FLAT>
+static int launch_wt(const CUtensorMap& tK, const CUtensorMap& tV, WindowTcParams& p, int tiles, cudaStream_t st) {
+  const size_t fixed = 1024 + static_cast<size_t>(p.D / 64 + 2) * kWtRows * 128 + 192, stage = static_cast<size_t>(p.D + p.DV) * 128;
+  const size_t limit = 227 * 1024;
+  p.stages = static_cast<int>((limit - fixed) / stage);
+  p.stages = p.stages > 4 ? 4 : p.stages;
+  DGPP_REQUIRE(p.stages >= 2, "window_attn_tc: head widths %d / %d do not fit shared memory", p.D, p.DV);
+  static bool attr = false;
+  if (!attr) {
+    DGPP_CUDA_OK(cudaFuncSetAttribute(window_attn_tc_kernel<FLAT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(limit)));
+    attr = true;
+  }
+  window_attn_tc_kernel<FLAT><<<dim3(tiles, p.hkv), kWtThreads, fixed + p.stages * stage, st>>>(tK, tV, p);
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// Runs of consecutive rows (run_start [runs + 1]); `tiles` = sum over the runs of ceil(length / (128 / group)).  The cache
+// (pages of 64 tokens) holds the runs' own positions already.
+DGPP_API int dgpp_window_attn_tc(const void* proj, int64_t stride, int q_off, const void* k_cache, const void* v_cache,
+                                 const void* block_table, const void* row_req, const void* positions, const void* run_start, void* out,
+                                 int64_t out_stride, int runs, int tiles, int hq, int hkv, int D, int DV, int page, int max_blocks,
+                                 int num_blocks, int window, float scale, float out_scale, cudaStream_t st) {
+  if (wt_check(proj, stride, q_off, out, out_stride, runs, hq, hkv, D, DV, page, window)) return -1;
   if (tiles == 0) return 0;
   WindowTcParams p;
+  memset(&p, 0, sizeof(p));
   p.proj = static_cast<const bf16*>(proj); p.stride = stride; p.q_off = q_off;
   p.block_table = static_cast<const int32_t*>(block_table);
   p.row_req = static_cast<const int32_t*>(row_req);
@@ -320,23 +368,45 @@ DGPP_API int dgpp_window_attn_tc(const void* proj, int64_t stride, int q_off, co
   p.status = device_status_ptr();
   p.runs = runs; p.hq = hq; p.hkv = hkv; p.D = D; p.DV = DV; p.max_blocks = max_blocks; p.window = window;
   p.scale = scale; p.out_scale = out_scale;
-  const size_t fixed = 1024 + static_cast<size_t>(D / 64 + 2) * kWtRows * 128 + 192, stage = static_cast<size_t>(D + DV) * 128;
-  const size_t limit = 227 * 1024;
-  p.stages = static_cast<int>((limit - fixed) / stage);
-  p.stages = p.stages > 4 ? 4 : p.stages;
-  DGPP_REQUIRE(p.stages >= 2, "window_attn_tc: head widths %d / %d do not fit shared memory", D, DV);
   const uint64_t rows = static_cast<uint64_t>(num_blocks) * hkv * page;
   CUtensorMap tK, tV;
   if (make_tmap_2d(&tK, k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, rows, static_cast<uint64_t>(D) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
   if (make_tmap_2d(&tV, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, DV, rows, static_cast<uint64_t>(DV) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
-  static bool attr = false;
-  if (!attr) {
-    DGPP_CUDA_OK(cudaFuncSetAttribute(window_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(limit)));
-    attr = true;
-  }
-  window_attn_tc_kernel<<<dim3(tiles, hkv), kWtThreads, fixed + p.stages * stage, st>>>(tK, tV, p);
-  DGPP_CUDA_OK(cudaGetLastError());
-  return 0;
+  return launch_wt<false>(tK, tV, p, tiles, st);
+}
+
+// The same over keys and values expanded from a latent cache: `flat` [flat_rows, heads * (dn + dv)] bf16, `lat` [flat_rows, lat_cols]
+// bf16 (the gathered cache rows, rotated key part from column rot_col), query head h at q_off + h * (dn + dr) of its row.  Runs:
+// run_start / run_len [runs]; flat row of position 0 of a run: flat_base (may be negative).  gate_off >= 0: sigmoid of that column
+// of a row, one per head, multiplies the head's output.
+DGPP_API int dgpp_latent_prefill_tc(const void* proj, int64_t stride, int q_off, int gate_off, const void* flat, const void* lat, int lat_cols,
+                                    int rot_col, const void* row_req, const void* positions, const void* run_start, const void* run_len,
+                                    const void* flat_base, void* out, int64_t out_stride, int runs, int tiles, int flat_rows, int heads, int dn,
+                                    int dr, int dv, int window, float scale, cudaStream_t st) {
+  if (wt_check(proj, stride, q_off, out, out_stride, runs, heads, heads, dn + dr, dv, kWtKeys, window)) return -1;
+  DGPP_REQUIRE(dn % 64 == 0 && dn >= 64 && dr % 64 == 0 && dr >= 0 && lat_cols % 8 == 0 && rot_col % 8 == 0 && rot_col + dr <= lat_cols,
+               "latent_prefill_tc: key widths %d + %d, cache rows of %d", dn, dr, lat_cols);
+  DGPP_REQUIRE(run_len && flat_base && flat_rows % kWtKeys == 0, "latent_prefill_tc: %d flat rows", flat_rows);
+  if (tiles == 0) return 0;
+  WindowTcParams p;
+  memset(&p, 0, sizeof(p));
+  p.proj = static_cast<const bf16*>(proj); p.stride = stride; p.q_off = q_off;
+  p.row_req = static_cast<const int32_t*>(row_req);
+  p.positions = static_cast<const int32_t*>(positions);
+  p.run_start = static_cast<const int32_t*>(run_start);
+  p.run_len = static_cast<const int32_t*>(run_len);
+  p.flat_base = static_cast<const int32_t*>(flat_base);
+  p.gate = gate_off >= 0 ? p.proj + gate_off : nullptr;
+  p.out = static_cast<bf16*>(out); p.out_stride = out_stride;
+  p.status = device_status_ptr();
+  p.runs = runs; p.hq = heads; p.hkv = heads; p.D = dn + dr; p.DV = dv; p.window = window;
+  p.DN = dn; p.rot_col = rot_col;
+  p.scale = scale; p.out_scale = 1.f;
+  const uint64_t cols = static_cast<uint64_t>(heads) * (dn + dv);
+  CUtensorMap tK, tV;
+  if (make_tmap_2d(&tK, flat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cols, flat_rows, cols * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
+  if (make_tmap_2d(&tV, lat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, lat_cols, flat_rows, static_cast<uint64_t>(lat_cols) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
+  return launch_wt<true>(tK, tV, p, tiles, st);
 }

@@ -3,8 +3,9 @@ under its path in the model object (`layers.3.qkv.payload`, `layers.3.moe.expert
 `config.json` that names the family (`model_type` = "dgpp-<family>") and carries the configuration and the format of
 every quantised matrix.  `save_family` writes one; `load_family` rebuilds the model on a device.  Quantised payloads
 and scales travel byte for byte.  The fixture writer of the per-family load / bind / forward checks, and the hand-off
-format between a conversion script and the server for these families.  The Sitirax family has a published layout of its
-own (`"architecture": "Sitirax"` in config.json, bf16 tensors named layer by layer); it is read and written as published.
+format between a conversion script and the server for these families.  The Sitirax and Potivik families have published layouts
+of their own (`"architecture": "Sitirax"` in config.json, bf16 tensors named layer by layer); they are read and written as
+published, and run in bf16 or in true fp32.
 (reference counterparts: src/models/*/loader.cpp + binding.cpp per family, tools' fixture writers; there every family
  binds its publisher's tensor names, which this build does for the dense family only.)
 """
@@ -71,20 +72,33 @@ def _walk(obj: Any, prefix: str = "") -> Iterator[Tuple[str, Any, Callable[[Any]
             yield from _walk(v, path + ".")
 
 
-def load_sitirax(ck, device="cuda", dtype: torch.dtype = torch.bfloat16) -> Any:
-    """A published Sitirax checkpoint -> the packed model (`dtype`: bf16, or fp32 to run everything in 32 bits)."""
-    from ..models.sitirax import SitiraxConfig, SitiraxModel, tensor_shapes
+def published(family: str):
+    """(configuration, model, runner, tensor_shapes, random_tensors) of a family with a published layout, or None."""
+    if family == "sitirax":
+        from ..models import sitirax as m
+        return m.SitiraxConfig, m.SitiraxModel, m.SitiraxRunner, m.tensor_shapes, m.random_tensors
+    if family == "potivik":
+        from ..models import potivik as m
+        return m.PotivikConfig, m.PotivikModel, m.PotivikRunner, m.tensor_shapes, m.random_tensors
+    return None
 
-    cfg = SitiraxConfig.from_dict(ck.config)
+
+PUBLISHED = ("sitirax", "potivik")
+
+
+def load_published(ck, device="cuda", dtype: torch.dtype = torch.bfloat16) -> Any:
+    """A published checkpoint -> the packed model (`dtype`: bf16, or fp32 to run everything in 32 bits)."""
+    config, model, _, tensor_shapes, _ = published(ck.family)
+    cfg = config.from_dict(ck.config)
     want = set(tensor_shapes(cfg))
     missing, stray = sorted(want - set(ck.names())), sorted(set(ck.names()) - want)
     if missing or stray:
         raise ValueError(f"{ck.dir}: missing tensors {missing[:4]}, tensors the configuration does not use {stray[:4]}")
-    return SitiraxModel.from_tensors(cfg, ck.tensor, device, dtype)
+    return model.from_tensors(cfg, ck.tensor, device, dtype)
 
 
-def save_sitirax(cfg: Any, tensors: Dict[str, torch.Tensor], out_dir: str) -> None:
-    """Writes config.json and the bf16 tensors of a Sitirax model in its published layout."""
+def save_published(cfg: Any, tensors: Dict[str, torch.Tensor], out_dir: str) -> None:
+    """Writes config.json and the bf16 tensors of a model in its family's published layout."""
     os.makedirs(out_dir, exist_ok=True)
     with open(os.path.join(out_dir, "config.json"), "w") as f:
         json.dump(cfg.to_dict(), f, indent=1)
@@ -139,12 +153,12 @@ def save_family(model: Any, out_dir: str) -> None:
 
 
 def load_family(spec: str, device="cuda", dtype: torch.dtype = torch.bfloat16) -> Any:
-    """Rebuilds the model a `save_family` directory (or a published Sitirax checkpoint) holds.  The object tree comes from the family's own constructor
+    """Rebuilds the model a `save_family` directory (or a published checkpoint) holds.  The object tree comes from the family's own constructor
     (every member then takes the stored bytes), so the configuration alone decides which tensors must exist: a missing
     or mis-shaped one is an error that names it."""
     ck = open_checkpoint(spec)
-    if ck.family == "sitirax":
-        return load_sitirax(ck, device, dtype)
+    if ck.family in PUBLISHED:
+        return load_published(ck, device, dtype)
     if dtype != torch.bfloat16:
         raise ValueError(f"{spec}: the {ck.family} family runs in bf16")
     mt = ck.config.get("model_type", "")
@@ -199,10 +213,10 @@ def _restack(obj: Any, device) -> None:
 def runner_for(model: Any, max_rows: int, slots: int, max_seq_len: int, device="cuda", pool_tokens: int = 0) -> Any:
     """The kernel runner of a family model (what `engine.adapters.RunnerEngine` drives).  pool_tokens: cache positions shared
     by all slots (families with a shared pool; 0: every slot at full length)."""
-    from ..models.sitirax import SitiraxModel, SitiraxRunner
-
-    if isinstance(model, SitiraxModel):
-        return SitiraxRunner(model, max_rows, slots, max_seq_len, device, pool_tokens)
+    for family in PUBLISHED:
+        _, cls, runner, _, _ = published(family)
+        if isinstance(model, cls):
+            return runner(model, max_rows, slots, max_seq_len, device, pool_tokens)
     if pool_tokens:
         raise ValueError(f"{type(model).__name__} lays its caches out per slot: no shared pool")
     from ..models.dory import DoryRunner
@@ -224,14 +238,21 @@ def _tiny_sitirax(vocab: int):
                                  DeltaSpec(4, 2, 64, 128, 4), 1024, logit_scale=0.25)
 
 
+def _tiny_potivik(vocab: int):
+    from ..models.potivik import ExpertsSpec, FeedForward, LatentSpec, PotivikConfig, StateSpaceSpec
+
+    return PotivikConfig.uniform(4, 512, vocab, LatentSpec(8, 64, 32, 64, 128, 0.1, 256, 10000.0, 32), StateSpaceSpec(8, 1, 64, 64, 4, 2),
+                                 ExpertsSpec(16, 2, FeedForward(256, 7.0), FeedForward(384, 7.0)), FeedForward(1024, 7.0), 64)
+
+
 def tiny_model(family: str, device="cpu", seed: int = 0, vocab: int = 4096) -> Any:
     """A small random-init model of `family` (the shapes the server's `--model <family>-tiny` choices use)."""
     from ..models.moe import MoEConfig
 
-    if family == "sitirax":
-        from ..models.sitirax import SitiraxModel, random_tensors
-        cfg = _tiny_sitirax(vocab)
-        return SitiraxModel.from_tensors(cfg, random_tensors(cfg, seed).__getitem__, device)
+    if family in PUBLISHED:
+        _, model, _, _, random_tensors = published(family)
+        cfg = {"sitirax": _tiny_sitirax, "potivik": _tiny_potivik}[family](vocab)
+        return model.from_tensors(cfg, random_tensors(cfg, seed).__getitem__, device)
     cfg_cls, model_cls = _registry()[family]
     moe = MoEConfig(hidden=512, experts=16, top_k=2, moe_ffn=512, shared_ffn=512)
     if family == "glm_flash":
@@ -256,17 +277,16 @@ def main(argv=None) -> int:
     import argparse
 
     ap = argparse.ArgumentParser(description=main.__doc__)
-    ap.add_argument("--family", required=True, choices=sorted(_registry()) + ["sitirax"])
+    ap.add_argument("--family", required=True, choices=sorted(_registry()) + list(PUBLISHED))
     ap.add_argument("--out", required=True)
     ap.add_argument("--seed", type=int, default=0)
     ap.add_argument("--vocab", type=int, default=4096)
     ap.add_argument("--check", action="store_true", help="load the directory back and compare the oracle logits of a short prompt")
     a = ap.parse_args(argv)
     model = tiny_model(a.family, "cpu", a.seed, a.vocab)
-    if a.family == "sitirax":
-        from ..models.sitirax import random_tensors
-        tensors = random_tensors(model.cfg, a.seed)
-        save_sitirax(model.cfg, tensors, a.out)
+    if a.family in PUBLISHED:
+        tensors = published(a.family)[4](model.cfg, a.seed)
+        save_published(model.cfg, tensors, a.out)
         report = {"family": a.family, "out": a.out, "tensors": len(tensors)}
     else:
         save_family(model, a.out)

@@ -1,0 +1,101 @@
+"""Mixture of experts over plain rows: bf16 (or fp32) expert matrices stacked for the grouped linear, a router and an optional
+gated shared expert that read the same input in one fp32-output linear.  The router's weight multiplies an expert's input; since
+the gate / up projection is linear it is applied to its fp32 result, in the activation kernel.
+
+Up to 16 rows: one launch routes and lists the experts in use, every listed expert reads all rows.  More rows: selection, counting
+sort into tiles, row scatter (`csrc/kernels/moe_prefill.cu`, `moe_rows.cu`).  Both are shapes fixed by the row count alone, so passes
+can be captured."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from ..ops import core as ops
+from ..ops import mixers as mx
+from ..quant.formats import QuantLinear
+
+
+@dataclass
+class RowExperts:
+    """Packed weights of one block."""
+    experts: int
+    top: int
+    ff: int                              # packed width of a routed expert (a multiple of 8)
+    limit: float
+    w_first: QuantLinear                 # [router rows | shared gate row | shared gate and up rows] over the input, fp32 results
+    w_gu: torch.Tensor                   # [experts * 2 ff, Hp]
+    w_down: torch.Tensor                 # [experts * Hp, ff]
+    hidden: int
+    sg_col: int = 0                      # columns of w_first's result
+    shared_col: int = 0
+    shared_ff: int = 0                   # 0: no shared expert
+    shared_limit: float = 0.0
+    shared_down: Optional[QuantLinear] = None
+
+    @property
+    def nbytes(self) -> int:
+        w = [self.w_gu, self.w_down]
+        return sum(t.numel() * t.element_size() for t in w) + self.w_first.nbytes + (self.shared_down.nbytes if self.shared_ff else 0)
+
+    def tile_rows(self, rows: int, f32: bool) -> int:
+        """Rows of a tile: about the experts' average share, as the linears take them."""
+        if rows <= mx.SMALL_TOKENS:
+            return 16
+        share = rows * self.top / self.experts
+        return next((bn for bn in (16, 32, 64) if share <= bn), 64 if f32 else 128)
+
+    def max_tiles(self, rows: int, bn: int) -> int:
+        pairs = rows * self.top
+        return min(self.experts, pairs) + (0 if rows <= mx.SMALL_TOKENS else pairs // bn)
+
+
+class RowExpertsScratch:
+    """Buffers for passes of up to `rows` rows, shared by the blocks of one runner."""
+
+    def __init__(self, blocks, rows: int, dtype: torch.dtype, device):
+        f32 = dtype == torch.float32
+        # every size grows with the row count while the tile stays the same: the largest count of every tile decides
+        counts = lambda b: {min(rows, n) for n in (mx.SMALL_TOKENS, rows, *(bn * b.experts // b.top for bn in (16, 32, 64)))}
+        need = lambda f: max([f(b, n) for b in blocks for n in counts(b)] + [1])
+        tiles = lambda b, n: b.max_tiles(n, b.tile_rows(n, f32))
+        tr = lambda b, n: tiles(b, n) * b.tile_rows(n, f32)
+        e = lambda n, dt: torch.empty(n, dtype=dt, device=device)
+        self.first = e(need(lambda b, n: n * b.w_first.n), torch.float32)
+        self.ids, self.wts = e(need(lambda b, n: n * b.top), torch.int32), e(need(lambda b, n: n * b.top), torch.float32)
+        self.pair_row, self.tiles, self.n_tiles = e(need(lambda b, n: n * b.top), torch.int32), e(need(tiles), torch.int32), e(1, torch.int32)
+        self.row_w = torch.zeros(need(tr), dtype=torch.float32, device=device)
+        self.xs = e(need(lambda b, n: tr(b, n) * b.hidden), dtype)
+        self.h = e(need(lambda b, n: tr(b, n) * 2 * b.ff), dtype)
+        self.act = e(need(lambda b, n: tr(b, n) * b.ff), dtype)
+        self.shared_act = e(need(lambda b, n: n * b.shared_ff), dtype)
+        self.y = e(need(lambda b, n: tr(b, n) * b.hidden), dtype)
+        self.shared = e(need(lambda b, n: n * b.hidden if b.shared_ff else 0), dtype)
+
+
+def run_experts(b: RowExperts, s: RowExpertsScratch, x: torch.Tensor) -> mx.MoeDelta:
+    """x [rows, hidden] -> the block's result as the rows ``stream_norm`` sums."""
+    rows, f32 = x.shape[0], x.dtype == torch.float32
+    view = lambda buf, *shape: buf[:torch.Size(shape).numel()].view(*shape)
+    first = view(s.first, rows, b.w_first.n)
+    ops.linear(x, b.w_first, out=first) if f32 else ops.gemm_tc(x, b.w_first, out32=first)
+    bn = b.tile_rows(rows, f32)
+    nt = b.max_tiles(rows, bn)
+    tiles, pair_row, row_w = s.tiles[:nt], s.pair_row[:rows * b.top], s.row_w[:nt * bn]
+    if rows <= mx.SMALL_TOKENS:
+        mx.moe_route_small(first, b.experts, b.top, pair_row, tiles, row_w)
+        xs = x
+    else:
+        ids, wts = view(s.ids, rows, b.top), view(s.wts, rows, b.top)
+        mx.moe_select(first, b.experts, b.top, ids, wts)
+        ops.moe_segment_sort(ids, bn, nt, 0, b.experts, pair_row, tiles, s.n_tiles)
+        xs = view(s.xs, nt * bn, b.hidden)
+        mx.moe_scatter_rows(x, pair_row, wts, xs, row_w, b.top)
+    h = mx.grouped_linear(xs, b.w_gu, 2 * b.ff, tiles, bn, view(s.h, nt * bn, 2 * b.ff), shared_rows=xs is x)
+    act = mx.clamped_glu(h, view(s.act, nt * bn, b.ff), b.limit, row_w=row_w, tiles=tiles, bn=bn)
+    y = mx.grouped_linear(act, b.w_down, b.hidden, tiles, bn, view(s.y, nt * bn, b.hidden))
+    if not b.shared_ff:
+        return mx.MoeDelta(y, pair_row, b.top)
+    act = mx.clamped_glu(first[:, b.shared_col:], view(s.shared_act, rows, b.shared_ff), b.shared_limit)
+    return mx.MoeDelta(y, pair_row, b.top, ops.linear(act, b.shared_down, out=view(s.shared, rows, b.hidden)), first[:, b.sg_col:])

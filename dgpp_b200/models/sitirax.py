@@ -31,14 +31,11 @@ import torch.nn.functional as F
 from ..ops import core as ops
 from ..ops import mixers as mx
 from ..quant.formats import QuantLinear
+from .packing import only_keys as _only, pad_cols as _pad_cols, pad_rows as _pad_rows, pad_vec as _pad_vec, up8
 from .rows import RowRunner, RowRuns
 
 BF = torch.bfloat16
 UNIT_EPS = 1e-6                 # inside the root of the delta rule's unit vectors
-
-
-def up8(n: int) -> int:
-    return (n + 7) // 8 * 8
 
 
 # ---------------------------------------------------------------------------------------------- configuration
@@ -82,11 +79,6 @@ class LayerSpec:
     mixer: Union[ParallelSpec, DeltaSpec]
     ff: Optional[int]            # None: the layer has no feed-forward sublayer
     source: int                  # the layer whose tensors it uses (itself, unless it shares)
-
-
-def _only(d: dict, keys, what: str) -> None:
-    if set(d) != set(keys):
-        raise ValueError(f"{what}: expected the keys {sorted(keys)}, got {sorted(d)}")
 
 
 @dataclass
@@ -230,21 +222,6 @@ def random_tensors(cfg: SitiraxConfig, seed: int = 0, rank_a: int = 0, rank_g: i
 
 
 # ---------------------------------------------------------------------------------------------- packed weights
-def _pad_rows(w: torch.Tensor, groups: int, n: int, npad: int) -> torch.Tensor:
-    """[groups * n, K] -> [groups * npad, K] with zero rows behind every group."""
-    if n == npad:
-        return w
-    return F.pad(w.reshape(groups, n, -1), (0, 0, 0, npad - n)).reshape(groups * npad, -1)
-
-
-def _pad_cols(w: torch.Tensor, groups: int, n: int, npad: int) -> torch.Tensor:
-    return _pad_rows(w.T, groups, n, npad).T
-
-
-def _pad_vec(v: torch.Tensor, groups: int, n: int, npad: int) -> torch.Tensor:
-    return _pad_rows(v.reshape(-1, 1), groups, n, npad).reshape(-1)
-
-
 @dataclass
 class Packed:
     """Kernel-ready weights of one layer (shared by the layers that use them)."""

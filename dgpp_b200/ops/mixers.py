@@ -1,6 +1,7 @@
-"""Front ends of the kernels behind models with an fp32 residual stream, sliding-window attention without rotation and
-fp32 linear-attention states (``csrc/kernels/stream_ops.cu``, ``window_attn.cu``, ``window_attn_tc.cu``,
-``linear_state.cu``).  Every operator exists for bf16 and for true fp32 activations; the dtype of the tensors decides."""
+"""Front ends of the kernels behind models with an fp32 residual stream, sliding-window attention (grouped heads, or a
+shared latent), fp32 linear-attention and state-space memories, and experts of plain rows (``csrc/kernels/stream_ops.cu``,
+``window_attn.cu``, ``window_attn_tc.cu``, ``latent_attn.cu``, ``mla_tc.cu``, ``linear_state.cu``, ``state_space.cu``,
+``moe_rows.cu``).  Every operator exists for bf16 and for true fp32 activations; the dtype of the tensors decides."""
 from __future__ import annotations
 
 from typing import Optional
@@ -16,6 +17,7 @@ _lib.declare("dgpp_gated_group_norm", [P, P, L, P, P, L, I, I, I, I, F, F, I, I,
 _lib.declare("dgpp_geglu", [P, P, I, I, I, P])
 _lib.declare("dgpp_qk_norm_append", [P, L, I, I, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P])
 _lib.declare("dgpp_window_attn", [P, L, I, I, I, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, I, I, I, F, F, F, I, P])
+_lib.declare("dgpp_state_space", [P, L, I, I, P, P, P, I, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, P])
 _lib.declare("dgpp_linear_state", [P, L, I, I, P, L, P, P, I, P, P, P, P, P, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, F, F,
                                    I, I, I, P])
 
@@ -70,6 +72,107 @@ def geglu(gate_up: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     return out
 
 
+NORMS = {None: 0, "rms": 1, "layer": 2}
+_lib.declare("dgpp_stream_norm", [P, P, P, P, I, P, P, L, I, P, I, P, P, I, I, I, F, I, P])
+_lib.declare("dgpp_gated_part_norm", [P, P, L, P, P, L, I, I, I, I, F, I, P])
+_lib.declare("dgpp_clamped_glu", [P, L, P, P, I, P, I, I, F, F, I, I, P])
+_lib.declare("dgpp_token_gate", [P, P, P, L, I, P, I, I, I, I, P])
+_lib.declare("dgpp_softcap", [P, L, F, P])
+
+
+def stream_norm(x: torch.Tensor, n: int, eps: float, out: torch.Tensor, delta=None, post=(None, None), pre=(None, None)) -> torch.Tensor:
+    """x [rows, cols] fp32 takes in post(delta) in place; out = pre(x).  post / pre: (None | "rms" | "layer", fp32 weight row)
+    over the n true columns.  delta: an fp32 row block, a ``MoeDelta`` or None."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous()
+    m = delta if isinstance(delta, MoeDelta) else None
+    d = None if m is not None else delta
+    assert d is None or (d.dtype == torch.float32 and d.is_contiguous())
+    call("dgpp_stream_norm", ptr(x), ptr(d), ptr(m and m.y), ptr(m and m.pair_row), m.top if m else 0, ptr(m and m.shared),
+         ptr(m and m.gate), m.gate.stride(0) if m and m.gate is not None else 0, NORMS[post[0]], ptr(post[1]), NORMS[pre[0]], ptr(pre[1]),
+         ptr(out), x.shape[0], x.shape[1], n, float(eps), _f32(out), stream_ptr())
+    return out
+
+
+def gated_part_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, out: torch.Tensor, parts: int, eps: float) -> torch.Tensor:
+    """a = y * silu(z) (y [rows, n] fp32, z's first n columns); out = a / rms of each of `parts` equal runs of columns * w [n]; the
+    columns of `out` behind n are cleared."""
+    n = y.shape[1]
+    assert y.dtype == torch.float32 and y.is_contiguous() and n % parts == 0 and w.numel() == n and out.shape[1] >= n
+    call("dgpp_gated_part_norm", ptr(y), ptr(z), z.stride(0), ptr(w), ptr(out), out.stride(0), y.shape[0], parts, n // parts, out.shape[1],
+         float(eps), _f32(out), stream_ptr())
+    return out
+
+
+def clamped_glu(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: float = 1.702, row_w=None, tiles=None, bn: int = 1) -> torch.Tensor:
+    """gate_up [rows, 2 I] -> min(s g, limit) sigmoid(alpha min(s g, limit)) (clamp(s u, +-limit) + 1) [rows, I]; s: `row_w` or one.
+    tiles [rows / bn]: rows of tiles with a negative entry are skipped."""
+    assert out.is_contiguous() and gate_up.shape[1] >= 2 * out.shape[1]
+    call("dgpp_clamped_glu", ptr(gate_up), gate_up.stride(0), ptr(row_w), ptr(tiles), bn, ptr(out), gate_up.shape[0], out.shape[1], float(limit),
+         float(alpha), _f32(out), _f32(gate_up), stream_ptr())
+    return out
+
+
+def token_gate(gate: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col: int, out: torch.Tensor) -> torch.Tensor:
+    """gelu_tanh(gate) * table[ids[r], col : col + dim] (gate [rows, dim] fp32)."""
+    assert gate.dtype == torch.float32 and gate.is_contiguous() and out.is_contiguous() and table.dtype == out.dtype
+    call("dgpp_token_gate", ptr(gate), ptr(ids), ptr(table), table.stride(0), col, ptr(out), gate.shape[0], out.shape[1], table.shape[0],
+         _f32(out), stream_ptr())
+    return out
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x (fp32, in place) = cap * tanh(x / cap)."""
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    call("dgpp_softcap", ptr(x), x.numel(), float(cap), stream_ptr())
+    return x
+
+
+# ---------------------------------------------------------------------------------------------- experts over plain rows
+_lib.declare("dgpp_moe_select", [P, L, P, P, I, I, I, I, I, F, P])
+_lib.declare("dgpp_moe_route_small", [P, L, P, P, P, I, I, I, I, I, P])
+_lib.declare("dgpp_moe_scatter_rows", [P, P, P, P, P, I, I, I, I, P])
+_lib.declare("dgpp_gemm_tc_grouped", [I, P, L, I, I, P, I, P, P, I, I, I, I, P])
+_lib.declare("dgpp_gemm_f32_grouped", [I, P, L, I, I, P, I, P, P, L, I, I, I, P])
+SMALL_TOKENS = 16                      # rows up to which routing is one launch and every listed expert reads all rows
+MAX_EXPERTS, MAX_TOP = 512, 16
+
+
+class MoeDelta:
+    """The rows of a mixture of experts as ``stream_norm`` takes them in: sum over j of y[pair_row[r * top + j]], plus
+    sigmoid(gate[r]) * shared[r]."""
+
+    def __init__(self, y, pair_row, top: int, shared=None, gate=None):
+        self.y, self.pair_row, self.top, self.shared, self.gate = y, pair_row, top, shared, gate
+
+
+def moe_select(logits: torch.Tensor, experts: int, top: int, ids: torch.Tensor, weights: torch.Tensor, softmax: bool = False,
+               norm_topk: bool = False, scaling: float = 1.0) -> None:
+    """The `top` best of the first `experts` columns of fp32 logits per row -> ids (ascending), weights (their scores)."""
+    call("dgpp_moe_select", ptr(logits), logits.stride(0), ptr(ids), ptr(weights), logits.shape[0], experts, top, int(softmax), int(norm_topk),
+         float(scaling), stream_ptr())
+
+
+def moe_route_small(logits: torch.Tensor, experts: int, top: int, pair_row, tiles, row_w, softmax: bool = False) -> None:
+    """Up to 16 rows: tiles (experts in use), pair_row [rows * top] = tile * 16 + row, row_w [tiles * 16]."""
+    call("dgpp_moe_route_small", ptr(logits), logits.stride(0), ptr(pair_row), ptr(tiles), ptr(row_w), logits.shape[0], experts, top,
+         tiles.numel(), int(softmax), stream_ptr())
+
+
+def moe_scatter_rows(x: torch.Tensor, pair_row, weights, xs, row_w, top: int) -> None:
+    """xs[pair_row[p]] = x[p // top], row_w[pair_row[p]] = weights[p]."""
+    assert x.is_contiguous() and xs.is_contiguous() and x.shape[1] == xs.shape[1]
+    call("dgpp_moe_scatter_rows", ptr(x), ptr(pair_row), ptr(weights), ptr(xs), ptr(row_w), x.shape[0], x.shape[1], top, _f32(x), stream_ptr())
+
+
+def grouped_linear(x: torch.Tensor, w: torch.Tensor, n: int, tiles: torch.Tensor, bn: int, out: torch.Tensor, shared_rows: bool = False) -> torch.Tensor:
+    """Tile t of `out` [tiles * bn, n] = its rows of x times matrix tiles[t] of the stack w [experts * n, k] (negative: skipped).
+    shared_rows: every tile reads the same x [<= bn, k]."""
+    assert w.dtype == x.dtype == out.dtype and w.shape[0] % n == 0 and w.shape[1] == x.shape[1] and w.is_contiguous()
+    call("dgpp_gemm_f32_grouped" if _f32(x) else "dgpp_gemm_tc_grouped", bn, ptr(x), x.stride(0), x.shape[0], int(not shared_rows), ptr(w),
+         w.shape[0] // n, ptr(tiles), ptr(out), out.stride(0), tiles.numel(), n, w.shape[1], stream_ptr())
+    return out
+
+
 class WindowHeads:
     """Static description of one window-attention block inside a fused projection row."""
 
@@ -107,15 +210,17 @@ def window_attn(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, posit
 
 class StateHeads:
     """Static description of one linear-attention block: widths (padded), offsets inside the fused projection row, and the
-    constants of its rule (`decay` per head: lightning; `A_log` / `dt_bias` / low-rank rows: channel delta rule)."""
+    constants of its rule (`decay` per head: lightning; `skip` per head with `A_log` / `dt_bias`: state space; `A_log` / `dt_bias` /
+    low-rank rows: channel delta rule)."""
 
     def __init__(self, heads: int, key_heads: int, dim: int, vdim: int, c_off: int, b_off: int = 0, eps: float = 0.0,
-                 conv_w=None, A_log=None, dt_bias=None, decay=None, norm_w=None):
+                 conv_w=None, A_log=None, dt_bias=None, decay=None, norm_w=None, conv_b=None, skip=None):
         self.hv, self.hk, self.dim, self.vdim = heads, key_heads, dim, vdim
         self.DK, self.DV = pad_to(dim, STATE_WIDTHS), pad_to(vdim, STATE_WIDTHS)
         self.c_off, self.b_off, self.eps = c_off, b_off, eps
         self.conv_w, self.A_log, self.dt_bias, self.decay, self.norm_w = conv_w, A_log, dt_bias, decay, norm_w
-        self.delta = decay is None
+        self.conv_b, self.skip = conv_b, skip
+        self.delta = decay is None and skip is None
         self.taps = 0 if conv_w is None else conv_w.shape[0]
 
     @property
@@ -131,6 +236,8 @@ class StateHeads:
     def prep_floats(self, rows: int, runs: int) -> int:
         """Scratch of a pass over `rows` rows in at most `runs` runs."""
         blocks = rows // 16 + runs
+        if self.skip is not None:
+            return rows * (self.channels + 2 * self.hv) + blocks * self.hv * 288
         return rows * (self.channels + self.hv * (3 * self.DK + 1)) + blocks * self.hv * (self.DK + 512)
 
 
@@ -141,6 +248,12 @@ def linear_state(g: StateHeads, proj, state, ring, row_slot, positions, low=None
     rows = proj.shape[0]
     blocks = 0 if runs is None else sum(-(-n // 16) for n in runs.lens)
     assert state.dtype == torch.float32 and (runs is None or prep.numel() >= g.prep_floats(rows, len(runs.lens)))
+    if g.skip is not None:                       # raw read-outs [rows, heads * vdim] to `o` either way
+        call("dgpp_state_space", ptr(proj), proj.stride(0), g.c_off, g.b_off, ptr(g.conv_w), ptr(g.conv_b), ptr(ring), g.taps, ptr(g.A_log),
+             ptr(g.dt_bias), ptr(g.skip), ptr(state), ptr(row_slot), ptr(positions), None if runs is None else ptr(runs.start),
+             None if runs is None else ptr(runs.row_run0), ptr(prep), ptr(o), rows, rows if runs is None else len(runs.lens), blocks, g.hk, g.hv,
+             g.DK, g.DV, g.vdim, int(runs is None), _f32(proj), stream_ptr())
+        return
     call("dgpp_linear_state", ptr(proj), proj.stride(0), g.c_off, g.b_off, ptr(low), 0 if low is None else low.stride(0),
          ptr(g.conv_w), ptr(ring), g.taps, ptr(g.A_log), ptr(g.dt_bias), ptr(g.decay), ptr(state), ptr(row_slot), ptr(positions),
          None if runs is None else ptr(runs.start), None if runs is None else ptr(runs.row_run0), ptr(prep), ptr(o), ptr(out),
@@ -164,4 +277,128 @@ def window_prefill(g: WindowHeads, proj, cache, block_table, row_req, positions,
     call("dgpp_window_attn_tc", ptr(proj), proj.stride(0), g.q_off, ptr(cache.k), ptr(cache.v), ptr(block_table), ptr(row_req),
          ptr(positions), ptr(runs.start), ptr(out), out.stride(0), len(runs.lens), tiles, g.hq, g.hkv, g.D, g.DV, cache.page,
          block_table.shape[1], cache.k.shape[0], g.window, float(g.scale), float(out_scale), stream_ptr())
+    return out
+
+
+# ---------------------------------------------------------------------------------------------- latent attention
+_LATENT = [P, L, I, I, P, P, P, P, P, P]
+_lib.declare("dgpp_latent_append", _LATENT + [I] * 12 + [F, I, P])
+_lib.declare("dgpp_latent_absorb", _LATENT + [P, P, P] + [I] * 13 + [F, I, P])
+_lib.declare("dgpp_latent_rows", [P] * 7 + [I] * 7 + [F, I, P])
+_lib.declare("dgpp_latent_decode_tc", [P] * 9 + [I] * 8 + [F, P])
+_lib.declare("dgpp_latent_up", [P, P, P, L, P, P, L, I, I, I, I, I, P])
+_lib.declare("dgpp_latent_gather", [P, P, P, I, I, I, P])
+_lib.declare("dgpp_latent_prefill_tc", [P, L, I, I, P, P, I, I, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, F, P])
+
+
+def rotation_freqs(base: float, dims: int, device) -> torch.Tensor:
+    """[2, dims / 2] fp32: base^(-2 i / dims) as a leading and a residual term."""
+    f = torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
+    hi = f.to(torch.float32)
+    return torch.stack([hi, (f - hi.double()).to(torch.float32)]).contiguous().to(device)
+
+
+class LatentHeads:
+    """Static description of one latent-attention block inside a fused projection row: queries [heads, DN | RP] from q_off, the
+    latent [KC | RP] from kv_off, one output gate per head from g_off.  w_up [heads * DN + heads * DV, KC]: key rows, then value
+    rows, of every head."""
+
+    def __init__(self, heads: int, dim: int, rot_dim: int, vdim: int, rank: int, window: int, scale: float, eps: float, base: float, rot: int,
+                 q_off: int, kv_off: int, g_off: int, norm_w: torch.Tensor, w_up: torch.Tensor):
+        self.heads, self.dim, self.rot_dim, self.vdim, self.rank = heads, dim, rot_dim, vdim, rank
+        self.window, self.scale, self.eps, self.rot = window, scale, eps, rot
+        self.DN, self.DV, self.KC, self.RP = latent_widths(dim, rot_dim, vdim, rank)
+        self.q_off, self.kv_off, self.g_off, self.norm_w, self.w_up = q_off, kv_off, g_off, norm_w, w_up
+        self.freq = rotation_freqs(base, rot, norm_w.device)
+
+    @property
+    def cache_cols(self) -> int:
+        return self.KC + self.RP
+
+    @property
+    def flat_cols(self) -> int:
+        return self.heads * (self.DN + self.DV)
+
+    def tc_rows(self, dtype) -> bool:
+        """Single rows run on the tensor cores."""
+        return dtype == torch.bfloat16 and self.KC % 128 == 0 and self.KC <= 512 and self.RP == 64
+
+    def tc_runs(self, dtype) -> bool:
+        """Prompt runs run on the tensor cores, over keys and values expanded from the latents."""
+        return dtype == torch.bfloat16 and self.DN + self.RP <= 256 and self.DV <= 256
+
+    def _args(self, proj, positions, row_req, block_table, cache):
+        assert cache.dtype == proj.dtype == self.w_up.dtype and cache.shape[-1] == self.cache_cols
+        return (ptr(proj), proj.stride(0), self.q_off, self.kv_off, ptr(self.norm_w), ptr(self.freq), ptr(positions), ptr(row_req), ptr(block_table),
+                ptr(cache))
+
+    def _sizes(self, page: int, block_table):
+        return (self.heads, self.DN, self.DV, self.dim, self.rank, self.KC, self.RP, self.rot_dim, self.rot, page, block_table.shape[1])
+
+
+def latent_widths(dim: int, rot_dim: int, vdim: int, rank: int):
+    """Padded widths (unrotated key part, value, latent, rotated part)."""
+    up = lambda n, m: (n + m - 1) // m * m
+    return up(dim, 64), up(vdim, 64), up(rank, 128) if rank <= 512 else up(rank, 64), max(64, up(rot_dim, 64))
+
+
+def latent_append(g: LatentHeads, proj, positions, row_req, block_table, cache, page: int) -> None:
+    """Appends the rows' latents and rotated key parts to the cache and rotates their queries in place."""
+    call("dgpp_latent_append", *g._args(proj, positions, row_req, block_table, cache), proj.shape[0], *g._sizes(page, block_table), float(g.eps),
+         _f32(proj), stream_ptr())
+
+
+def latent_absorb(g: LatentHeads, proj, positions, row_req, block_table, cache, page: int, q_abs, rows: int, row_list=None, fused: bool = False):
+    """q_abs [rows, heads, KC + RP] fp32 of the rows (`row_list`: of these pass rows).  fused: the rows are new tokens; their queries are
+    rotated here and their latents appended."""
+    assert q_abs.dtype == torch.float32 and q_abs.numel() >= rows * g.heads * g.cache_cols
+    call("dgpp_latent_absorb", *g._args(proj, positions, row_req, block_table, cache), ptr(row_list), ptr(g.w_up), ptr(q_abs), rows,
+         *g._sizes(page, block_table), int(fused), float(g.eps), _f32(proj), stream_ptr())
+    return q_abs
+
+
+def latent_attn(g: LatentHeads, q_abs, cache, block_table, row_req, positions, page: int, lat, rows: int, row_list=None, splits: int = 1,
+                scratch=None) -> torch.Tensor:
+    """Windowed attention of absorbed rows -> lat [rows, heads, KC] fp32; on the tensor cores where the kernel takes the widths."""
+    if g.tc_rows(cache.dtype):
+        ml, acc = scratch if splits > 1 else (None, None)
+        call("dgpp_latent_decode_tc", ptr(q_abs), ptr(cache), ptr(block_table), ptr(row_req), ptr(positions), ptr(row_list), ptr(ml), ptr(acc),
+             ptr(lat), rows, g.heads, g.KC, page, block_table.shape[1], cache.shape[0], splits, g.window, float(g.scale), stream_ptr())
+    else:
+        call("dgpp_latent_rows", ptr(q_abs), ptr(cache), ptr(block_table), ptr(row_req), ptr(positions), ptr(row_list), ptr(lat), rows, g.heads,
+             g.KC, g.RP, page, block_table.shape[1], g.window, float(g.scale), _f32(cache), stream_ptr())
+    return lat
+
+
+def latent_up(g: LatentHeads, lat, proj, out, rows: int, row_list=None) -> torch.Tensor:
+    """out[row, h * DV + v] = (W_uv lat)[v] * sigmoid(gate of head h)."""
+    w = g.w_up[g.heads * g.DN:]
+    gate = proj[:, g.g_off:]
+    call("dgpp_latent_up", ptr(lat), ptr(w), ptr(gate), proj.stride(0), ptr(row_list), ptr(out), out.stride(0), rows, g.heads, g.DV, g.KC,
+         _f32(out), stream_ptr())
+    return out
+
+
+def latent_gather(cache, pages, out, page: int) -> torch.Tensor:
+    """out [n * page, cols] bf16 = the cache's pages pages[0 .. n - 1]."""
+    assert cache.dtype == torch.bfloat16 and out.is_contiguous()
+    call("dgpp_latent_gather", ptr(cache), ptr(pages), ptr(out), pages.numel(), page, cache.shape[-1], stream_ptr())
+    return out
+
+
+class LatentRuns:
+    """The longer runs of a pass for ``latent_prefill`` with one window: int32 device arrays first row, length, flat row of position 0
+    per run; physical ids of the pages to expand; 128-row tiles."""
+
+    def __init__(self, start, lens, base, pages, tiles: int):
+        self.start, self.lens, self.base, self.pages, self.tiles = start, lens, base, pages, tiles
+
+
+def latent_prefill(g: LatentHeads, proj, flat, gathered, row_req, positions, runs: LatentRuns, out) -> torch.Tensor:
+    """Windowed attention of prompt runs over expanded keys and values (flat [n, flat_cols], gathered [n, KC + RP]), gate included.
+    `latent_append` comes before it."""
+    assert proj.dtype == flat.dtype == gathered.dtype == out.dtype == torch.bfloat16 and flat.is_contiguous() and gathered.is_contiguous()
+    call("dgpp_latent_prefill_tc", ptr(proj), proj.stride(0), g.q_off, g.g_off, ptr(flat), ptr(gathered), gathered.shape[1], g.KC, ptr(row_req),
+         ptr(positions), ptr(runs.start), ptr(runs.lens), ptr(runs.base), ptr(out), out.stride(0), runs.lens.numel(), runs.tiles, flat.shape[0],
+         g.heads, g.DN, g.RP, g.DV, g.window, float(g.scale), stream_ptr())
     return out

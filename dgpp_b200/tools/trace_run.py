@@ -73,11 +73,12 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", type=int, required=True)
     a = ap.parse_args(argv)
     from .. import build
+    from ..loaders.family_io import PUBLISHED
 
     with open(os.path.join(a.model, "config.json")) as f:
         cfg = json.load(f)
     family = str(cfg.get("architecture", "")).lower()
-    if a.dtype == "float32" and family != "sitirax":
+    if a.dtype == "float32" and family not in PUBLISHED:
         print("this model's family does not run in float32", file=sys.stderr)
         return 3
     kernels = build.ensure(family)

@@ -47,12 +47,12 @@ def test_refused_configurations():
 
 def test_checkpoint_round_trip_and_refusals(tmp_path):
     from dgpp_b200.loaders.checkpoint import open_checkpoint, write_safetensors
-    from dgpp_b200.loaders.family_io import load_family, save_sitirax
+    from dgpp_b200.loaders.family_io import load_family, save_published
 
     cfg = sc.CONFIGS["odd"]
     c, w = SitiraxConfig.from_dict(cfg), sc.tensors(cfg, 2)
     out = str(tmp_path / "ck")
-    save_sitirax(c, w, out)
+    save_published(c, w, out)
     assert open_checkpoint(out).family == "sitirax"
     assert json.load(open(out + "/config.json")) == cfg
     toks = torch.tensor(sc.token_ids(cfg, 20))

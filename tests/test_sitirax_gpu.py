@@ -219,12 +219,12 @@ def test_generation_with_sampling_parameters(dev):
 def test_trace_replay(dev, dtype, tmp_path):
     """The replay program over its standard input: mixed steps, a request left out and resumed, slots and pages given back and
     taken again, logits where they are wanted."""
-    from dgpp_b200.loaders.family_io import save_sitirax
+    from dgpp_b200.loaders.family_io import save_published
     from dgpp_b200.models.sitirax import SitiraxConfig
 
     name = "odd"
     cfg = sc.CONFIGS[name]
-    save_sitirax(SitiraxConfig.from_dict(cfg), sc.tensors(cfg, 1), str(tmp_path / "ck"))
+    save_published(SitiraxConfig.from_dict(cfg), sc.tensors(cfg, 1), str(tmp_path / "ck"))
     t = {c: sc.token_ids(cfg, n, s) for c, n, s in (("a", 90, 1), ("b", 40, 2), ("c", 100, 3))}
     cuts = [({"a": (0, 60), "b": (0, 7)}, []), ({"b": (7, 8)}, []), ({"a": (60, 61), "b": (8, 40)}, ["b"]),
             ({"a": (61, 62), "c": (0, 2)}, []), ({"a": (62, 90), "c": (2, 3)}, ["a"]), ({"c": (3, 100)}, ["c"])]
