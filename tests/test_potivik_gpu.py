@@ -54,9 +54,10 @@ def _close(got, want, dtype):
 
     ops.check_status()
     rms = (got.double().cpu() - want).pow(2).mean(-1).sqrt() / want.std()
-    limit, typical = (4e-5, 2e-5) if dtype == torch.float32 else (0.15, 0.05)      # fp32 is the sharp comparison
+    # fp32 is the sharp comparison; bf16: rounding, and single rows where it moves a close routing decision
+    limit, most, typical = (4e-5, 4e-5, 2e-5) if dtype == torch.float32 else (0.3, 0.15, 0.05)
     assert rms.max().item() <= limit, (rms.max().item(), int(rms.argmax()))
-    assert len(rms) < 8 or rms.median().item() <= typical, rms.median().item()
+    assert len(rms) < 8 or (rms.quantile(0.9).item() <= most and rms.median().item() <= typical), (rms.quantile(0.9).item(), rms.median().item())
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
