@@ -119,7 +119,7 @@ def _latent_rows(dev, batch: int, rows: int, heads: int = 32, dim: int = 128, ro
 
         def attn(j):
             r = runners[j]
-            splits = max(1, -(-148 // (n * -(-heads // 16))))
+            splits = mx.latent_splits(n, heads, window, r.max_splits)
             mx.latent_attn(r.m.layers[0].latent, r.q_abs, r.kv.layers[0].k, r.kv.block_table, req, pos, 64, r.lat, n, None, splits, r.scratch)
 
         def ups(j):

@@ -31,6 +31,32 @@ __device__ __forceinline__ void st_elem4(bf16* p, float4 v) {
   *reinterpret_cast<uint2*>(p) = w;
 }
 
+// Eight consecutive elements (16-byte aligned).
+__device__ __forceinline__ void ld_elem8(const float* p, float* f) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void ld_elem8(const bf16* p, float* f) {
+  Pack16 v;
+  v.u = *reinterpret_cast<const uint4*>(p);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 t = __bfloat1622float2(v.h2[j]);
+    f[2 * j] = t.x;
+    f[2 * j + 1] = t.y;
+  }
+}
+__device__ __forceinline__ void st_elem8(float* p, const float* f) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+}
+__device__ __forceinline__ void st_elem8(bf16* p, const float* f) {
+  Pack16 v;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) v.h2[j] = __floats2bfloat162_rn(f[2 * j], f[2 * j + 1]);
+  *reinterpret_cast<uint4*>(p) = v.u;
+}
+
 // 16 bytes of elements: 8 bf16 or 4 fp32, converted to fp32.
 template <typename T>
 struct Vec16;

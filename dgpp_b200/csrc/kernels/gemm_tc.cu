@@ -79,6 +79,9 @@ struct GemmParams {
   // with a negative entry do nothing.  group_x: every tile has its own BN activation rows, else all tiles read the rows from 0.
   const int32_t* groups;
   int group_x;
+  // bf16 weights, one output (bf16 or fp32), 16-byte aligned rows, no split: the finished tile is turned around in shared memory
+  // (all eight spare warps read the accumulator) and leaves as 16-byte vectors along N
+  int staged;
 };
 
 template <int BN>
@@ -390,8 +393,53 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA,   // bf16 weights, or pa
     }
   }
 
+  // ------------------------------------------------------------------ staged epilogue (warps 2..9, bf16 weights)
+  if constexpr (!kQuant) {
+    if (p.staged && warp >= 2) {
+      const int q = warp & 3, half = (warp - 2) >> 2;
+      const bool ok = wait_bar(acc_full, 0) && !*abort_flag;
+      if (!ok) { report(p.status, kTimeoutAccum, 7); *abort_flag = 1; }
+      tc_fence_after();
+      const int cols = min(BN, p.T - m0), at = q * 32 + lane;
+      // the operand rings are idle once the accumulator is complete (sB and sA are one block of shared memory)
+      if (ok) {
+#pragma unroll 1
+        for (int c0 = half * 16; c0 < cols; c0 += 32) {
+          uint32_t r[16];
+          tmem_ld_x16(tmem_base + (static_cast<uint32_t>(q * 32) << 16) + c0, r);
+          if (p.out != nullptr) {
+            bf16* d = reinterpret_cast<bf16*>(sB) + c0 * kBM + at;
+#pragma unroll
+            for (int j = 0; j < 16; ++j) d[j * kBM] = f32_to_bf16(__uint_as_float(r[j]) * p.alpha);
+          } else {
+            float* d = reinterpret_cast<float*>(sB) + c0 * kBM + at;
+#pragma unroll
+            for (int j = 0; j < 16; ++j) d[j * kBM] = __uint_as_float(r[j]) * p.alpha;
+          }
+        }
+      }
+      asm volatile("bar.sync 2, 256;" ::: "memory");
+      if (ok) {
+        const int et = static_cast<int>(threadIdx.x) - 64;
+        const uint4* tile = reinterpret_cast<const uint4*>(sB);
+        if (p.out != nullptr) {
+          const int seg = et % (kBM / 8);
+          bf16* dst = p.out + static_cast<size_t>(m0) * p.ldc + n0 + seg * 8;
+          if (n0 + seg * 8 < p.N)
+            for (int m = et / (kBM / 8); m < cols; m += 256 / (kBM / 8))
+              *reinterpret_cast<uint4*>(dst + static_cast<size_t>(m) * p.ldc) = tile[m * (kBM / 8) + seg];
+        } else {
+          const int seg = et % (kBM / 4);
+          float* dst = p.out32 + static_cast<size_t>(m0) * p.ldc + n0 + seg * 4;
+          if (n0 + seg * 4 < p.N)
+            for (int m = et / (kBM / 4); m < cols; m += 256 / (kBM / 4))
+              *reinterpret_cast<uint4*>(dst + static_cast<size_t>(m) * p.ldc) = tile[m * (kBM / 4) + seg];
+        }
+      }
+    }
+  }
   // ------------------------------------------------------------------ epilogue (warps 2..5)
-  if (warp >= 2 && warp < 6) {
+  if ((kQuant || !p.staged) && warp >= 2 && warp < 6) {
     const int q = warp & 3;  // TMEM lane quadrant this warp may read
     const bool ok = nkb > 0 ? wait_bar(acc_full, 0) : true;
     if (!ok) { report(p.status, kTimeoutAccum, 6); *abort_flag = 1; }
@@ -553,6 +601,7 @@ static int launch_gemm(const CUtensorMap& tA, const CUtensorMap& tB, const CUten
   static bool attr = false;
   constexpr size_t smem = C::smem();
   static_assert(smem <= 227 * 1024, "shared memory budget exceeded");
+  static_assert(WMODE != 0 || static_cast<size_t>(C::SB) * (BN + kBM) * 128 >= static_cast<size_t>(BN) * kBM * 4, "a tile fits the rings");
   if (!attr) {
     DGPP_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     attr = true;
@@ -641,6 +690,8 @@ static int gemm_tc_impl(int wmode, int a_f16, int bn, const void* x, int64_t x_s
   per = dgpp_ceil_div(per, align) * align;
   p.kb_per_split = per;
   splits = dgpp_ceil_div(num_kb, per);
+  const uintptr_t dst = reinterpret_cast<uintptr_t>(out ? out : out32);
+  p.staged = wmode == 0 && splits == 1 && !comm_push && !resid && (out == nullptr) != (out32 == nullptr) && N % 8 == 0 && ldc % 8 == 0 && dst % 16 == 0;
 
   CUtensorMap tA, tB, tSf;
   memset(&tSf, 0, sizeof(tSf));

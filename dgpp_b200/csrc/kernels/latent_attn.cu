@@ -99,14 +99,14 @@ __global__ void __launch_bounds__(256) latent_append_kernel(LatentArgs a) {
 
 constexpr int kLatRows = 8;
 
-// grid (heads (+ 1 when fused), ceil(n / 8), KC / 64), 256 threads: a CTA owns 64 latent columns of one head for up to 8 rows; a
-// warp sums an eighth of the head's key rows (lane = two columns), the eight partial sums are added in warp order.  The CTAs
-// behind the last head write the cache rows.
+// grid (heads (+ 1 when fused), ceil(n / 8), KC / 128 rounded up), 256 threads: a CTA owns 128 latent columns of one head for up to
+// 8 rows; a warp sums an eighth of the head's key rows (lane = four columns), the eight partial sums are added in warp order.  The
+// CTAs behind the last head write the cache rows.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a) {
-  extern __shared__ float ab_smem[];
-  float* qs = ab_smem;                                    // [8][dim]
-  float* part = ab_smem + kLatRows * a.dim;               // [8 warps][8 rows][64]
+  extern __shared__ __align__(16) float ab_smem[];
+  float* qs = ab_smem;                                    // [dim][8 rows]
+  float* part = ab_smem + kLatRows * a.dim;               // [8 warps][8 rows][128]
   pdl_wait();
   const int h = blockIdx.x, r0 = blockIdx.y * kLatRows, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int nr = min(kLatRows, a.n - r0);
@@ -117,38 +117,47 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a) {
   }
   const T* proj = static_cast<const T*>(a.proj);
   const size_t qcol = a.q_off + static_cast<size_t>(h) * (a.DN + a.RP);
-  for (int i = tid; i < kLatRows * a.dim; i += 256) {
-    const int r = i / a.dim, c = i % a.dim;
-    qs[i] = r < nr ? ld_elem(proj + static_cast<size_t>(pass_row(r)) * a.stride + qcol + c) : 0.f;
+  if (warp < kLatRows) {
+    const T* src = proj + static_cast<size_t>(pass_row(min(warp, nr - 1))) * a.stride + qcol;
+    for (int c = lane; c < a.dim; c += 32) qs[c * kLatRows + warp] = warp < nr ? ld_elem(src + c) : 0.f;
   }
   __syncthreads();
-  const int d0 = blockIdx.z * 64 + lane * 2;
-  const int per = (a.dim + 7) / 8, n0 = warp * per, n1 = min(a.dim, n0 + per);
-  float acc[kLatRows][2];
+  const int d0 = blockIdx.z * 128 + lane * 4;
+  const bool live = d0 < a.KC;
+  const int per = (a.dim + 7) / 8, n0 = warp * per, n1 = live ? min(a.dim, n0 + per) : n0;
+  float acc[kLatRows][4];
 #pragma unroll
-  for (int r = 0; r < kLatRows; ++r) acc[r][0] = acc[r][1] = 0.f;
-  const T* wp = static_cast<const T*>(a.w_up) + static_cast<size_t>(h) * a.DN * a.KC + d0;
+  for (int r = 0; r < kLatRows; ++r) acc[r][0] = acc[r][1] = acc[r][2] = acc[r][3] = 0.f;
+  const T* wp = static_cast<const T*>(a.w_up) + static_cast<size_t>(h) * a.DN * a.KC + (live ? d0 : 0);
 #pragma unroll 8
   for (int c = n0; c < n1; ++c) {
-    const float2 w = ld_elem2(wp + static_cast<size_t>(c) * a.KC);
+    const float4 w = ld_elem4(wp + static_cast<size_t>(c) * a.KC);
+    const float4 qa = *reinterpret_cast<const float4*>(qs + c * kLatRows), qb = *reinterpret_cast<const float4*>(qs + c * kLatRows + 4);
+    const float q[kLatRows] = {qa.x, qa.y, qa.z, qa.w, qb.x, qb.y, qb.z, qb.w};
 #pragma unroll
     for (int r = 0; r < kLatRows; ++r) {
-      const float q = qs[r * a.dim + c];
-      acc[r][0] = fmaf(q, w.x, acc[r][0]);
-      acc[r][1] = fmaf(q, w.y, acc[r][1]);
+      acc[r][0] = fmaf(q[r], w.x, acc[r][0]);
+      acc[r][1] = fmaf(q[r], w.y, acc[r][1]);
+      acc[r][2] = fmaf(q[r], w.z, acc[r][2]);
+      acc[r][3] = fmaf(q[r], w.w, acc[r][3]);
     }
   }
 #pragma unroll
   for (int r = 0; r < kLatRows; ++r)
-    *reinterpret_cast<float2*>(part + (warp * kLatRows + r) * 64 + lane * 2) = make_float2(acc[r][0], acc[r][1]);
+    *reinterpret_cast<float4*>(part + (warp * kLatRows + r) * 128 + lane * 4) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
   __syncthreads();
   const int D = a.KC + a.RP;
-  for (int i = tid; i < nr * 64; i += 256) {
-    const int r = i / 64, d = i % 64;
-    float sum = 0.f;
+  {
+    const int r = warp, d = lane * 4;                     // 8 warps = 8 rows
+    if (r < nr && live) {
+      float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int w = 0; w < 8; ++w) sum += part[(w * kLatRows + r) * 64 + d];
-    a.q_abs[(static_cast<size_t>(r0 + r) * a.heads + h) * D + blockIdx.z * 64 + d] = sum;
+      for (int w = 0; w < 8; ++w) {
+        const float4 v = *reinterpret_cast<const float4*>(part + (w * kLatRows + r) * 128 + d);
+        sum.x += v.x; sum.y += v.y; sum.z += v.z; sum.w += v.w;
+      }
+      *reinterpret_cast<float4*>(a.q_abs + (static_cast<size_t>(r0 + r) * a.heads + h) * D + d0) = sum;
+    }
   }
   if (blockIdx.z != 0) return;
   for (int i = tid; i < nr * (a.RP / 2); i += 256) {
@@ -240,45 +249,60 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(LatentRowsArgs a) {
     if (lane + 32 * j < a.KC) a.out[(static_cast<size_t>(i0) * a.heads + h) * a.KC + lane + 32 * j] = acc[j] / l;
 }
 
-// grid (heads, ceil(n / 8), ceil(DV / 16)), 256 threads: a CTA owns 16 outputs of one head for up to 8 rows; 16 lanes share an
-// output and take its 16-byte chunks in turns.
+constexpr int kUpOut = 4;        // outputs of a lane
+
+// grid (heads, ceil(n / 8), ceil(DV / 64)), 256 threads: a CTA owns 64 outputs of one head for up to 8 rows.  Sixteen lanes take the
+// 16-byte chunks of four weight rows in turns, so a value read from shared memory meets four weights.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_up_kernel(const float* __restrict__ lat, const T* __restrict__ w, const T* __restrict__ gate,
                                                         int64_t gate_stride, const int32_t* __restrict__ row_list, T* __restrict__ out,
                                                         int64_t out_stride, int n, int heads, int DV, int KC) {
-  constexpr int VN = Vec16<T>::N;
-  extern __shared__ float lu_smem[];                       // [8][chunks][VN + 1]
+  constexpr int VN = Vec16<T>::N, CS = VN + 4;             // a chunk of VN values takes CS words: 16-byte reads without bank conflicts
+  extern __shared__ __align__(16) float lu_smem[];         // [8][chunks][CS]
   pdl_wait();
   const int h = blockIdx.x, r0 = blockIdx.y * kLatRows, tid = threadIdx.x, nr = min(kLatRows, n - r0), chunks = KC / VN;
-  for (int i = tid; i < kLatRows * KC; i += 256) {
-    const int r = i / KC, d = i % KC;
-    lu_smem[(r * chunks + d / VN) * (VN + 1) + d % VN] = r < nr ? lat[(static_cast<size_t>(r0 + r) * heads + h) * KC + d] : 0.f;
+  const int warp = tid >> 5, lane = tid & 31, g = lane & 15;
+  {
+    const int r = warp;                                    // 8 warps = 8 rows
+    const float* src = lat + (static_cast<size_t>(r0 + min(r, nr - 1)) * heads + h) * KC;
+    for (int d = lane * 4; d < KC; d += 128)
+      *reinterpret_cast<float4*>(lu_smem + (r * chunks + d / VN) * CS + d % VN) = r < nr ? *reinterpret_cast<const float4*>(src + d) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   __syncthreads();
-  const int warp = tid >> 5, lane = tid & 31, g = lane & 15, v = blockIdx.z * 16 + warp * 2 + (lane >> 4);
-  const T* wp = w + (static_cast<size_t>(h) * DV + min(v, DV - 1)) * KC;
-  float acc[kLatRows];
+  const int v0 = blockIdx.z * 64 + (warp * 2 + (lane >> 4)) * kUpOut;
+  const T* wp = w + static_cast<size_t>(h) * DV * KC;
+  float acc[kUpOut][kLatRows];
 #pragma unroll
-  for (int r = 0; r < kLatRows; ++r) acc[r] = 0.f;
-#pragma unroll 4
+  for (int o = 0; o < kUpOut; ++o)
+#pragma unroll
+    for (int r = 0; r < kLatRows; ++r) acc[o][r] = 0.f;
   for (int c = g; c < chunks; c += 16) {
-    float f[VN];
-    Vec16<T>::load(wp + c * VN, f);
+    float f[kUpOut][VN];
 #pragma unroll
-    for (int j = 0; j < VN; ++j)
+    for (int o = 0; o < kUpOut; ++o) Vec16<T>::load(wp + static_cast<size_t>(min(v0 + o, DV - 1)) * KC + c * VN, f[o]);
 #pragma unroll
-      for (int r = 0; r < kLatRows; ++r) acc[r] = fmaf(lu_smem[(r * chunks + c) * (VN + 1) + j], f[j], acc[r]);
-  }
+    for (int r = 0; r < kLatRows; ++r) {
 #pragma unroll
-  for (int r = 0; r < kLatRows; ++r) {
-    float s = acc[r];
+      for (int j = 0; j < VN; j += 4) {
+        const float4 x = *reinterpret_cast<const float4*>(lu_smem + (r * chunks + c) * CS + j);
 #pragma unroll
-    for (int o = 8; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-    if (g == 0 && v < DV && r < nr) {
-      const size_t row = row_list != nullptr ? row_list[r0 + r] : r0 + r;
-      st_elem(out + row * out_stride + static_cast<size_t>(h) * DV + v, s * sigmoid_f32(ld_elem(gate + row * gate_stride + h)));
+        for (int o = 0; o < kUpOut; ++o)
+          acc[o][r] = fmaf(x.w, f[o][j + 3], fmaf(x.z, f[o][j + 2], fmaf(x.y, f[o][j + 1], fmaf(x.x, f[o][j], acc[o][r]))));
+      }
     }
   }
+#pragma unroll
+  for (int o = 0; o < kUpOut; ++o)
+#pragma unroll
+    for (int r = 0; r < kLatRows; ++r) {
+      float s = acc[o][r];
+#pragma unroll
+      for (int k = 8; k > 0; k >>= 1) s += __shfl_xor_sync(0xffffffffu, s, k);
+      if (g == r && v0 + o < DV && r < nr) {               // lane r of the sixteen finishes row r
+        const size_t row = row_list != nullptr ? row_list[r0 + r] : r0 + r;
+        st_elem(out + row * out_stride + static_cast<size_t>(h) * DV + v0 + o, s * sigmoid_f32(ld_elem(gate + row * gate_stride + h)));
+      }
+    }
 }
 
 // grid (pages), 256 threads
@@ -340,12 +364,12 @@ DGPP_API int dgpp_latent_absorb(void* proj, int64_t stride, int q_off, int kv_of
   DGPP_REQUIRE(dim <= 1024, "latent_absorb: heads of %d columns (at most 1024)", dim);
   if (n == 0) return 0;
   a.row_list = static_cast<const int32_t*>(row_list); a.w_up = w_up; a.q_abs = static_cast<float*>(q_abs); a.fused = fused;
-  const dim3 grid(heads + (fused ? 1 : 0), dgpp_ceil_div(n, kLatRows), KC / 64);
-  const size_t smem = static_cast<size_t>(kLatRows * dim + 8 * kLatRows * 64 + 2) * sizeof(float);
+  const dim3 grid(heads + (fused ? 1 : 0), dgpp_ceil_div(n, kLatRows), dgpp_ceil_div(KC, 128));
+  const size_t smem = static_cast<size_t>(kLatRows * dim + 8 * kLatRows * 128) * sizeof(float);
   static bool attr = false;
   if (!attr) {
-    DGPP_CUDA_OK(cudaFuncSetAttribute(latent_absorb_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
-    DGPP_CUDA_OK(cudaFuncSetAttribute(latent_absorb_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(latent_absorb_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(latent_absorb_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
     attr = true;
   }
   if (f32) latent_absorb_kernel<float><<<grid, 256, smem, st>>>(a);
@@ -396,9 +420,15 @@ DGPP_API int dgpp_latent_up(const void* lat, const void* w, const void* gate, in
                             int64_t out_stride, int n, int heads, int DV, int KC, int f32, cudaStream_t st) {
   DGPP_REQUIRE(KC % 64 == 0 && KC <= 1024 && DV >= 1, "latent_up: %d columns from %d", DV, KC);
   if (n == 0) return 0;
-  const dim3 grid(heads, dgpp_ceil_div(n, kLatRows), dgpp_ceil_div(DV, 16));
+  const dim3 grid(heads, dgpp_ceil_div(n, kLatRows), dgpp_ceil_div(DV, 64));
   const int vn = f32 ? 4 : 8;
-  const size_t smem = static_cast<size_t>(kLatRows) * (KC / vn) * (vn + 1) * sizeof(float);
+  const size_t smem = static_cast<size_t>(kLatRows) * (KC / vn) * (vn + 4) * sizeof(float);
+  static bool attr = false;
+  if (!attr) {
+    DGPP_CUDA_OK(cudaFuncSetAttribute(latent_up_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(latent_up_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
+    attr = true;
+  }
   const float* lp = static_cast<const float*>(lat);
   const int32_t* rl = static_cast<const int32_t*>(row_list);
   if (f32) latent_up_kernel<float><<<grid, 256, smem, st>>>(lp, static_cast<const float*>(w), static_cast<const float*>(gate), gate_stride, rl, static_cast<float*>(out), out_stride, n, heads, DV, KC);

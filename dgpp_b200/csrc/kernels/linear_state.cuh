@@ -13,7 +13,8 @@
 //
 //   lin_decode   runs of one token: convolution, norms, gates, state update and read-out of a (row, head) in one CTA with
 //                the whole S in registers; the delta rule's output norm and gate are fused in as well
-//   lin_prep     token-parallel part of longer runs -> fp32 scratch (unit q / k, v, decays, strengths)
+//   lin_prep     token-parallel part of longer runs -> fp32 scratch (unit q / k, v, decays, strengths); ssd_prep: the same for the
+//                state-space rule, convolution windows in registers
 //   lin_block    16-token blocks in parallel: the block's decay products and token-pair matrices (ssd_block: the same for the
 //                state-space rule, whose scalar decays leave q and k as they are, shared by a group of heads)
 //   lin_scan     block-sequential part: one CTA per (32 state columns, head, run), S in registers, the next block's operands
@@ -463,6 +464,56 @@ __global__ void __launch_bounds__(256) lin_block_kernel(LinearArgs a) {
   }
 }
 
+// The state-space rule's lin_prep for convolutions of up to four taps: a thread owns four channels of a 16-token block and slides the
+// window along in registers.  grid (ceil(C / 512) + 1, blocks), 128 threads; the last column of CTAs makes steps and decays.
+template <typename T, int DK, int DV, int TAPS>
+__global__ void __launch_bounds__(128) ssd_prep_kernel(LinearArgs a) {
+  pdl_wait();
+  int row0 = 0, n = 0;
+  if (!find_block(a, blockIdx.y, row0, n)) return;
+  const PrepView pv = prep_view<DK, DV, kStateSpace>(a);
+  const T* proj = static_cast<const T*>(a.proj) + static_cast<size_t>(row0) * a.stride;
+  if (blockIdx.x == gridDim.x - 1) {
+    for (int i = threadIdx.x; i < n * a.hv; i += 128) {
+      const int t = i / a.hv, h = i % a.hv;
+      const float dt = softplus_f32(ld_elem(proj + t * a.stride + a.b_off + h) + a.dt_bias[h]);
+      pv.b[static_cast<size_t>(row0) * a.hv + i] = dt;
+      pv.g[static_cast<size_t>(row0) * a.hv + i] = expf(-expf(a.A_log[h]) * dt);
+    }
+    return;
+  }
+  const int nk = a.hk * DK, C = 2 * nk + a.hv * DV, ch = (blockIdx.x * 128 + threadIdx.x) * 4;
+  if (ch >= C) return;
+  const int pos = a.positions[row0], back = row0 - a.row_run0[row0];
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  const T* x = proj + a.c_off + ch;
+  const float* ring = a.ring + static_cast<size_t>(a.row_slot[row0]) * TAPS * C + ch;
+  float4 w[TAPS], h[TAPS];                                 // h[j]: the input j tokens back
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) {
+    w[j] = ld_elem4(a.conv_w + static_cast<size_t>(TAPS - 1 - j) * C + ch);
+    h[j] = zero;
+    if (j >= 1 && j <= pos) h[j] = j <= back ? ld_elem4(x - j * a.stride) : ld_elem4(ring + static_cast<size_t>((pos - j) % TAPS) * C);
+  }
+  const float4 bias = a.conv_b != nullptr ? ld_elem4(a.conv_b + ch) : zero;
+  float* dst = ch < nk ? pv.q + static_cast<size_t>(row0) * nk + ch
+                       : (ch < 2 * nk ? pv.k + static_cast<size_t>(row0) * nk + ch - nk : pv.v + static_cast<size_t>(row0) * a.hv * DV + ch - 2 * nk);
+  const int step = ch < 2 * nk ? nk : a.hv * DV;
+#pragma unroll 4
+  for (int t = 0; t < n; ++t) {
+    h[0] = ld_elem4(x + t * a.stride);
+    float4 acc = bias;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      acc.x = fmaf(w[j].x, h[j].x, acc.x); acc.y = fmaf(w[j].y, h[j].y, acc.y);
+      acc.z = fmaf(w[j].z, h[j].z, acc.z); acc.w = fmaf(w[j].w, h[j].w, acc.w);
+    }
+    *reinterpret_cast<float4*>(dst + static_cast<size_t>(t) * step) = make_float4(silu_f32(acc.x), silu_f32(acc.y), silu_f32(acc.z), silu_f32(acc.w));
+#pragma unroll
+    for (int j = TAPS - 1; j > 0; --j) h[j] = h[j - 1];
+  }
+}
+
 constexpr int kSsdHeads = 8;
 
 // grid (hk * ceil(heads per group / 8), blocks), 256 threads: thread (t, s) holds q_t . k_s and walks up to 8 heads of the group.
@@ -725,7 +776,17 @@ static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
     DGPP_CUDA_OK(cudaFuncSetAttribute(lin_scan_kernel<DK, DV, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     attr = true;
   }
-  lin_prep_kernel<T, DK, DV, RULE><<<dgpp_ceil_div(a.rows * (a.hk + a.hv), 8), 256, 0, st>>>(a);
+  bool prepared = false;
+  if constexpr (RULE == kStateSpace) {
+    const dim3 grid(dgpp_ceil_div(2 * a.hk * DK + a.hv * DV, 512) + 1, a.blocks);
+    prepared = a.taps <= 4 && a.stride % 4 == 0 && a.c_off % 4 == 0;
+    if (!prepared) {}
+    else if (a.taps == 1) ssd_prep_kernel<T, DK, DV, 1><<<grid, 128, 0, st>>>(a);
+    else if (a.taps == 2) ssd_prep_kernel<T, DK, DV, 2><<<grid, 128, 0, st>>>(a);
+    else if (a.taps == 3) ssd_prep_kernel<T, DK, DV, 3><<<grid, 128, 0, st>>>(a);
+    else ssd_prep_kernel<T, DK, DV, 4><<<grid, 128, 0, st>>>(a);
+  }
+  if (!prepared) lin_prep_kernel<T, DK, DV, RULE><<<dgpp_ceil_div(a.rows * (a.hk + a.hv), 8), 256, 0, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   if constexpr (RULE == kStateSpace) ssd_block_kernel<DK, DV><<<dim3(a.hk * dgpp_ceil_div(a.hv / a.hk, kSsdHeads), a.blocks), 256, 0, st>>>(a);
   else lin_block_kernel<DK, DV, RULE><<<dim3(a.hv, a.blocks), 256, bsmem, st>>>(a);

@@ -264,18 +264,20 @@ clamped_glu_kernel(const TI* __restrict__ gate_up, int64_t stride, const float* 
   pdl_wait();
   const size_t row = blockIdx.y;
   if (tiles != nullptr && tiles[row / bn] < 0) return;
-  const int i = (blockIdx.x * kStreamThreads + threadIdx.x) * 4;
+  const int i = (blockIdx.x * kStreamThreads + threadIdx.x) * 8;
   if (i >= inter) return;
   const float s = row_w != nullptr ? row_w[row] : 1.f;
-  const float4 g4 = ld_elem4(gate_up + row * stride + i), u4 = ld_elem4(gate_up + row * stride + inter + i);
-  const float gi[4] = {g4.x, g4.y, g4.z, g4.w}, ui[4] = {u4.x, u4.y, u4.z, u4.w};
-  float o[4];
+  const TI* gp = gate_up + row * stride + i;
+  float g[8], u[8];
+  ld_elem8(gp, g);
+  ld_elem8(gp + inter, u);
 #pragma unroll
-  for (int e = 0; e < 4; ++e) {
-    const float g = fminf(gi[e] * s, limit), u = fminf(fmaxf(ui[e] * s, -limit), limit);
-    o[e] = g * sigmoid_f32(alpha * g) * (u + 1.f);
+  for (int e = 0; e < 8; ++e) {
+    const float a = fminf(g[e] * s, limit), b = fminf(fmaxf(u[e] * s, -limit), limit);
+    const float sg = sizeof(T) == 4 ? sigmoid_f32(alpha * a) : __fdividef(1.f, 1.f + __expf(-alpha * a));
+    g[e] = a * sg * (b + 1.f);
   }
-  st_elem4(out + row * inter + i, make_float4(o[0], o[1], o[2], o[3]));
+  st_elem8(out + row * inter + i, g);
 }
 
 template <typename T>
@@ -402,10 +404,10 @@ DGPP_API int dgpp_gated_part_norm(const void* y, const void* z, int64_t z_stride
 // in_f32: gate_up is fp32 although the output is bf16.
 DGPP_API int dgpp_clamped_glu(const void* gate_up, int64_t stride, const void* row_w, const void* tiles, int bn, void* out, int rows, int inter,
                               float limit, float alpha, int f32, int in_f32, cudaStream_t st) {
-  DGPP_REQUIRE(inter % 8 == 0 && stride % 4 == 0 && bn >= 1, "clamped_glu: width %d (a multiple of 8)", inter);
+  DGPP_REQUIRE(inter % 8 == 0 && stride % 8 == 0 && bn >= 1, "clamped_glu: width %d (a multiple of 8)", inter);
   if (rows == 0) return 0;
   DGPP_REQUIRE(rows <= 65535, "clamped_glu: %d rows", rows);
-  const dim3 grid(dgpp_ceil_div(inter / 4, kStreamThreads), rows);
+  const dim3 grid(dgpp_ceil_div(inter / 8, kStreamThreads), rows);
   const float* rw = static_cast<const float*>(row_w);
   const int32_t* tl = static_cast<const int32_t*>(tiles);
 #define DGPP_CG(TI, TT) clamped_glu_kernel<TI, TT><<<grid, kStreamThreads, 0, st>>>(static_cast<const TI*>(gate_up), stride, rw, tl, bn, \

@@ -555,10 +555,7 @@ class PotivikRunner(RowRunner):
     def _absorbed(self, g: mx.LatentHeads, proj, mixed, positions, row_req, cache, rows: int, row_list, fused: bool) -> None:
         bt, page = self.kv.block_table, self.c.page
         mx.latent_absorb(g, proj, positions, row_req, bt, cache, page, self.q_abs, rows, row_list, fused)
-        tiles = -(-(min(g.window, self.max_span) + 127) // 128)
-        splits = 1
-        if rows <= self.slots:
-            splits = max(1, min(self.max_splits, tiles, -(-148 // (rows * -(-g.heads // 16)))))
+        splits = mx.latent_splits(rows, g.heads, min(g.window, self.max_span), self.max_splits) if rows <= self.slots else 1
         mx.latent_attn(g, self.q_abs, cache, bt, row_req, positions, page, self.lat, rows, row_list, splits, self.scratch)
         mx.latent_up(g, self.lat, proj, mixed, rows, row_list)
 

@@ -357,6 +357,14 @@ def latent_absorb(g: LatentHeads, proj, positions, row_req, block_table, cache, 
     return q_abs
 
 
+def latent_splits(rows: int, heads: int, span: int, most: int, sms: int = 148) -> int:
+    """Window splits of single rows: the fewest that finish soonest, counting 128-token tiles one after the other per CTA, one CTA
+    per SM at a time, and a tile's time for the merge of the splits."""
+    tiles, units = -(-(span + 127) // 128), rows * -(-heads // 16)
+    cost = lambda s: -(-units * s // sms) * -(-tiles // s) + (s > 1)
+    return min(range(1, max(1, min(most, tiles)) + 1), key=cost)
+
+
 def latent_attn(g: LatentHeads, q_abs, cache, block_table, row_req, positions, page: int, lat, rows: int, row_list=None, splits: int = 1,
                 scratch=None) -> torch.Tensor:
     """Windowed attention of absorbed rows -> lat [rows, heads, KC] fp32; on the tensor cores where the kernel takes the widths."""
