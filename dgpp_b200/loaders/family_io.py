@@ -19,6 +19,7 @@ from typing import Any, Callable, Dict, Iterator, Tuple
 import torch
 
 from ..quant.formats import QuantLinear
+from . import PUBLISHED
 from .checkpoint import open_checkpoint, write_safetensors
 
 
@@ -81,9 +82,6 @@ def published(family: str):
         from ..models import potivik as m
         return m.PotivikConfig, m.PotivikModel, m.PotivikRunner, m.tensor_shapes, m.random_tensors
     return None
-
-
-PUBLISHED = ("sitirax", "potivik")
 
 
 def load_published(ck, device="cuda", dtype: torch.dtype = torch.bfloat16) -> Any:

@@ -73,7 +73,7 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", type=int, required=True)
     a = ap.parse_args(argv)
     from .. import build
-    from ..loaders.family_io import PUBLISHED
+    from ..loaders import PUBLISHED
 
     with open(os.path.join(a.model, "config.json")) as f:
         cfg = json.load(f)
