@@ -40,6 +40,8 @@ KERNEL_SETS = {
     "sitirax": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "window_attn", "window_attn_tc", "linear_state", "graph_exec"],
     "potivik": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "moe", "moe_prefill", "moe_rows", "latent_attn", "mla_tc", "window_attn_tc",
                 "state_space", "graph_exec"],
+    "vevapel": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "moe", "moe_prefill", "moe_rows", "window_attn", "window_attn_tc",
+                "gated_delta", "graph_exec"],
 }
 # Translation units that must not contract a*b+c into fma (sampler parity with the host oracle).
 NO_FMA = {"sample.cu"}

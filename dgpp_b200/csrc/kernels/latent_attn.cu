@@ -12,13 +12,14 @@
 //   latent_up       out[row, head] = W_uv lat[row, head] * sigmoid(gate[row, head])
 //   latent_gather   pages of the cache into consecutive rows (the input of the up-projection that expands a prompt's keys)
 //
-// Angles: position * f as an fp32 product plus its rounding error (f itself in two terms), so far positions lose nothing.
+// Angles: common/rope.cuh.
 #include <math.h>
 
 #include "common/common.h"
 #include "common/dtypes.cuh"
 #include "common/elem.cuh"
 #include "common/ptx.cuh"
+#include "common/rope.cuh"
 
 namespace dgpp {
 
@@ -39,15 +40,6 @@ struct LatentArgs {
   float eps;
 };
 
-__device__ __forceinline__ void latent_angle(const LatentArgs& a, int pos, int i, float& s, float& c) {
-  const float p = static_cast<float>(pos), hi = a.freq[i], ang = p * hi;
-  const float err = fmaf(p, hi, -ang) + p * a.freq[a.rot / 2 + i];
-  float s0, c0;
-  sincosf(ang, &s0, &c0);
-  s = fmaf(c0, err, s0);
-  c = fmaf(-s0, err, c0);
-}
-
 // One warp: the cache row of one token.
 template <typename T>
 __device__ __forceinline__ void latent_cache_row(const LatentArgs& a, int row, int lane) {
@@ -67,7 +59,7 @@ __device__ __forceinline__ void latent_cache_row(const LatentArgs& a, int row, i
     float u = ld_elem(kr + 2 * i), v = ld_elem(kr + 2 * i + 1);
     if (2 * i < a.rot) {
       float s, c;
-      latent_angle(a, pos, i, s, c);
+      rope_angle(a.freq, a.rot / 2, pos, i, s, c);
       const float t = u * c - v * s;
       v = v * c + u * s;
       u = t;
@@ -83,7 +75,7 @@ __global__ void __launch_bounds__(256) latent_append_kernel(LatentArgs a) {
   extern __shared__ float la_cs[];                        // [rot / 2][2]
   pdl_wait();
   const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int i = threadIdx.x; i < a.rot / 2; i += 256) latent_angle(a, a.positions[row], i, la_cs[2 * i], la_cs[2 * i + 1]);
+  for (int i = threadIdx.x; i < a.rot / 2; i += 256) rope_angle(a.freq, a.rot / 2, a.positions[row], i, la_cs[2 * i], la_cs[2 * i + 1]);
   __syncthreads();
   if (warp == 0) latent_cache_row<T>(a, row, lane);
   T* q = static_cast<T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.q_off;
@@ -166,7 +158,7 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a) {
     float u = ld_elem(qr), v = ld_elem(qr + 1);
     if (a.fused && 2 * j < a.rot) {
       float s, c;
-      latent_angle(a, a.positions[row], j, s, c);
+      rope_angle(a.freq, a.rot / 2, a.positions[row], j, s, c);
       const float t = u * c - v * s;
       v = v * c + u * s;
       u = t;

@@ -3,20 +3,23 @@
 //   channel delta rule   S <- g_t * S (a decay per key channel);  u = b_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
 //                        q, k, v pass a causal depthwise convolution and silu, q and k become unit vectors, q is scaled;
 //                        g_t = exp(-exp(A) softplus(a_t + dt)),  b_t = sigmoid(beta_t)
+//   scalar delta rule    the same with one decay per token and head, g_t = exp(-exp(A_h) softplus(a_t + dt_h)); its output gate is a
+//                        silu of plain columns of the projection
 //   lightning            S <- d_h * S + k_t v_t^T (a constant decay per head);  o_t = S^T q_t;  q, k, v = silu(projection)
 //   state space          S <- a_t S + dt_t k_t v_t^T (a decay per token and head);  o_t = S^T q_t + D_h v_t
 //                        q, k (shared by groups of heads), v pass a causal depthwise convolution with bias and silu;
 //                        dt_t = softplus(raw step + bias),  a_t = exp(-exp(A) dt_t)
 //
-// All are one kernel family (template parameter RULE; linear_state.cu and state_space.cu hold the entry points).  A pass carries runs of consecutive tokens of any number of requests:
+// All are one kernel family (template parameter RULE; linear_state.cu, state_space.cu and gated_delta.cu hold the entry points).  A pass
+// carries runs of consecutive tokens of any number of requests:
 // run r = rows [run_start[r], run_start[r + 1]) of the request in state slot row_slot[first row].
 //
 //   lin_decode   runs of one token: convolution, norms, gates, state update and read-out of a (row, head) in one CTA with
 //                the whole S in registers; the delta rule's output norm and gate are fused in as well
 //   lin_prep     token-parallel part of longer runs -> fp32 scratch (unit q / k, v, decays, strengths); ssd_prep: the same for the
-//                state-space rule, convolution windows in registers
-//   lin_block    16-token blocks in parallel: the block's decay products and token-pair matrices (ssd_block: the same for the
-//                state-space rule, whose scalar decays leave q and k as they are, shared by a group of heads)
+//                rules with scalar decays, convolution windows in registers
+//   lin_block    16-token blocks in parallel: the block's decay products and token-pair matrices (ssd_block, gated_block:
+//                the same for scalar decays, which leave q and k as they are, shared by a group of heads)
 //   lin_scan     block-sequential part: one CTA per (32 state columns, head, run), S in registers, the next block's operands
 //                streaming in with cp.async while the current one is consumed
 //   lin_tail     the newest inputs of the convolution go to the request's ring after every reader is done
@@ -36,19 +39,23 @@
 
 namespace dgpp {
 
-enum LinearRule { kLightning = 0, kDelta = 1, kStateSpace = 2 };
+enum LinearRule { kLightning = 0, kDelta = 1, kStateSpace = 2, kScalarDelta = 3 };
+
+__host__ __device__ constexpr bool is_delta(int rule) { return rule == kDelta || rule == kScalarDelta; }
+__host__ __device__ constexpr bool scalar_decay(int rule) { return rule == kStateSpace || rule == kScalarDelta; }
 
 struct LinearArgs {
   const void* proj;         // [rows, stride] (T): conv channels q (hk * DK) | k (hk * DK) | v (hv * DV) from column c_off
   int64_t stride;
   int c_off, b_off;         // b_off: raw write strengths (delta) or raw step sizes (state space) [hv]
+  int a_off, g_off;         // raw decays [hv], raw output gates [hv * DV] (scalar delta)
   const float* low;         // [rows, low_stride] fp32: raw decays [hv * DK], then raw output gates [hv * DV] (delta)
   int64_t low_stride;
   const float* conv_w;      // [taps, C] (last row: the current token); null: no convolution
   const float* conv_b;      // [C] or null
   float* ring;              // [slots, taps, C]
   const float* A_log;       // [hv]
-  const float* dt_bias;     // [hv * DK] (delta), [hv] (state space)
+  const float* dt_bias;     // [hv * DK] (channel delta), [hv] (state space, scalar delta)
   const float* skip;        // [hv] D (state space)
   const float* decay;       // [hv] (lightning)
   float* state;             // [slots, hv, DK, DV]
@@ -118,7 +125,7 @@ __device__ __forceinline__ float4 fma4(float4 s, float a, float4 acc) {
 // grid (hv, rows)
 template <typename T, int DK, int DV, int RULE>
 __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(LinearArgs a) {
-  constexpr bool DELTA = RULE == kDelta, SSD = RULE == kStateSpace;
+  constexpr bool DELTA = is_delta(RULE), CH = RULE == kDelta, SSD = RULE == kStateSpace;
   using G = LinGeom<DK, DV>;
   constexpr int NT = G::kThreads, PER = G::kPer, PARTS = G::kParts;
   extern __shared__ __align__(16) float ld_smem[];
@@ -160,13 +167,17 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
     beta = softplus_f32(ld_elem(static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.b_off + h) + a.dt_bias[h]);
     dh = expf(-expf(a.A_log[h]) * beta);
     skip = a.skip[h];
-  } else if (!DELTA) {
+  } else if (RULE == kLightning) {
     dh = a.decay[h];
   }
   if (DELTA) {
     const float ea = -expf(a.A_log[h]);
-    const float* ar = a.low + static_cast<size_t>(row) * a.low_stride + h * DK;
-    for (int c = tid; c < DK; c += NT) gs[c] = expf(ea * softplus_f32(ar[c] + a.dt_bias[h * DK + c]));
+    if (CH) {
+      const float* ar = a.low + static_cast<size_t>(row) * a.low_stride + h * DK;
+      for (int c = tid; c < DK; c += NT) gs[c] = expf(ea * softplus_f32(ar[c] + a.dt_bias[h * DK + c]));
+    } else {
+      dh = expf(ea * softplus_f32(ld_elem(static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.a_off + h) + a.dt_bias[h]));
+    }
     beta = sigmoid_f32(ld_elem(static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.b_off + h));
   }
   __syncthreads();
@@ -185,7 +196,7 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int r = part + PARTS * i;
-    const float g = DELTA ? gs[r] : dh;
+    const float g = CH ? gs[r] : dh;
     s[i].x *= g; s[i].y *= g; s[i].z *= g; s[i].w *= g;
     n4 = fma4(s[i], qs[r], n4);
     if (DELTA) m4 = fma4(s[i], ks[r], m4);
@@ -219,34 +230,42 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
   }
   if (DELTA) {
     const float r = 1.f / sqrtf(block_sum_f32(ss, scratch) / static_cast<float>(a.vdim) + a.eps);
-    const float* gt = a.low + static_cast<size_t>(row) * a.low_stride + a.hv * DK + h * DV;
     T* dst = static_cast<T*>(a.out) + static_cast<size_t>(row) * a.out_stride + h * DV;
-    for (int c = tid; c < DV; c += NT) st_elem(dst + c, vs[c] * r * a.norm_w[c] * sigmoid_f32(gt[c]));
+    if (CH) {
+      const float* gt = a.low + static_cast<size_t>(row) * a.low_stride + a.hv * DK + h * DV;
+      for (int c = tid; c < DV; c += NT) st_elem(dst + c, vs[c] * r * a.norm_w[c] * sigmoid_f32(gt[c]));
+    } else {
+      const T* gt = static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.g_off + h * DV;
+      for (int c = tid; c < DV; c += NT) st_elem(dst + c, vs[c] * r * a.norm_w[c] * silu_f32(ld_elem(gt + c)));
+    }
   }
 }
 
 // Scratch of a pass over runs (fp32): per row q, k [hk, DK], v [hv, DV], decays [hv, DK] (delta; lin_block replaces them by
 // K * gamma), Q * gamma and the suffix-weighted keys [hv, DK]; per block gamma_16 [hv, DK], P and (delta) T B [hv, 16, 16]; the
 // strengths [rows, hv] (delta) at the end.  State space: per row q, k, v, decay and step [hv] each; per block and head P with the
-// steps and the skip folded in [16, 16] and 16 prefix products, then 16 write weights.
+// steps and the skip folded in [16, 16] and 16 prefix products, then 16 write weights.  Scalar delta: per row q, k (not yet unit
+// vectors), v, decay and strength; per block and head P and T B [16, 16], then 16 factors each of Q S, of the writes and of K S, and
+// gamma_16; the lengths of q and k ride in all of these.
 struct PrepView {
   float *q, *k, *v, *g, *kt, *qt, *kh, *gam, *pm, *tb, *b;
 };
 template <int DK, int DV, int RULE>
 __device__ __forceinline__ PrepView prep_view(const LinearArgs& a) {
-  constexpr bool DELTA = RULE == kDelta;
+  constexpr bool DELTA = RULE == kDelta;              // (the scalar rule has its own layout)
   PrepView p;
   const size_t R = a.rows, B = a.blocks;
   p.q = a.prep;
   p.k = p.q + R * a.hk * DK;
   p.v = p.k + R * a.hk * DK;
   p.g = p.v + R * a.hv * DV;
-  if (RULE == kStateSpace) {
+  if (scalar_decay(RULE)) {
     p.pm = p.g;
-    p.gam = p.pm + B * a.hv * 256;
-    p.g = p.gam + B * a.hv * 32;
+    p.tb = p.pm + B * a.hv * 256;
+    p.gam = RULE == kScalarDelta ? p.tb + B * a.hv * 256 : p.tb;
+    p.g = p.gam + B * a.hv * (RULE == kScalarDelta ? 64 : 32);
     p.b = p.g + R * a.hv;
-    p.kt = p.qt = p.kh = p.tb = nullptr;
+    p.kt = p.qt = p.kh = nullptr;
     return p;
   }
   p.kt = p.g;
@@ -304,6 +323,11 @@ __global__ void __launch_bounds__(256) lin_prep_kernel(LinearArgs a) {
     pv.b[rh] = dt;
     pv.g[rh] = expf(-expf(a.A_log[h]) * dt);
   }
+  if (RULE == kScalarDelta && lane == 0) {
+    const T* x = static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + h;
+    pv.b[rh] = sigmoid_f32(ld_elem(x + a.b_off));
+    pv.g[rh] = expf(-expf(a.A_log[h]) * softplus_f32(ld_elem(x + a.a_off) + a.dt_bias[h]));
+  }
   if (DELTA) {
     const float ea = -expf(a.A_log[h]);
     const float* ar = a.low + static_cast<size_t>(row) * a.low_stride + h * DK + lane;
@@ -332,6 +356,7 @@ __global__ void __launch_bounds__(256) lin_tail_kernel(LinearArgs a, int C) {
 //     lightning  U = V
 //     O = (Q * gamma) S + P U,            P_ts = sum_c q_t k_s (g_(s+1) .. g_t)                                      (s <= t)
 //     S <- gamma_16 * S + (K * g_(t+1) .. g_16)^T U
+//     scalar     as delta, with gamma_t a number: gamma_t (K S) instead of (K * gamma) S
 //     state sp.  U = V,  P_ts = (q_t . k_s) (a_(s+1) .. a_t) dt_s + [s = t] D,  O = (a_1 .. a_t) (Q S) + P U,
 //                S <- (a_1 .. a_16) S + K^T (dt_s a_(s+1) .. a_16 U)
 // lin_block (parallel over blocks and heads) makes K * gamma, Q * gamma, the suffix-weighted keys, gamma_16, T B and P.
@@ -464,20 +489,20 @@ __global__ void __launch_bounds__(256) lin_block_kernel(LinearArgs a) {
   }
 }
 
-// The state-space rule's lin_prep for convolutions of up to four taps: a thread owns four channels of a 16-token block and slides the
-// window along in registers.  grid (ceil(C / 512) + 1, blocks), 128 threads; the last column of CTAs makes steps and decays.
-template <typename T, int DK, int DV, int TAPS>
+// lin_prep of the rules with scalar decays for convolutions of up to four taps: a thread owns four channels of a 16-token block and slides the
+// window along in registers.  grid (ceil(C / 512) + 1, blocks), 128 threads; the last column of CTAs makes steps (strengths) and decays.
+template <typename T, int DK, int DV, int RULE, int TAPS>
 __global__ void __launch_bounds__(128) ssd_prep_kernel(LinearArgs a) {
   pdl_wait();
   int row0 = 0, n = 0;
   if (!find_block(a, blockIdx.y, row0, n)) return;
-  const PrepView pv = prep_view<DK, DV, kStateSpace>(a);
+  const PrepView pv = prep_view<DK, DV, RULE>(a);
   const T* proj = static_cast<const T*>(a.proj) + static_cast<size_t>(row0) * a.stride;
   if (blockIdx.x == gridDim.x - 1) {
     for (int i = threadIdx.x; i < n * a.hv; i += 128) {
       const int t = i / a.hv, h = i % a.hv;
-      const float dt = softplus_f32(ld_elem(proj + t * a.stride + a.b_off + h) + a.dt_bias[h]);
-      pv.b[static_cast<size_t>(row0) * a.hv + i] = dt;
+      const float dt = softplus_f32(ld_elem(proj + t * a.stride + (RULE == kScalarDelta ? a.a_off : a.b_off) + h) + a.dt_bias[h]);
+      pv.b[static_cast<size_t>(row0) * a.hv + i] = RULE == kScalarDelta ? sigmoid_f32(ld_elem(proj + t * a.stride + a.b_off + h)) : dt;
       pv.g[static_cast<size_t>(row0) * a.hv + i] = expf(-expf(a.A_log[h]) * dt);
     }
     return;
@@ -570,19 +595,104 @@ __global__ void __launch_bounds__(256) ssd_block_kernel(LinearArgs a) {
   }
 }
 
+// The same for the scalar delta rule: thread (t, s) holds q_t . k_s and k_t . k_s of the raw vectors, whose lengths become factors;
+// (I + A)^-1 of up to 8 heads side by side, one lane per column.
+template <int DK, int DV>
+__global__ void __launch_bounds__(256) gated_block_kernel(LinearArgs a) {
+  __shared__ float ks[kBlk][DK + 1], qs[kBlk][DK + 1];
+  __shared__ float as[kSsdHeads][kBlk], bs[kSsdHeads][kBlk], rq[kBlk], rk[kBlk];
+  __shared__ float A[kSsdHeads][kBlk][kBlk + 1];
+  pdl_wait();
+  const int ratio = a.hv / a.hk, chunks = (ratio + kSsdHeads - 1) / kSsdHeads;
+  const int hk = blockIdx.x / chunks, h0 = hk * ratio + (blockIdx.x % chunks) * kSsdHeads;
+  const int nh = min(kSsdHeads, (hk + 1) * ratio - h0), blk = blockIdx.y, tid = threadIdx.x;
+  int row0 = 0, n = 0;
+  if (!find_block(a, blk, row0, n)) return;
+  const PrepView pv = prep_view<DK, DV, kScalarDelta>(a);
+  for (int i = tid; i < kBlk * DK; i += 256) {
+    const int t = i / DK, c = i % DK;
+    const size_t o = (static_cast<size_t>(row0 + t) * a.hk + hk) * DK + c;
+    ks[t][c] = t < n ? pv.k[o] : 0.f;
+    qs[t][c] = t < n ? pv.q[o] : 0.f;
+  }
+  for (int i = tid; i < nh * kBlk; i += 256) {
+    const int h = i / kBlk, t = i % kBlk;
+    const size_t o = static_cast<size_t>(row0 + t) * a.hv + h0 + h;
+    as[h][t] = t < n ? pv.g[o] : 1.f;
+    bs[h][t] = t < n ? pv.b[o] : 0.f;
+  }
+  __syncthreads();
+  for (int t = tid / 32; t < kBlk; t += 8) {
+    float q2 = 0.f, k2 = 0.f;
+    for (int c = tid & 31; c < DK; c += 32) {
+      q2 = fmaf(qs[t][c], qs[t][c], q2);
+      k2 = fmaf(ks[t][c], ks[t][c], k2);
+    }
+    q2 = warp_sum_f32(q2); k2 = warp_sum_f32(k2);
+    if ((tid & 31) == 0) { rq[t] = a.q_scale / sqrtf(q2 + 1e-6f); rk[t] = 1.f / sqrtf(k2 + 1e-6f); }
+  }
+  const int t = tid / kBlk, s = tid % kBlk;
+  float dq = 0.f, dk = 0.f;
+  if (s <= t) {
+#pragma unroll 8
+    for (int c = 0; c < DK; ++c) {
+      dq = fmaf(qs[t][c], ks[s][c], dq);
+      dk = fmaf(ks[t][c], ks[s][c], dk);
+    }
+  }
+  __syncthreads();
+  dq *= rq[t] * rk[s];
+  dk *= rk[t] * rk[s];
+  for (int h = 0; h < nh; ++h) {
+    const size_t bh = static_cast<size_t>(blk) * a.hv + h0 + h;
+    float w = 1.f;
+    if (s <= t)
+      for (int j = s + 1; j <= t; ++j) w *= as[h][j];
+    pv.pm[bh * kBlk * kBlk + tid] = s <= t ? dq * w : 0.f;
+    A[h][t][s] = s < t ? bs[h][t] * dk * w : 0.f;
+    if (tid < 4 * kBlk) {                                  // factors of Q S, of the writes, of K S; gamma_16
+      const int i = tid % kBlk, what = tid / kBlk;
+      float f = 1.f;
+      if (what == 1) {
+        for (int j = kBlk - 1; j > i; --j) f *= as[h][j];
+        f *= rk[i];
+      } else {
+        for (int j = 0; j <= (what == 3 ? kBlk - 1 : i); ++j) f *= as[h][j];
+        f *= what == 0 ? rq[i] : (what == 2 ? rk[i] : 1.f);
+      }
+      pv.gam[bh * 4 * kBlk + tid] = f;
+    }
+  }
+  __syncthreads();
+  if (tid < nh * kBlk) {
+    const int h = tid / kBlk, c = tid % kBlk;
+    float* tb = pv.tb + (static_cast<size_t>(blk) * a.hv + h0 + h) * kBlk * kBlk;
+    float col[kBlk];
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) {
+      float acc = i == c ? 1.f : 0.f;
+#pragma unroll
+      for (int j = 0; j < i; ++j) acc = fmaf(-A[h][i][j], col[j], acc);
+      col[i] = acc;
+      tb[i * kBlk + c] = acc * bs[h][c];
+    }
+  }
+}
+
 constexpr int kScanCols = 32;
 
-template <int DK, bool DELTA>
+template <int DK, int RULE>
 struct ScanGeom {
   static constexpr int kParts = DK >= 128 ? 32 : DK / 4;    // threads that share a column
   static constexpr int kThreads = kParts * (kScanCols / 4);
   static constexpr int kNI = DK / (4 * kParts);
   // floats of one staging buffer
   static constexpr int kQ = 0, kH = kBlk * DK, kK = 2 * kBlk * DK;
-  static constexpr int kV = kK + (DELTA ? kBlk * DK : 0);
+  static constexpr int kV = kK + (RULE == kDelta ? kBlk * DK : 0);
   static constexpr int kP = kV + kBlk * kScanCols, kT = kP + kBlk * kBlk;
-  static constexpr int kG = kT + (DELTA ? kBlk * kBlk : 0);
-  static constexpr int kTotal = kG + DK;
+  static constexpr int kG = kT + (is_delta(RULE) ? kBlk * kBlk : 0);
+  static constexpr int kGam = RULE == kStateSpace ? 2 * kBlk : (RULE == kScalarDelta ? 4 * kBlk : DK);   // factors of a block and head
+  static constexpr int kTotal = kG + kGam;
 };
 
 // Block-sequential pass.  A CTA owns 32 columns of one head's state in registers: a thread 4 columns and the rows
@@ -590,9 +700,9 @@ struct ScanGeom {
 // the CTA only meets at the staging buffers (the next block streams in with cp.async meanwhile).
 // grid (DV / 32, hv, runs)
 template <int DK, int DV, int RULE>
-__global__ void __launch_bounds__(ScanGeom<DK, RULE == kDelta>::kThreads) lin_scan_kernel(LinearArgs a) {
-  constexpr bool DELTA = RULE == kDelta, SSD = RULE == kStateSpace;
-  using G = ScanGeom<DK, DELTA>;
+__global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(LinearArgs a) {
+  constexpr bool DELTA = is_delta(RULE), CH = RULE == kDelta, SCALAR = scalar_decay(RULE);
+  using G = ScanGeom<DK, RULE>;
   constexpr int NI = G::kNI, PARTS = G::kParts, NT = G::kThreads;
   constexpr int NV = 4 * kBlk, CNT = NV / PARTS;            // values of a group's block; totals per lane (2, 4 or 8)
   extern __shared__ __align__(16) float sc_smem[];          // [2][G::kTotal], then W and U of every group [8][2][64]
@@ -602,7 +712,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE == kDelta>::kThreads) lin_sc
   const int first = a.run_start[blockIdx.z], last = a.run_start[blockIdx.z + 1];
   int blk = 0;
   for (int r = 0; r < static_cast<int>(blockIdx.z); ++r) blk += (a.run_start[r + 1] - a.run_start[r] + kBlk - 1) / kBlk;
-  const int slot = a.row_slot[first], hk = SSD ? h / (a.hv / a.hk) : 0;
+  const int slot = a.row_slot[first], hk = SCALAR ? h / (a.hv / a.hk) : 0;
   const PrepView pv = prep_view<DK, DV, RULE>(a);
   float* ws = sc_smem + 2 * G::kTotal + cg * 2 * NV;        // [16][4] W
   float* us = ws + NV;                                      // [16][4] U
@@ -623,15 +733,15 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE == kDelta>::kThreads) lin_sc
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int i = tid; i < kBlk * (DK / 4); i += NT) {
       const int t = i / (DK / 4), c = (i % (DK / 4)) * 4;
-      const size_t o = SSD ? (static_cast<size_t>(t0 + t) * a.hk + hk) * DK + c : (static_cast<size_t>(t0 + t) * a.hv + h) * DK + c;
+      const size_t o = SCALAR ? (static_cast<size_t>(t0 + t) * a.hk + hk) * DK + c : (static_cast<size_t>(t0 + t) * a.hv + h) * DK + c;
       if (t < n) {
-        cp_async_16(d + G::kQ + t * DK + c, (SSD ? pv.q : pv.qt) + o);
-        cp_async_16(d + G::kH + t * DK + c, (SSD ? pv.k : pv.kh) + o);
-        if (DELTA) cp_async_16(d + G::kK + t * DK + c, pv.kt + o);
+        cp_async_16(d + G::kQ + t * DK + c, (SCALAR ? pv.q : pv.qt) + o);
+        cp_async_16(d + G::kH + t * DK + c, (SCALAR ? pv.k : pv.kh) + o);
+        if (CH) cp_async_16(d + G::kK + t * DK + c, pv.kt + o);
       } else {
         *reinterpret_cast<float4*>(d + G::kQ + t * DK + c) = zero;
         *reinterpret_cast<float4*>(d + G::kH + t * DK + c) = zero;
-        if (DELTA) *reinterpret_cast<float4*>(d + G::kK + t * DK + c) = zero;
+        if (CH) *reinterpret_cast<float4*>(d + G::kK + t * DK + c) = zero;
       }
     }
     for (int i = tid; i < kBlk * (kScanCols / 4); i += NT) {
@@ -644,8 +754,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE == kDelta>::kThreads) lin_sc
       cp_async_16(d + G::kP + i, pv.pm + bh * kBlk * kBlk + i);
       if (DELTA) cp_async_16(d + G::kT + i, pv.tb + bh * kBlk * kBlk + i);
     }
-    constexpr int kGam = SSD ? 2 * kBlk : DK;
-    for (int i = tid * 4; i < kGam; i += NT * 4) cp_async_16(d + G::kG + i, pv.gam + bh * kGam + i);
+    for (int i = tid * 4; i < G::kGam; i += NT * 4) cp_async_16(d + G::kG + i, pv.gam + bh * G::kGam + i);
     cp_async_group_commit();
   };
   // partial products of 16 staged rows with this thread's part of the state, summed over the group
@@ -698,11 +807,11 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE == kDelta>::kThreads) lin_sc
     const int n = min(kBlk, last - t0);
     float val[NV], x[CNT];
     if (DELTA) {
-      rows_times_state(d + G::kK, val);
+      rows_times_state(d + (CH ? G::kK : G::kH), val);
 #pragma unroll
       for (int i = 0; i < CNT; ++i) {
         const int idx = part * CNT + i;
-        ws[idx] = vb[(idx / 4) * kScanCols + idx % 4] - val[i];
+        ws[idx] = fmaf(CH ? -1.f : -d[G::kG + 2 * kBlk + idx / 4], val[i], vb[(idx / 4) * kScanCols + idx % 4]);
       }
       __syncwarp();
       pairs_times(d + G::kT, ws, 4, x);
@@ -717,13 +826,13 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE == kDelta>::kThreads) lin_sc
 #pragma unroll
     for (int i = 0; i < CNT; ++i) {
       const int idx = part * CNT + i;
-      const float w = SSD ? d[G::kG + idx / 4] : 1.f;
+      const float w = SCALAR ? d[G::kG + idx / 4] : 1.f;
       if (idx / 4 < n && j0 + idx % 4 < a.ow) a.o[(static_cast<size_t>(t0 + idx / 4) * a.hv + h) * a.ow + j0 + idx % 4] = fmaf(w, val[i], x[i]);
     }
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
       float4 g4;
-      if (SSD) g4.x = g4.y = g4.z = g4.w = d[G::kG + kBlk - 1];
+      if (SCALAR) g4.x = g4.y = g4.z = g4.w = d[G::kG + (DELTA ? 3 * kBlk : kBlk - 1)];
       else g4 = *reinterpret_cast<const float4*>(d + G::kG + 4 * PARTS * i + 4 * part);
       const float gf[4] = {g4.x, g4.y, g4.z, g4.w};
 #pragma unroll
@@ -734,7 +843,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE == kDelta>::kThreads) lin_sc
 #pragma unroll
     for (int t = 0; t < kBlk; ++t) {
       const float4 u4 = *reinterpret_cast<const float4*>(u + t * ustride);
-      const float w = SSD ? d[G::kG + kBlk + t] : 1.f;
+      const float w = SCALAR ? d[G::kG + kBlk + t] : 1.f;
       const float uf[4] = {u4.x * w, u4.y * w, u4.z * w, u4.w * w};
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
@@ -758,7 +867,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE == kDelta>::kThreads) lin_sc
 
 template <typename T, int DK, int DV, int RULE>
 static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
-  constexpr bool DELTA = RULE == kDelta;
+  constexpr bool DELTA = is_delta(RULE);
   using G = LinGeom<DK, DV>;
   if (decode) {
     const size_t smem = static_cast<size_t>(G::kParts) * DV * sizeof(float) * (DELTA ? 2 : 1);
@@ -767,31 +876,33 @@ static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
     DGPP_CUDA_OK(cudaGetLastError());
     return 0;
   }
-  constexpr size_t smem = (2 * ScanGeom<DK, DELTA>::kTotal + 8 * 2 * 4 * kBlk) * sizeof(float);
+  constexpr size_t smem = (2 * ScanGeom<DK, RULE>::kTotal + 8 * 2 * 4 * kBlk) * sizeof(float);
   constexpr size_t bsmem = (DELTA ? 3 : 2) * static_cast<size_t>(kBlk) * DK * sizeof(float);
   static bool attr = false;
   if (!attr) {
-    if constexpr (RULE != kStateSpace)
+    if constexpr (!scalar_decay(RULE))
       DGPP_CUDA_OK(cudaFuncSetAttribute(lin_block_kernel<DK, DV, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bsmem)));
     DGPP_CUDA_OK(cudaFuncSetAttribute(lin_scan_kernel<DK, DV, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     attr = true;
   }
   bool prepared = false;
-  if constexpr (RULE == kStateSpace) {
+  if constexpr (scalar_decay(RULE)) {
     const dim3 grid(dgpp_ceil_div(2 * a.hk * DK + a.hv * DV, 512) + 1, a.blocks);
     prepared = a.taps <= 4 && a.stride % 4 == 0 && a.c_off % 4 == 0;
     if (!prepared) {}
-    else if (a.taps == 1) ssd_prep_kernel<T, DK, DV, 1><<<grid, 128, 0, st>>>(a);
-    else if (a.taps == 2) ssd_prep_kernel<T, DK, DV, 2><<<grid, 128, 0, st>>>(a);
-    else if (a.taps == 3) ssd_prep_kernel<T, DK, DV, 3><<<grid, 128, 0, st>>>(a);
-    else ssd_prep_kernel<T, DK, DV, 4><<<grid, 128, 0, st>>>(a);
+    else if (a.taps == 1) ssd_prep_kernel<T, DK, DV, RULE, 1><<<grid, 128, 0, st>>>(a);
+    else if (a.taps == 2) ssd_prep_kernel<T, DK, DV, RULE, 2><<<grid, 128, 0, st>>>(a);
+    else if (a.taps == 3) ssd_prep_kernel<T, DK, DV, RULE, 3><<<grid, 128, 0, st>>>(a);
+    else ssd_prep_kernel<T, DK, DV, RULE, 4><<<grid, 128, 0, st>>>(a);
   }
   if (!prepared) lin_prep_kernel<T, DK, DV, RULE><<<dgpp_ceil_div(a.rows * (a.hk + a.hv), 8), 256, 0, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
-  if constexpr (RULE == kStateSpace) ssd_block_kernel<DK, DV><<<dim3(a.hk * dgpp_ceil_div(a.hv / a.hk, kSsdHeads), a.blocks), 256, 0, st>>>(a);
+  const dim3 groups(a.hk * dgpp_ceil_div(a.hv / a.hk, kSsdHeads), a.blocks);
+  if constexpr (RULE == kStateSpace) ssd_block_kernel<DK, DV><<<groups, 256, 0, st>>>(a);
+  else if constexpr (RULE == kScalarDelta) gated_block_kernel<DK, DV><<<groups, 256, 0, st>>>(a);
   else lin_block_kernel<DK, DV, RULE><<<dim3(a.hv, a.blocks), 256, bsmem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
-  lin_scan_kernel<DK, DV, RULE><<<dim3(DV / kScanCols, a.hv, a.runs), ScanGeom<DK, DELTA>::kThreads, smem, st>>>(a);
+  lin_scan_kernel<DK, DV, RULE><<<dim3(DV / kScanCols, a.hv, a.runs), ScanGeom<DK, RULE>::kThreads, smem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   if (a.conv_w != nullptr) {
     const int C = 2 * a.hk * DK + a.hv * DV;

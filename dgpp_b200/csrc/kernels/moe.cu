@@ -30,12 +30,13 @@ struct RouterArgs {
   int64_t x_stride;
   const bf16* gate;      // [E, H]
   const float* bias;     // [E] selection correction, may be null
+  const float* logit_bias;  // [E] added to the logits, may be null
   int32_t* ids;          // [T, k] ascending
   float* weights;        // [T, k]
   float* logits_out;     // [T, logits_stride]
   int64_t logits_stride;
   int T, H, E, k, n_group, topk_group;
-  int softmax, norm_topk;
+  int softmax, norm_topk;   // softmax 0: sigmoid scores, 1: softmax over all experts, 2: selection by logit, softmax over the chosen
   float scaling;
 };
 
@@ -91,9 +92,9 @@ __global__ void __launch_bounds__(kRouterThreads) moe_router_select_kernel(Route
   __shared__ int pick_id[kMoeMaxTopK];
   pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
-  for (int e = tid; e < a.E; e += kRouterThreads) score[e] = a.logits_out[t * a.logits_stride + e];
+  for (int e = tid; e < a.E; e += kRouterThreads) score[e] = a.logits_out[t * a.logits_stride + e] + (a.logit_bias ? a.logit_bias[e] : 0.f);
   __syncthreads();
-  if (a.softmax) {
+  if (a.softmax == 1) {
     // softmax over all experts: max, then the sum of exp, each by a fixed tree (thread-strided partials, xor-shuffle
     // within the warp, the 8 warp results in warp order), so the value does not depend on timing
     __shared__ float mx_s, sum_s;
@@ -122,7 +123,7 @@ __global__ void __launch_bounds__(kRouterThreads) moe_router_select_kernel(Route
     }
     __syncthreads();
     for (int e = tid; e < a.E; e += kRouterThreads) score[e] = expf(score[e] - mx_s) / sum_s;
-  } else {
+  } else if (a.softmax == 0) {
     for (int e = tid; e < a.E; e += kRouterThreads) score[e] = 1.f / (1.f + expf(-score[e]));
   }
   __syncthreads();
@@ -184,11 +185,16 @@ __global__ void __launch_bounds__(kRouterThreads) moe_router_select_kernel(Route
         while (j >= 0 && pick_id[j] > v) { pick_id[j + 1] = pick_id[j]; --j; }
         pick_id[j + 1] = v;
       }
+      if (a.softmax == 2) {
+        float m = -INFINITY;
+        for (int i = 0; i < a.k; ++i) m = fmaxf(m, score[pick_id[i]]);
+        for (int i = 0; i < a.k; ++i) score[pick_id[i]] = expf(score[pick_id[i]] - m);
+      }
       float sum = 0.f;
       for (int i = 0; i < a.k; ++i) sum += score[pick_id[i]];
       for (int i = 0; i < a.k; ++i) {
         float w = score[pick_id[i]];
-        if (a.norm_topk) w = w / (sum + 1e-20f);
+        if (a.norm_topk || a.softmax == 2) w = w / (sum + 1e-20f);
         a.ids[t * a.k + i] = pick_id[i];
         a.weights[t * a.k + i] = w * a.scaling;
       }
@@ -346,8 +352,9 @@ DGPP_API int dgpp_moe_route(const void* x, int64_t x_stride, const void* gate, c
   return 0;
 }
 
-// Selection alone, over logits [T, E] (row stride logits_stride) that another kernel made; no correction, no groups.
-DGPP_API int dgpp_moe_select(const void* logits, int64_t logits_stride, void* ids, void* weights, int T, int E, int k, int softmax, int norm_topk,
+// Selection alone, over logits [T, E] (row stride logits_stride) that another kernel made, plus `bias` [E] fp32 where it is given; no
+// correction, no groups.
+DGPP_API int dgpp_moe_select(const void* logits, int64_t logits_stride, const void* bias, void* ids, void* weights, int T, int E, int k, int softmax, int norm_topk,
                              float scaling, cudaStream_t st) {
   DGPP_REQUIRE(E >= 1 && E <= kMoeMaxExperts && k >= 1 && k <= kMoeMaxTopK && k <= E, "moe_select: E %d / k %d unsupported", E, k);
   if (T == 0) return 0;
@@ -356,6 +363,7 @@ DGPP_API int dgpp_moe_select(const void* logits, int64_t logits_stride, void* id
   a.weights = static_cast<float*>(weights);
   a.logits_out = static_cast<float*>(const_cast<void*>(logits));
   a.logits_stride = logits_stride;
+  a.logit_bias = static_cast<const float*>(bias);
   a.T = T; a.E = E; a.k = k; a.n_group = 1; a.topk_group = 1;
   a.softmax = softmax; a.norm_topk = norm_topk; a.scaling = scaling;
   moe_router_select_kernel<<<T, kRouterThreads, 0, st>>>(a);

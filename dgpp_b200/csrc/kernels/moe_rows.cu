@@ -1,7 +1,7 @@
 // Mixture of experts over plain 16-bit or 32-bit rows (expert matrices without block scales): the launches between the router
 // logits and the grouped linears.
 //
-//   moe_route_small    up to 16 tokens, one CTA: picks every token's experts from its logits (sigmoid or softmax scores, ties to
+//   moe_route_small    up to 16 tokens, one CTA: picks every token's experts from its logits (sigmoid or softmax weights, ties to
 //                      the lower id), lists the experts in use as tiles of 16 rows over the SAME activation rows, and writes the
 //                      row of every (token, choice) pair and every tile row's weight (0: the token did not choose the expert)
 //   moe_scatter_rows   any number of tokens, after the counting sort of moe_prefill.cu: copies a pair's activation row to its place
@@ -24,7 +24,8 @@ struct RouteSmall {
   int32_t* pair_row;       // [T * top]
   int32_t* tiles;          // [max_tiles]
   float* row_w;            // [max_tiles * 16]
-  int T, E, top, max_tiles, softmax;
+  const float* bias;       // [E] added to the logits, or null
+  int T, E, top, max_tiles, score;   // score: 0 sigmoid, 1 softmax over all experts, 2 softmax over the chosen ones
 };
 
 __global__ void __launch_bounds__(kSmallThreads) moe_route_small_kernel(RouteSmall a) {
@@ -43,11 +44,11 @@ __global__ void __launch_bounds__(kSmallThreads) moe_route_small_kernel(RouteSma
 #pragma unroll
     for (int i = 0; i < kSmallExperts / 32; ++i) {
       const int e = lane + 32 * i;
-      z[i] = e < a.E ? a.logits[t * a.stride + e] : -INFINITY;
+      z[i] = e < a.E ? a.logits[t * a.stride + e] + (a.bias != nullptr ? a.bias[e] : 0.f) : -INFINITY;
       mx = fmaxf(mx, z[i]);
     }
     float norm = 1.f;
-    if (a.softmax) {
+    if (a.score == 1) {
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       float sum = 0.f;
@@ -78,9 +79,15 @@ __global__ void __launch_bounds__(kSmallThreads) moe_route_small_kernel(RouteSma
         int j = r;                                     // ascending ids: the order of the sum
         while (j > 0 && ids[t][j - 1] > be) { ids[t][j] = ids[t][j - 1]; wts[t][j] = wts[t][j - 1]; --j; }
         ids[t][j] = be;
-        wts[t][j] = a.softmax ? expf(bv - mx) / norm : sigmoid_f32(bv);
+        if (r == 0 && a.score == 2) mx = bv;           // the largest comes first
+        wts[t][j] = a.score == 0 ? sigmoid_f32(bv) : expf(bv - mx) / norm;
         slot[be] = 1;
       }
+    }
+    if (a.score == 2 && lane == 0) {
+      float sum = 0.f;
+      for (int j = 0; j < a.top; ++j) sum += wts[t][j];
+      for (int j = 0; j < a.top; ++j) wts[t][j] /= sum;
     }
   }
   __syncthreads();
@@ -125,14 +132,15 @@ __global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const T* __restri
 
 using namespace dgpp;
 
-// logits [T, E] fp32 with row stride `stride`, T <= 16.  max_tiles >= min(E, T * top).
-DGPP_API int dgpp_moe_route_small(const void* logits, int64_t stride, void* pair_row, void* tiles, void* row_w, int T, int E, int top, int max_tiles,
-                                  int softmax, cudaStream_t st) {
+// logits [T, E] fp32 with row stride `stride` (bias [E] fp32 or null is added), T <= 16.  max_tiles >= min(E, T * top).
+DGPP_API int dgpp_moe_route_small(const void* logits, int64_t stride, const void* bias, void* pair_row, void* tiles, void* row_w, int T, int E, int top, int max_tiles,
+                                  int score, cudaStream_t st) {
+  DGPP_REQUIRE(score >= 0 && score <= 2, "moe_route_small: score %d", score);
   DGPP_REQUIRE(E >= 1 && E <= kSmallExperts && top >= 1 && top <= kSmallTop && top <= E, "moe_route_small: %d of %d experts", top, E);
   DGPP_REQUIRE(T <= kSmallTokens && max_tiles >= (E < T * top ? E : T * top), "moe_route_small: %d tokens in %d tiles", T, max_tiles);
   if (T == 0) return 0;
   const RouteSmall a = {static_cast<const float*>(logits), stride, static_cast<int32_t*>(pair_row), static_cast<int32_t*>(tiles),
-                        static_cast<float*>(row_w), T, E, top, max_tiles, softmax};
+                        static_cast<float*>(row_w), static_cast<const float*>(bias), T, E, top, max_tiles, score};
   moe_route_small_kernel<<<1, kSmallThreads, 0, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;

@@ -1,13 +1,15 @@
 // Row operators of models that keep the residual stream in fp32 (activations T = bf16 or fp32):
-//   embed_rows        out[r] = table[ids[r]]                                                   (fp32 rows)
+//   embed_rows        out[r] = scale * table[ids[r]]                           (fp32 rows; on request a second time in T)
 //   resid_norm        x += delta (fp32, optional); out = x / sqrt(mean(x^2) + eps) * w           (out in T)
-//   gated_group_norm  per group of columns: out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) * scale
+//   gated_group_norm  per group of columns: out = o / sqrt(mean(o^2) + eps) * w * act(gate) * scale; act: sigmoid or silu
 //   geglu             out = gelu_tanh(gate) * up
-//   stream_norm       x += post(delta); out = pre(x); post and pre each nothing, an RMS norm or a layer norm (weight, no bias);
-//                     delta is a row of fp32 or the weighed rows of a mixture of experts plus its gated shared expert
+//   stream_norm       x += mult * post(delta + bias) + vec; out = pre(x); post and pre each nothing, an RMS norm or a layer norm
+//                     (weight, perhaps a bias); delta is a row of fp32 or the weighed rows of a mixture of experts plus its gated
+//                     shared expert; vec is one row for all
 //   gated_part_norm   a = y * silu(z); every one of `parts` runs of columns by its own root mean square, times w
-//   clamped_glu       g = min(s gate, limit), u = clamp(s up, -limit, limit); out = g * sigmoid(alpha g) * (u + 1); s: a factor per
-//                     row (the input weight of a routed expert; the product with the weights is linear) or one
+//   clamped_glu       g = min(s gate, limit), u = clamp(s up, -limit, limit); out = r * g * sigmoid(alpha g) * (u + shift); s or r: a
+//                     factor per row (the weight of a routed expert on its input or on its output; the products with the weights
+//                     are linear), else one
 //   token_gate        out = gelu_tanh(gate) * table[ids[r]][columns of one layer]
 //   softcap           x = cap * tanh(x / cap)
 // Rows may carry zero columns behind their `n` true ones (the padding of the tensor-core GEMM): means divide by the true
@@ -25,14 +27,20 @@ constexpr int kStreamThreads = 256;
 
 template <typename T>
 __global__ void __launch_bounds__(kStreamThreads)
-embed_rows_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, int cols, int vocab) {
+embed_rows_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, T* __restrict__ copy, int64_t copy_stride,
+                  int cols, int vocab, float scale) {
   pdl_wait();
   const int row = blockIdx.x;
   int id = ids[row];
   id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
   const T* src = table + static_cast<size_t>(id) * cols;
   float* dst = out + static_cast<size_t>(row) * cols;
-  for (int i = threadIdx.x * 4; i < cols; i += kStreamThreads * 4) st_elem4(dst + i, ld_elem4(src + i));
+  for (int i = threadIdx.x * 4; i < cols; i += kStreamThreads * 4) {
+    float4 v = ld_elem4(src + i);
+    v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+    st_elem4(dst + i, v);
+    if (copy != nullptr) st_elem4(copy + row * copy_stride + i, v);
+  }
 }
 
 template <typename T>
@@ -64,7 +72,7 @@ resid_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, const 
 template <typename T, typename TG>
 __global__ void __launch_bounds__(kStreamThreads)
 gated_group_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int64_t gate_stride, const float* __restrict__ w,
-                        T* __restrict__ out, int64_t out_stride, int rows, int groups, int gp, int n, float eps, float scale, int team) {
+                        T* __restrict__ out, int64_t out_stride, int rows, int groups, int gp, int n, float eps, float scale, int silu, int team) {
   __shared__ float scratch[kStreamThreads / 32];
   pdl_wait();
   const size_t unit = (static_cast<size_t>(blockIdx.x) * kStreamThreads + threadIdx.x) / team;
@@ -85,8 +93,8 @@ gated_group_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate
   const float r = scale / sqrtf(ss / static_cast<float>(n) + eps);
   for (int i = me * 4; i < gp; i += team * 4) {
     const float4 v = ld_elem4(op + i), a = ld_elem4(gt + i), ww = ld_elem4(w + i);
-    st_elem4(dst + i, make_float4(v.x * r * ww.x * sigmoid_f32(a.x), v.y * r * ww.y * sigmoid_f32(a.y),
-                                  v.z * r * ww.z * sigmoid_f32(a.z), v.w * r * ww.w * sigmoid_f32(a.w)));
+    auto act = [silu](float z) { return silu ? silu_f32(z) : sigmoid_f32(z); };
+    st_elem4(dst + i, make_float4(v.x * r * ww.x * act(a.x), v.y * r * ww.y * act(a.y), v.z * r * ww.z * act(a.z), v.w * r * ww.w * act(a.w)));
   }
 }
 
@@ -122,9 +130,15 @@ struct MoeRows {
   int top;
 };
 
-// Norm of a row held in registers; columns at or beyond n are zero and stay zero (their weights are zero).
+struct RowNorm {
+  int kind;
+  const float *w, *b;        // weights; bias or null
+};
+
+// Norm of a row held in registers; columns at or beyond n are zero and stay zero (their weights and biases are zero).
 template <int NT, int NV>
-__device__ __forceinline__ void norm_row(float4 (&v)[NV], int kind, const float* __restrict__ w, int cols, int n, float eps, float* scratch) {
+__device__ __forceinline__ void norm_row(float4 (&v)[NV], const RowNorm& norm, int cols, int n, float eps, float* scratch) {
+  const int kind = norm.kind;
   if (kind == kNormNone) return;
   float mean = 0.f;
   if (kind == kNormLayer) {
@@ -148,18 +162,32 @@ __device__ __forceinline__ void norm_row(float4 (&v)[NV], int kind, const float*
   for (int j = 0; j < NV; ++j) {
     const int i = (threadIdx.x + NT * j) * 4;
     if (i < cols) {
-      const float4 g = ld_elem4(w + i);
-      v[j].x *= r * g.x; v[j].y *= r * g.y; v[j].z *= r * g.z; v[j].w *= r * g.w;
+      const float4 g = ld_elem4(norm.w + i), b = norm.b != nullptr ? ld_elem4(norm.b + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[j].x = fmaf(v[j].x, r * g.x, b.x); v[j].y = fmaf(v[j].y, r * g.y, b.y);
+      v[j].z = fmaf(v[j].z, r * g.z, b.z); v[j].w = fmaf(v[j].w, r * g.w, b.w);
     }
   }
 }
 
+struct StreamNorm {
+  float* x;                  // [rows, cols]
+  const float* delta;        // [rows, cols] or null
+  const float* delta_b;      // [cols] or null: added to the delta
+  const float* vec;          // [cols] or null: added to every row
+  float mult, eps;
+  RowNorm post, pre;
+  int64_t out_stride;
+  int cols, n;
+};
+
 template <typename T, int NT, int NV>
 __global__ void __launch_bounds__(NT)
-stream_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, MoeRows<T> moe, int post, const float* __restrict__ wp, int pre,
-                   const float* __restrict__ wn, T* __restrict__ out, int cols, int n, float eps) {
+stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
   __shared__ float scratch[NT / 32];
   pdl_wait();
+  float* __restrict__ x = p.x;
+  const float* __restrict__ delta = p.delta;
+  const int cols = p.cols, n = p.n;
   const size_t row = blockIdx.x, base = row * cols;
   float4 v[NV];
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -171,7 +199,12 @@ stream_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, MoeRo
       const int i = (threadIdx.x + NT * j) * 4;
       v[j] = zero;
       if (i >= cols) continue;
-      if (delta != nullptr) { v[j] = ld_elem4(delta + base + i); continue; }
+      if (p.delta_b != nullptr) v[j] = ld_elem4(p.delta_b + i);
+      if (delta != nullptr) {
+        const float4 a = ld_elem4(delta + base + i);
+        v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
+        continue;
+      }
       for (int k = 0; k < moe.top; ++k) {
         const float4 a = ld_elem4(moe.y + static_cast<size_t>(moe.pair_row[row * moe.top + k]) * cols + i);
         v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
@@ -181,28 +214,32 @@ stream_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, MoeRo
         v[j].x = fmaf(sg, a.x, v[j].x); v[j].y = fmaf(sg, a.y, v[j].y); v[j].z = fmaf(sg, a.z, v[j].z); v[j].w = fmaf(sg, a.w, v[j].w);
       }
     }
-    norm_row<NT, NV>(v, post, wp, cols, n, eps, scratch);
+    norm_row<NT, NV>(v, p.post, cols, n, p.eps, scratch);
   }
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     const int i = (threadIdx.x + NT * j) * 4;
-    const float4 a = i < cols ? ld_elem4(x + base + i) : zero;
-    if (!add) { v[j] = a; continue; }
-    v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
-    if (i < cols) st_elem4(x + base + i, v[j]);
+    float4 a = i < cols ? ld_elem4(x + base + i) : zero;
+    if (p.vec != nullptr && i < cols) {
+      const float4 e = ld_elem4(p.vec + i);
+      a.x += e.x; a.y += e.y; a.z += e.z; a.w += e.w;
+    }
+    if (add) { a.x = fmaf(p.mult, v[j].x, a.x); a.y = fmaf(p.mult, v[j].y, a.y); a.z = fmaf(p.mult, v[j].z, a.z); a.w = fmaf(p.mult, v[j].w, a.w); }
+    v[j] = a;
+    if (i < cols && (add || p.vec != nullptr)) st_elem4(x + base + i, a);
   }
-  norm_row<NT, NV>(v, pre, wn, cols, n, eps, scratch);
+  norm_row<NT, NV>(v, p.pre, cols, n, p.eps, scratch);
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     const int i = (threadIdx.x + NT * j) * 4;
-    if (i < cols) st_elem4(out + base + i, v[j]);
+    if (i < cols) st_elem4(out + row * p.out_stride + i, v[j]);
   }
 }
 
 template <typename T>
-static int launch_stream_norm(float* x, const float* delta, const MoeRows<T>& moe, int post, const float* wp, int pre, const float* wn,
-                              T* out, int rows, int cols, int n, float eps, cudaStream_t st) {
-#define DGPP_SN(NT, NV) stream_norm_kernel<T, NT, NV><<<rows, NT, 0, st>>>(x, delta, moe, post, wp, pre, wn, out, cols, n, eps)
+static int launch_stream_norm(const StreamNorm& p, const MoeRows<T>& moe, T* out, int rows, cudaStream_t st) {
+  const int cols = p.cols;
+#define DGPP_SN(NT, NV) stream_norm_kernel<T, NT, NV><<<rows, NT, 0, st>>>(p, moe, out)
   if (cols <= 1024) DGPP_SN(256, 1);
   else if (cols <= 2048) DGPP_SN(256, 2);
   else if (cols <= 4096) DGPP_SN(256, 4);
@@ -260,13 +297,13 @@ gated_part_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, int
 template <typename TI, typename T>
 __global__ void __launch_bounds__(kStreamThreads)
 clamped_glu_kernel(const TI* __restrict__ gate_up, int64_t stride, const float* __restrict__ row_w, const int32_t* __restrict__ tiles, int bn,
-                   T* __restrict__ out, int inter, float limit, float alpha) {
+                   T* __restrict__ out, int inter, float limit, float alpha, float shift, int weigh_out) {
   pdl_wait();
   const size_t row = blockIdx.y;
   if (tiles != nullptr && tiles[row / bn] < 0) return;
   const int i = (blockIdx.x * kStreamThreads + threadIdx.x) * 8;
   if (i >= inter) return;
-  const float s = row_w != nullptr ? row_w[row] : 1.f;
+  const float w = row_w != nullptr ? row_w[row] : 1.f, s = weigh_out ? 1.f : w, r = weigh_out ? w : 1.f;
   const TI* gp = gate_up + row * stride + i;
   float g[8], u[8];
   ld_elem8(gp, g);
@@ -275,7 +312,7 @@ clamped_glu_kernel(const TI* __restrict__ gate_up, int64_t stride, const float* 
   for (int e = 0; e < 8; ++e) {
     const float a = fminf(g[e] * s, limit), b = fminf(fmaxf(u[e] * s, -limit), limit);
     const float sg = sizeof(T) == 4 ? sigmoid_f32(alpha * a) : __fdividef(1.f, 1.f + __expf(-alpha * a));
-    g[e] = a * sg * (b + 1.f);
+    g[e] = r * a * sg * (b + shift);
   }
   st_elem8(out + row * inter + i, g);
 }
@@ -306,11 +343,14 @@ __global__ void __launch_bounds__(kStreamThreads) softcap_kernel(float* __restri
 using namespace dgpp;
 
 // `f32` selects fp32 activations (else bf16) in every entry point below.
-DGPP_API int dgpp_embed_rows(const void* ids, const void* table, void* out, int rows, int cols, int vocab, int f32, cudaStream_t st) {
+// copy: optional second place of the rows, in the activations' type with a row stride of its own.
+DGPP_API int dgpp_embed_rows(const void* ids, const void* table, void* out, void* copy, int64_t copy_stride, int rows, int cols, int vocab, float scale,
+                             int f32, cudaStream_t st) {
+  DGPP_REQUIRE(copy_stride % 8 == 0, "embed_rows: row stride %lld", static_cast<long long>(copy_stride));
   DGPP_REQUIRE(cols % 8 == 0, "embed_rows: %d columns (a multiple of 8)", cols);
   if (rows == 0) return 0;
-  if (f32) embed_rows_kernel<float><<<rows, kStreamThreads, 0, st>>>(static_cast<const int32_t*>(ids), static_cast<const float*>(table), static_cast<float*>(out), cols, vocab);
-  else embed_rows_kernel<bf16><<<rows, kStreamThreads, 0, st>>>(static_cast<const int32_t*>(ids), static_cast<const bf16*>(table), static_cast<float*>(out), cols, vocab);
+  if (f32) embed_rows_kernel<float><<<rows, kStreamThreads, 0, st>>>(static_cast<const int32_t*>(ids), static_cast<const float*>(table), static_cast<float*>(out), static_cast<float*>(copy), copy_stride, cols, vocab, scale);
+  else embed_rows_kernel<bf16><<<rows, kStreamThreads, 0, st>>>(static_cast<const int32_t*>(ids), static_cast<const bf16*>(table), static_cast<float*>(out), static_cast<bf16*>(copy), copy_stride, cols, vocab, scale);
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -326,16 +366,16 @@ DGPP_API int dgpp_resid_norm(void* x, const void* delta, const void* w, void* ou
   return 0;
 }
 
-// gate_f32: the gate rows are fp32 although the activations are bf16.
+// gate_f32: the gate rows are fp32 although the activations are bf16.  silu: the gate passes silu, else a sigmoid.
 DGPP_API int dgpp_gated_group_norm(const void* o, const void* gate, int64_t gate_stride, const void* w, void* out, int64_t out_stride,
-                                   int rows, int groups, int gp, int n, float eps, float scale, int f32, int gate_f32, cudaStream_t st) {
+                                   int rows, int groups, int gp, int n, float eps, float scale, int silu, int f32, int gate_f32, cudaStream_t st) {
   DGPP_REQUIRE(gp % 8 == 0 && gate_stride % 8 == 0 && out_stride % 8 == 0 && n >= 1 && n <= gp, "gated_group_norm: %d of %d columns", n, gp);
   if (rows == 0) return 0;
   const int team = gp <= 512 ? 32 : kStreamThreads;
   const int64_t blocks = dgpp_ceil_div64(static_cast<int64_t>(rows) * groups * team, kStreamThreads);
   const float *op = static_cast<const float*>(o), *wp = static_cast<const float*>(w);
 #define DGPP_GGN(TT, TG) gated_group_norm_kernel<TT, TG><<<static_cast<unsigned>(blocks), kStreamThreads, 0, st>>>( \
-      op, static_cast<const TG*>(gate), gate_stride, wp, static_cast<TT*>(out), out_stride, rows, groups, gp, n, eps, scale, team)
+      op, static_cast<const TG*>(gate), gate_stride, wp, static_cast<TT*>(out), out_stride, rows, groups, gp, n, eps, scale, silu, team)
   if (f32) DGPP_GGN(float, float);
   else if (gate_f32) DGPP_GGN(bf16, float);
   else DGPP_GGN(bf16, bf16);
@@ -355,25 +395,29 @@ DGPP_API int dgpp_geglu(const void* gate_up, void* out, int rows, int inter, int
   return 0;
 }
 
-// post / pre: 0 nothing, 1 RMS norm, 2 layer norm, each with its weights.  The delta is `delta` (fp32 [rows, cols]), or the
-// expert rows y[pair_row[r * top + j]] plus sigmoid(gate) * shared (y, shared: activations), or absent.
+// post / pre: 0 nothing, 1 RMS norm, 2 layer norm, each with its weights and perhaps a bias.  The delta is `delta` (fp32 [rows, cols]),
+// or the expert rows y[pair_row[r * top + j]] plus sigmoid(gate) * shared (y, shared: activations), or absent; delta_b [cols] is added
+// to it.  vec [cols]: added to every row of x.
 DGPP_API int dgpp_stream_norm(void* x, const void* delta, const void* y, const void* pair_row, int top, const void* shared, const void* gate,
-                              int64_t gate_stride, int post, const void* post_w, int pre, const void* pre_w, void* out, int rows, int cols,
-                              int n, float eps, int f32, cudaStream_t st) {
+                              int64_t gate_stride, const void* delta_b, const void* vec, float mult, int post, const void* post_w,
+                              const void* post_b, int pre, const void* pre_w, const void* pre_b, void* out, int64_t out_stride, int rows,
+                              int cols, int n, float eps, int f32, cudaStream_t st) {
   DGPP_REQUIRE(cols % 8 == 0 && cols <= 16384 && n >= 1 && n <= cols, "stream_norm: %d of %d columns (at most 16384)", n, cols);
   DGPP_REQUIRE(post >= 0 && post <= 2 && pre >= 0 && pre <= 2 && (!post || post_w) && (!pre || pre_w), "stream_norm: norms %d / %d", post, pre);
   DGPP_REQUIRE(!(delta && y) && (!y || (pair_row && top >= 1)) && (!shared || (y && gate)), "stream_norm: one delta only");
+  DGPP_REQUIRE(out_stride % 8 == 0 && out_stride >= cols && (!delta_b || delta || y), "stream_norm: output rows of %lld", static_cast<long long>(out_stride));
   if (rows == 0) return 0;
-  float* xp = static_cast<float*>(x);
-  const float *dp = static_cast<const float*>(delta), *wp = static_cast<const float*>(post_w), *wn = static_cast<const float*>(pre_w);
+  auto f = [](const void* q) { return static_cast<const float*>(q); };
+  const StreamNorm p = {static_cast<float*>(x), f(delta), f(delta_b), f(vec), mult, eps, {post, f(post_w), f(post_b)}, {pre, f(pre_w), f(pre_b)},
+                        out_stride, cols, n};
   const int32_t* pr = static_cast<const int32_t*>(pair_row);
   const float* gp = static_cast<const float*>(gate);
   if (f32) {
     const MoeRows<float> m = {static_cast<const float*>(y), pr, static_cast<const float*>(shared), gp, gate_stride, top};
-    return launch_stream_norm<float>(xp, dp, m, post, wp, pre, wn, static_cast<float*>(out), rows, cols, n, eps, st);
+    return launch_stream_norm<float>(p, m, static_cast<float*>(out), rows, st);
   }
   const MoeRows<bf16> m = {static_cast<const bf16*>(y), pr, static_cast<const bf16*>(shared), gp, gate_stride, top};
-  return launch_stream_norm<bf16>(xp, dp, m, post, wp, pre, wn, static_cast<bf16*>(out), rows, cols, n, eps, st);
+  return launch_stream_norm<bf16>(p, m, static_cast<bf16*>(out), rows, st);
 }
 
 DGPP_API int dgpp_gated_part_norm(const void* y, const void* z, int64_t z_stride, const void* w, void* out, int64_t out_stride, int rows,
@@ -401,9 +445,9 @@ DGPP_API int dgpp_gated_part_norm(const void* y, const void* z, int64_t z_stride
   return 0;
 }
 
-// in_f32: gate_up is fp32 although the output is bf16.
+// in_f32: gate_up is fp32 although the output is bf16.  weigh_out: row_w multiplies the result, else the inputs.
 DGPP_API int dgpp_clamped_glu(const void* gate_up, int64_t stride, const void* row_w, const void* tiles, int bn, void* out, int rows, int inter,
-                              float limit, float alpha, int f32, int in_f32, cudaStream_t st) {
+                              float limit, float alpha, float shift, int weigh_out, int f32, int in_f32, cudaStream_t st) {
   DGPP_REQUIRE(inter % 8 == 0 && stride % 8 == 0 && bn >= 1, "clamped_glu: width %d (a multiple of 8)", inter);
   if (rows == 0) return 0;
   DGPP_REQUIRE(rows <= 65535, "clamped_glu: %d rows", rows);
@@ -411,7 +455,7 @@ DGPP_API int dgpp_clamped_glu(const void* gate_up, int64_t stride, const void* r
   const float* rw = static_cast<const float*>(row_w);
   const int32_t* tl = static_cast<const int32_t*>(tiles);
 #define DGPP_CG(TI, TT) clamped_glu_kernel<TI, TT><<<grid, kStreamThreads, 0, st>>>(static_cast<const TI*>(gate_up), stride, rw, tl, bn, \
-                                                                                   static_cast<TT*>(out), inter, limit, alpha)
+                                                                                   static_cast<TT*>(out), inter, limit, alpha, shift, weigh_out)
   if (f32) DGPP_CG(float, float);
   else if (in_f32) DGPP_CG(float, bf16);
   else DGPP_CG(bf16, bf16);

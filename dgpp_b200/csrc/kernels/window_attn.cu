@@ -1,23 +1,36 @@
-// Sliding-window GQA over a paged cache of 16-bit or true 32-bit keys and values, with per-head query / key norms, no
-// rotation, a softmax scale of its own and value heads that may be wider or narrower than the key heads.
+// GQA over a paged cache of 16-bit or true 32-bit keys and values, of a sliding window, of the row's own chunk of positions, or of
+// the whole sequence (a window nobody fills), with a softmax scale of its own and value heads that may be wider or narrower than the
+// key heads.
 //
-//   query head h reads key/value head g = h / (hq / hkv);  qn = rms(q_h) * wq, kn = rms(k_g) * wk (fp32)
-//   row at position i attends to positions max(0, i - window + 1) .. i:  p = softmax(scale * qn . kn),  out = sum p v
+//   query head h reads key/value head g = h / (hq / hkv)
+//   row at position i attends to positions lo(i) .. i:  p = softmax(scale * q . k),  out = sum p v
+//   lo(i) = max(0, i - window + 1), or i - i % window (chunked)
+//
+// What comes before the scores (each part optional, fp32, in this order): biases of q, k and v; RMS norm of q and k per head or over
+// the whole projection; rotation of the first `rot` columns of a head, column i < rot / 2 with column i + rot / 2; a factor on q that
+// grows with the position, 1 + coef * ln(floor((i + 1) / every) + 1).  Behind them, optional: a sigmoid gate per head.
+//
+// Differential attention (maps = 2): a value head has two key heads, and every output head two query heads, whose attentions a1, a2
+// over the same values make one output o = a1 - lambda a2, divided by its root mean square, times a factor and a sigmoid gate per
+// column.  Query heads are laid out [kv head][map][head of the group], key heads [kv head][map].
 //
 // The projections of a row sit in one fused row (T = bf16 or fp32); head widths are padded to multiples of 64 with zero
 // columns (D for queries / keys, DV for values), `dim` is the true key width that the norms divide by.
-// Cache: k [blocks, hkv, page, D], v [blocks, hkv, page, DV].
+// Cache: k [blocks, hkv * maps, page, D], v [blocks, hkv, page, DV].
 //
-//   qk_norm_append   prompt rows: norms q in place, appends normed k and v to the cache (one warp per row and head)
+//   qk_norm_append   prompt rows: prepares q in place, appends prepared k and v to the cache (one CTA per row)
 //   window_attn      one (row, kv head, split of the window) per CTA; `fused` = every row is the newest token of its
-//                    request and the CTA norms q, norms and appends k / v itself (decode: one launch per layer)
+//                    request and the CTA prepares q, prepares and appends k / v itself (decode: one launch per layer)
+//   diff_combine     the merge of the splits and the combination of the two maps, one warp per (row, head)
 // Softmax statistics and sums are fp32; the partials of the splits merge in ascending order.
 #include <math.h>
+#include <string.h>
 
 #include "common/common.h"
 #include "common/dtypes.cuh"
 #include "common/elem.cuh"
 #include "common/ptx.cuh"
+#include "common/rope.cuh"
 
 namespace dgpp {
 
@@ -25,20 +38,24 @@ struct WindowAttnParams {
   void* proj;               // [rows, stride]: q heads at q_off + h * D, k heads at k_off + g * D, v heads at v_off + g * DV
   int64_t stride;
   int q_off, k_off, v_off;
-  const float* wq;          // [D] fp32 norm weights (zero beyond dim)
+  const float* wq;          // fp32 norm weights, zero beyond dim: [D], or one row of the whole projection [hq * D] / [hkv * maps * D]
   const float* wk;
+  const float *bq, *bk, *bv;  // fp32 biases [hq * D], [hkv * maps * D], [hkv * DV], or null
+  const float* freq;        // [2, rot / 2]: rotation frequencies, leading and residual term
   void* k_cache;
   void* v_cache;
   const int32_t* block_table;
   const int32_t* row_req;
   const int32_t* positions;
   const int32_t* row_list;  // optional: the rows of this launch (else 0 .. grid - 1)
-  float* part_ml;           // [rows, hq, splits, 2]   (splits > 1)
-  float* part_acc;          // [rows, hq, splits, DV]
+  float* part_ml;           // [launch rows, hq, splits, 2]   (splits > 1 or two maps; else null)
+  float* part_acc;          // [launch rows, hq, splits, DV]
   void* out;                // [rows, out_stride] head h at column h * DV
   int64_t out_stride;
-  int hq, hkv, D, DV, dim, page, max_blocks, splits, window, fused;
-  float scale, eps, out_scale;
+  int hq, hkv, maps, D, DV, dim, page, max_blocks, splits, window, chunked, fused;
+  int norm;                 // 0: none, 1: per head, 2: over the whole projection
+  int rot, temp_every, gate_off;   // gate_off: column of the row with the gate of head 0 (negative: no gate)
+  float scale, eps, out_scale, temp_coef;
 };
 
 constexpr int kWaWarps = 4;
@@ -50,67 +67,130 @@ __device__ __forceinline__ float wa_exp<float>(float x) { return expf(x); }
 template <>
 __device__ __forceinline__ float wa_exp<bf16>(float x) { return __expf(x); }
 
-__device__ __forceinline__ size_t wa_token(const WindowAttnParams& p, const int32_t* bt, int g, int t) {
-  return (static_cast<size_t>(bt[t / p.page]) * p.hkv + g) * p.page + t % p.page;
+__device__ __forceinline__ size_t wa_token(const WindowAttnParams& p, const int32_t* bt, int heads, int g, int t) {
+  return (static_cast<size_t>(bt[t / p.page]) * heads + g) * p.page + t % p.page;
 }
 
-// 1 / rms of one head, by one warp
+__device__ __forceinline__ float wa_temperature(const WindowAttnParams& p, int pos) {
+  return p.temp_coef == 0.f ? 1.f : fmaf(p.temp_coef, logf(static_cast<float>((pos + 1) / p.temp_every) + 1.f), 1.f);
+}
+
+// Sum of squares of n columns (bias added), this thread's part.
 template <typename T>
-__device__ __forceinline__ float wa_rstd(const T* src, int D, int dim, float eps, int lane) {
+__device__ __forceinline__ float wa_squares(const T* src, const float* bias, int n, int first, int step) {
+  constexpr int VN = Vec16<T>::N;
   float ss = 0.f;
-  for (int d = lane; d < D; d += 32) {
-    const float f = ld_elem(src + d);
-    ss += f * f;
+  for (int c = first * VN; c < n; c += step * VN) {
+    float f[VN];
+    Vec16<T>::load(src + c, f);
+#pragma unroll
+    for (int j = 0; j < VN; ++j) {
+      const float v = f[j] + (bias != nullptr ? bias[c + j] : 0.f);
+      ss = fmaf(v, v, ss);
+    }
   }
-  return 1.f / sqrtf(warp_sum_f32(ss) / static_cast<float>(dim) + eps);
+  return ss;
+}
+
+// One query or key head by one warp: bias, norm (`rstd` of the whole projection, or the head's own), rotation and a factor into dst,
+// which may be src (a lane holds both columns of a rotated pair).
+template <typename T, typename D>
+__device__ __noinline__ void wa_head(const WindowAttnParams& p, const T* src, const float* bias, const float* w, float rstd, float factor, int pos,
+                                        int lane, D* dst) {
+  float r = factor;
+  if (p.norm == 1) r *= 1.f / sqrtf(warp_sum_f32(wa_squares(src, bias, p.D, lane, 32)) / static_cast<float>(p.dim) + p.eps);
+  else if (p.norm == 2) r *= rstd;
+  auto value = [&](int d) { return (ld_elem(src + d) + (bias != nullptr ? bias[d] : 0.f)) * (p.norm ? r * w[d] : r); };
+  const int half = p.rot / 2;
+#pragma unroll 1
+  for (int i = lane; i < half; i += 32) {
+    float s, c;
+    rope_angle(p.freq, half, pos, i, s, c);
+    const float a = value(i), b = value(i + half);
+    st_elem(dst + i, a * c - b * s);
+    st_elem(dst + i + half, b * c + a * s);
+  }
+#pragma unroll 2
+  for (int d = p.rot + lane; d < p.D; d += 32) st_elem(dst + d, value(d));
 }
 
 template <typename T>
-__global__ void __launch_bounds__(128) qk_norm_append_kernel(WindowAttnParams p, int rows) {
-  pdl_wait();
-  const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
-  const int heads = p.hq + 2 * p.hkv;
-  if (warp >= rows * heads) return;
-  const int row = warp / heads, head = warp % heads;
-  T* base = static_cast<T*>(p.proj) + static_cast<size_t>(row) * p.stride;
-  if (head < p.hq) {
-    T* q = base + p.q_off + static_cast<size_t>(head) * p.D;
-    const float r = wa_rstd(q, p.D, p.dim, p.eps, lane);
-    for (int d = lane; d < p.D; d += 32) st_elem(q + d, ld_elem(q + d) * r * p.wq[d]);
-    return;
-  }
-  const int32_t* bt = p.block_table + static_cast<size_t>(p.row_req[row]) * p.max_blocks;
-  const int g = (head - p.hq) % p.hkv;
-  const size_t tok = wa_token(p, bt, g, p.positions[row]);
-  if (head < p.hq + p.hkv) {
-    const T* k = base + p.k_off + static_cast<size_t>(g) * p.D;
-    T* dst = static_cast<T*>(p.k_cache) + tok * p.D;
-    const float r = wa_rstd(k, p.D, p.dim, p.eps, lane);
-    for (int d = lane; d < p.D; d += 32) st_elem(dst + d, ld_elem(k + d) * r * p.wk[d]);
-  } else {
-    const T* v = base + p.v_off + static_cast<size_t>(g) * p.DV;
-    T* dst = static_cast<T*>(p.v_cache) + tok * p.DV;
-    for (int d = lane; d < p.DV; d += 32) dst[d] = v[d];
+__device__ __noinline__ void wa_append_key(const WindowAttnParams& p, const T* base, const int32_t* bt, int g, float rstd, int pos, int lane) {
+  const size_t o = static_cast<size_t>(g) * p.D;
+  wa_head(p, base + p.k_off + o, p.bk ? p.bk + o : nullptr, p.norm == 2 ? p.wk + o : p.wk, rstd, 1.f, pos, lane,
+          static_cast<T*>(p.k_cache) + wa_token(p, bt, p.hkv * p.maps, g, pos) * p.D);
+}
+
+template <typename T>
+__device__ __forceinline__ void wa_append_value(const WindowAttnParams& p, const T* base, const int32_t* bt, int g, int pos, int lane) {
+  const T* v = base + p.v_off + static_cast<size_t>(g) * p.DV;
+  T* dst = static_cast<T*>(p.v_cache) + wa_token(p, bt, p.hkv, g, pos) * p.DV;
+  for (int d = lane; d < p.DV; d += 32) {
+    if (p.bv == nullptr) dst[d] = v[d];
+    else st_elem(dst + d, ld_elem(v + d) + p.bv[g * p.DV + d]);
   }
 }
 
-// grid (hkv * head_chunks, splits, rows).  NG query heads of one kv head per CTA; a warp scores 32 keys at a time (lane =
-// key), then the lanes take value columns 2 * lane + 64 * j.
-template <typename T, int NV, int NG>
-__global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(WindowAttnParams p) {
-  constexpr int DV = NV * 64, VN = Vec16<T>::N;
+// 1 / root mean square of all query columns (part 0) or all key columns (part 1) of a row, by the whole CTA.
+template <typename T>
+__device__ __forceinline__ float wa_row_rstd(const WindowAttnParams& p, const T* base, int part, float* scratch) {
+  const int heads = part ? p.hkv * p.maps : p.hq;
+  const float ss = wa_squares(base + (part ? p.k_off : p.q_off), part ? p.bk : p.bq, heads * p.D, threadIdx.x, blockDim.x);
+  return 1.f / sqrtf(block_sum_f32(ss, scratch) / static_cast<float>(heads * p.dim) + p.eps);
+}
+
+// grid (rows)
+template <typename T>
+__global__ void __launch_bounds__(256) qk_norm_append_kernel(const __grid_constant__ WindowAttnParams p) {
+  __shared__ float scratch[8];
+  pdl_wait();
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hk = p.hkv * p.maps;
+  T* base = static_cast<T*>(p.proj) + static_cast<size_t>(row) * p.stride;
+  float rq = 1.f, rk = 1.f;
+  if (p.norm == 2) {
+    rq = wa_row_rstd(p, base, 0, scratch);
+    rk = wa_row_rstd(p, base, 1, scratch);
+  }
+  const int pos = p.positions[row];
+  const float temp = wa_temperature(p, pos);
+  const int32_t* bt = p.block_table + static_cast<size_t>(p.row_req[row]) * p.max_blocks;
+  for (int head = warp; head < p.hq + hk + p.hkv; head += 8) {
+    if (head < p.hq) {
+      const size_t o = static_cast<size_t>(head) * p.D;
+      T* q = base + p.q_off + o;
+      wa_head(p, q, p.bq ? p.bq + o : nullptr, p.norm == 2 ? p.wq + o : p.wq, rq, temp, pos, lane, q);
+    } else if (head < p.hq + hk) {
+      wa_append_key(p, base, bt, head - p.hq, rk, pos, lane);
+    } else {
+      wa_append_value(p, base, bt, head - p.hq - hk, pos, lane);
+    }
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ float wa_gate(const WindowAttnParams& p, int row, int h) {
+  return p.gate_off < 0 ? p.out_scale
+                        : p.out_scale * sigmoid_f32(ld_elem(static_cast<const T*>(p.proj) + static_cast<size_t>(row) * p.stride + p.gate_off + h));
+}
+
+// grid (hkv * head_chunks, splits, rows).  NG query heads of one kv head per CTA, NG / MAPS of every map; a warp scores 32 keys at a
+// time (lane = key), then the lanes take value columns 2 * lane + 64 * j.
+template <typename T, int NV, int NG, int MAPS>
+__global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(const __grid_constant__ WindowAttnParams p) {
+  constexpr int DV = NV * 64, VN = Vec16<T>::N, NGM = NG / MAPS;
   extern __shared__ __align__(16) float wa_smem[];
   float* q_s = wa_smem;                                   // [NG][D]
   float* red_acc = q_s + NG * p.D;                        // [warps][NG][DV]
-  __shared__ float red_m[kWaWarps][NG], red_l[kWaWarps][NG];
+  __shared__ float red_m[kWaWarps][NG], red_l[kWaWarps][NG], scratch[kWaWarps];
   pdl_wait();
-  const int group = p.hq / p.hkv, chunks = (group + NG - 1) / NG;
-  const int kvh = blockIdx.x / chunks, g0 = (blockIdx.x % chunks) * NG;
+  const int group = p.hq / (p.hkv * MAPS), chunks = (group + NGM - 1) / NGM, hk = p.hkv * MAPS;
+  const int kvh = blockIdx.x / chunks, g0 = (blockIdx.x % chunks) * NGM;
   const int split = blockIdx.y, row = p.row_list ? p.row_list[blockIdx.z] : static_cast<int>(blockIdx.z);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pos = p.positions[row];
-  const int ng = min(NG, group - g0), h0 = kvh * group + g0;
-  const int first = max(0, pos + 1 - p.window), len = pos + 1;
+  const int ng = min(NGM, group - g0);
+  auto head_of = [&](int i) { return (kvh * MAPS + i / NGM) * group + g0 + min(i % NGM, ng - 1); };
+  const int first = p.chunked ? pos - pos % p.window : max(0, pos + 1 - p.window), len = pos + 1;
   int per = (len - first + p.splits - 1) / p.splits;
   per = (per + 31) & ~31;
   const int t_begin = first + split * per;
@@ -120,21 +200,30 @@ __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(WindowAttnPa
   const T* kc = static_cast<const T*>(p.k_cache);
   const T* vc = static_cast<const T*>(p.v_cache);
 
-  for (int g = warp; g < NG; g += kWaWarps) {
-    const T* q = base + p.q_off + static_cast<size_t>(h0 + min(g, ng - 1)) * p.D;
-    const float r = p.fused ? wa_rstd(q, p.D, p.dim, p.eps, lane) * p.scale : p.scale;
-    for (int d = lane; d < p.D; d += 32) q_s[g * p.D + d] = ld_elem(q + d) * r * (p.fused ? p.wq[d] : 1.f);
-  }
-  if (p.fused && t_begin < len && t_end == len && warp == kWaWarps - 1) {
-    // the CTA that reads the row's own position appends it (head chunks of one kv head write the same bytes)
-    const size_t tok = wa_token(p, bt, kvh, pos);
-    const T* k = base + p.k_off + static_cast<size_t>(kvh) * p.D;
-    const T* v = base + p.v_off + static_cast<size_t>(kvh) * p.DV;
-    const float r = wa_rstd(k, p.D, p.dim, p.eps, lane);
-    T* kd = static_cast<T*>(p.k_cache) + tok * p.D;
-    T* vd = static_cast<T*>(p.v_cache) + tok * p.DV;
-    for (int d = lane; d < p.D; d += 32) st_elem(kd + d, ld_elem(k + d) * r * p.wk[d]);
-    for (int d = lane; d < p.DV; d += 32) vd[d] = v[d];
+  // the CTA that reads the row's own position appends it (head chunks of one kv head write the same bytes)
+  const bool append = p.fused && t_begin < len && t_end == len;
+  if (p.fused) {
+    float rq = 1.f, rk = 1.f;
+    if (p.norm == 2) {
+      rq = wa_row_rstd(p, base, 0, scratch);
+      if (append) rk = wa_row_rstd(p, base, 1, scratch);
+    }
+    const float f = p.scale * wa_temperature(p, pos);
+    for (int i = warp; i < NG + (append ? MAPS + 1 : 0); i += kWaWarps) {
+      if (i < NG) {
+        const size_t o = static_cast<size_t>(head_of(i)) * p.D;
+        wa_head(p, base + p.q_off + o, p.bq ? p.bq + o : nullptr, p.norm == 2 ? p.wq + o : p.wq, rq, f, pos, lane, q_s + i * p.D);
+      } else if (i < NG + MAPS) {
+        wa_append_key(p, base, bt, kvh * MAPS + i - NG, rk, pos, lane);
+      } else {
+        wa_append_value(p, base, bt, kvh, pos, lane);
+      }
+    }
+  } else {
+    for (int i = warp; i < NG; i += kWaWarps) {
+      const T* q = base + p.q_off + static_cast<size_t>(head_of(i)) * p.D;
+      for (int d = lane; d < p.D; d += 32) q_s[i * p.D + d] = ld_elem(q + d) * p.scale;
+    }
   }
   __syncthreads();
 
@@ -149,24 +238,29 @@ __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(WindowAttnPa
   for (int t0 = t_begin + warp * 32; t0 < t_end; t0 += kWaWarps * 32) {
     const int t = t0 + lane;
     const bool valid = t < t_end;
-    const size_t tok = wa_token(p, bt, kvh, valid ? t : t_end - 1);
+    const int tv = valid ? t : t_end - 1;
+    const size_t tok = wa_token(p, bt, p.hkv, kvh, tv);
     float s[NG];
 #pragma unroll
     for (int g = 0; g < NG; ++g) s[g] = 0.f;
-    const T* kr = kc + tok * p.D;
+#pragma unroll
+    for (int m0 = 0; m0 < MAPS; ++m0) {
+      const T* kr = kc + (MAPS == 1 ? tok : wa_token(p, bt, hk, kvh * MAPS + m0, tv)) * p.D;
 #pragma unroll 4
-    for (int c = 0; c < p.D; c += VN) {
-      float kf[VN];
-      Vec16<T>::load(kr + c, kf);
+      for (int c = 0; c < p.D; c += VN) {
+        float kf[VN];
+        Vec16<T>::load(kr + c, kf);
 #pragma unroll
-      for (int g = 0; g < NG; ++g) {
+        for (int gm = 0; gm < NGM; ++gm) {
+          const int g = m0 * NGM + gm;
 #pragma unroll
-        for (int j = 0; j < VN; j += 4) {
-          const float4 q4 = *reinterpret_cast<const float4*>(q_s + g * p.D + c + j);
-          s[g] = fmaf(kf[j], q4.x, s[g]);
-          s[g] = fmaf(kf[j + 1], q4.y, s[g]);
-          s[g] = fmaf(kf[j + 2], q4.z, s[g]);
-          s[g] = fmaf(kf[j + 3], q4.w, s[g]);
+          for (int j = 0; j < VN; j += 4) {
+            const float4 q4 = *reinterpret_cast<const float4*>(q_s + g * p.D + c + j);
+            s[g] = fmaf(kf[j], q4.x, s[g]);
+            s[g] = fmaf(kf[j + 1], q4.y, s[g]);
+            s[g] = fmaf(kf[j + 2], q4.z, s[g]);
+            s[g] = fmaf(kf[j + 3], q4.w, s[g]);
+          }
         }
       }
     }
@@ -212,8 +306,9 @@ __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(WindowAttnPa
     for (int j = 0; j < NV; ++j)
       *reinterpret_cast<float2*>(red_acc + (warp * NG + g) * DV + 64 * j + 2 * lane) = make_float2(acc[g][2 * j], acc[g][2 * j + 1]);
   __syncthreads();
-  for (int i = threadIdx.x; i < ng * DV; i += blockDim.x) {
+  for (int i = threadIdx.x; i < NG * DV; i += blockDim.x) {
     const int g = i / DV, d = i % DV;
+    if (g % NGM >= ng) continue;
     float mm = -INFINITY;
     for (int w = 0; w < kWaWarps; ++w) mm = fmaxf(mm, red_m[w][g]);
     float ll = 0.f, a = 0.f;
@@ -222,12 +317,12 @@ __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(WindowAttnPa
       ll += red_l[w][g] * c;
       a += red_acc[(w * NG + g) * DV + d] * c;
     }
-    const int h = h0 + g;
-    if (p.splits == 1) {
+    const int h = head_of(g);
+    if (p.part_ml == nullptr) {
       st_elem(static_cast<T*>(p.out) + static_cast<size_t>(row) * p.out_stride + static_cast<size_t>(h) * DV + d,
-              ll > 0.f ? a / ll * p.out_scale : 0.f);
+              ll > 0.f ? a / ll * wa_gate<T>(p, row, h) : 0.f);
     } else {
-      const size_t pi = (static_cast<size_t>(row) * p.hq + h) * p.splits + split;
+      const size_t pi = (static_cast<size_t>(blockIdx.z) * p.hq + h) * p.splits + split;
       p.part_acc[pi * DV + d] = a;
       if (d == 0) { p.part_ml[pi * 2] = mm; p.part_ml[pi * 2 + 1] = ll; }
     }
@@ -240,7 +335,7 @@ __global__ void __launch_bounds__(256) window_attn_combine_kernel(WindowAttnPara
   pdl_wait();
   const int row = p.row_list ? p.row_list[blockIdx.y] : static_cast<int>(blockIdx.y);
   const int h = blockIdx.x, d = threadIdx.x;
-  const size_t rh = static_cast<size_t>(row) * p.hq + h;
+  const size_t rh = static_cast<size_t>(blockIdx.y) * p.hq + h;
   float mm = -INFINITY;
   for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, p.part_ml[(rh * p.splits + s) * 2]);
   float ll = 0.f, a = 0.f;
@@ -251,21 +346,83 @@ __global__ void __launch_bounds__(256) window_attn_combine_kernel(WindowAttnPara
     a += p.part_acc[(rh * p.splits + s) * p.DV + d] * c;
   }
   st_elem(static_cast<T*>(p.out) + static_cast<size_t>(row) * p.out_stride + static_cast<size_t>(h) * p.DV + d,
-          ll > 0.f ? a / ll * p.out_scale : 0.f);
+          ll > 0.f ? a / ll * wa_gate<T>(p, row, h) : 0.f);
 }
 
-template <typename T, int NV, int NG>
+struct DiffCombine {
+  const float* ml;          // [n, 2 heads, splits, 2], or null: acc holds finished outputs [rows, 2 heads, DV]
+  const float* acc;         // [n, 2 heads, splits, DV]
+  const void* gate;         // [rows, gate_stride] (T), column h * DV + d
+  int64_t gate_stride;
+  void* out;                // [rows, out_stride] (T)
+  int64_t out_stride;
+  const int32_t* row_list;
+  int n, heads, group, vdim, splits;
+  float lambda, factor, eps;
+};
+
+// One warp per (row, output head), four warps per CTA; value columns 2 * lane + 64 * j.
+template <typename T, int NV>
+__global__ void __launch_bounds__(128) diff_combine_kernel(DiffCombine p) {
+  constexpr int DV = NV * 64;
+  pdl_wait();
+  const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= p.n * p.heads) return;
+  const int i = unit / p.heads, h = unit % p.heads, row = p.row_list ? p.row_list[i] : i;
+  float2 o[NV];
+#pragma unroll
+  for (int map = 0; map < 2; ++map) {
+    const size_t rh = static_cast<size_t>(p.ml != nullptr ? i : row) * 2 * p.heads + (h / p.group * 2 + map) * p.group + h % p.group;
+    float2 a[NV];
+#pragma unroll
+    for (int j = 0; j < NV; ++j) a[j] = make_float2(0.f, 0.f);
+    float mm = -INFINITY, ll = 0.f;
+    if (p.ml != nullptr)
+      for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, p.ml[(rh * p.splits + s) * 2]);
+    for (int s = 0; s < p.splits; ++s) {
+      float c = 1.f;
+      if (p.ml != nullptr) {
+        const float ms = p.ml[(rh * p.splits + s) * 2];
+        c = ms == -INFINITY ? 0.f : wa_exp<T>(ms - mm);
+        ll += p.ml[(rh * p.splits + s) * 2 + 1] * c;
+      }
+#pragma unroll
+      for (int j = 0; j < NV; ++j) {
+        const float2 v = *reinterpret_cast<const float2*>(p.acc + (rh * p.splits + s) * DV + 64 * j + 2 * lane);
+        a[j].x = fmaf(v.x, c, a[j].x);
+        a[j].y = fmaf(v.y, c, a[j].y);
+      }
+    }
+    const float r = p.ml == nullptr ? 1.f : (ll > 0.f ? 1.f / ll : 0.f), f = map ? -p.lambda * r : r;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) o[j] = map ? make_float2(fmaf(a[j].x, f, o[j].x), fmaf(a[j].y, f, o[j].y)) : make_float2(a[j].x * f, a[j].y * f);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) ss = fmaf(o[j].x, o[j].x, fmaf(o[j].y, o[j].y, ss));
+  const float r = p.factor / sqrtf(warp_sum_f32(ss) / static_cast<float>(p.vdim) + p.eps);
+  const T* gate = static_cast<const T*>(p.gate) + row * p.gate_stride + static_cast<size_t>(h) * DV + 2 * lane;
+  T* dst = static_cast<T*>(p.out) + row * p.out_stride + static_cast<size_t>(h) * DV + 2 * lane;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const float2 g = ld_elem2(gate + 64 * j);
+    st_elem(dst + 64 * j, o[j].x * r * sigmoid_f32(g.x));
+    st_elem(dst + 64 * j + 1, o[j].y * r * sigmoid_f32(g.y));
+  }
+}
+
+template <typename T, int NV, int NG, int MAPS>
 static int launch_wa(const WindowAttnParams& p, int rows, cudaStream_t st) {
-  const int chunks = dgpp_ceil_div(p.hq / p.hkv, NG);
+  const int chunks = dgpp_ceil_div(p.hq / (p.hkv * MAPS), NG / MAPS);
   const size_t smem = (static_cast<size_t>(NG) * p.D + static_cast<size_t>(kWaWarps) * NG * NV * 64) * sizeof(float);
   static bool attr = false;
   if (!attr) {
-    DGPP_CUDA_OK(cudaFuncSetAttribute(window_attn_kernel<T, NV, NG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(window_attn_kernel<T, NV, NG, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
     attr = true;
   }
-  window_attn_kernel<T, NV, NG><<<dim3(p.hkv * chunks, p.splits, rows), kWaWarps * 32, smem, st>>>(p);
+  window_attn_kernel<T, NV, NG, MAPS><<<dim3(p.hkv * chunks, p.splits, rows), kWaWarps * 32, smem, st>>>(p);
   DGPP_CUDA_OK(cudaGetLastError());
-  if (p.splits > 1) {
+  if (MAPS == 1 && p.splits > 1) {
     window_attn_combine_kernel<T><<<dim3(p.hq, rows), NV * 64, 0, st>>>(p);
     DGPP_CUDA_OK(cudaGetLastError());
   }
@@ -274,11 +431,16 @@ static int launch_wa(const WindowAttnParams& p, int rows, cudaStream_t st) {
 
 template <typename T, int NV>
 static int launch_wa_g(const WindowAttnParams& p, int rows, cudaStream_t st) {
-  const int g = p.hq / p.hkv;
-  if (g == 1) return launch_wa<T, NV, 1>(p, rows, st);
-  if (g == 2) return launch_wa<T, NV, 2>(p, rows, st);
-  if (g <= 4) return launch_wa<T, NV, 4>(p, rows, st);
-  return launch_wa<T, NV, 8>(p, rows, st);
+  const int g = p.hq / (p.hkv * p.maps);
+  if (p.maps == 2) {
+    if (g == 1) return launch_wa<T, NV, 2, 2>(p, rows, st);
+    if (g == 2) return launch_wa<T, NV, 4, 2>(p, rows, st);
+    return launch_wa<T, NV, 8, 2>(p, rows, st);
+  }
+  if (g == 1) return launch_wa<T, NV, 1, 1>(p, rows, st);
+  if (g == 2) return launch_wa<T, NV, 2, 1>(p, rows, st);
+  if (g <= 4) return launch_wa<T, NV, 4, 1>(p, rows, st);
+  return launch_wa<T, NV, 8, 1>(p, rows, st);
 }
 
 template <typename T>
@@ -290,12 +452,15 @@ static int launch_wa_v(const WindowAttnParams& p, int rows, cudaStream_t st) {
 }
 
 static int wa_check(const WindowAttnParams& p, int rows) {
-  DGPP_REQUIRE(p.hkv > 0 && p.hq % p.hkv == 0, "window_attn: %d query heads over %d key heads", p.hq, p.hkv);
+  DGPP_REQUIRE((p.maps == 1 || p.maps == 2) && p.hkv > 0 && p.hq % (p.hkv * p.maps) == 0, "window_attn: %d query heads over %d x %d key heads", p.hq, p.hkv, p.maps);
+  DGPP_REQUIRE(p.norm >= 0 && p.norm <= 2 && (!p.norm || (p.wq && p.wk)), "window_attn: norm %d needs its weights", p.norm);
+  DGPP_REQUIRE(p.rot >= 0 && p.rot % 2 == 0 && p.rot <= p.dim && (p.rot == 0 || p.freq), "window_attn: %d of %d columns rotated", p.rot, p.dim);
+  DGPP_REQUIRE(p.temp_coef == 0.f || p.temp_every >= 1, "window_attn: temperature every %d", p.temp_every);
   DGPP_REQUIRE(p.D % 64 == 0 && p.D >= 64 && p.D <= 256 && p.DV % 64 == 0 && p.DV >= 64 && p.DV <= 256,
                "window_attn: head widths %d / %d (padded to multiples of 64, at most 256)", p.D, p.DV);
   DGPP_REQUIRE(p.stride % 8 == 0 && p.q_off % 8 == 0 && p.k_off % 8 == 0 && p.v_off % 8 == 0, "window_attn: unaligned projection rows");
   DGPP_REQUIRE(p.window >= 1 && p.splits >= 1 && p.page >= 1 && p.dim >= 1 && p.dim <= p.D, "window_attn: window %d splits %d", p.window, p.splits);
-  DGPP_REQUIRE(p.splits == 1 || (p.part_ml && p.part_acc), "window_attn: scratch required when splits > 1");
+  DGPP_REQUIRE(p.part_ml ? p.part_acc != nullptr : p.splits == 1, "window_attn: scratch required when splits > 1");
   DGPP_REQUIRE(rows >= 0 && rows <= 65535, "window_attn: %d rows", rows);
   return 0;
 }
@@ -304,51 +469,73 @@ static int wa_check(const WindowAttnParams& p, int rows) {
 
 using namespace dgpp;
 
-static WindowAttnParams wa_params(void* proj, int64_t stride, int q_off, int k_off, int v_off, const void* wq, const void* wk,
-                                  void* k_cache, void* v_cache, const void* block_table, const void* row_req,
-                                  const void* positions, int hq, int hkv, int D, int DV, int dim, int page, int max_blocks, float eps) {
+// What every entry point takes: see WindowAttnParams.  bq / bk / bv, freq (rot = 0) and the norm weights (norm = 0) may be null.
+#define WA_COMMON                                                                                                                      \
+  void *proj, int64_t stride, int q_off, int k_off, int v_off, const void *wq, const void *wk, const void *bq, const void *bk,          \
+      const void *bv, const void *freq, void *k_cache, void *v_cache, const void *block_table, const void *row_req,                    \
+      const void *positions, int rows, int hq, int hkv, int maps, int D, int DV, int dim, int page, int max_blocks, int norm, int rot,  \
+      int temp_every, float temp_coef, float eps
+
+static WindowAttnParams wa_params(WA_COMMON) {
   WindowAttnParams p;
+  memset(&p, 0, sizeof(p));
   p.proj = proj; p.stride = stride; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off;
-  p.wq = static_cast<const float*>(wq); p.wk = static_cast<const float*>(wk);
+  auto f = [](const void* q) { return static_cast<const float*>(q); };
+  p.wq = f(wq); p.wk = f(wk); p.bq = f(bq); p.bk = f(bk); p.bv = f(bv); p.freq = f(freq);
   p.k_cache = k_cache; p.v_cache = v_cache;
   p.block_table = static_cast<const int32_t*>(block_table);
   p.row_req = static_cast<const int32_t*>(row_req);
   p.positions = static_cast<const int32_t*>(positions);
-  p.row_list = nullptr; p.part_ml = nullptr; p.part_acc = nullptr; p.out = nullptr; p.out_stride = 0;
-  p.hq = hq; p.hkv = hkv; p.D = D; p.DV = DV; p.dim = dim; p.page = page; p.max_blocks = max_blocks;
-  p.splits = 1; p.window = 1; p.fused = 0; p.scale = 1.f; p.eps = eps; p.out_scale = 1.f;
+  p.hq = hq; p.hkv = hkv; p.maps = maps; p.D = D; p.DV = DV; p.dim = dim; p.page = page; p.max_blocks = max_blocks;
+  p.norm = norm; p.rot = rot; p.temp_every = temp_every; p.temp_coef = temp_coef; p.eps = eps;
+  p.splits = 1; p.window = 1; p.scale = 1.f; p.out_scale = 1.f; p.gate_off = -1;
   return p;
 }
+#define WA_ARGS                                                                                                                   \
+  proj, stride, q_off, k_off, v_off, wq, wk, bq, bk, bv, freq, k_cache, v_cache, block_table, row_req, positions, rows, hq, hkv, maps, D, \
+      DV, dim, page, max_blocks, norm, rot, temp_every, temp_coef, eps
 
-DGPP_API int dgpp_qk_norm_append(void* proj, int64_t stride, int q_off, int k_off, int v_off, const void* wq, const void* wk,
-                                 void* k_cache, void* v_cache, const void* block_table, const void* row_req, const void* positions,
-                                 int rows, int hq, int hkv, int D, int DV, int dim, int page, int max_blocks, float eps, int f32,
-                                 cudaStream_t st) {
-  const WindowAttnParams p = wa_params(proj, stride, q_off, k_off, v_off, wq, wk, k_cache, v_cache, block_table, row_req, positions,
-                                       hq, hkv, D, DV, dim, page, max_blocks, eps);
+DGPP_API int dgpp_qk_norm_append(WA_COMMON, int f32, cudaStream_t st) {
+  const WindowAttnParams p = wa_params(WA_ARGS);
   if (wa_check(p, rows)) return -1;
   if (rows == 0) return 0;
-  const int blocks = dgpp_ceil_div(rows * (hq + 2 * hkv), 4);
-  if (f32) qk_norm_append_kernel<float><<<blocks, 128, 0, st>>>(p, rows);
-  else qk_norm_append_kernel<bf16><<<blocks, 128, 0, st>>>(p, rows);
+  if (f32) qk_norm_append_kernel<float><<<rows, 256, 0, st>>>(p);
+  else qk_norm_append_kernel<bf16><<<rows, 256, 0, st>>>(p);
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;
 }
 
 // rows: rows of this launch (row_list, int32, names them when given).  fused: see the header.  out_scale multiplies the
-// outputs before they are rounded.  part_ml / part_acc: rows of the whole pass * hq * splits * (2 | DV) floats.
-DGPP_API int dgpp_window_attn(void* proj, int64_t stride, int q_off, int k_off, int v_off, const void* wq, const void* wk,
-                              void* k_cache, void* v_cache, const void* block_table, const void* row_req, const void* positions,
-                              const void* row_list, void* part_ml, void* part_acc, void* out, int64_t out_stride, int rows,
-                              int hq, int hkv, int D, int DV, int dim, int page, int max_blocks, int splits, int window, int fused,
-                              float scale, float eps, float out_scale, int f32, cudaStream_t st) {
-  WindowAttnParams p = wa_params(proj, stride, q_off, k_off, v_off, wq, wk, k_cache, v_cache, block_table, row_req, positions,
-                                 hq, hkv, D, DV, dim, page, max_blocks, eps);
+// outputs before they are rounded.  part_ml / part_acc: rows * hq * splits * (2 | DV) floats; with two maps they are the result (null
+// out), which `dgpp_diff_combine` finishes.
+DGPP_API int dgpp_window_attn(WA_COMMON, const void* row_list, void* part_ml, void* part_acc, void* out, int64_t out_stride, int splits,
+                              int window, int chunked, int fused, int gate_off, float scale, float out_scale, int f32, cudaStream_t st) {
+  WindowAttnParams p = wa_params(WA_ARGS);
   p.row_list = static_cast<const int32_t*>(row_list);
   p.part_ml = static_cast<float*>(part_ml); p.part_acc = static_cast<float*>(part_acc);
   p.out = out; p.out_stride = out_stride;
-  p.splits = splits; p.window = window; p.fused = fused; p.scale = scale; p.out_scale = out_scale;
+  p.splits = splits; p.window = window; p.chunked = chunked; p.fused = fused; p.gate_off = gate_off; p.scale = scale; p.out_scale = out_scale;
   if (wa_check(p, rows)) return -1;
+  DGPP_REQUIRE(maps == 1 ? out != nullptr && (splits > 1) == (part_ml != nullptr) : part_ml != nullptr, "window_attn: no place for the result");
   if (rows == 0) return 0;
   return f32 ? launch_wa_v<float>(p, rows, st) : launch_wa_v<bf16>(p, rows, st);
+}
+
+// out[row, h] = rms-normed (a1 - lambda a2) * factor * sigmoid(gate) for n rows (row_list names them when given) of `heads` output
+// heads, `group` per kv head; ml null: acc holds finished outputs of all rows of the pass (one split).
+DGPP_API int dgpp_diff_combine(const void* ml, const void* acc, const void* gate, int64_t gate_stride, const void* row_list, void* out,
+                               int64_t out_stride, int n, int heads, int group, int DV, int vdim, int splits, float lambda, float factor, float eps,
+                               int f32, cudaStream_t st) {
+  DGPP_REQUIRE(DV % 64 == 0 && DV >= 64 && DV <= 256 && vdim >= 1 && vdim <= DV && group >= 1 && heads % group == 0 && splits >= 1 && (ml || splits == 1),
+               "diff_combine: %d heads of %d columns, %d splits", heads, DV, splits);
+  if (n == 0) return 0;
+  const DiffCombine p = {static_cast<const float*>(ml), static_cast<const float*>(acc), gate, gate_stride, out, out_stride,
+                         static_cast<const int32_t*>(row_list), n, heads, group, vdim, splits, lambda, factor, eps};
+  const int64_t grid = dgpp_ceil_div64(static_cast<int64_t>(n) * heads, 4);
+#define DGPP_DC(NV) if (DV == NV * 64) { if (f32) diff_combine_kernel<float, NV><<<static_cast<unsigned>(grid), 128, 0, st>>>(p); \
+                                         else diff_combine_kernel<bf16, NV><<<static_cast<unsigned>(grid), 128, 0, st>>>(p); }
+  DGPP_DC(1) DGPP_DC(2) DGPP_DC(3) DGPP_DC(4)
+#undef DGPP_DC
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
 }

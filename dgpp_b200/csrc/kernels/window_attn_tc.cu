@@ -1,8 +1,8 @@
-// Sliding-window GQA for prompt rows on the 5th-generation tensor cores (bf16 queries, keys and values; see window_attn.cu
-// for the layer and the cache, whose new positions and normed queries `qk_norm_append` has written).
+// GQA for prompt rows on the 5th-generation tensor cores (bf16 queries, keys and values; see window_attn.cu for the layer, its windows,
+// chunks and maps, and for the cache, whose new positions and prepared queries `qk_norm_append` has written).
 //
-// One CTA = 128 query rows of one kv head: 128 / G consecutive tokens of one run with their G = hq / hkv query heads, row
-// r = token r / G, head r % G.  It walks the cache pages from the first key its first token sees to its last token:
+// One CTA = 128 query rows of one key head: 128 / G consecutive tokens of one run with their G = hq / hkv query heads, row
+// r = token r / G, head r % G (differential attention: `maps` key heads read the same values; finished fp32 outputs go to `raw`).  It walks the cache pages from the first key its first token sees to its last token:
 //
 //   MMA1     S[r, t] = q_r . k_t              (fp32 in TMEM, double buffered: tile i + 1 overlaps the softmax of tile i)
 //   softmax  one thread per row: running maximum, p = 2^(s - m), window and causal mask; p goes to shared memory as two
@@ -44,10 +44,11 @@ struct WindowTcParams {
   const int32_t* run_len;   // optional [runs]: the runs are not back to back
   const int32_t* flat_base; // [runs] (FLAT)
   const bf16* gate;         // optional [rows, stride]: sigmoid(gate[row, head]) multiplies the output
+  float* raw;               // optional [rows, hq, DV] fp32: the outputs instead of `out`
   bf16* out;
   int64_t out_stride;
   DeviceStatus* status;
-  int runs, hq, hkv, D, DV, max_blocks, window, stages;
+  int runs, hq, hkv, maps, D, DV, max_blocks, window, chunked, stages;   // hkv: key heads; value heads: hkv / maps
   int DN, rot_col;          // FLAT: key columns from the expanded rows; first rotated column of a gathered cache row
   float scale, out_scale;
 };
@@ -55,6 +56,9 @@ struct WindowTcParams {
 __device__ __forceinline__ uint32_t wt_sw128(uint32_t row, uint32_t byte_in_row) {
   return row * 128u + ((((byte_in_row >> 4) ^ (row & 7u)) << 4) | (byte_in_row & 15u));
 }
+
+// First position that the query at position i sees
+__device__ __forceinline__ int wt_first_key(const WindowTcParams& p, int i) { return p.chunked ? i - i % p.window : max(0, i + 1 - p.window); }
 
 // Largest masked score of 64 keys (row of this thread)
 template <bool kMask>
@@ -153,7 +157,7 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   }
   const int first_pos = p.positions[row0], last_pos = first_pos + ntok - 1;
   const int32_t* bt = p.block_table + static_cast<size_t>(p.row_req[row0]) * p.max_blocks;
-  const int page0 = max(0, first_pos + 1 - p.window) / kWtKeys, base = page0 * kWtKeys;
+  const int page0 = wt_first_key(p, first_pos) / kWtKeys, base = page0 * kWtKeys;
   const int ntiles = ntok > 0 ? last_pos / kWtKeys - page0 + 1 : 0;
   if (warp >= 2) {
     // ---- this thread's query row into the swizzled A operand
@@ -186,9 +190,9 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
           for (int a = nn; a < natom; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmV, p.rot_col + (a - nn) * 64, y, &kv_full[s]);
           for (int a = 0; a < vatom; ++a) tma_load_2d(sV + (s * vatom + a) * kblk, &tmK, p.hq * p.DN + kvh * p.DV + a * 64, y, &kv_full[s]);
         } else {
-          const int y = (bt[page0 + i] * p.hkv + kvh) * kWtKeys;
+          const int y = (bt[page0 + i] * p.hkv + kvh) * kWtKeys, yv = (bt[page0 + i] * (p.hkv / p.maps) + kvh / p.maps) * kWtKeys;
           for (int a = 0; a < natom; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmK, a * 64, y, &kv_full[s]);
-          for (int a = 0; a < vatom; ++a) tma_load_2d(sV + (s * vatom + a) * kblk, &tmV, a * 64, y, &kv_full[s]);
+          for (int a = 0; a < vatom; ++a) tma_load_2d(sV + (s * vatom + a) * kblk, &tmV, a * 64, yv, &kv_full[s]);
         }
         if (*abort_flag) break;
       }
@@ -245,7 +249,7 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     const int quad = warp & 3, r = quad * 32 + lane, tok = r / group;
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const bool live = tok < ntok;
-    const int hi = first_pos + (live ? tok : 0), lo = max(0, hi + 1 - p.window);
+    const int hi = first_pos + (live ? tok : 0), lo = wt_first_key(p, hi);
     const float sm = p.scale * 1.4426950408889634f;
     float m_used = -INFINITY, l_run = 0.f;
     bool ok = true;
@@ -296,12 +300,18 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       } else {
         tc_fence_after();
         float f = l_run > 0.f ? p.out_scale / l_run : 0.f;
-        if (FLAT && p.gate != nullptr && live) f *= sigmoid_f32(bf16_to_f32(p.gate[static_cast<size_t>(row0 + tok) * p.stride + kvh * group + r % group]));
+        if (p.gate != nullptr && live) f *= sigmoid_f32(bf16_to_f32(p.gate[static_cast<size_t>(row0 + tok) * p.stride + kvh * group + r % group]));
+        float* dst32 = p.raw != nullptr ? p.raw + (static_cast<size_t>(row0 + (live ? tok : 0)) * p.hq + kvh * group + r % group) * p.DV : nullptr;
         bf16* dst = p.out + static_cast<size_t>(row0 + (live ? tok : 0)) * p.out_stride + static_cast<size_t>(kvh * group + r % group) * p.DV;
         for (int c0 = 0; c0 < p.DV; c0 += 16) {
           uint32_t raw[16];
           tmem_ld_x16(tmem_o + lane_addr + c0, raw);
-          if (live) {
+          if (live && dst32 != nullptr) {
+#pragma unroll
+            for (int j = 0; j < 16; j += 4)
+              *reinterpret_cast<float4*>(dst32 + c0 + j) = make_float4(__uint_as_float(raw[j]) * f, __uint_as_float(raw[j + 1]) * f,
+                                                                     __uint_as_float(raw[j + 2]) * f, __uint_as_float(raw[j + 3]) * f);
+          } else if (live) {
             Pack16 o[2];
 #pragma unroll
             for (int j = 0; j < 16; ++j) o[j >> 3].h[j & 7] = f32_to_bf16(__uint_as_float(raw[j]) * f);
@@ -322,7 +332,7 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 using namespace dgpp;
 
 static int wt_check(const void* proj, int64_t stride, int q_off, const void* out, int64_t out_stride, int runs, int hq, int hkv, int D, int DV,
-                    int page, int window) {
+                    int page, int window) {                    // hkv: key heads
   DGPP_REQUIRE(hkv > 0 && hq % hkv == 0 && hq / hkv <= kWtRows, "window_attn_tc: %d query heads over %d key heads", hq, hkv);
   DGPP_REQUIRE(D % 64 == 0 && D >= 64 && D <= 256 && DV % 64 == 0 && DV >= 64 && DV <= 256, "window_attn_tc: head widths %d / %d", D, DV);
   DGPP_REQUIRE(page == kWtKeys, "window_attn_tc: page %d (64)", page);
@@ -349,13 +359,17 @@ static int launch_wt(const CUtensorMap& tK, const CUtensorMap& tV, WindowTcParam
   return 0;
 }
 
-// Runs of consecutive rows (run_start [runs + 1]); `tiles` = sum over the runs of ceil(length / (128 / group)).  The cache
-// (pages of 64 tokens) holds the runs' own positions already.
+// Runs of consecutive rows (run_start [runs + 1], or run_start / run_len [runs]); `tiles` = sum over the runs of ceil(length / (128 /
+// group)), group = hq / (hkv * maps).  The cache (pages of 64 tokens) holds the runs' own positions already.  chunked: `window` is the
+// size of the chunks.  gate_off >= 0: the sigmoid of that column of a row, one per head, multiplies the head's output.  raw: fp32
+// outputs [rows, hq, DV] instead of `out`.
 DGPP_API int dgpp_window_attn_tc(const void* proj, int64_t stride, int q_off, const void* k_cache, const void* v_cache,
-                                 const void* block_table, const void* row_req, const void* positions, const void* run_start, void* out,
-                                 int64_t out_stride, int runs, int tiles, int hq, int hkv, int D, int DV, int page, int max_blocks,
-                                 int num_blocks, int window, float scale, float out_scale, cudaStream_t st) {
-  if (wt_check(proj, stride, q_off, out, out_stride, runs, hq, hkv, D, DV, page, window)) return -1;
+                                 const void* block_table, const void* row_req, const void* positions, const void* run_start, const void* run_len,
+                                 void* out, int64_t out_stride, void* raw, int runs, int tiles, int hq, int hkv, int maps, int D, int DV, int page,
+                                 int max_blocks, int num_blocks, int window, int chunked, int gate_off, float scale, float out_scale,
+                                 cudaStream_t st) {
+  DGPP_REQUIRE(maps == 1 || (maps == 2 && raw), "window_attn_tc: %d maps", maps);
+  if (wt_check(proj, stride, q_off, out, out_stride, runs, hq, hkv * maps, D, DV, page, window)) return -1;
   if (tiles == 0) return 0;
   WindowTcParams p;
   memset(&p, 0, sizeof(p));
@@ -364,13 +378,16 @@ DGPP_API int dgpp_window_attn_tc(const void* proj, int64_t stride, int q_off, co
   p.row_req = static_cast<const int32_t*>(row_req);
   p.positions = static_cast<const int32_t*>(positions);
   p.run_start = static_cast<const int32_t*>(run_start);
+  p.run_len = static_cast<const int32_t*>(run_len);
+  p.gate = gate_off >= 0 ? p.proj + gate_off : nullptr;
+  p.raw = static_cast<float*>(raw);
   p.out = static_cast<bf16*>(out); p.out_stride = out_stride;
   p.status = device_status_ptr();
-  p.runs = runs; p.hq = hq; p.hkv = hkv; p.D = D; p.DV = DV; p.max_blocks = max_blocks; p.window = window;
+  p.runs = runs; p.hq = hq; p.hkv = hkv * maps; p.maps = maps; p.chunked = chunked; p.D = D; p.DV = DV; p.max_blocks = max_blocks; p.window = window;
   p.scale = scale; p.out_scale = out_scale;
   const uint64_t rows = static_cast<uint64_t>(num_blocks) * hkv * page;
   CUtensorMap tK, tV;
-  if (make_tmap_2d(&tK, k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, rows, static_cast<uint64_t>(D) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B))
+  if (make_tmap_2d(&tK, k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, rows * maps, static_cast<uint64_t>(D) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
   if (make_tmap_2d(&tV, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, DV, rows, static_cast<uint64_t>(DV) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
@@ -401,7 +418,7 @@ DGPP_API int dgpp_latent_prefill_tc(const void* proj, int64_t stride, int q_off,
   p.gate = gate_off >= 0 ? p.proj + gate_off : nullptr;
   p.out = static_cast<bf16*>(out); p.out_stride = out_stride;
   p.status = device_status_ptr();
-  p.runs = runs; p.hq = heads; p.hkv = heads; p.D = dn + dr; p.DV = dv; p.window = window;
+  p.runs = runs; p.hq = heads; p.hkv = heads; p.maps = 1; p.D = dn + dr; p.DV = dv; p.window = window;
   p.DN = dn; p.rot_col = rot_col;
   p.scale = scale; p.out_scale = 1.f;
   const uint64_t cols = static_cast<uint64_t>(heads) * (dn + dv);

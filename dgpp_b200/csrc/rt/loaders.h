@@ -288,7 +288,7 @@ inline std::string resolve_model(const std::string& spec, const std::string& cac
 }
 
 // ------------------------------------------------------------------------------------------- architecture detect
-enum class Family { Unknown, QwenHybrid, QwenFlashNext, Glm4, GlmFlash, GlmDsa, DeepSeekV4, DeepSeekV41, MiMo, MiniMax, Flint, Dory, Sitirax, Potivik, DenseGqa };
+enum class Family { Unknown, QwenHybrid, QwenFlashNext, Glm4, GlmFlash, GlmDsa, DeepSeekV4, DeepSeekV41, MiMo, MiniMax, Flint, Dory, Sitirax, Potivik, Vevapel, DenseGqa };
 
 inline const char* family_name(Family f) {
   switch (f) {
@@ -305,6 +305,7 @@ inline const char* family_name(Family f) {
     case Family::Dory: return "dory";
     case Family::Sitirax: return "sitirax";
     case Family::Potivik: return "potivik";
+    case Family::Vevapel: return "vevapel";
     case Family::DenseGqa: return "dense_gqa";
     default: return "unknown";
   }
@@ -337,6 +338,7 @@ inline Family detect_family(const json::Value& config) {
   if (has("dory")) return Family::Dory;
   if (has("sitirax")) return Family::Sitirax;
   if (has("potivik")) return Family::Potivik;
+  if (has("vevapel")) return Family::Vevapel;
   if (has("qwen3") || has("qwen2") || has("llama") || has("mistral")) return Family::DenseGqa;
   throw std::runtime_error("detect_family: unsupported architecture '" + arch + "' / model_type '" + type + "'");
 }

@@ -53,7 +53,8 @@ class _PyBlockTable:
 class PagedKV:
     def __init__(self, layers: int, hkv: int, d: int, num_blocks: int, max_requests: int, max_blocks_per_req: int,
                  page: int = 64, fp8: bool = True, device="cuda", shapes=None, dtype=None):
-        """`shapes`: [(kv heads, key width, value width)] per layer when the layers differ (or values are not as wide as keys);
+        """`shapes`: [(kv heads, key width, value width[, value heads])] per layer when the layers differ (or values are not as wide as
+        keys, or fewer);
         `dtype`: storage of an unscaled cache (bf16 by default, fp32 for models that run in 32 bits)."""
         shapes = [(hkv, d, d)] * layers if shapes is None else list(shapes)
         assert len(shapes) == layers and (dtype is None or not fp8)
@@ -61,9 +62,9 @@ class PagedKV:
         self.num_blocks, self.max_requests, self.max_blocks = num_blocks, max_requests, max_blocks_per_req
         dt = torch.uint8 if fp8 else (dtype or torch.bfloat16)
         self.layers: List[KVLayer] = []
-        for hkv, d, dv in shapes:
+        for hkv, d, dv, *hv in shapes:
             k = torch.zeros(num_blocks, hkv, page, d, dtype=dt, device=device)
-            v = torch.zeros(num_blocks, hkv, page, dv, dtype=dt, device=device)
+            v = torch.zeros(num_blocks, hv[0] if hv else hkv, page, dv, dtype=dt, device=device)
             ks = torch.ones(num_blocks, hkv, page, dtype=torch.float32, device=device) if fp8 else None
             vs = torch.ones(num_blocks, hkv, page, dtype=torch.float32, device=device) if fp8 else None
             self.layers.append(KVLayer(k, v, ks, vs, page, fp8))

@@ -3,7 +3,7 @@ under its path in the model object (`layers.3.qkv.payload`, `layers.3.moe.expert
 `config.json` that names the family (`model_type` = "dgpp-<family>") and carries the configuration and the format of
 every quantised matrix.  `save_family` writes one; `load_family` rebuilds the model on a device.  Quantised payloads
 and scales travel byte for byte.  The fixture writer of the per-family load / bind / forward checks, and the hand-off
-format between a conversion script and the server for these families.  The Sitirax and Potivik families have published layouts
+format between a conversion script and the server for these families.  The Sitirax, Potivik and Vevapel families have published layouts
 of their own (`"architecture": "Sitirax"` in config.json, bf16 tensors named layer by layer); they are read and written as
 published, and run in bf16 or in true fp32.
 (reference counterparts: src/models/*/loader.cpp + binding.cpp per family, tools' fixture writers; there every family
@@ -81,6 +81,9 @@ def published(family: str):
     if family == "potivik":
         from ..models import potivik as m
         return m.PotivikConfig, m.PotivikModel, m.PotivikRunner, m.tensor_shapes, m.random_tensors
+    if family == "vevapel":
+        from ..models import vevapel as m
+        return m.VevapelConfig, m.VevapelModel, m.VevapelRunner, m.tensor_shapes, m.random_tensors
     return None
 
 
@@ -243,13 +246,21 @@ def _tiny_potivik(vocab: int):
                                  ExpertsSpec(16, 2, FeedForward(256, 7.0), FeedForward(384, 7.0)), FeedForward(1024, 7.0), 64)
 
 
+def _tiny_vevapel(vocab: int):
+    from ..models.vevapel import AttentionSpec, DeltaSpec, DiffSpec, ExpertsSpec, LoopSpec, VevapelConfig
+
+    return VevapelConfig.cycle(4, 512, vocab, (DeltaSpec(4, 2, 64, 128, 4), DiffSpec(4, 2, 64, 128, 0.125, 128, 10000.0, 64, 0.3),
+                                               AttentionSpec(8, 2, 64, 64, 0.125, 0.1, 256)), ExpertsSpec(16, 2, 256), LoopSpec(1, 3, 2),
+                               embed_scale=4.0, residual=0.8)
+
+
 def tiny_model(family: str, device="cpu", seed: int = 0, vocab: int = 4096) -> Any:
     """A small random-init model of `family` (the shapes the server's `--model <family>-tiny` choices use)."""
     from ..models.moe import MoEConfig
 
     if family in PUBLISHED:
         _, model, _, _, random_tensors = published(family)
-        cfg = {"sitirax": _tiny_sitirax, "potivik": _tiny_potivik}[family](vocab)
+        cfg = {"sitirax": _tiny_sitirax, "potivik": _tiny_potivik, "vevapel": _tiny_vevapel}[family](vocab)
         return model.from_tensors(cfg, random_tensors(cfg, seed).__getitem__, device)
     cfg_cls, model_cls = _registry()[family]
     moe = MoEConfig(hidden=512, experts=16, top_k=2, moe_ffn=512, shared_ffn=512)

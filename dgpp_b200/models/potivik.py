@@ -529,11 +529,8 @@ class PotivikRunner(RowRunner):
     def _plan_runs(self, runs: RowRuns):
         """Splits a pass into runs that attend over expanded keys (per window: which pages, where) and single rows that attend in
         the absorbed form; one upload for all tables."""
-        page, start = self.c.page, [0]
-        for n in runs.lens:
-            start.append(start[-1] + n)
-        long = [r for r, n in enumerate(runs.lens) if n > ABSORB_RUN]
-        short = [start[r] + k for r, n in enumerate(runs.lens) if n <= ABSORB_RUN for k in range(n)]
+        page = self.c.page
+        short, long, start = runs.split(ABSORB_RUN)
         windows = sorted({P.latent.window for P in self.m.layers if P.latent is not None and P.latent.tc_runs(self.m.dtype)})
         host = short + [start[r] for r in long] + [runs.lens[r] for r in long]
         parts = []

@@ -1,6 +1,6 @@
 """Mixture of experts over plain rows: bf16 (or fp32) expert matrices stacked for the grouped linear, a router and an optional
-gated shared expert that read the same input in one fp32-output linear.  The router's weight multiplies an expert's input; since
-the gate / up projection is linear it is applied to its fp32 result, in the activation kernel.
+gated shared expert that read the same input in one fp32-output linear.  The router's weight multiplies an expert's input or its
+output; since the projections around the activation are linear it is applied in the activation kernel either way.
 
 Up to 16 rows: one launch routes and lists the experts in use, every listed expert reads all rows.  More rows: selection, counting
 sort into tiles, row scatter (`csrc/kernels/moe_prefill.cu`, `moe_rows.cu`).  Both are shapes fixed by the row count alone, so passes
@@ -33,6 +33,11 @@ class RowExperts:
     shared_ff: int = 0                   # 0: no shared expert
     shared_limit: float = 0.0
     shared_down: Optional[QuantLinear] = None
+    alpha: float = 1.702                 # activation: min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, +-limit) + shift)
+    shift: float = 1.0
+    score: str = "sigmoid"               # the router's weights (ops.mixers.SCORES)
+    weigh_out: bool = False              # they multiply the experts' outputs instead of their inputs
+    router_b: Optional[torch.Tensor] = None   # fp32 [experts]: added to the logits
 
     @property
     def nbytes(self) -> int:
@@ -84,18 +89,18 @@ def run_experts(b: RowExperts, s: RowExpertsScratch, x: torch.Tensor) -> mx.MoeD
     nt = b.max_tiles(rows, bn)
     tiles, pair_row, row_w = s.tiles[:nt], s.pair_row[:rows * b.top], s.row_w[:nt * bn]
     if rows <= mx.SMALL_TOKENS:
-        mx.moe_route_small(first, b.experts, b.top, pair_row, tiles, row_w)
+        mx.moe_route_small(first, b.experts, b.top, pair_row, tiles, row_w, b.score, b.router_b)
         xs = x
     else:
         ids, wts = view(s.ids, rows, b.top), view(s.wts, rows, b.top)
-        mx.moe_select(first, b.experts, b.top, ids, wts)
+        mx.moe_select(first, b.experts, b.top, ids, wts, b.score, bias=b.router_b)
         ops.moe_segment_sort(ids, bn, nt, 0, b.experts, pair_row, tiles, s.n_tiles)
         xs = view(s.xs, nt * bn, b.hidden)
         mx.moe_scatter_rows(x, pair_row, wts, xs, row_w, b.top)
     h = mx.grouped_linear(xs, b.w_gu, 2 * b.ff, tiles, bn, view(s.h, nt * bn, 2 * b.ff), shared_rows=xs is x)
-    act = mx.clamped_glu(h, view(s.act, nt * bn, b.ff), b.limit, row_w=row_w, tiles=tiles, bn=bn)
+    act = mx.clamped_glu(h, view(s.act, nt * bn, b.ff), b.limit, b.alpha, row_w, tiles, bn, b.shift, b.weigh_out)
     y = mx.grouped_linear(act, b.w_down, b.hidden, tiles, bn, view(s.y, nt * bn, b.hidden))
     if not b.shared_ff:
         return mx.MoeDelta(y, pair_row, b.top)
-    act = mx.clamped_glu(first[:, b.shared_col:], view(s.shared_act, rows, b.shared_ff), b.shared_limit)
+    act = mx.clamped_glu(first[:, b.shared_col:], view(s.shared_act, rows, b.shared_ff), b.shared_limit, b.alpha, shift=b.shift)
     return mx.MoeDelta(y, pair_row, b.top, ops.linear(act, b.shared_down, out=view(s.shared, rows, b.hidden)), first[:, b.sg_col:])

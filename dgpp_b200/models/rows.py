@@ -27,6 +27,14 @@ class RowRuns:
     slots: List[int]
     pos0: List[int]              # position of every run's first token
 
+    def split(self, limit: int):
+        """(rows of the runs of up to `limit` tokens, indices of the longer runs, first row of every run and behind the last)."""
+        start = [0]
+        for n in self.lens:
+            start.append(start[-1] + n)
+        return ([start[r] + k for r, n in enumerate(self.lens) if n <= limit for k in range(n)],
+                [r for r, n in enumerate(self.lens) if n > limit], start)
+
 
 class RowRunner:
     mixed_runs = False           # True: `forward_runs` exists and `step` may be used
@@ -35,7 +43,7 @@ class RowRunner:
     def _init_pool(self, slots: int, device, kv_shapes, kv_dtype, page: int, max_seq_len: int, max_rows: int,
                    pool_tokens: int = 0) -> None:
         """Rows over one shared pool of `pool_tokens` cache positions (default: every slot at full length); kv_shapes lists
-        (kv heads, key width, value width) per attention layer."""
+        (kv heads, key width, value width[, value heads]) per attention layer."""
         from ..engine.kv_cache import PagedKV
 
         self._init_rows(slots, device, max_rows=max_rows)

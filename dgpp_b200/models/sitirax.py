@@ -422,7 +422,7 @@ class SitiraxRunner(RowRunner):
         T = model.dtype
         self.kv_index = {i: j for j, i in enumerate(i for i, P in enumerate(model.layers) if P.window is not None)}
         heads = [model.layers[i].window for i in self.kv_index]
-        self._init_pool(slots, device, [(g.hkv, g.D, g.DV) for g in heads], T, c.page, max_seq_len, max_rows, pool_tokens)
+        self._init_pool(slots, device, [g.kv_shape for g in heads], T, c.page, max_seq_len, max_rows, pool_tokens)
         self.states = [P.state.new_state(slots, device) for P in model.layers]
         e = lambda n, dt: torch.empty(n, dtype=dt, device=device)
         R, Hp = max_rows, model.hp
@@ -450,12 +450,6 @@ class SitiraxRunner(RowRunner):
             return ops.gemm_tc(x, w, out32=out)
         return ops.linear(x, w, out=out)
 
-    def _splits(self, g: mx.WindowHeads, rows: int) -> int:
-        """Window splits of a decode pass: about two CTAs per SM, at least 64 keys each."""
-        span = min(g.window, self.max_span)
-        chunks = -(-(g.hq // g.hkv) // 8)
-        return max(1, min(self.max_splits, -(-296 // (g.hkv * chunks * rows)), span // 64))
-
     def _parallel(self, i: int, P: Packed, proj, mixed, positions, row_req, runs: Optional[RowRuns]) -> None:
         m, g, s = self.c.plan[i].mixer, P.window, P.state
         rows, n_left = proj.shape[0], g.hq * g.DV
@@ -463,7 +457,7 @@ class SitiraxRunner(RowRunner):
         o = self.o[:rows * s.hv * s.DV].view(rows, s.hv * s.DV)
         if runs is None:
             mx.window_attn(g, proj, P.q_norm, P.k_norm, cache, bt, row_req, positions, mixed, m.left_scale, fused=True,
-                           splits=self._splits(g, rows), scratch=self.scratch)
+                           splits=g.splits(rows, self.max_span, self.max_splits), scratch=self.scratch)
             mx.linear_state(s, proj, *self.states[i], row_req, positions, o=o)
         else:
             mx.qk_norm_append(g, proj, P.q_norm, P.k_norm, cache, bt, row_req, positions)

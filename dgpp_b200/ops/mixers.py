@@ -1,7 +1,7 @@
 """Front ends of the kernels behind models with an fp32 residual stream, sliding-window attention (grouped heads, or a
 shared latent), fp32 linear-attention and state-space memories, and experts of plain rows (``csrc/kernels/stream_ops.cu``,
-``window_attn.cu``, ``window_attn_tc.cu``, ``latent_attn.cu``, ``mla_tc.cu``, ``linear_state.cu``, ``state_space.cu``,
-``moe_rows.cu``).  Every operator exists for bf16 and for true fp32 activations; the dtype of the tensors decides."""
+``window_attn.cu``, ``window_attn_tc.cu``, ``latent_attn.cu``, ``mla_tc.cu``, ``linear_state.cu``, ``gated_delta.cu``,
+``state_space.cu``, ``moe_rows.cu``).  Every operator exists for bf16 and for true fp32 activations; the dtype of the tensors decides."""
 from __future__ import annotations
 
 from typing import Optional
@@ -11,13 +11,16 @@ import torch
 from . import _lib
 from ._lib import F, I, L, P, call, ptr, stream_ptr
 
-_lib.declare("dgpp_embed_rows", [P, P, P, I, I, I, I, P])
+_lib.declare("dgpp_embed_rows", [P, P, P, P, L, I, I, I, F, I, P])
 _lib.declare("dgpp_resid_norm", [P, P, P, P, I, I, I, F, I, P])
-_lib.declare("dgpp_gated_group_norm", [P, P, L, P, P, L, I, I, I, I, F, F, I, I, P])
+_lib.declare("dgpp_gated_group_norm", [P, P, L, P, P, L, I, I, I, I, F, F, I, I, I, P])
 _lib.declare("dgpp_geglu", [P, P, I, I, I, P])
-_lib.declare("dgpp_qk_norm_append", [P, L, I, I, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P])
-_lib.declare("dgpp_window_attn", [P, L, I, I, I, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, I, I, I, F, F, F, I, P])
+_WINDOW = [P, L, I, I, I] + [P] * 11 + [I] * 12 + [F, F]
+_lib.declare("dgpp_qk_norm_append", _WINDOW + [I, P])
+_lib.declare("dgpp_window_attn", _WINDOW + [P, P, P, P, L, I, I, I, I, I, F, F, I, P])
+_lib.declare("dgpp_diff_combine", [P, P, P, L, P, P, L, I, I, I, I, I, I, F, F, F, I, P])
 _lib.declare("dgpp_state_space", [P, L, I, I, P, P, P, I, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, P])
+_lib.declare("dgpp_gated_delta", [P, L, I, I, I, I, P, P, I, P, P, P, P, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, F, F, I, I, P])
 _lib.declare("dgpp_linear_state", [P, L, I, I, P, L, P, P, I, P, P, P, P, P, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, F, F,
                                    I, I, I, P])
 
@@ -42,9 +45,11 @@ ATTN_WIDTHS = (64, 128, 192, 256)      # padded head widths of the window attent
 STATE_WIDTHS = (32, 64, 128, 256)      # padded key / value widths of the linear-state kernels
 
 
-def embed_rows(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """fp32 rows out[r] = table[ids[r]] (table [vocab, cols] bf16 or fp32)."""
-    call("dgpp_embed_rows", ptr(ids), ptr(table), ptr(out), ids.numel(), table.shape[1], table.shape[0], _f32(table), stream_ptr())
+def embed_rows(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0, copy: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 rows out[r] = scale * table[ids[r]] (table [vocab, cols] bf16 or fp32); copy [rows, cols] receives them in the table's type."""
+    assert copy is None or copy.dtype == table.dtype
+    call("dgpp_embed_rows", ptr(ids), ptr(table), ptr(out), ptr(copy), 0 if copy is None else copy.stride(0), ids.numel(), table.shape[1],
+         table.shape[0], float(scale), _f32(table), stream_ptr())
     return out
 
 
@@ -57,11 +62,11 @@ def resid_norm(x: torch.Tensor, w: torch.Tensor, n: int, eps: float, out: torch.
 
 
 def gated_group_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, out: torch.Tensor, groups: int, n: int, eps: float,
-                     scale: float = 1.0) -> torch.Tensor:
-    """o [rows, groups * gp] fp32 -> rms norm per group (n true columns) * w [gp] * sigmoid(gate) * scale."""
+                     scale: float = 1.0, silu: bool = False) -> torch.Tensor:
+    """o [rows, groups * gp] fp32 -> rms norm per group (n true columns) * w [gp] * sigmoid(gate) (or silu(gate)) * scale."""
     assert o.dtype == torch.float32 and o.is_contiguous() and o.shape[1] % groups == 0
     call("dgpp_gated_group_norm", ptr(o), ptr(gate), gate.stride(0), ptr(w), ptr(out), out.stride(0), o.shape[0], groups,
-         o.shape[1] // groups, n, float(eps), float(scale), _f32(out), _f32(gate), stream_ptr())
+         o.shape[1] // groups, n, float(eps), float(scale), int(silu), _f32(out), _f32(gate), stream_ptr())
     return out
 
 
@@ -73,23 +78,26 @@ def geglu(gate_up: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
 
 
 NORMS = {None: 0, "rms": 1, "layer": 2}
-_lib.declare("dgpp_stream_norm", [P, P, P, P, I, P, P, L, I, P, I, P, P, I, I, I, F, I, P])
+_lib.declare("dgpp_stream_norm", [P, P, P, P, I, P, P, L, P, P, F, I, P, P, I, P, P, P, L, I, I, I, F, I, P])
 _lib.declare("dgpp_gated_part_norm", [P, P, L, P, P, L, I, I, I, I, F, I, P])
-_lib.declare("dgpp_clamped_glu", [P, L, P, P, I, P, I, I, F, F, I, I, P])
+_lib.declare("dgpp_clamped_glu", [P, L, P, P, I, P, I, I, F, F, F, I, I, I, P])
 _lib.declare("dgpp_token_gate", [P, P, P, L, I, P, I, I, I, I, P])
 _lib.declare("dgpp_softcap", [P, L, F, P])
 
 
-def stream_norm(x: torch.Tensor, n: int, eps: float, out: torch.Tensor, delta=None, post=(None, None), pre=(None, None)) -> torch.Tensor:
-    """x [rows, cols] fp32 takes in post(delta) in place; out = pre(x).  post / pre: (None | "rms" | "layer", fp32 weight row)
-    over the n true columns.  delta: an fp32 row block, a ``MoeDelta`` or None."""
-    assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous()
+def stream_norm(x: torch.Tensor, n: int, eps: float, out: torch.Tensor, delta=None, post=(None, None), pre=(None, None), mult: float = 1.0,
+                delta_b=None, vec=None) -> torch.Tensor:
+    """x [rows, cols] fp32 takes in mult * post(delta + delta_b) + vec in place; out [rows, >= cols] = pre(x).  post / pre:
+    (None | "rms" | "layer", fp32 weight row[, fp32 bias row]) over the n true columns.  delta: an fp32 row block, a ``MoeDelta`` or
+    None; delta_b, vec: fp32 rows or None."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.stride(1) == 1
+    post, pre = (tuple(t) + (None,) * (3 - len(t)) for t in (post, pre))
     m = delta if isinstance(delta, MoeDelta) else None
     d = None if m is not None else delta
     assert d is None or (d.dtype == torch.float32 and d.is_contiguous())
     call("dgpp_stream_norm", ptr(x), ptr(d), ptr(m and m.y), ptr(m and m.pair_row), m.top if m else 0, ptr(m and m.shared),
-         ptr(m and m.gate), m.gate.stride(0) if m and m.gate is not None else 0, NORMS[post[0]], ptr(post[1]), NORMS[pre[0]], ptr(pre[1]),
-         ptr(out), x.shape[0], x.shape[1], n, float(eps), _f32(out), stream_ptr())
+         ptr(m and m.gate), m.gate.stride(0) if m and m.gate is not None else 0, ptr(delta_b), ptr(vec), float(mult), NORMS[post[0]], ptr(post[1]),
+         ptr(post[2]), NORMS[pre[0]], ptr(pre[1]), ptr(pre[2]), ptr(out), out.stride(0), x.shape[0], x.shape[1], n, float(eps), _f32(out), stream_ptr())
     return out
 
 
@@ -103,12 +111,13 @@ def gated_part_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, out: torc
     return out
 
 
-def clamped_glu(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: float = 1.702, row_w=None, tiles=None, bn: int = 1) -> torch.Tensor:
-    """gate_up [rows, 2 I] -> min(s g, limit) sigmoid(alpha min(s g, limit)) (clamp(s u, +-limit) + 1) [rows, I]; s: `row_w` or one.
-    tiles [rows / bn]: rows of tiles with a negative entry are skipped."""
+def clamped_glu(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: float = 1.702, row_w=None, tiles=None, bn: int = 1,
+                shift: float = 1.0, weigh_out: bool = False) -> torch.Tensor:
+    """gate_up [rows, 2 I] -> min(s g, limit) sigmoid(alpha min(s g, limit)) (clamp(s u, +-limit) + shift) [rows, I]; s: `row_w` or one
+    (weigh_out: the row's weight multiplies the result instead).  limit inf, alpha 1, shift 0: silu(g) u.  tiles [rows / bn]: rows of tiles with a negative entry are skipped."""
     assert out.is_contiguous() and gate_up.shape[1] >= 2 * out.shape[1]
     call("dgpp_clamped_glu", ptr(gate_up), gate_up.stride(0), ptr(row_w), ptr(tiles), bn, ptr(out), gate_up.shape[0], out.shape[1], float(limit),
-         float(alpha), _f32(out), _f32(gate_up), stream_ptr())
+         float(alpha), float(shift), int(weigh_out), _f32(out), _f32(gate_up), stream_ptr())
     return out
 
 
@@ -128,13 +137,14 @@ def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
 
 
 # ---------------------------------------------------------------------------------------------- experts over plain rows
-_lib.declare("dgpp_moe_select", [P, L, P, P, I, I, I, I, I, F, P])
-_lib.declare("dgpp_moe_route_small", [P, L, P, P, P, I, I, I, I, I, P])
+_lib.declare("dgpp_moe_select", [P, L, P, P, P, I, I, I, I, I, F, P])
+_lib.declare("dgpp_moe_route_small", [P, L, P, P, P, P, I, I, I, I, I, P])
 _lib.declare("dgpp_moe_scatter_rows", [P, P, P, P, P, I, I, I, I, P])
 _lib.declare("dgpp_gemm_tc_grouped", [I, P, L, I, I, P, I, P, P, I, I, I, I, P])
 _lib.declare("dgpp_gemm_f32_grouped", [I, P, L, I, I, P, I, P, P, L, I, I, I, P])
 SMALL_TOKENS = 16                      # rows up to which routing is one launch and every listed expert reads all rows
 MAX_EXPERTS, MAX_TOP = 512, 16
+SCORES = {"sigmoid": 0, "softmax": 1, "chosen": 2}      # of the logit; softmax over all experts; softmax over the chosen ones only
 
 
 class MoeDelta:
@@ -145,17 +155,17 @@ class MoeDelta:
         self.y, self.pair_row, self.top, self.shared, self.gate = y, pair_row, top, shared, gate
 
 
-def moe_select(logits: torch.Tensor, experts: int, top: int, ids: torch.Tensor, weights: torch.Tensor, softmax: bool = False,
-               norm_topk: bool = False, scaling: float = 1.0) -> None:
-    """The `top` best of the first `experts` columns of fp32 logits per row -> ids (ascending), weights (their scores)."""
-    call("dgpp_moe_select", ptr(logits), logits.stride(0), ptr(ids), ptr(weights), logits.shape[0], experts, top, int(softmax), int(norm_topk),
+def moe_select(logits: torch.Tensor, experts: int, top: int, ids: torch.Tensor, weights: torch.Tensor, score: str = "sigmoid",
+               norm_topk: bool = False, scaling: float = 1.0, bias=None) -> None:
+    """The `top` best of the first `experts` columns of fp32 logits (+ bias [experts] fp32) per row -> ids (ascending), weights."""
+    call("dgpp_moe_select", ptr(logits), logits.stride(0), ptr(bias), ptr(ids), ptr(weights), logits.shape[0], experts, top, SCORES[score], int(norm_topk),
          float(scaling), stream_ptr())
 
 
-def moe_route_small(logits: torch.Tensor, experts: int, top: int, pair_row, tiles, row_w, softmax: bool = False) -> None:
+def moe_route_small(logits: torch.Tensor, experts: int, top: int, pair_row, tiles, row_w, score: str = "sigmoid", bias=None) -> None:
     """Up to 16 rows: tiles (experts in use), pair_row [rows * top] = tile * 16 + row, row_w [tiles * 16]."""
-    call("dgpp_moe_route_small", ptr(logits), logits.stride(0), ptr(pair_row), ptr(tiles), ptr(row_w), logits.shape[0], experts, top,
-         tiles.numel(), int(softmax), stream_ptr())
+    call("dgpp_moe_route_small", ptr(logits), logits.stride(0), ptr(bias), ptr(pair_row), ptr(tiles), ptr(row_w), logits.shape[0], experts, top,
+         tiles.numel(), SCORES[score], stream_ptr())
 
 
 def moe_scatter_rows(x: torch.Tensor, pair_row, weights, xs, row_w, top: int) -> None:
@@ -173,53 +183,94 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, n: int, tiles: torch.Tensor
     return out
 
 
+NO_WINDOW = 1 << 30                    # a window that nobody fills: every earlier key is visible
+
+
 class WindowHeads:
-    """Static description of one window-attention block inside a fused projection row."""
+    """Static description of one attention block inside a fused projection row.  `window` keys (chunked: the keys of the row's own
+    chunk of `window` positions, counted from 0).  norm: "head" or "row" (over the whole projection) or None; biases fp32, padded as
+    the heads are; freq: ``rotation_freqs`` of the first `rot` columns, paired (i, i + rot / 2); temp: (coef, every) of the query
+    temperature; gate_off: column with one output gate per head.  maps 2: differential attention, query heads laid out
+    [kv head][map][head of the group], `heads` counts output heads."""
 
     def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, window: int, scale: float, eps: float,
-                 q_off: int, k_off: int, v_off: int):
-        self.hq, self.hkv, self.dim, self.window, self.scale, self.eps = heads, kv_heads, dim, window, scale, eps
+                 q_off: int, k_off: int, v_off: int, norm: Optional[str] = "head", bias=(None, None, None), freq=None, rot: int = 0,
+                 temp=(0.0, 1), gate_off: int = -1, maps: int = 1, chunked: bool = False):
+        self.hq, self.hkv, self.dim, self.vdim, self.window, self.scale, self.eps = heads * maps, kv_heads, dim, vdim, window, scale, eps
         self.D, self.DV = pad_to(dim, ATTN_WIDTHS), pad_to(vdim, ATTN_WIDTHS)
         self.q_off, self.k_off, self.v_off = q_off, k_off, v_off
+        self.norm, self.bias, self.freq, self.rot, self.temp, self.gate_off = norm, bias, freq, rot, temp, gate_off
+        self.maps, self.chunked, self.group = maps, chunked, heads // kv_heads
+
+    @property
+    def kv_shape(self):
+        """(key heads, key width, value width, value heads) of the cache."""
+        return self.hkv * self.maps, self.D, self.DV, self.hkv
+
+    def splits(self, rows: int, max_span: int, most: int) -> int:
+        """Splits of single rows' keys: about two CTAs per SM, at least 64 keys each."""
+        chunks = -(-self.group // (8 // self.maps))
+        return max(1, min(most, -(-296 // (self.hkv * chunks * rows)), min(self.window, max_span) // 64))
 
 
-def _wa_common(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, positions):
-    return (ptr(proj), proj.stride(0), g.q_off, g.k_off, g.v_off, ptr(wq), ptr(wk), ptr(cache.k), ptr(cache.v),
-            ptr(block_table), ptr(row_req), ptr(positions))
+def _wa_common(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, positions, rows: int):
+    coef, every = g.temp
+    norm = {None: 0, "head": 1, "row": 2}[g.norm]
+    return (ptr(proj), proj.stride(0), g.q_off, g.k_off, g.v_off, ptr(wq), ptr(wk), *(ptr(b) for b in g.bias), ptr(g.freq), ptr(cache.k), ptr(cache.v),
+            ptr(block_table), ptr(row_req), ptr(positions), rows, g.hq, g.hkv, g.maps, g.D, g.DV, g.dim, cache.page, block_table.shape[1], norm,
+            g.rot, int(every), float(coef), float(g.eps))
 
 
 def qk_norm_append(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, positions) -> None:
-    """Norms the query heads of `proj` in place and appends normed keys and values to the paged cache."""
+    """Prepares the query heads of `proj` in place (bias, norm, rotation, temperature) and appends prepared keys and values to the
+    paged cache."""
     assert cache.k.dtype == proj.dtype
-    call("dgpp_qk_norm_append", *_wa_common(g, proj, wq, wk, cache, block_table, row_req, positions), proj.shape[0], g.hq, g.hkv,
-         g.D, g.DV, g.dim, cache.page, block_table.shape[1], float(g.eps), _f32(proj), stream_ptr())
+    call("dgpp_qk_norm_append", *_wa_common(g, proj, wq, wk, cache, block_table, row_req, positions, proj.shape[0]), _f32(proj), stream_ptr())
 
 
 def window_attn(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, positions, out, out_scale: float = 1.0,
-                fused: bool = False, splits: int = 1, scratch=None, row_list=None) -> torch.Tensor:
-    """Every row attends to the last `window` positions of its request, its own included -> out [rows, >= hq * DV].
-    fused: the rows are single new tokens; the kernel norms and appends them itself.  row_list: int32 subset of rows."""
-    assert cache.k.dtype == proj.dtype and out.dtype == proj.dtype
-    ml, acc = scratch if splits > 1 else (None, None)
+                fused: bool = False, splits: int = 1, scratch=None, row_list=None) -> Optional[torch.Tensor]:
+    """Every row attends to the positions of its request that it sees, its own included -> out [rows, >= hq * DV].
+    fused: the rows are single new tokens; the kernel prepares and appends them itself.  row_list: int32 subset of rows.
+    scratch: (fp32 launch rows * hq * splits * 2, * DV) where splits > 1; with two maps always, and the result stays there for
+    ``diff_combine`` (out unused)."""
+    assert cache.k.dtype == proj.dtype and (g.maps == 2 or out.dtype == proj.dtype)
     rows = proj.shape[0] if row_list is None else row_list.numel()
-    call("dgpp_window_attn", *_wa_common(g, proj, wq, wk, cache, block_table, row_req, positions), ptr(row_list), ptr(ml), ptr(acc),
-         ptr(out), out.stride(0), rows, g.hq, g.hkv, g.D, g.DV, g.dim, cache.page, block_table.shape[1], splits, g.window,
-         int(fused), float(g.scale), float(g.eps), float(out_scale), _f32(proj), stream_ptr())
+    ml, acc = scratch if splits > 1 or g.maps == 2 else (None, None)
+    assert ml is None or (ml.numel() >= rows * g.hq * splits * 2 and acc.numel() >= rows * g.hq * splits * g.DV)
+    out = None if g.maps == 2 else out
+    call("dgpp_window_attn", *_wa_common(g, proj, wq, wk, cache, block_table, row_req, positions, rows), ptr(row_list), ptr(ml), ptr(acc),
+         ptr(out), 0 if out is None else out.stride(0), splits, g.window, int(g.chunked), int(fused), g.gate_off, float(g.scale), float(out_scale),
+         _f32(proj), stream_ptr())
+    return out
+
+
+def diff_combine(g: WindowHeads, scratch, proj, gate_off: int, out, lam: float, factor: float, splits: int = 1, row_list=None,
+                 finished: bool = False) -> torch.Tensor:
+    """out [rows, >= heads * DV] = (a1 - lam * a2) / its root mean square per head * factor * sigmoid(gate columns of proj).  scratch as
+    ``window_attn`` left it, or (finished) the fp32 outputs [rows, hq, DV] of ``window_prefill``."""
+    ml, acc = (None, scratch) if finished else scratch
+    rows = proj.shape[0] if row_list is None else row_list.numel()
+    gate = proj[:, gate_off:]
+    call("dgpp_diff_combine", ptr(ml), ptr(acc), ptr(gate), proj.stride(0), ptr(row_list), ptr(out), out.stride(0), rows, g.hq // 2, g.group, g.DV,
+         g.vdim, splits, float(lam), float(factor), float(g.eps), _f32(out), stream_ptr())
     return out
 
 
 class StateHeads:
     """Static description of one linear-attention block: widths (padded), offsets inside the fused projection row, and the
-    constants of its rule (`decay` per head: lightning; `skip` per head with `A_log` / `dt_bias`: state space; `A_log` / `dt_bias` /
-    low-rank rows: channel delta rule)."""
+    constants of its rule (`decay` per head: lightning; `skip` per head with `A_log` / `dt_bias`: state space; a_off / gate_off, the
+    columns of the raw decays and output gates: delta rule with a decay per head; `A_log` / `dt_bias` / low-rank rows: channel delta
+    rule)."""
 
     def __init__(self, heads: int, key_heads: int, dim: int, vdim: int, c_off: int, b_off: int = 0, eps: float = 0.0,
-                 conv_w=None, A_log=None, dt_bias=None, decay=None, norm_w=None, conv_b=None, skip=None):
+                 conv_w=None, A_log=None, dt_bias=None, decay=None, norm_w=None, conv_b=None, skip=None, a_off: int = -1, gate_off: int = 0):
         self.hv, self.hk, self.dim, self.vdim = heads, key_heads, dim, vdim
         self.DK, self.DV = pad_to(dim, STATE_WIDTHS), pad_to(vdim, STATE_WIDTHS)
         self.c_off, self.b_off, self.eps = c_off, b_off, eps
         self.conv_w, self.A_log, self.dt_bias, self.decay, self.norm_w = conv_w, A_log, dt_bias, decay, norm_w
         self.conv_b, self.skip = conv_b, skip
+        self.a_off, self.gate_off = a_off, gate_off
         self.delta = decay is None and skip is None
         self.taps = 0 if conv_w is None else conv_w.shape[0]
 
@@ -238,6 +289,8 @@ class StateHeads:
         blocks = rows // 16 + runs
         if self.skip is not None:
             return rows * (self.channels + 2 * self.hv) + blocks * self.hv * 288
+        if self.a_off >= 0:
+            return rows * (self.channels + 2 * self.hv) + blocks * self.hv * 576
         return rows * (self.channels + self.hv * (3 * self.DK + 1)) + blocks * self.hv * (self.DK + 512)
 
 
@@ -254,6 +307,13 @@ def linear_state(g: StateHeads, proj, state, ring, row_slot, positions, low=None
              None if runs is None else ptr(runs.row_run0), ptr(prep), ptr(o), rows, rows if runs is None else len(runs.lens), blocks, g.hk, g.hv,
              g.DK, g.DV, g.vdim, int(runs is None), _f32(proj), stream_ptr())
         return
+    if g.a_off >= 0:
+        call("dgpp_gated_delta", ptr(proj), proj.stride(0), g.c_off, g.b_off, g.a_off, g.gate_off, ptr(g.conv_w), ptr(ring), g.taps, ptr(g.A_log),
+             ptr(g.dt_bias), ptr(state), ptr(row_slot), ptr(positions), None if runs is None else ptr(runs.start),
+             None if runs is None else ptr(runs.row_run0), ptr(prep), ptr(o), ptr(out), 0 if out is None else out.stride(0), ptr(g.norm_w), rows,
+             rows if runs is None else len(runs.lens), blocks, g.hk, g.hv, g.DK, g.DV, g.vdim, float(g.dim ** -0.5), float(g.eps),
+             int(runs is None), _f32(proj), stream_ptr())
+        return
     call("dgpp_linear_state", ptr(proj), proj.stride(0), g.c_off, g.b_off, ptr(low), 0 if low is None else low.stride(0),
          ptr(g.conv_w), ptr(ring), g.taps, ptr(g.A_log), ptr(g.dt_bias), ptr(g.decay), ptr(state), ptr(row_slot), ptr(positions),
          None if runs is None else ptr(runs.start), None if runs is None else ptr(runs.row_run0), ptr(prep), ptr(o), ptr(out),
@@ -261,22 +321,30 @@ def linear_state(g: StateHeads, proj, state, ring, row_slot, positions, low=None
          g.vdim, float(g.dim ** -0.5), float(g.eps), int(g.delta), int(runs is None), _f32(proj), stream_ptr())
 
 
-_lib.declare("dgpp_window_attn_tc", [P, L, I, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, I, I, F, F, P])
+_lib.declare("dgpp_window_attn_tc", [P, L, I] + [P] * 8 + [L, P] + [I] * 13 + [F, F, P])
 
 
 def window_prefill_usable(g: WindowHeads, proj, page: int = 64) -> bool:
     """Whether the tensor-core kernel takes these rows (bf16, pages of 64 tokens, at most 128 query heads per key head)."""
-    return proj.dtype == torch.bfloat16 and page == 64 and g.hq // g.hkv <= 128
+    return proj.dtype == torch.bfloat16 and page == 64 and g.group <= 128
 
 
-def window_prefill(g: WindowHeads, proj, cache, block_table, row_req, positions, runs, out, out_scale: float = 1.0) -> torch.Tensor:
-    """`window_attn` for runs of prompt rows on the tensor cores (tcgen05); `qk_norm_append` comes before it."""
-    assert cache.k.dtype == proj.dtype == out.dtype == torch.bfloat16
-    per = 128 // (g.hq // g.hkv)
-    tiles = sum(-(-n // per) for n in runs.lens)
+def window_tiles(g: WindowHeads, lens) -> int:
+    """CTAs per key head of ``window_prefill`` over runs of these lengths."""
+    per = 128 // g.group
+    return sum(-(-n // per) for n in lens)
+
+
+def window_prefill(g: WindowHeads, proj, cache, block_table, row_req, positions, runs, out, out_scale: float = 1.0, raw=None,
+                   some=None) -> torch.Tensor:
+    """`window_attn` for runs of prompt rows on the tensor cores (tcgen05); `qk_norm_append` comes before it.  raw: fp32 [rows, hq, DV]
+    takes the outputs instead of `out` (two maps: required).  some: (int32 first rows, int32 lengths, lengths on the host) of the runs
+    to take, else all of them."""
+    assert cache.k.dtype == proj.dtype == torch.bfloat16 and (raw is not None or out.dtype == torch.bfloat16)
+    start, lens_dev, lens = (runs.start, None, runs.lens) if some is None else some
     call("dgpp_window_attn_tc", ptr(proj), proj.stride(0), g.q_off, ptr(cache.k), ptr(cache.v), ptr(block_table), ptr(row_req),
-         ptr(positions), ptr(runs.start), ptr(out), out.stride(0), len(runs.lens), tiles, g.hq, g.hkv, g.D, g.DV, cache.page,
-         block_table.shape[1], cache.k.shape[0], g.window, float(g.scale), float(out_scale), stream_ptr())
+         ptr(positions), ptr(start), ptr(lens_dev), ptr(out), out.stride(0), ptr(raw), len(lens), window_tiles(g, lens), g.hq, g.hkv, g.maps, g.D, g.DV,
+         cache.page, block_table.shape[1], cache.k.shape[0], g.window, int(g.chunked), g.gate_off, float(g.scale), float(out_scale), stream_ptr())
     return out
 
 
