@@ -143,7 +143,9 @@ MIXERS = {"attention": mixer_attention, "attention_2": mixer_attention_2, "delta
 
 def schedule(cfg):
     """[(layer, pass or None)] in the order they run; the pass where a layer is the first of one."""
-    n, lp = len(cfg["layers"]), cfg["loop"]
+    n, lp = len(cfg["layers"]), cfg.get("loop")
+    if lp is None:
+        return [(i, None) for i in range(n)]
     order = [(i, None) for i in range(lp["start"])]
     for t in range(lp["times"]):
         order += [(i, t if i == lp["start"] else None) for i in range(lp["start"], lp["stop"])]
