@@ -333,7 +333,7 @@ DGPP_API int dgpp_moe_route(const void* x, int64_t x_stride, const void* gate, c
   DGPP_REQUIRE(n_group <= 1 || (n_group <= 64 && E % n_group == 0 && topk_group >= 1 && topk_group <= n_group),
                "moe_route: bad grouping %d / %d", n_group, topk_group);
   if (T == 0) return 0;
-  RouterArgs a;
+  RouterArgs a = {};
   a.x = static_cast<const bf16*>(x); a.x_stride = x_stride;
   a.gate = static_cast<const bf16*>(gate);
   a.bias = static_cast<const float*>(bias);

@@ -177,7 +177,7 @@ __device__ __forceinline__ float wa_gate(const WindowAttnParams& p, int row, int
 // time (lane = key), then the lanes take value columns 2 * lane + 64 * j.
 template <typename T, int NV, int NG, int MAPS>
 __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(const __grid_constant__ WindowAttnParams p) {
-  constexpr int DV = NV * 64, VN = Vec16<T>::N, NGM = NG / MAPS;
+  constexpr int DV = NV * 64, VN = Vec16<T>::N, NGM = NG / MAPS, VU = NV <= 2 ? 8 : 4;
   extern __shared__ __align__(16) float wa_smem[];
   float* q_s = wa_smem;                                   // [NG][D]
   float* red_acc = q_s + NG * p.D;                        // [warps][NG][DV]
@@ -192,7 +192,7 @@ __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(const __grid
   auto head_of = [&](int i) { return (kvh * MAPS + i / NGM) * group + g0 + min(i % NGM, ng - 1); };
   const int first = p.chunked ? pos - pos % p.window : max(0, pos + 1 - p.window), len = pos + 1;
   int per = (len - first + p.splits - 1) / p.splits;
-  per = (per + 31) & ~31;
+  per = (per + kWaWarps * 32 - 1) / (kWaWarps * 32) * (kWaWarps * 32);   // every warp scores as many keys; the last splits may be empty
   const int t_begin = first + split * per;
   const int t_end = min(len, t_begin + per);
   const int32_t* bt = p.block_table + static_cast<size_t>(p.row_req[row]) * p.max_blocks;
@@ -279,21 +279,26 @@ __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(const __grid
       for (int j = 0; j < 2 * NV; ++j) acc[g][j] *= corr;
     }
     const int n = min(32, t_end - t0);
-    for (int tt = 0; tt < n; ++tt) {
-      const size_t vtok = __shfl_sync(0xffffffffu, static_cast<unsigned long long>(tok), tt);
-      const T* vr = vc + vtok * DV + 2 * lane;
-      float2 vf[NV];
+    for (int tt = 0; tt < n; tt += VU) {                  // VU keys' values in flight; lanes behind the last key weigh 0
+      float2 vf[VU][NV];
 #pragma unroll
-      for (int j = 0; j < NV; ++j) vf[j] = ld_elem2(vr + 64 * j);
+      for (int u = 0; u < VU; ++u) {
+        const size_t vtok = __shfl_sync(0xffffffffu, static_cast<unsigned long long>(tok), tt + u);
+        const T* vr = vc + vtok * DV + 2 * lane;
 #pragma unroll
-      for (int g = 0; g < NG; ++g) {
-        const float pg = __shfl_sync(0xffffffffu, pr[g], tt);
-#pragma unroll
-        for (int j = 0; j < NV; ++j) {
-          acc[g][2 * j] = fmaf(pg, vf[j].x, acc[g][2 * j]);
-          acc[g][2 * j + 1] = fmaf(pg, vf[j].y, acc[g][2 * j + 1]);
-        }
+        for (int j = 0; j < NV; ++j) vf[u][j] = ld_elem2(vr + 64 * j);
       }
+#pragma unroll
+      for (int u = 0; u < VU; ++u)
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+          const float pg = __shfl_sync(0xffffffffu, pr[g], tt + u);
+#pragma unroll
+          for (int j = 0; j < NV; ++j) {
+            acc[g][2 * j] = fmaf(pg, vf[u][j].x, acc[g][2 * j]);
+            acc[g][2 * j + 1] = fmaf(pg, vf[u][j].y, acc[g][2 * j + 1]);
+          }
+        }
     }
   }
   if (lane == 0) {

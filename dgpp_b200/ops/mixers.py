@@ -208,9 +208,9 @@ class WindowHeads:
         return self.hkv * self.maps, self.D, self.DV, self.hkv
 
     def splits(self, rows: int, max_span: int, most: int) -> int:
-        """Splits of single rows' keys: about two CTAs per SM, at least 64 keys each."""
+        """Splits of single rows' keys: at most one wave of CTAs (four per SM, three with two maps), at least 128 keys each."""
         chunks = -(-self.group // (8 // self.maps))
-        return max(1, min(most, -(-296 // (self.hkv * chunks * rows)), min(self.window, max_span) // 64))
+        return max(1, min(most, 148 * (5 - self.maps) // (self.hkv * chunks * rows), min(self.window, max_span) // 128))
 
 
 def _wa_common(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, positions, rows: int):
