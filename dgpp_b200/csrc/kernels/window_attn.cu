@@ -92,32 +92,53 @@ __device__ __forceinline__ float wa_squares(const T* src, const float* bias, int
   return ss;
 }
 
+// Cosine and sine of the row's rotated pairs, by the whole CTA (a barrier follows).
+__device__ __forceinline__ void wa_angles(const WindowAttnParams& p, int pos, float2* cs) {
+  const int half = p.rot / 2;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, c;
+    rope_angle(p.freq, half, pos, i, sn, c);
+    cs[i] = make_float2(c, sn);
+  }
+}
+
 // One query or key head by one warp: bias, norm (`rstd` of the whole projection, or the head's own), rotation and a factor into dst,
 // which may be src (a lane holds both columns of a rotated pair).
 template <typename T, typename D>
-__device__ __noinline__ void wa_head(const WindowAttnParams& p, const T* src, const float* bias, const float* w, float rstd, float factor, int pos,
-                                        int lane, D* dst) {
+__device__ __noinline__ void wa_head(const WindowAttnParams& p, const T* src, const float* bias, const float* w, const float2* cs, float rstd,
+                                     float factor, int lane, D* dst) {
   float r = factor;
   if (p.norm == 1) r *= 1.f / sqrtf(warp_sum_f32(wa_squares(src, bias, p.D, lane, 32)) / static_cast<float>(p.dim) + p.eps);
   else if (p.norm == 2) r *= rstd;
   auto value = [&](int d) { return (ld_elem(src + d) + (bias != nullptr ? bias[d] : 0.f)) * (p.norm ? r * w[d] : r); };
   const int half = p.rot / 2;
-#pragma unroll 1
-  for (int i = lane; i < half; i += 32) {
-    float s, c;
-    rope_angle(p.freq, half, pos, i, s, c);
-    const float a = value(i), b = value(i + half);
-    st_elem(dst + i, a * c - b * s);
-    st_elem(dst + i + half, b * c + a * s);
-  }
 #pragma unroll 2
-  for (int d = p.rot + lane; d < p.D; d += 32) st_elem(dst + d, value(d));
+  for (int i = lane; i < half; i += 32) {
+    const float a = value(i), b = value(i + half);
+    st_elem(dst + i, a * cs[i].x - b * cs[i].y);
+    st_elem(dst + i + half, b * cs[i].x + a * cs[i].y);
+  }
+  int d = p.rot;
+  for (; d % 4 != 0; d += 2)                              // (rot is even)
+    if (lane < 2) st_elem(dst + d + lane, value(d + lane));
+  for (d += lane * 4; d < p.D; d += 128) {
+    float4 v = ld_elem4(src + d), m = make_float4(r, r, r, r);
+    if (bias != nullptr) {
+      const float4 e = ld_elem4(bias + d);
+      v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+    }
+    if (p.norm) {
+      const float4 e = ld_elem4(w + d);
+      m.x *= e.x; m.y *= e.y; m.z *= e.z; m.w *= e.w;
+    }
+    st_elem4(dst + d, make_float4(v.x * m.x, v.y * m.y, v.z * m.z, v.w * m.w));
+  }
 }
 
 template <typename T>
-__device__ __noinline__ void wa_append_key(const WindowAttnParams& p, const T* base, const int32_t* bt, int g, float rstd, int pos, int lane) {
+__device__ __noinline__ void wa_append_key(const WindowAttnParams& p, const T* base, const int32_t* bt, const float2* cs, int g, float rstd, int pos, int lane) {
   const size_t o = static_cast<size_t>(g) * p.D;
-  wa_head(p, base + p.k_off + o, p.bk ? p.bk + o : nullptr, p.norm == 2 ? p.wk + o : p.wk, rstd, 1.f, pos, lane,
+  wa_head(p, base + p.k_off + o, p.bk ? p.bk + o : nullptr, p.norm == 2 ? p.wk + o : p.wk, cs, rstd, 1.f, lane,
           static_cast<T*>(p.k_cache) + wa_token(p, bt, p.hkv * p.maps, g, pos) * p.D);
 }
 
@@ -125,9 +146,13 @@ template <typename T>
 __device__ __forceinline__ void wa_append_value(const WindowAttnParams& p, const T* base, const int32_t* bt, int g, int pos, int lane) {
   const T* v = base + p.v_off + static_cast<size_t>(g) * p.DV;
   T* dst = static_cast<T*>(p.v_cache) + wa_token(p, bt, p.hkv, g, pos) * p.DV;
-  for (int d = lane; d < p.DV; d += 32) {
-    if (p.bv == nullptr) dst[d] = v[d];
-    else st_elem(dst + d, ld_elem(v + d) + p.bv[g * p.DV + d]);
+  for (int d = lane * 4; d < p.DV; d += 128) {
+    float4 x = ld_elem4(v + d);
+    if (p.bv != nullptr) {
+      const float4 e = ld_elem4(p.bv + g * p.DV + d);
+      x.x += e.x; x.y += e.y; x.z += e.z; x.w += e.w;
+    }
+    st_elem4(dst + d, x);
   }
 }
 
@@ -143,6 +168,7 @@ __device__ __forceinline__ float wa_row_rstd(const WindowAttnParams& p, const T*
 template <typename T>
 __global__ void __launch_bounds__(256) qk_norm_append_kernel(const __grid_constant__ WindowAttnParams p) {
   __shared__ float scratch[8];
+  __shared__ float2 cs[128];
   pdl_wait();
   const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hk = p.hkv * p.maps;
   T* base = static_cast<T*>(p.proj) + static_cast<size_t>(row) * p.stride;
@@ -152,15 +178,19 @@ __global__ void __launch_bounds__(256) qk_norm_append_kernel(const __grid_consta
     rk = wa_row_rstd(p, base, 1, scratch);
   }
   const int pos = p.positions[row];
+  if (p.rot) {
+    wa_angles(p, pos, cs);
+    __syncthreads();
+  }
   const float temp = wa_temperature(p, pos);
   const int32_t* bt = p.block_table + static_cast<size_t>(p.row_req[row]) * p.max_blocks;
   for (int head = warp; head < p.hq + hk + p.hkv; head += 8) {
     if (head < p.hq) {
       const size_t o = static_cast<size_t>(head) * p.D;
       T* q = base + p.q_off + o;
-      wa_head(p, q, p.bq ? p.bq + o : nullptr, p.norm == 2 ? p.wq + o : p.wq, rq, temp, pos, lane, q);
+      wa_head(p, q, p.bq ? p.bq + o : nullptr, p.norm == 2 ? p.wq + o : p.wq, cs, rq, temp, lane, q);
     } else if (head < p.hq + hk) {
-      wa_append_key(p, base, bt, head - p.hq, rk, pos, lane);
+      wa_append_key(p, base, bt, cs, head - p.hq, rk, pos, lane);
     } else {
       wa_append_value(p, base, bt, head - p.hq - hk, pos, lane);
     }
@@ -182,6 +212,7 @@ __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(const __grid
   float* q_s = wa_smem;                                   // [NG][D]
   float* red_acc = q_s + NG * p.D;                        // [warps][NG][DV]
   __shared__ float red_m[kWaWarps][NG], red_l[kWaWarps][NG], scratch[kWaWarps];
+  __shared__ float2 cs[128];
   pdl_wait();
   const int group = p.hq / (p.hkv * MAPS), chunks = (group + NGM - 1) / NGM, hk = p.hkv * MAPS;
   const int kvh = blockIdx.x / chunks, g0 = (blockIdx.x % chunks) * NGM;
@@ -208,13 +239,17 @@ __global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(const __grid
       rq = wa_row_rstd(p, base, 0, scratch);
       if (append) rk = wa_row_rstd(p, base, 1, scratch);
     }
+    if (p.rot) {
+      wa_angles(p, pos, cs);
+      __syncthreads();
+    }
     const float f = p.scale * wa_temperature(p, pos);
     for (int i = warp; i < NG + (append ? MAPS + 1 : 0); i += kWaWarps) {
       if (i < NG) {
         const size_t o = static_cast<size_t>(head_of(i)) * p.D;
-        wa_head(p, base + p.q_off + o, p.bq ? p.bq + o : nullptr, p.norm == 2 ? p.wq + o : p.wq, rq, f, pos, lane, q_s + i * p.D);
+        wa_head(p, base + p.q_off + o, p.bq ? p.bq + o : nullptr, p.norm == 2 ? p.wq + o : p.wq, cs, rq, f, lane, q_s + i * p.D);
       } else if (i < NG + MAPS) {
-        wa_append_key(p, base, bt, kvh * MAPS + i - NG, rk, pos, lane);
+        wa_append_key(p, base, bt, cs, kvh * MAPS + i - NG, rk, pos, lane);
       } else {
         wa_append_value(p, base, bt, kvh, pos, lane);
       }
