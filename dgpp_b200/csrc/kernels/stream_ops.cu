@@ -135,6 +135,20 @@ struct RowNorm {
   const float *w, *b;        // weights; bias or null
 };
 
+// v += one row of fp32 (or nothing)
+template <int NT, int NV>
+__device__ __forceinline__ void add_row(float4 (&v)[NV], const float* __restrict__ b, int cols) {
+  if (b == nullptr) return;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + NT * j) * 4;
+    if (i < cols) {
+      const float4 e = ld_elem4(b + i);
+      v[j].x += e.x; v[j].y += e.y; v[j].z += e.z; v[j].w += e.w;
+    }
+  }
+}
+
 // Norm of a row held in registers; columns at or beyond n are zero and stay zero (their weights and biases are zero).
 template <int NT, int NV>
 __device__ __forceinline__ void norm_row(float4 (&v)[NV], const RowNorm& norm, int cols, int n, float eps, float* scratch) {
@@ -162,11 +176,11 @@ __device__ __forceinline__ void norm_row(float4 (&v)[NV], const RowNorm& norm, i
   for (int j = 0; j < NV; ++j) {
     const int i = (threadIdx.x + NT * j) * 4;
     if (i < cols) {
-      const float4 g = ld_elem4(norm.w + i), b = norm.b != nullptr ? ld_elem4(norm.b + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-      v[j].x = fmaf(v[j].x, r * g.x, b.x); v[j].y = fmaf(v[j].y, r * g.y, b.y);
-      v[j].z = fmaf(v[j].z, r * g.z, b.z); v[j].w = fmaf(v[j].w, r * g.w, b.w);
+      const float4 g = ld_elem4(norm.w + i);
+      v[j].x *= r * g.x; v[j].y *= r * g.y; v[j].z *= r * g.z; v[j].w *= r * g.w;
     }
   }
+  add_row<NT, NV>(v, norm.b, cols);
 }
 
 struct StreamNorm {
@@ -199,12 +213,7 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
       const int i = (threadIdx.x + NT * j) * 4;
       v[j] = zero;
       if (i >= cols) continue;
-      if (p.delta_b != nullptr) v[j] = ld_elem4(p.delta_b + i);
-      if (delta != nullptr) {
-        const float4 a = ld_elem4(delta + base + i);
-        v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
-        continue;
-      }
+      if (delta != nullptr) { v[j] = ld_elem4(delta + base + i); continue; }
       for (int k = 0; k < moe.top; ++k) {
         const float4 a = ld_elem4(moe.y + static_cast<size_t>(moe.pair_row[row * moe.top + k]) * cols + i);
         v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
@@ -214,19 +223,24 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
         v[j].x = fmaf(sg, a.x, v[j].x); v[j].y = fmaf(sg, a.y, v[j].y); v[j].z = fmaf(sg, a.z, v[j].z); v[j].w = fmaf(sg, a.w, v[j].w);
       }
     }
+    add_row<NT, NV>(v, p.delta_b, cols);
     norm_row<NT, NV>(v, p.post, cols, n, p.eps, scratch);
   }
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     const int i = (threadIdx.x + NT * j) * 4;
     float4 a = i < cols ? ld_elem4(x + base + i) : zero;
-    if (p.vec != nullptr && i < cols) {
-      const float4 e = ld_elem4(p.vec + i);
-      a.x += e.x; a.y += e.y; a.z += e.z; a.w += e.w;
-    }
     if (add) { a.x = fmaf(p.mult, v[j].x, a.x); a.y = fmaf(p.mult, v[j].y, a.y); a.z = fmaf(p.mult, v[j].z, a.z); a.w = fmaf(p.mult, v[j].w, a.w); }
     v[j] = a;
-    if (i < cols && (add || p.vec != nullptr)) st_elem4(x + base + i, a);
+    if (i < cols && add && p.vec == nullptr) st_elem4(x + base + i, a);
+  }
+  if (p.vec != nullptr) {
+    add_row<NT, NV>(v, p.vec, cols);
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int i = (threadIdx.x + NT * j) * 4;
+      if (i < cols) st_elem4(x + base + i, v[j]);
+    }
   }
   norm_row<NT, NV>(v, p.pre, cols, n, p.eps, scratch);
 #pragma unroll
