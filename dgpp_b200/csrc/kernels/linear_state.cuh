@@ -9,8 +9,13 @@
 //   state space          S <- a_t S + dt_t k_t v_t^T (a decay per token and head);  o_t = S^T q_t + D_h v_t
 //                        q, k (shared by groups of heads), v pass a causal depthwise convolution with bias and silu;
 //                        dt_t = softplus(raw step + bias),  a_t = exp(-exp(A) dt_t)
+//   matrix memory        S <- d_t S + w_t k_t v_t^T,  n <- d_t n + w_t k_t,  o_t = S^T q_t / (max(|n . q_t|, exp(-m_t)) + 1e-6)
+//                        (the mLSTM of xLSTM); log gates i = cap tanh((raw + bias) / cap), f = logsigmoid(cap tanh((raw + bias) / cap)),
+//                        running maximum m_t = max(f + m_(t-1), i) from m = 0, d_t = exp(f + m_(t-1) - m_t), w_t = exp(i - m_t);
+//                        a norm per head and a sigmoid gate per column behind it; q, k, v as projected, q scaled
 //
-// All are one kernel family (template parameter RULE; linear_state.cu, state_space.cu and gated_delta.cu hold the entry points).  A pass
+// All are one kernel family (template parameter RULE; linear_state.cu, state_space.cu, gated_delta.cu and matrix_memory.cu hold the entry
+// points).  A pass
 // carries runs of consecutive tokens of any number of requests:
 // run r = rows [run_start[r], run_start[r + 1]) of the request in state slot row_slot[first row].
 //
@@ -21,7 +26,8 @@
 //   lin_block    16-token blocks in parallel: the block's decay products and token-pair matrices (ssd_block, gated_block:
 //                the same for scalar decays, which leave q and k as they are, shared by a group of heads)
 //   lin_scan     block-sequential part: one CTA per (32 state columns, head, run), S in registers, the next block's operands
-//                streaming in with cp.async while the current one is consumed
+//                streaming in with cp.async while the current one is consumed.  Matrix memory: one more CTA per head carries n as the
+//                state's column for a value that is always one, and finishes the denominators
 //   lin_tail     the newest inputs of the convolution go to the request's ring after every reader is done
 //
 // The decode kernel takes o_t as (g S)^T q + (k . q) u, the read-out after the write, so both reductions over the key channels
@@ -39,10 +45,10 @@
 
 namespace dgpp {
 
-enum LinearRule { kLightning = 0, kDelta = 1, kStateSpace = 2, kScalarDelta = 3 };
+enum LinearRule { kLightning = 0, kDelta = 1, kStateSpace = 2, kScalarDelta = 3, kMatrix = 4 };
 
 __host__ __device__ constexpr bool is_delta(int rule) { return rule == kDelta || rule == kScalarDelta; }
-__host__ __device__ constexpr bool scalar_decay(int rule) { return rule == kStateSpace || rule == kScalarDelta; }
+__host__ __device__ constexpr bool scalar_decay(int rule) { return rule == kStateSpace || rule == kScalarDelta || rule == kMatrix; }
 
 struct LinearArgs {
   const void* proj;         // [rows, stride] (T): conv channels q (hk * DK) | k (hk * DK) | v (hv * DV) from column c_off
@@ -67,7 +73,11 @@ struct LinearArgs {
   float* o;                 // [rows, hv * ow] fp32 read-outs (scan; lightning and state-space decode)
   void* out;                // [rows, out_stride] (T): normed and gated read-outs (delta decode)
   int64_t out_stride;
-  const float* norm_w;      // [DV]
+  const float* norm_w;      // [DV] (matrix memory: [hv * DV])
+  float* nstate;            // [slots, hv, DK + 4]: n, then the running maximum m (matrix memory)
+  float* den;               // [rows, hv] denominators of the read-outs in `o` (matrix memory)
+  const float *i_bias, *f_bias;   // [hv]; raw input gates at b_off, raw forget gates at a_off (matrix memory)
+  float gate_cap;
   int rows, runs, blocks, hk, hv, taps, vdim, ow;   // ow: columns of a head's read-out in `o` (DV; state space: vdim)
   float q_scale, eps;
 };
@@ -117,6 +127,17 @@ __device__ __forceinline__ float conv_channel(const LinearArgs& a, const T* x, i
   return acc;
 }
 
+// Log gates of a row and head (matrix memory).
+template <typename T>
+__device__ __forceinline__ float2 matrix_gates(const LinearArgs& a, int row, int h) {
+  const T* x = static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + h;
+  const float i = a.gate_cap * tanhf((ld_elem(x + a.b_off) + a.i_bias[h]) / a.gate_cap);
+  const float f = a.gate_cap * tanhf((ld_elem(x + a.a_off) + a.f_bias[h]) / a.gate_cap);
+  return make_float2(i, -softplus_f32(-f));
+}
+
+__device__ __forceinline__ float matrix_den(float nq, float floor) { return fmaxf(fabsf(nq), floor) + 1e-6f; }
+
 __device__ __forceinline__ float4 fma4(float4 s, float a, float4 acc) {
   acc.x = fmaf(s.x, a, acc.x); acc.y = fmaf(s.y, a, acc.y); acc.z = fmaf(s.z, a, acc.z); acc.w = fmaf(s.w, a, acc.w);
   return acc;
@@ -125,7 +146,7 @@ __device__ __forceinline__ float4 fma4(float4 s, float a, float4 acc) {
 // grid (hv, rows)
 template <typename T, int DK, int DV, int RULE>
 __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(LinearArgs a) {
-  constexpr bool DELTA = is_delta(RULE), CH = RULE == kDelta, SSD = RULE == kStateSpace;
+  constexpr bool DELTA = is_delta(RULE), CH = RULE == kDelta, SSD = RULE == kStateSpace, MAT = RULE == kMatrix;
   using G = LinGeom<DK, DV>;
   constexpr int NT = G::kThreads, PER = G::kPer, PARTS = G::kParts;
   extern __shared__ __align__(16) float ld_smem[];
@@ -133,7 +154,7 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
   float* red_m = red_n + PARTS * DV;                      // [PARTS][DV] (delta)
   __shared__ float qs[DK], ks[DK], gs[DK];
   __shared__ __align__(16) float vs[DV], us[DV];
-  __shared__ float scal[3];                               // |q|^2, |k|^2, q . k
+  __shared__ float scal[3];                               // |q|^2 (matrix memory: n . q), |k|^2, q . k
   __shared__ float scratch[32];
   pdl_wait();
   const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x;
@@ -157,12 +178,20 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
       acc = conv_channel(a, x + ch, a.stride, xv, 0, C, slot, pos, base, ch);
       if (c >= 2 * DK || h % ratio == 0) a.ring[(static_cast<size_t>(slot) * a.taps + base) * C + ch] = xv;
     }
-    acc = silu_f32(acc);
+    if (!MAT) acc = silu_f32(acc);
     if (c < DK) qs[c] = acc;
     else if (c < 2 * DK) ks[c - DK] = acc;
     else vs[c - 2 * DK] = acc;
   }
-  float beta = 1.f, dh = 1.f, skip = 0.f;
+  float beta = 1.f, dh = 1.f, skip = 0.f, m_new = 0.f;
+  float* ns = MAT ? a.nstate + (static_cast<size_t>(slot) * a.hv + h) * (DK + 4) : nullptr;
+  if (MAT) {
+    const float2 g = matrix_gates<T>(a, row, h);
+    const float past = g.y + (pos > 0 ? ns[DK] : 0.f);
+    m_new = fmaxf(past, g.x);
+    dh = expf(past - m_new);
+    beta = expf(g.x - m_new);
+  }
   if (SSD) {
     beta = softplus_f32(ld_elem(static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.b_off + h) + a.dt_bias[h]);
     dh = expf(-expf(a.A_log[h]) * beta);
@@ -182,14 +211,23 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
   }
   __syncthreads();
   if (tid < 32) {
-    float q2 = 0.f, k2 = 0.f, qk = 0.f;
+    float q2 = 0.f, k2 = 0.f, qk = 0.f, nq = 0.f;
     for (int c = tid; c < DK; c += 32) {
       q2 = fmaf(qs[c], qs[c], q2);
       k2 = fmaf(ks[c], ks[c], k2);
       qk = fmaf(qs[c], ks[c], qk);
+      if (MAT) {
+        const float n = fmaf(beta, ks[c], pos > 0 ? dh * ns[c] : 0.f);
+        ns[c] = n;
+        nq = fmaf(n, qs[c], nq);
+      }
     }
+    if (MAT) nq = warp_sum_f32(nq);
     q2 = warp_sum_f32(q2); k2 = warp_sum_f32(k2); qk = warp_sum_f32(qk);
-    if (tid == 0) { scal[0] = q2; scal[1] = k2; scal[2] = qk; }
+    if (tid == 0) {
+      scal[0] = MAT ? nq : q2; scal[1] = k2; scal[2] = qk;
+      if (MAT) ns[DK] = m_new;
+    }
   }
   // ---- decay, both reductions
   float4 n4 = make_float4(0.f, 0.f, 0.f, 0.f), m4 = n4;
@@ -204,8 +242,9 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
   *reinterpret_cast<float4*>(red_n + part * DV + 4 * cg) = n4;
   if (DELTA) *reinterpret_cast<float4*>(red_m + part * DV + 4 * cg) = m4;
   __syncthreads();
-  const float rq = DELTA ? a.q_scale / sqrtf(scal[0] + 1e-6f) : 1.f, rk = DELTA ? 1.f / sqrtf(scal[1] + 1e-6f) : 1.f;
+  const float rq = DELTA ? a.q_scale / sqrtf(scal[0] + 1e-6f) : (MAT ? a.q_scale : 1.f), rk = DELTA ? 1.f / sqrtf(scal[1] + 1e-6f) : 1.f;
   const float qk = scal[2] * rq * rk;
+  const float inv = MAT ? 1.f / matrix_den(scal[0] * rq, expf(-m_new)) : 1.f;
   float ss = 0.f;
   for (int c = tid; c < DV; c += NT) {
     float n = 0.f, m = 0.f;
@@ -214,11 +253,11 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
       n += red_n[w * DV + c];
       if (DELTA) m += red_m[w * DV + c];
     }
-    const float u = DELTA ? beta * (vs[c] - m * rk) : (SSD ? beta * vs[c] : vs[c]);
-    const float o = n * rq + qk * u + (SSD ? skip * vs[c] : 0.f);
+    const float u = DELTA ? beta * (vs[c] - m * rk) : (SSD || MAT ? beta * vs[c] : vs[c]);
+    const float o = (n * rq + qk * u + (SSD ? skip * vs[c] : 0.f)) * inv;
     us[c] = u * rk;                              // the key's norm rides on u
     ss = fmaf(o, o, ss);
-    if (DELTA) vs[c] = o;
+    if (DELTA || MAT) vs[c] = o;
     else if (c < a.ow) a.o[(static_cast<size_t>(row) * a.hv + h) * a.ow + c] = o;
   }
   __syncthreads();
@@ -228,10 +267,13 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
     const int r = part + PARTS * i;
     sp[static_cast<size_t>(r) * G::kCols4] = fma4(u4, ks[r], s[i]);
   }
-  if (DELTA) {
+  if (DELTA || MAT) {
     const float r = 1.f / sqrtf(block_sum_f32(ss, scratch) / static_cast<float>(a.vdim) + a.eps);
     T* dst = static_cast<T*>(a.out) + static_cast<size_t>(row) * a.out_stride + h * DV;
-    if (CH) {
+    if (MAT) {
+      const T* gt = static_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.stride + a.g_off + h * DV;
+      for (int c = tid; c < DV; c += NT) st_elem(dst + c, vs[c] * r * a.norm_w[h * DV + c] * sigmoid_f32(ld_elem(gt + c)));
+    } else if (CH) {
       const float* gt = a.low + static_cast<size_t>(row) * a.low_stride + a.hv * DK + h * DV;
       for (int c = tid; c < DV; c += NT) st_elem(dst + c, vs[c] * r * a.norm_w[c] * sigmoid_f32(gt[c]));
     } else {
@@ -246,9 +288,10 @@ __global__ void __launch_bounds__(LinGeom<DK, DV>::kThreads) lin_decode_kernel(L
 // strengths [rows, hv] (delta) at the end.  State space: per row q, k, v, decay and step [hv] each; per block and head P with the
 // steps and the skip folded in [16, 16] and 16 prefix products, then 16 write weights.  Scalar delta: per row q, k (not yet unit
 // vectors), v, decay and strength; per block and head P and T B [16, 16], then 16 factors each of Q S, of the writes and of K S, and
-// gamma_16; the lengths of q and k ride in all of these.
+// gamma_16; the lengths of q and k ride in all of these.  Matrix memory: as state space (d_t and w_t for decay and step), then exp(-m_t)
+// [rows, hv].
 struct PrepView {
-  float *q, *k, *v, *g, *kt, *qt, *kh, *gam, *pm, *tb, *b;
+  float *q, *k, *v, *g, *kt, *qt, *kh, *gam, *pm, *tb, *b, *fl;
 };
 template <int DK, int DV, int RULE>
 __device__ __forceinline__ PrepView prep_view(const LinearArgs& a) {
@@ -266,8 +309,10 @@ __device__ __forceinline__ PrepView prep_view(const LinearArgs& a) {
     p.g = p.gam + B * a.hv * (RULE == kScalarDelta ? 64 : 32);
     p.b = p.g + R * a.hv;
     p.kt = p.qt = p.kh = nullptr;
+    p.fl = p.b + R * a.hv;
     return p;
   }
+  p.fl = nullptr;
   p.kt = p.g;
   p.qt = p.g + (DELTA ? R * a.hv * DK : 0);
   p.kh = p.qt + R * a.hv * DK;
@@ -357,6 +402,7 @@ __global__ void __launch_bounds__(256) lin_tail_kernel(LinearArgs a, int C) {
 //     O = (Q * gamma) S + P U,            P_ts = sum_c q_t k_s (g_(s+1) .. g_t)                                      (s <= t)
 //     S <- gamma_16 * S + (K * g_(t+1) .. g_16)^T U
 //     scalar     as delta, with gamma_t a number: gamma_t (K S) instead of (K * gamma) S
+//     matrix m.  as state sp. with D = 0, dt_s = w_s
 //     state sp.  U = V,  P_ts = (q_t . k_s) (a_(s+1) .. a_t) dt_s + [s = t] D,  O = (a_1 .. a_t) (Q S) + P U,
 //                S <- (a_1 .. a_16) S + K^T (dt_s a_(s+1) .. a_16 U)
 // lin_block (parallel over blocks and heads) makes K * gamma, Q * gamma, the suffix-weighted keys, gamma_16, T B and P.
@@ -539,10 +585,63 @@ __global__ void __launch_bounds__(128) ssd_prep_kernel(LinearArgs a) {
   }
 }
 
+// Matrix memory: q (scaled), k and v as fp32 rows.  grid (ceil(C / 1024), rows), 256 threads.
+template <typename T, int DK, int DV>
+__global__ void __launch_bounds__(256) matrix_prep_kernel(LinearArgs a) {
+  pdl_wait();
+  const int nk = a.hk * DK, nv = a.hv * DV, ch = (blockIdx.x * 256 + threadIdx.x) * 4;
+  const size_t row = blockIdx.y;
+  if (ch >= 2 * nk + nv) return;
+  const PrepView pv = prep_view<DK, DV, kMatrix>(a);
+  float4 x = ld_elem4(static_cast<const T*>(a.proj) + row * a.stride + a.c_off + ch);
+  if (ch < nk) { x.x *= a.q_scale; x.y *= a.q_scale; x.z *= a.q_scale; x.w *= a.q_scale; }
+  float* dst = ch < nk ? pv.q + row * nk + ch : (ch < 2 * nk ? pv.k + row * nk + ch - nk : pv.v + row * nv + ch - 2 * nk);
+  *reinterpret_cast<float4*>(dst) = x;
+}
+
+// The running maximum of a run and head, 32 tokens at a time: (F, M) of consecutive tokens combine to (F1 + F2, max(M1 + F2, M2)), and
+// m_t = max(m + F, M).  grid (ceil(hv / 4), runs), one warp per head; the next tokens' gates are loaded while these are scanned.
+template <typename T, int DK, int DV>
+__global__ void __launch_bounds__(128) matrix_gates_kernel(LinearArgs a) {
+  pdl_wait();
+  const int h = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= a.hv) return;
+  const int first = a.run_start[blockIdx.y], last = a.run_start[blockIdx.y + 1];
+  const PrepView pv = prep_view<DK, DV, kMatrix>(a);
+  float* ns = a.nstate + (static_cast<size_t>(a.row_slot[first]) * a.hv + h) * (DK + 4) + DK;
+  float m = a.positions[first] == 0 ? 0.f : *ns;
+  const float2 none = make_float2(-INFINITY, 0.f);
+  float2 next = first + lane < last ? matrix_gates<T>(a, first + lane, h) : none;
+  for (int t0 = first; t0 < last; t0 += 32) {
+    const float2 g = next;
+    next = t0 + 32 + lane < last ? matrix_gates<T>(a, t0 + 32 + lane, h) : none;
+    float F = g.y, M = g.x;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
+      if (lane >= o) {
+        M = fmaxf(Mp + F, M);
+        F += Fp;
+      }
+    }
+    const float mt = fmaxf(m + F, M);
+    float before = __shfl_up_sync(0xffffffffu, mt, 1);
+    if (lane == 0) before = m;
+    if (t0 + lane < last) {
+      const size_t o = static_cast<size_t>(t0 + lane) * a.hv + h;
+      pv.g[o] = expf(fminf(g.y + before - mt, 0.f));
+      pv.b[o] = expf(g.x - mt);
+      pv.fl[o] = expf(-mt);
+    }
+    m = __shfl_sync(0xffffffffu, mt, 31);
+  }
+  if (lane == 0) *ns = m;
+}
+
 constexpr int kSsdHeads = 8;
 
 // grid (hk * ceil(heads per group / 8), blocks), 256 threads: thread (t, s) holds q_t . k_s and walks up to 8 heads of the group.
-template <int DK, int DV>
+template <int DK, int DV, int RULE>
 __global__ void __launch_bounds__(256) ssd_block_kernel(LinearArgs a) {
   __shared__ float ks[kBlk][DK + 1], qs[kBlk][DK + 1];
   __shared__ float as[kSsdHeads][kBlk], ds[kSsdHeads][kBlk];
@@ -552,7 +651,7 @@ __global__ void __launch_bounds__(256) ssd_block_kernel(LinearArgs a) {
   const int nh = min(kSsdHeads, (hk + 1) * ratio - h0), blk = blockIdx.y, tid = threadIdx.x;
   int row0 = 0, n = 0;
   if (!find_block(a, blk, row0, n)) return;
-  const PrepView pv = prep_view<DK, DV, kStateSpace>(a);
+  const PrepView pv = prep_view<DK, DV, RULE>(a);
   for (int i = tid; i < kBlk * DK; i += 256) {
     const int t = i / DK, c = i % DK;
     const size_t o = (static_cast<size_t>(row0 + t) * a.hk + hk) * DK + c;
@@ -579,7 +678,7 @@ __global__ void __launch_bounds__(256) ssd_block_kernel(LinearArgs a) {
       p = dot;
       for (int j = s + 1; j <= t; ++j) p *= as[h][j];
       p *= ds[h][s];
-      if (s == t && t < n) p += a.skip[h0 + h];
+      if (RULE == kStateSpace && s == t && t < n) p += a.skip[h0 + h];
     }
     pv.pm[bh * kBlk * kBlk + tid] = p;
     if (tid < 2 * kBlk) {
@@ -691,14 +790,14 @@ struct ScanGeom {
   static constexpr int kV = kK + (RULE == kDelta ? kBlk * DK : 0);
   static constexpr int kP = kV + kBlk * kScanCols, kT = kP + kBlk * kBlk;
   static constexpr int kG = kT + (is_delta(RULE) ? kBlk * kBlk : 0);
-  static constexpr int kGam = RULE == kStateSpace ? 2 * kBlk : (RULE == kScalarDelta ? 4 * kBlk : DK);   // factors of a block and head
+  static constexpr int kGam = RULE == kStateSpace || RULE == kMatrix ? 2 * kBlk : (RULE == kScalarDelta ? 4 * kBlk : DK);   // factors of a block and head
   static constexpr int kTotal = kG + kGam;
 };
 
 // Block-sequential pass.  A CTA owns 32 columns of one head's state in registers: a thread 4 columns and the rows
 // 4 part + 4 PARTS i + e; the PARTS lanes of a column group sit in one warp, so a group works through a block on its own and
 // the CTA only meets at the staging buffers (the next block streams in with cp.async meanwhile).
-// grid (DV / 32, hv, runs)
+// grid (DV / 32, hv, runs); matrix memory: one more column of CTAs for n
 template <int DK, int DV, int RULE>
 __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(LinearArgs a) {
   constexpr bool DELTA = is_delta(RULE), CH = RULE == kDelta, SCALAR = scalar_decay(RULE);
@@ -718,11 +817,18 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
   float* us = ws + NV;                                      // [16][4] U
   float* sp = a.state + (static_cast<size_t>(slot) * a.hv + h) * DK * DV + j0;
   const bool fresh = a.positions[first] == 0;
+  const bool ones = RULE == kMatrix && jb >= DV;            // this CTA carries n, in its first column
+  float* ns = ones ? a.nstate + (static_cast<size_t>(slot) * a.hv + h) * (DK + 4) : nullptr;
   float s[NI][4][4];                                        // [i][row e][column]
 #pragma unroll
   for (int i = 0; i < NI; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
+      if (ones) {
+        s[i][e][0] = cg == 0 && !fresh ? ns[4 * PARTS * i + 4 * part + e] : 0.f;
+        s[i][e][1] = s[i][e][2] = s[i][e][3] = 0.f;
+        continue;
+      }
       const float4 v = fresh ? make_float4(0.f, 0.f, 0.f, 0.f)
                              : *reinterpret_cast<const float4*>(sp + static_cast<size_t>(4 * PARTS * i + 4 * part + e) * DV);
       s[i][e][0] = v.x; s[i][e][1] = v.y; s[i][e][2] = v.z; s[i][e][3] = v.w;
@@ -746,7 +852,8 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
     }
     for (int i = tid; i < kBlk * (kScanCols / 4); i += NT) {
       const int t = i / (kScanCols / 4), c = (i % (kScanCols / 4)) * 4;
-      if (t < n) cp_async_16(d + G::kV + t * kScanCols + c, pv.v + (static_cast<size_t>(t0 + t) * a.hv + h) * DV + jb + c);
+      if (ones) *reinterpret_cast<float4*>(d + G::kV + t * kScanCols + c) = make_float4(c == 0 && t < n ? 1.f : 0.f, 0.f, 0.f, 0.f);
+      else if (t < n) cp_async_16(d + G::kV + t * kScanCols + c, pv.v + (static_cast<size_t>(t0 + t) * a.hv + h) * DV + jb + c);
       else *reinterpret_cast<float4*>(d + G::kV + t * kScanCols + c) = zero;
     }
     const size_t bh = static_cast<size_t>(b) * a.hv + h;
@@ -805,6 +912,10 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
     const float* d = sc_smem + buf * G::kTotal;
     const float* vb = d + G::kV + 4 * cg;                   // [16] rows of 32 columns, this group's 4
     const int n = min(kBlk, last - t0);
+    if (ones && tid >= 32) {                                // columns of zeros
+      __syncthreads();
+      continue;
+    }
     float val[NV], x[CNT];
     if (DELTA) {
       rows_times_state(d + (CH ? G::kK : G::kH), val);
@@ -827,7 +938,10 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
     for (int i = 0; i < CNT; ++i) {
       const int idx = part * CNT + i;
       const float w = SCALAR ? d[G::kG + idx / 4] : 1.f;
-      if (idx / 4 < n && j0 + idx % 4 < a.ow) a.o[(static_cast<size_t>(t0 + idx / 4) * a.hv + h) * a.ow + j0 + idx % 4] = fmaf(w, val[i], x[i]);
+      if (ones) {
+        const size_t rh = static_cast<size_t>(t0 + idx / 4) * a.hv + h;
+        if (idx / 4 < n && cg == 0 && idx % 4 == 0) a.den[rh] = matrix_den(fmaf(w, val[i], x[i]), pv.fl[rh]);
+      } else if (idx / 4 < n && j0 + idx % 4 < a.ow) a.o[(static_cast<size_t>(t0 + idx / 4) * a.hv + h) * a.ow + j0 + idx % 4] = fmaf(w, val[i], x[i]);
     }
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
@@ -860,9 +974,14 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
 #pragma unroll
   for (int i = 0; i < NI; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
-      *reinterpret_cast<float4*>(sp + static_cast<size_t>(4 * PARTS * i + 4 * part + e) * DV) =
-          make_float4(s[i][e][0], s[i][e][1], s[i][e][2], s[i][e][3]);
+    for (int e = 0; e < 4; ++e) {
+      if (ones) {
+        if (cg == 0) ns[4 * PARTS * i + 4 * part + e] = s[i][e][0];
+      } else {
+        *reinterpret_cast<float4*>(sp + static_cast<size_t>(4 * PARTS * i + 4 * part + e) * DV) =
+            make_float4(s[i][e][0], s[i][e][1], s[i][e][2], s[i][e][3]);
+      }
+    }
 }
 
 template <typename T, int DK, int DV, int RULE>
@@ -886,7 +1005,12 @@ static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
     attr = true;
   }
   bool prepared = false;
-  if constexpr (scalar_decay(RULE)) {
+  if constexpr (RULE == kMatrix) {
+    matrix_prep_kernel<T, DK, DV><<<dim3(dgpp_ceil_div(2 * a.hk * DK + a.hv * DV, 1024), a.rows), 256, 0, st>>>(a);
+    DGPP_CUDA_OK(cudaGetLastError());
+    matrix_gates_kernel<T, DK, DV><<<dim3(dgpp_ceil_div(a.hv, 4), a.runs), 128, 0, st>>>(a);
+    prepared = true;
+  } else if constexpr (scalar_decay(RULE)) {
     const dim3 grid(dgpp_ceil_div(2 * a.hk * DK + a.hv * DV, 512) + 1, a.blocks);
     prepared = a.taps <= 4 && a.stride % 4 == 0 && a.c_off % 4 == 0;
     if (!prepared) {}
@@ -895,14 +1019,15 @@ static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
     else if (a.taps == 3) ssd_prep_kernel<T, DK, DV, RULE, 3><<<grid, 128, 0, st>>>(a);
     else ssd_prep_kernel<T, DK, DV, RULE, 4><<<grid, 128, 0, st>>>(a);
   }
-  if (!prepared) lin_prep_kernel<T, DK, DV, RULE><<<dgpp_ceil_div(a.rows * (a.hk + a.hv), 8), 256, 0, st>>>(a);
+  if constexpr (RULE != kMatrix)
+    if (!prepared) lin_prep_kernel<T, DK, DV, RULE><<<dgpp_ceil_div(a.rows * (a.hk + a.hv), 8), 256, 0, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   const dim3 groups(a.hk * dgpp_ceil_div(a.hv / a.hk, kSsdHeads), a.blocks);
-  if constexpr (RULE == kStateSpace) ssd_block_kernel<DK, DV><<<groups, 256, 0, st>>>(a);
+  if constexpr (RULE == kStateSpace || RULE == kMatrix) ssd_block_kernel<DK, DV, RULE><<<groups, 256, 0, st>>>(a);
   else if constexpr (RULE == kScalarDelta) gated_block_kernel<DK, DV><<<groups, 256, 0, st>>>(a);
   else lin_block_kernel<DK, DV, RULE><<<dim3(a.hv, a.blocks), 256, bsmem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
-  lin_scan_kernel<DK, DV, RULE><<<dim3(DV / kScanCols, a.hv, a.runs), ScanGeom<DK, RULE>::kThreads, smem, st>>>(a);
+  lin_scan_kernel<DK, DV, RULE><<<dim3(DV / kScanCols + (RULE == kMatrix ? 1 : 0), a.hv, a.runs), ScanGeom<DK, RULE>::kThreads, smem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   if (a.conv_w != nullptr) {
     const int C = 2 * a.hk * DK + a.hv * DV;

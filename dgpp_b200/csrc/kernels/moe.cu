@@ -353,8 +353,8 @@ DGPP_API int dgpp_moe_route(const void* x, int64_t x_stride, const void* gate, c
 }
 
 // Selection alone, over logits [T, E] (row stride logits_stride) that another kernel made, plus `bias` [E] fp32 where it is given; no
-// correction, no groups.
-DGPP_API int dgpp_moe_select(const void* logits, int64_t logits_stride, const void* bias, void* ids, void* weights, int T, int E, int k, int softmax, int norm_topk,
+// groups.  correction [E] or null: added to the scores for the choice alone.
+DGPP_API int dgpp_moe_select(const void* logits, int64_t logits_stride, const void* bias, const void* correction, void* ids, void* weights, int T, int E, int k, int softmax, int norm_topk,
                              float scaling, cudaStream_t st) {
   DGPP_REQUIRE(E >= 1 && E <= kMoeMaxExperts && k >= 1 && k <= kMoeMaxTopK && k <= E, "moe_select: E %d / k %d unsupported", E, k);
   if (T == 0) return 0;
@@ -364,6 +364,7 @@ DGPP_API int dgpp_moe_select(const void* logits, int64_t logits_stride, const vo
   a.logits_out = static_cast<float*>(const_cast<void*>(logits));
   a.logits_stride = logits_stride;
   a.logit_bias = static_cast<const float*>(bias);
+  a.bias = static_cast<const float*>(correction);
   a.T = T; a.E = E; a.k = k; a.n_group = 1; a.topk_group = 1;
   a.softmax = softmax; a.norm_topk = norm_topk; a.scaling = scaling;
   moe_router_select_kernel<<<T, kRouterThreads, 0, st>>>(a);

@@ -3,7 +3,8 @@
 //
 //   moe_route_small    up to 16 tokens, one CTA: picks every token's experts from its logits (sigmoid or softmax weights, ties to
 //                      the lower id), lists the experts in use as tiles of 16 rows over the SAME activation rows, and writes the
-//                      row of every (token, choice) pair and every tile row's weight (0: the token did not choose the expert)
+//                      row of every (token, choice) pair and every tile row's weight (0: the token did not choose the expert);
+//                      choices at or beyond `experts` are identity experts, whose output is the token's input: row -1
 //   moe_scatter_rows   any number of tokens, after the counting sort of moe_prefill.cu: copies a pair's activation row to its place
 //                      in the sorted tiles and writes the row's weight there
 // The weights ride along per tile row, so the activation kernel can scale what an expert sees.
@@ -24,8 +25,11 @@ struct RouteSmall {
   int32_t* pair_row;       // [T * top]
   int32_t* tiles;          // [max_tiles]
   float* row_w;            // [max_tiles * 16]
+  float* wts;              // [T * top] weight of every pair, or null
   const float* bias;       // [E] added to the logits, or null
+  const float* correction; // [E] added to the scores for the choice alone, or null
   int T, E, top, max_tiles, score;   // score: 0 sigmoid, 1 softmax over all experts, 2 softmax over the chosen ones
+  int experts, norm_topk;            // outputs with matrices (the others are identity experts); weights divided by their sum
 };
 
 __global__ void __launch_bounds__(kSmallThreads) moe_route_small_kernel(RouteSmall a) {
@@ -56,6 +60,17 @@ __global__ void __launch_bounds__(kSmallThreads) moe_route_small_kernel(RouteSma
       for (int i = 0; i < kSmallExperts / 32; ++i) sum += expf(z[i] - mx);
       norm = warp_sum_f32(sum);
     }
+    // with a correction the choice goes by score + correction, and the scores are kept
+    float sc[kSmallExperts / 32];
+    if (a.correction != nullptr) {
+#pragma unroll
+      for (int i = 0; i < kSmallExperts / 32; ++i) {
+        const int e = lane + 32 * i;
+        if (e >= a.E) continue;
+        sc[i] = a.score == 0 ? sigmoid_f32(z[i]) : expf(z[i] - mx) / norm;
+        z[i] = sc[i] + a.correction[e];
+      }
+    }
     // both scores grow with the logit; equal scores of different logits go to the larger logit
     for (int r = 0; r < a.top; ++r) {
       float bv = -INFINITY;
@@ -72,20 +87,25 @@ __global__ void __launch_bounds__(kSmallThreads) moe_route_small_kernel(RouteSma
         if (ov > bv || (ov == bv && oe < be)) { bv = ov; be = oe; }
       }
       if (be >= a.E) be = 0;                           // only with logits that are not numbers
+      float chosen = 0.f;
 #pragma unroll
       for (int i = 0; i < kSmallExperts / 32; ++i)
-        if (lane + 32 * i == be) z[i] = -INFINITY;
+        if (lane + 32 * i == be) {
+          z[i] = -INFINITY;
+          if (a.correction != nullptr) chosen = sc[i];
+        }
+      if (a.correction != nullptr) chosen = __shfl_sync(0xffffffffu, chosen, be & 31);
       if (lane == 0) {
         int j = r;                                     // ascending ids: the order of the sum
         while (j > 0 && ids[t][j - 1] > be) { ids[t][j] = ids[t][j - 1]; wts[t][j] = wts[t][j - 1]; --j; }
         ids[t][j] = be;
         if (r == 0 && a.score == 2) mx = bv;           // the largest comes first
-        wts[t][j] = a.score == 0 ? sigmoid_f32(bv) : expf(bv - mx) / norm;
-        slot[be] = 1;
+        wts[t][j] = a.correction != nullptr ? chosen : (a.score == 0 ? sigmoid_f32(bv) : expf(bv - mx) / norm);
+        if (be < a.experts) slot[be] = 1;
       }
     }
-    if (a.score == 2 && lane == 0) {
-      float sum = 0.f;
+    if ((a.score == 2 || a.norm_topk) && lane == 0) {
+      float sum = 1e-20f;
       for (int j = 0; j < a.top; ++j) sum += wts[t][j];
       for (int j = 0; j < a.top; ++j) wts[t][j] /= sum;
     }
@@ -106,9 +126,14 @@ __global__ void __launch_bounds__(kSmallThreads) moe_route_small_kernel(RouteSma
   for (int i = total + tid; i < a.max_tiles; i += kSmallThreads) a.tiles[i] = -1;
   __syncthreads();
   if (t < a.T && lane < a.top) {
-    const int row = min(slot[ids[t][lane]], a.max_tiles - 1) * kSmallTokens + t;
-    a.pair_row[t * a.top + lane] = row;
-    a.row_w[row] = wts[t][lane];
+    if (a.wts != nullptr) a.wts[t * a.top + lane] = wts[t][lane];
+    if (ids[t][lane] >= a.experts) {
+      a.pair_row[t * a.top + lane] = -1;
+    } else {
+      const int row = min(slot[ids[t][lane]], a.max_tiles - 1) * kSmallTokens + t;
+      a.pair_row[t * a.top + lane] = row;
+      a.row_w[row] = wts[t][lane];
+    }
   }
 }
 
@@ -132,15 +157,19 @@ __global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const T* __restri
 
 using namespace dgpp;
 
-// logits [T, E] fp32 with row stride `stride` (bias [E] fp32 or null is added), T <= 16.  max_tiles >= min(E, T * top).
-DGPP_API int dgpp_moe_route_small(const void* logits, int64_t stride, const void* bias, void* pair_row, void* tiles, void* row_w, int T, int E, int top, int max_tiles,
-                                  int score, cudaStream_t st) {
-  DGPP_REQUIRE(score >= 0 && score <= 2, "moe_route_small: score %d", score);
+// logits [T, E] fp32 with row stride `stride` (bias [E] fp32 or null is added), T <= 16.  The first `experts` outputs have matrices;
+// max_tiles >= min(experts, T * top).  correction [E] or null: added to the scores for the choice alone; norm_topk: weights divided by
+// their sum.  wts [T * top] or null: the pairs' weights.
+DGPP_API int dgpp_moe_route_small(const void* logits, int64_t stride, const void* bias, const void* correction, void* pair_row, void* tiles,
+                                  void* row_w, void* wts, int T, int E, int experts, int top, int max_tiles, int score, int norm_topk, cudaStream_t st) {
+  DGPP_REQUIRE(score >= 0 && score <= 2 && (!correction || score < 2), "moe_route_small: score %d", score);
   DGPP_REQUIRE(E >= 1 && E <= kSmallExperts && top >= 1 && top <= kSmallTop && top <= E, "moe_route_small: %d of %d experts", top, E);
-  DGPP_REQUIRE(T <= kSmallTokens && max_tiles >= (E < T * top ? E : T * top), "moe_route_small: %d tokens in %d tiles", T, max_tiles);
+  DGPP_REQUIRE(experts >= 1 && experts <= E && (experts == E || wts), "moe_route_small: %d of %d outputs with matrices", experts, E);
+  DGPP_REQUIRE(T <= kSmallTokens && max_tiles >= (experts < T * top ? experts : T * top), "moe_route_small: %d tokens in %d tiles", T, max_tiles);
   if (T == 0) return 0;
   const RouteSmall a = {static_cast<const float*>(logits), stride, static_cast<int32_t*>(pair_row), static_cast<int32_t*>(tiles),
-                        static_cast<float*>(row_w), static_cast<const float*>(bias), T, E, top, max_tiles, score};
+                        static_cast<float*>(row_w), static_cast<float*>(wts), static_cast<const float*>(bias),
+                        static_cast<const float*>(correction), T, E, top, max_tiles, score, experts, norm_topk};
   moe_route_small_kernel<<<1, kSmallThreads, 0, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;

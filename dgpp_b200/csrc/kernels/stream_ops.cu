@@ -1,15 +1,18 @@
 // Row operators of models that keep the residual stream in fp32 (activations T = bf16 or fp32):
 //   embed_rows        out[r] = scale * table[ids[r]]                           (fp32 rows; on request a second time in T)
 //   resid_norm        x += delta (fp32, optional); out = x / sqrt(mean(x^2) + eps) * w           (out in T)
-//   gated_group_norm  per group of columns: out = o / sqrt(mean(o^2) + eps) * w * act(gate) * scale; act: sigmoid or silu
+//   gated_group_norm  per group of columns: out = o / sqrt(mean(o^2) + eps) * w * act(gate) * scale; act: sigmoid or silu; o may first be
+//                     divided by a number per row and group
 //   geglu             out = gelu_tanh(gate) * up
-//   stream_norm       x += mult * post(delta + bias) + vec; out = pre(x); post and pre each nothing, an RMS norm or a layer norm
-//                     (weight, perhaps a bias); delta is a row of fp32 or the weighed rows of a mixture of experts plus its gated
-//                     shared expert; vec is one row for all
+//   stream_norm       x += mult * post(delta + bias) + vec; out = pre(x); post and pre each nothing, an RMS norm (over the row, or over
+//                     each of several equal parts of it) or a layer norm (weight, perhaps a bias); delta is a row of fp32, or the sum of
+//                     two such rows, each behind an RMS norm and a bias of its own, or the weighed rows of a mixture of experts (some of
+//                     which may be the block's input itself) plus its shared expert, gated or not; vec is one row for all
 //   gated_part_norm   a = y * silu(z); every one of `parts` runs of columns by its own root mean square, times w
 //   clamped_glu       g = min(s gate, limit), u = clamp(s up, -limit, limit); out = r * g * sigmoid(alpha g) * (u + shift); s or r: a
 //                     factor per row (the weight of a routed expert on its input or on its output; the products with the weights
 //                     are linear), else one
+//   act_rows          out = r * act(x); act: square of relu, or gelu (erf form); r: a factor per row, else one
 //   token_gate        out = gelu_tanh(gate) * table[ids[r]][columns of one layer]
 //   softcap           x = cap * tanh(x / cap)
 // Rows may carry zero columns behind their `n` true ones (the padding of the tensor-core GEMM): means divide by the true
@@ -67,12 +70,13 @@ resid_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, const 
   }
 }
 
-// o [rows, groups * gp] fp32, gate [rows, gate_stride] (TG), w [gp] shared by the groups.  A group is handled by `team` threads
+// o [rows, groups * gp] fp32, gate [rows, gate_stride] (TG), w [gp] shared by the groups, or one row per group w_stride apart; den [rows,
+// groups] or null.  A group is handled by `team` threads
 // (a warp, or the whole CTA for wide groups).
 template <typename T, typename TG>
 __global__ void __launch_bounds__(kStreamThreads)
-gated_group_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int64_t gate_stride, const float* __restrict__ w,
-                        T* __restrict__ out, int64_t out_stride, int rows, int groups, int gp, int n, float eps, float scale, int silu, int team) {
+gated_group_norm_kernel(const float* __restrict__ o, const float* __restrict__ den, const TG* __restrict__ gate, int64_t gate_stride,
+                        const float* __restrict__ w, int w_stride, T* __restrict__ out, int64_t out_stride, int rows, int groups, int gp, int n, float eps, float scale, int silu, int team) {
   __shared__ float scratch[kStreamThreads / 32];
   pdl_wait();
   const size_t unit = (static_cast<size_t>(blockIdx.x) * kStreamThreads + threadIdx.x) / team;
@@ -90,7 +94,9 @@ gated_group_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate
   }
   ss = team == 32 ? warp_sum_f32(ss) : block_sum_f32(ss, scratch);
   if (!live) return;
-  const float r = scale / sqrtf(ss / static_cast<float>(n) + eps);
+  const float inv = den != nullptr ? 1.f / den[row * groups + g] : 1.f;
+  const float r = scale * inv / sqrtf(ss * inv * inv / static_cast<float>(n) + eps);
+  w += static_cast<size_t>(g) * w_stride;
   for (int i = me * 4; i < gp; i += team * 4) {
     const float4 v = ld_elem4(op + i), a = ld_elem4(gt + i), ww = ld_elem4(w + i);
     auto act = [silu](float z) { return silu ? silu_f32(z) : sigmoid_f32(z); };
@@ -116,10 +122,11 @@ geglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter) {
                                               gelu_tanh_f32(g.z) * u.z, gelu_tanh_f32(g.w) * u.w));
 }
 
-enum NormKind { kNormNone = 0, kNormRms = 1, kNormLayer = 2 };
+enum NormKind { kNormNone = 0, kNormRms = 1, kNormLayer = 2, kNormParts = 3 };
 
 // The rows of a mixture of experts that make up a delta: sum over j of y[pair_row[r * top + j]] (fp32, ascending j) and, with a
-// shared expert, sigmoid(gate[r]) * shared[r].
+// shared expert, sigmoid(gate[r]) * shared[r] (no gate: shared[r]).  A negative pair_row is the block's input `self` itself, times
+// its weight wts[r * top + j].
 template <typename T>
 struct MoeRows {
   const T* y;
@@ -127,7 +134,15 @@ struct MoeRows {
   const T* shared;
   const float* gate;
   int64_t gate_stride;
+  const T* self;
+  const float* wts;
   int top;
+};
+
+// A delta that is the sum of two rows: half (rms(delta + bias) * w + rms(second + second_b) * second_w) with half = factor.
+struct SecondRow {
+  const float *row, *bias, *w, *first_w;
+  float factor;
 };
 
 struct RowNorm {
@@ -183,6 +198,48 @@ __device__ __forceinline__ void norm_row(float4 (&v)[NV], const RowNorm& norm, i
   add_row<NT, NV>(v, norm.b, cols);
 }
 
+// RMS norm of `parts` equal runs of a row's n true columns.  smem: cols + parts floats, shared by the calls of a kernel.
+template <int NT, int NV>
+__device__ __forceinline__ void norm_parts(float4 (&v)[NV], const RowNorm& norm, int cols, int n, int parts, float eps, float* smem) {
+  const int len = n / parts, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool quad = len % 4 == 0;                          // four columns always belong to one part
+  float* rs = smem + cols;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + NT * j) * 4;
+    if (i >= cols) continue;
+    const float4 q = make_float4(v[j].x * v[j].x, v[j].y * v[j].y, v[j].z * v[j].z, v[j].w * v[j].w);
+    if (quad) smem[i >> 2] = (q.x + q.y) + (q.z + q.w);
+    else *reinterpret_cast<float4*>(smem + i) = q;
+  }
+  __syncthreads();
+  const int entries = quad ? len >> 2 : len;
+  for (int g = warp; g < parts; g += NT / 32) {
+    float ss = 0.f;
+    for (int k = lane; k < entries; k += 32) ss += smem[g * entries + k];
+    ss = warp_sum_f32(ss);
+    if (lane == 0) rs[g] = 1.f / sqrtf(ss / static_cast<float>(len) + eps);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + NT * j) * 4;
+    if (i >= cols) continue;
+    const float4 w = ld_elem4(norm.w + i);
+    const int g = min(i / len, parts - 1);
+    if (quad) {
+      const float r = rs[g];
+      v[j].x *= r * w.x; v[j].y *= r * w.y; v[j].z *= r * w.z; v[j].w *= r * w.w;
+    } else {                                               // (weights of padded columns are zero)
+      v[j].x *= rs[g] * w.x;
+      v[j].y *= rs[min((i + 1) / len, parts - 1)] * w.y;
+      v[j].z *= rs[min((i + 2) / len, parts - 1)] * w.z;
+      v[j].w *= rs[min((i + 3) / len, parts - 1)] * w.w;
+    }
+  }
+  add_row<NT, NV>(v, norm.b, cols);
+}
+
 struct StreamNorm {
   float* x;                  // [rows, cols]
   const float* delta;        // [rows, cols] or null
@@ -191,12 +248,14 @@ struct StreamNorm {
   float mult, eps;
   RowNorm post, pre;
   int64_t out_stride;
-  int cols, n;
+  int cols, n, parts;        // parts: of the norms over parts
 };
 
-template <typename T, int NT, int NV>
+// PARTS: post and pre are norms over parts.  PAIR: the delta is the sum of two rows.
+template <typename T, int NT, int NV, bool PARTS, bool PAIR>
 __global__ void __launch_bounds__(NT)
-stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
+stream_norm_kernel(StreamNorm p, MoeRows<T> moe, SecondRow pair, T* __restrict__ out) {
+  extern __shared__ __align__(16) float sn_smem[];         // PARTS: [cols + parts]
   __shared__ float scratch[NT / 32];
   pdl_wait();
   float* __restrict__ x = p.x;
@@ -206,7 +265,11 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
   float4 v[NV];
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   const bool add = delta != nullptr || moe.y != nullptr;
-  const float sg = moe.shared != nullptr ? sigmoid_f32(moe.gate[row * moe.gate_stride]) : 0.f;
+  const float sg = moe.gate != nullptr ? sigmoid_f32(moe.gate[row * moe.gate_stride]) : 1.f;
+  auto norm = [&](float4 (&u)[NV], const RowNorm& w) {
+    if (PARTS) norm_parts<NT, NV>(u, w, cols, n, p.parts, p.eps, sn_smem);
+    else norm_row<NT, NV>(u, w, cols, n, p.eps, scratch);
+  };
   if (add) {
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
@@ -215,7 +278,15 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
       if (i >= cols) continue;
       if (delta != nullptr) { v[j] = ld_elem4(delta + base + i); continue; }
       for (int k = 0; k < moe.top; ++k) {
-        const float4 a = ld_elem4(moe.y + static_cast<size_t>(moe.pair_row[row * moe.top + k]) * cols + i);
+        const int pr = moe.pair_row[row * moe.top + k];
+        if (pr < 0) {                                      // the input itself
+          if (moe.self == nullptr) continue;
+          const float4 a = ld_elem4(moe.self + base + i);
+          const float f = moe.wts[row * moe.top + k];
+          v[j].x = fmaf(f, a.x, v[j].x); v[j].y = fmaf(f, a.y, v[j].y); v[j].z = fmaf(f, a.z, v[j].z); v[j].w = fmaf(f, a.w, v[j].w);
+          continue;
+        }
+        const float4 a = ld_elem4(moe.y + static_cast<size_t>(pr) * cols + i);
         v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
       }
       if (moe.shared != nullptr) {
@@ -224,7 +295,23 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
       }
     }
     add_row<NT, NV>(v, p.delta_b, cols);
-    norm_row<NT, NV>(v, p.post, cols, n, p.eps, scratch);
+    if (PAIR) {
+      float4 u[NV];
+#pragma unroll
+      for (int j = 0; j < NV; ++j) {
+        const int i = (threadIdx.x + NT * j) * 4;
+        u[j] = i < cols ? ld_elem4(pair.row + base + i) : zero;
+      }
+      add_row<NT, NV>(u, pair.bias, cols);
+      norm_row<NT, NV>(v, {kNormRms, pair.first_w, nullptr}, cols, n, p.eps, scratch);
+      norm_row<NT, NV>(u, {kNormRms, pair.w, nullptr}, cols, n, p.eps, scratch);
+#pragma unroll
+      for (int j = 0; j < NV; ++j) {
+        v[j].x = pair.factor * (v[j].x + u[j].x); v[j].y = pair.factor * (v[j].y + u[j].y);
+        v[j].z = pair.factor * (v[j].z + u[j].z); v[j].w = pair.factor * (v[j].w + u[j].w);
+      }
+    }
+    norm(v, p.post);
   }
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
@@ -242,7 +329,7 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
       if (i < cols) st_elem4(x + base + i, v[j]);
     }
   }
-  norm_row<NT, NV>(v, p.pre, cols, n, p.eps, scratch);
+  norm(v, p.pre);
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     const int i = (threadIdx.x + NT * j) * 4;
@@ -250,10 +337,16 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, T* __restrict__ out) {
   }
 }
 
-template <typename T>
-static int launch_stream_norm(const StreamNorm& p, const MoeRows<T>& moe, T* out, int rows, cudaStream_t st) {
+template <typename T, bool PARTS, bool PAIR>
+static int launch_stream_norm(const StreamNorm& p, const MoeRows<T>& moe, const SecondRow& pair, T* out, int rows, cudaStream_t st) {
   const int cols = p.cols;
-#define DGPP_SN(NT, NV) stream_norm_kernel<T, NT, NV><<<rows, NT, 0, st>>>(p, moe, out)
+  const size_t smem = PARTS ? static_cast<size_t>(cols + p.parts) * sizeof(float) : 0;
+#define DGPP_SN(NT, NV)                                                                                                              \
+  do {                                                                                                                               \
+    if (smem > 48 * 1024)                                                                                                            \
+      DGPP_CUDA_OK(cudaFuncSetAttribute(stream_norm_kernel<T, NT, NV, PARTS, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)); \
+    stream_norm_kernel<T, NT, NV, PARTS, PAIR><<<rows, NT, smem, st>>>(p, moe, pair, out);                                           \
+  } while (0)
   if (cols <= 1024) DGPP_SN(256, 1);
   else if (cols <= 2048) DGPP_SN(256, 2);
   else if (cols <= 4096) DGPP_SN(256, 4);
@@ -262,6 +355,13 @@ static int launch_stream_norm(const StreamNorm& p, const MoeRows<T>& moe, T* out
 #undef DGPP_SN
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;
+}
+
+template <typename T>
+static int launch_stream_norm_kind(const StreamNorm& p, const MoeRows<T>& moe, const SecondRow& pair, T* out, int rows, cudaStream_t st) {
+  const bool two = pair.row != nullptr;
+  if (p.parts > 0) return two ? launch_stream_norm<T, true, true>(p, moe, pair, out, rows, st) : launch_stream_norm<T, true, false>(p, moe, pair, out, rows, st);
+  return two ? launch_stream_norm<T, false, true>(p, moe, pair, out, rows, st) : launch_stream_norm<T, false, false>(p, moe, pair, out, rows, st);
 }
 
 // grid (parts, rows); y [rows, parts * gp] fp32.  The last part's CTA also clears the columns up to `pad`.
@@ -331,6 +431,29 @@ clamped_glu_kernel(const TI* __restrict__ gate_up, int64_t stride, const float* 
   st_elem8(out + row * inter + i, g);
 }
 
+enum RowAct { kRelu2 = 0, kGeluErf = 1 };
+
+// x [rows, stride] (TI) -> out [rows, inter]; tiles: rows come in tiles of `bn`, and those whose entry is negative are skipped.
+template <typename TI, typename T, int ACT>
+__global__ void __launch_bounds__(kStreamThreads)
+act_rows_kernel(const TI* __restrict__ x, int64_t stride, const float* __restrict__ row_w, const int32_t* __restrict__ tiles, int bn,
+                T* __restrict__ out, int inter) {
+  pdl_wait();
+  const size_t row = blockIdx.y;
+  if (tiles != nullptr && tiles[row / bn] < 0) return;
+  const int i = (blockIdx.x * kStreamThreads + threadIdx.x) * 8;
+  if (i >= inter) return;
+  const float r = row_w != nullptr ? row_w[row] : 1.f;
+  float v[8];
+  ld_elem8(x + row * stride + i, v);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    const float z = ACT == kRelu2 ? fmaxf(v[e], 0.f) : v[e];
+    v[e] = r * (ACT == kRelu2 ? z * z : 0.5f * z * (1.f + erff(z * 0.70710678118654752f)));
+  }
+  st_elem8(out + row * inter + i, v);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kStreamThreads)
 token_gate_kernel(const float* __restrict__ gate, const int32_t* __restrict__ ids, const T* __restrict__ table, int64_t table_stride, int col,
@@ -380,16 +503,17 @@ DGPP_API int dgpp_resid_norm(void* x, const void* delta, const void* w, void* ou
   return 0;
 }
 
-// gate_f32: the gate rows are fp32 although the activations are bf16.  silu: the gate passes silu, else a sigmoid.
-DGPP_API int dgpp_gated_group_norm(const void* o, const void* gate, int64_t gate_stride, const void* w, void* out, int64_t out_stride,
+// gate_f32: the gate rows are fp32 although the activations are bf16.  silu: the gate passes silu, else a sigmoid.  den: optional fp32
+// [rows, groups], divides o.  w_stride: 0, or columns between the groups' weights.
+DGPP_API int dgpp_gated_group_norm(const void* o, const void* den, const void* gate, int64_t gate_stride, const void* w, int w_stride, void* out, int64_t out_stride,
                                    int rows, int groups, int gp, int n, float eps, float scale, int silu, int f32, int gate_f32, cudaStream_t st) {
-  DGPP_REQUIRE(gp % 8 == 0 && gate_stride % 8 == 0 && out_stride % 8 == 0 && n >= 1 && n <= gp, "gated_group_norm: %d of %d columns", n, gp);
+  DGPP_REQUIRE(gp % 8 == 0 && gate_stride % 8 == 0 && out_stride % 8 == 0 && w_stride % 4 == 0 && n >= 1 && n <= gp, "gated_group_norm: %d of %d columns", n, gp);
   if (rows == 0) return 0;
   const int team = gp <= 512 ? 32 : kStreamThreads;
   const int64_t blocks = dgpp_ceil_div64(static_cast<int64_t>(rows) * groups * team, kStreamThreads);
-  const float *op = static_cast<const float*>(o), *wp = static_cast<const float*>(w);
+  const float *op = static_cast<const float*>(o), *wp = static_cast<const float*>(w), *dp = static_cast<const float*>(den);
 #define DGPP_GGN(TT, TG) gated_group_norm_kernel<TT, TG><<<static_cast<unsigned>(blocks), kStreamThreads, 0, st>>>( \
-      op, static_cast<const TG*>(gate), gate_stride, wp, static_cast<TT*>(out), out_stride, rows, groups, gp, n, eps, scale, silu, team)
+      op, dp, static_cast<const TG*>(gate), gate_stride, wp, w_stride, static_cast<TT*>(out), out_stride, rows, groups, gp, n, eps, scale, silu, team)
   if (f32) DGPP_GGN(float, float);
   else if (gate_f32) DGPP_GGN(bf16, float);
   else DGPP_GGN(bf16, bf16);
@@ -409,29 +533,37 @@ DGPP_API int dgpp_geglu(const void* gate_up, void* out, int rows, int inter, int
   return 0;
 }
 
-// post / pre: 0 nothing, 1 RMS norm, 2 layer norm, each with its weights and perhaps a bias.  The delta is `delta` (fp32 [rows, cols]),
-// or the expert rows y[pair_row[r * top + j]] plus sigmoid(gate) * shared (y, shared: activations), or absent; delta_b [cols] is added
-// to it.  vec [cols]: added to every row of x.
+// post / pre: 0 nothing, 1 RMS norm, 2 layer norm, 3 RMS norm over each of `parts` equal parts (both of them then), each with its weights
+// and perhaps a bias.  The delta is `delta` (fp32 [rows, cols]), or the expert rows y[pair_row[r * top + j]] (negative: wts[r * top + j]
+// times `self`, or nothing) plus sigmoid(gate) * shared (no gate: shared; y, shared, self: activations), or absent; delta_b [cols] is
+// added to it.  delta2: the delta is pair_factor * (rms(delta + delta_b) * pair_w1 + rms(delta2 + delta2_b) * pair_w2).  vec [cols]: added to every
+// row of x.
 DGPP_API int dgpp_stream_norm(void* x, const void* delta, const void* y, const void* pair_row, int top, const void* shared, const void* gate,
-                              int64_t gate_stride, const void* delta_b, const void* vec, float mult, int post, const void* post_w,
-                              const void* post_b, int pre, const void* pre_w, const void* pre_b, void* out, int64_t out_stride, int rows,
-                              int cols, int n, float eps, int f32, cudaStream_t st) {
+                              int64_t gate_stride, const void* self, const void* wts, const void* delta_b, const void* delta2,
+                              const void* delta2_b, const void* pair_w1, const void* pair_w2, float pair_factor, const void* vec, float mult, int post,
+                              const void* post_w, const void* post_b, int pre, const void* pre_w, const void* pre_b, int parts, void* out,
+                              int64_t out_stride, int rows, int cols, int n, float eps, int f32, cudaStream_t st) {
   DGPP_REQUIRE(cols % 8 == 0 && cols <= 16384 && n >= 1 && n <= cols, "stream_norm: %d of %d columns (at most 16384)", n, cols);
-  DGPP_REQUIRE(post >= 0 && post <= 2 && pre >= 0 && pre <= 2 && (!post || post_w) && (!pre || pre_w), "stream_norm: norms %d / %d", post, pre);
-  DGPP_REQUIRE(!(delta && y) && (!y || (pair_row && top >= 1)) && (!shared || (y && gate)), "stream_norm: one delta only");
+  DGPP_REQUIRE(post >= 0 && post <= 3 && pre >= 0 && pre <= 3 && (!post || post_w) && (!pre || pre_w), "stream_norm: norms %d / %d", post, pre);
+  DGPP_REQUIRE(!(delta && y) && (!y || (pair_row && top >= 1)) && (!shared || y) && (!gate || shared) && (!self || (y && wts)), "stream_norm: one delta only");
+  DGPP_REQUIRE(!delta2 || (delta && pair_w1 && pair_w2), "stream_norm: the second row needs a first one, and weights");
   DGPP_REQUIRE(out_stride % 8 == 0 && out_stride >= cols && (!delta_b || delta || y), "stream_norm: output rows of %lld", static_cast<long long>(out_stride));
+  const bool in_parts = post == kNormParts || pre == kNormParts;
+  DGPP_REQUIRE(!in_parts || ((post == kNormParts || !(delta || y)) && pre == kNormParts && parts >= 1 && n % parts == 0),
+               "stream_norm: norms %d / %d over %d parts of %d columns", post, pre, parts, n);
   if (rows == 0) return 0;
   auto f = [](const void* q) { return static_cast<const float*>(q); };
   const StreamNorm p = {static_cast<float*>(x), f(delta), f(delta_b), f(vec), mult, eps, {post, f(post_w), f(post_b)}, {pre, f(pre_w), f(pre_b)},
-                        out_stride, cols, n};
+                        out_stride, cols, n, in_parts ? parts : 0};
+  const SecondRow pair = {f(delta2), f(delta2_b), f(pair_w2), f(pair_w1), pair_factor};
   const int32_t* pr = static_cast<const int32_t*>(pair_row);
-  const float* gp = static_cast<const float*>(gate);
   if (f32) {
-    const MoeRows<float> m = {static_cast<const float*>(y), pr, static_cast<const float*>(shared), gp, gate_stride, top};
-    return launch_stream_norm<float>(p, m, static_cast<float*>(out), rows, st);
+    const MoeRows<float> m = {f(y), pr, f(shared), f(gate), gate_stride, f(self), f(wts), top};
+    return launch_stream_norm_kind<float>(p, m, pair, static_cast<float*>(out), rows, st);
   }
-  const MoeRows<bf16> m = {static_cast<const bf16*>(y), pr, static_cast<const bf16*>(shared), gp, gate_stride, top};
-  return launch_stream_norm<bf16>(p, m, static_cast<bf16*>(out), rows, st);
+  auto h = [](const void* q) { return static_cast<const bf16*>(q); };
+  const MoeRows<bf16> m = {h(y), pr, h(shared), f(gate), gate_stride, h(self), f(wts), top};
+  return launch_stream_norm_kind<bf16>(p, m, pair, static_cast<bf16*>(out), rows, st);
 }
 
 DGPP_API int dgpp_gated_part_norm(const void* y, const void* z, int64_t z_stride, const void* w, void* out, int64_t out_stride, int rows,
@@ -474,6 +606,30 @@ DGPP_API int dgpp_clamped_glu(const void* gate_up, int64_t stride, const void* r
   else if (in_f32) DGPP_CG(float, bf16);
   else DGPP_CG(bf16, bf16);
 #undef DGPP_CG
+  DGPP_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// act: 0 square of relu, 1 gelu (erf form).  in_f32: x is fp32 although the output is bf16.  row_w [rows] or null multiplies the result.
+DGPP_API int dgpp_act_rows(const void* x, int64_t stride, const void* row_w, const void* tiles, int bn, void* out, int rows, int inter, int act, int f32,
+                           int in_f32, cudaStream_t st) {
+  DGPP_REQUIRE(inter % 8 == 0 && stride % 8 == 0 && bn >= 1 && (act == kRelu2 || act == kGeluErf), "act_rows: width %d (a multiple of 8), activation %d", inter, act);
+  if (rows == 0) return 0;
+  DGPP_REQUIRE(rows <= 65535, "act_rows: %d rows", rows);
+  const dim3 grid(dgpp_ceil_div(inter / 8, kStreamThreads), rows);
+  const float* rw = static_cast<const float*>(row_w);
+  const int32_t* tl = static_cast<const int32_t*>(tiles);
+#define DGPP_AR(TI, TT)                                                                                                                        \
+  do {                                                                                                                                         \
+    const TI* xp = static_cast<const TI*>(x);                                                                                                  \
+    TT* op = static_cast<TT*>(out);                                                                                                            \
+    if (act == kRelu2) act_rows_kernel<TI, TT, kRelu2><<<grid, kStreamThreads, 0, st>>>(xp, stride, rw, tl, bn, op, inter);                    \
+    else act_rows_kernel<TI, TT, kGeluErf><<<grid, kStreamThreads, 0, st>>>(xp, stride, rw, tl, bn, op, inter);                                \
+  } while (0)
+  if (f32) DGPP_AR(float, float);
+  else if (in_f32) DGPP_AR(float, bf16);
+  else DGPP_AR(bf16, bf16);
+#undef DGPP_AR
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;
 }

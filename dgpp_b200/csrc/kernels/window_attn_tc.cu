@@ -14,6 +14,9 @@
 // softmax either way.
 // Warps: 0 = TMA producer (one page of keys and values per stage), 1 = MMA issuer / TMEM owner, 2..5 = softmax.
 //
+// Kept first tokens: their pages come before those of the window.  CAP: scores pass cap * tanh(s / cap).  A sink joins the sum of the weights
+// at the end; rotated values are turned back there too, columns m and m + DV / 2 of a row together.
+//
 // FLAT is the form for latent attention, whose keys and values are expanded from the cached latents before the launch: every head
 // is its own kv head; key columns 0 .. DN - 1 and the values come from the expanded rows [flat rows, hq * DN + hq * DV], the other
 // key columns (the rotated part that all heads share) from the gathered cache rows.  A run's page g starts at flat row
@@ -49,6 +52,10 @@ struct WindowTcParams {
   int64_t out_stride;
   DeviceStatus* status;
   int runs, hq, hkv, maps, D, DV, max_blocks, window, chunked, stages;   // hkv: key heads; value heads: hkv / maps
+  const float* sink;        // optional [hq]: exp(sink) joins the sum of a row's weights
+  const float2* turn;       // optional [rows, DV / 2]: cosines and sines by which a row's outputs are turned back
+  int keep_first;           // positions below are seen from everywhere
+  float softcap;            // CAP
   int DN, rot_col;          // FLAT: key columns from the expanded rows; first rotated column of a gathered cache row
   float scale, out_scale;
 };
@@ -60,9 +67,9 @@ __device__ __forceinline__ uint32_t wt_sw128(uint32_t row, uint32_t byte_in_row)
 // First position that the query at position i sees
 __device__ __forceinline__ int wt_first_key(const WindowTcParams& p, int i) { return p.chunked ? i - i % p.window : max(0, i + 1 - p.window); }
 
-// Largest masked score of 64 keys (row of this thread)
+// Largest masked score of 64 keys (row of this thread); keys below `keep` are seen although they lie before lo
 template <bool kMask>
-__device__ __forceinline__ float wt_row_max(uint32_t taddr, int t0, int lo, int hi) {
+__device__ __forceinline__ float wt_row_max(uint32_t taddr, int t0, int lo, int hi, int keep) {
   float mt = -INFINITY;
 #pragma unroll
   for (int c0 = 0; c0 < kWtKeys; c0 += 16) {
@@ -71,15 +78,18 @@ __device__ __forceinline__ float wt_row_max(uint32_t taddr, int t0, int lo, int 
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
       const int t = t0 + c0 + j;
-      mt = fmaxf(mt, (!kMask || (t <= hi && t >= lo)) ? __uint_as_float(raw[j]) : -INFINITY);
+      mt = fmaxf(mt, (!kMask || (t <= hi && (t >= lo || t < keep))) ? __uint_as_float(raw[j]) : -INFINITY);
     }
   }
   return mt;
 }
 
-// p = 2^(s * sm - m) as two bf16 terms into row r of the A operand; returns the row's sum
-template <bool kMask>
-__device__ __forceinline__ float wt_probs(uint32_t taddr, unsigned char* sP, int r, float sm, float neg_m, int t0, int lo, int hi) {
+// cap * tanh(s / cap) in binary orders: top - 2 top / (1 + 2^(s in)), in = 2 scale log2(e) / cap, top = cap log2(e)
+__device__ __forceinline__ float wt_cap(float s, float in, float top) { return top - __fdividef(2.f * top, 1.f + fast_exp2(s * in)); }
+
+// p = 2^(s * sm - m) (CAP: 2^(wt_cap(s, sm, top) - m)) as two bf16 terms into row r of the A operand; returns the row's sum
+template <bool kMask, bool CAP>
+__device__ __forceinline__ float wt_probs(uint32_t taddr, unsigned char* sP, int r, float sm, float top, float neg_m, int t0, int lo, int hi, int keep) {
   float sum = 0.f;
 #pragma unroll
   for (int c0 = 0; c0 < kWtKeys; c0 += 16) {
@@ -89,7 +99,8 @@ __device__ __forceinline__ float wt_probs(uint32_t taddr, unsigned char* sP, int
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
       const int t = t0 + c0 + j;
-      const float p = (!kMask || (t <= hi && t >= lo)) ? fast_exp2(fmaf(__uint_as_float(raw[j]), sm, neg_m)) : 0.f;
+      const float s = __uint_as_float(raw[j]);
+      const float p = (!kMask || (t <= hi && (t >= lo || t < keep))) ? fast_exp2(CAP ? wt_cap(s, sm, top) + neg_m : fmaf(s, sm, neg_m)) : 0.f;
       sum += p;
       const bf16 h = f32_to_bf16(p);
       a[j >> 3].h[j & 7] = h;
@@ -105,7 +116,7 @@ __device__ __forceinline__ float wt_probs(uint32_t taddr, unsigned char* sP, int
 }
 
 // grid (tiles of all runs, hkv)
-template <bool FLAT>
+template <bool FLAT, bool CAP>
 __global__ void __launch_bounds__(kWtThreads, 1)
 window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, WindowTcParams p) {
   extern __shared__ __align__(1024) unsigned char smem_dyn[];
@@ -157,8 +168,10 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   }
   const int first_pos = p.positions[row0], last_pos = first_pos + ntok - 1;
   const int32_t* bt = p.block_table + static_cast<size_t>(p.row_req[row0]) * p.max_blocks;
-  const int page0 = wt_first_key(p, first_pos) / kWtKeys, base = page0 * kWtKeys;
-  const int ntiles = ntok > 0 ? last_pos / kWtKeys - page0 + 1 : 0;
+  // pages in order: those of the kept first tokens, then from the first one that the window of the tile's first token reaches
+  const int page0 = wt_first_key(p, first_pos) / kWtKeys, nkeep = min((p.keep_first + kWtKeys - 1) / kWtKeys, page0);
+  const int ntiles = ntok > 0 ? last_pos / kWtKeys - page0 + 1 + nkeep : 0;
+  auto page_of = [&](int i) { return i < nkeep ? i : page0 - nkeep + i; };
   if (warp >= 2) {
     // ---- this thread's query row into the swizzled A operand
     const int r = (warp & 3) * 32 + lane, tok = r / group;
@@ -185,12 +198,12 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         if (!wait_bar(&kv_empty[s], ((i / p.stages) & 1) ^ 1)) { report(p.status, kTimeoutStageEmpty, 71); *abort_flag = 1; break; }
         mbar_expect_tx(&kv_full[s], (natom + vatom) * kblk);
         if (FLAT) {                              // tmK: expanded rows, tmV: gathered cache rows
-          const int y = flat0 + (page0 + i) * kWtKeys, nn = p.DN / 64;
+          const int y = flat0 + page_of(i) * kWtKeys, nn = p.DN / 64;
           for (int a = 0; a < nn; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmK, kvh * p.DN + a * 64, y, &kv_full[s]);
           for (int a = nn; a < natom; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmV, p.rot_col + (a - nn) * 64, y, &kv_full[s]);
           for (int a = 0; a < vatom; ++a) tma_load_2d(sV + (s * vatom + a) * kblk, &tmK, p.hq * p.DN + kvh * p.DV + a * 64, y, &kv_full[s]);
         } else {
-          const int y = (bt[page0 + i] * p.hkv + kvh) * kWtKeys, yv = (bt[page0 + i] * (p.hkv / p.maps) + kvh / p.maps) * kWtKeys;
+          const int pg = bt[page_of(i)], y = (pg * p.hkv + kvh) * kWtKeys, yv = (pg * (p.hkv / p.maps) + kvh / p.maps) * kWtKeys;
           for (int a = 0; a < natom; ++a) tma_load_2d(sK + (s * natom + a) * kblk, &tmK, a * 64, y, &kv_full[s]);
           for (int a = 0; a < vatom; ++a) tma_load_2d(sV + (s * vatom + a) * kblk, &tmV, a * 64, yv, &kv_full[s]);
         }
@@ -250,19 +263,21 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const bool live = tok < ntok;
     const int hi = first_pos + (live ? tok : 0), lo = wt_first_key(p, hi);
-    const float sm = p.scale * 1.4426950408889634f;
+    const float log2e = 1.4426950408889634f, top = CAP ? p.softcap * log2e : 0.f;
+    const float sm = CAP ? 2.f * p.scale * log2e / p.softcap : p.scale * log2e;
+    const int keep = p.keep_first;
     float m_used = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int i = 0; i < ntiles; ++i) {
-      const int b = i & 1, t0 = base + i * kWtKeys;
+      const int b = i & 1, t0 = page_of(i) * kWtKeys;
       ok = __all_sync(0xffffffffu, wait_bar(&s_full[b], (i >> 1) & 1) && !*abort_flag) != 0;
       if (!ok) { report(p.status, kTimeoutAccum, 75); *abort_flag = 1; break; }
       tc_fence_after();
       // warp-uniform choices: the TMEM accesses are .sync.aligned
-      const bool full = __all_sync(0xffffffffu, t0 + kWtKeys - 1 <= hi && t0 >= lo) != 0;
-      const float mt = full ? wt_row_max<false>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi)
-                            : wt_row_max<true>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi);
-      const float mn = fmaxf(m_used, mt == -INFINITY ? -INFINITY : mt * sm);
+      const bool full = __all_sync(0xffffffffu, t0 + kWtKeys - 1 <= hi && (t0 >= lo || t0 + kWtKeys <= keep)) != 0;
+      const float mt = full ? wt_row_max<false>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep)
+                            : wt_row_max<true>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep);
+      const float mn = fmaxf(m_used, mt == -INFINITY ? -INFINITY : (CAP ? wt_cap(mt, sm, top) : mt * sm));
       const bool grow = mn > m_used + 8.f || (m_used == -INFINITY && mn != -INFINITY);
       if (i > 0) {
         // the previous tile's product is complete: its weights may be overwritten, O may be rescaled
@@ -285,8 +300,8 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         }
       }
       const float neg_m = m_used == -INFINITY ? 0.f : -m_used;
-      l_run += full ? wt_probs<false>(tmem_s + b * kWtKeys + lane_addr, sP, r, sm, neg_m, t0, lo, hi)
-                    : wt_probs<true>(tmem_s + b * kWtKeys + lane_addr, sP, r, sm, neg_m, t0, lo, hi);
+      l_run += full ? wt_probs<false, CAP>(tmem_s + b * kWtKeys + lane_addr, sP, r, sm, top, neg_m, t0, lo, hi, keep)
+                    : wt_probs<true, CAP>(tmem_s + b * kWtKeys + lane_addr, sP, r, sm, top, neg_m, t0, lo, hi, keep);
       fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
@@ -299,12 +314,36 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         *abort_flag = 1;
       } else {
         tc_fence_after();
+        if (p.sink != nullptr && l_run > 0.f) l_run += fast_exp2(fmaf(p.sink[kvh * group + r % group], log2e, -m_used));
         float f = l_run > 0.f ? p.out_scale / l_run : 0.f;
         if (p.gate != nullptr && live) f *= sigmoid_f32(bf16_to_f32(p.gate[static_cast<size_t>(row0 + tok) * p.stride + kvh * group + r % group]));
         float* dst32 = p.raw != nullptr ? p.raw + (static_cast<size_t>(row0 + (live ? tok : 0)) * p.hq + kvh * group + r % group) * p.DV : nullptr;
         bf16* dst = p.out + static_cast<size_t>(row0 + (live ? tok : 0)) * p.out_stride + static_cast<size_t>(kvh * group + r % group) * p.DV;
+        const int half = p.DV / 2;
+        const float2* turn = p.turn != nullptr ? p.turn + static_cast<size_t>(row0 + (live ? tok : 0)) * half : nullptr;
         for (int c0 = 0; c0 < p.DV; c0 += 16) {
           uint32_t raw[16];
+          if (turn != nullptr) {                                 // 16 columns of both halves (DV / 2 is a multiple of 32)
+            if (c0 >= half) break;
+            uint32_t other[16];
+            tmem_ld_x16(tmem_o + lane_addr + c0, raw);
+            tmem_ld_x16(tmem_o + lane_addr + half + c0, other);
+            if (live) {
+              Pack16 o[2], q[2];
+#pragma unroll
+              for (int j = 0; j < 16; ++j) {
+                const float2 cs = turn[c0 + j];
+                const float a = __uint_as_float(raw[j]) * f, b = __uint_as_float(other[j]) * f;
+                o[j >> 3].h[j & 7] = f32_to_bf16(fmaf(b, cs.y, a * cs.x));
+                q[j >> 3].h[j & 7] = f32_to_bf16(fmaf(-a, cs.y, b * cs.x));
+              }
+              *reinterpret_cast<uint4*>(dst + c0) = o[0].u;
+              *reinterpret_cast<uint4*>(dst + c0 + 8) = o[1].u;
+              *reinterpret_cast<uint4*>(dst + half + c0) = q[0].u;
+              *reinterpret_cast<uint4*>(dst + half + c0 + 8) = q[1].u;
+            }
+            continue;
+          }
           tmem_ld_x16(tmem_o + lane_addr + c0, raw);
           if (live && dst32 != nullptr) {
 #pragma unroll
@@ -342,7 +381,7 @@ static int wt_check(const void* proj, int64_t stride, int q_off, const void* out
   return 0;
 }
 
-template <bool FLAT>
+template <bool FLAT, bool CAP>
 static int launch_wt(const CUtensorMap& tK, const CUtensorMap& tV, WindowTcParams& p, int tiles, cudaStream_t st) {
   const size_t fixed = 1024 + static_cast<size_t>(p.D / 64 + 2) * kWtRows * 128 + 192, stage = static_cast<size_t>(p.D + p.DV) * 128;
   const size_t limit = 227 * 1024;
@@ -351,10 +390,10 @@ static int launch_wt(const CUtensorMap& tK, const CUtensorMap& tV, WindowTcParam
   DGPP_REQUIRE(p.stages >= 2, "window_attn_tc: head widths %d / %d do not fit shared memory", p.D, p.DV);
   static bool attr = false;
   if (!attr) {
-    DGPP_CUDA_OK(cudaFuncSetAttribute(window_attn_tc_kernel<FLAT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(limit)));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(window_attn_tc_kernel<FLAT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(limit)));
     attr = true;
   }
-  window_attn_tc_kernel<FLAT><<<dim3(tiles, p.hkv), kWtThreads, fixed + p.stages * stage, st>>>(tK, tV, p);
+  window_attn_tc_kernel<FLAT, CAP><<<dim3(tiles, p.hkv), kWtThreads, fixed + p.stages * stage, st>>>(tK, tV, p);
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -362,13 +401,16 @@ static int launch_wt(const CUtensorMap& tK, const CUtensorMap& tV, WindowTcParam
 // Runs of consecutive rows (run_start [runs + 1], or run_start / run_len [runs]); `tiles` = sum over the runs of ceil(length / (128 /
 // group)), group = hq / (hkv * maps).  The cache (pages of 64 tokens) holds the runs' own positions already.  chunked: `window` is the
 // size of the chunks.  gate_off >= 0: the sigmoid of that column of a row, one per head, multiplies the head's output.  raw: fp32
-// outputs [rows, hq, DV] instead of `out`.
+// outputs [rows, hq, DV] instead of `out`.  sink [hq], turn [rows, DV / 2] pairs (see qk_norm_append): optional; keep_first: that many first
+// positions are seen from everywhere; softcap 0: none.
 DGPP_API int dgpp_window_attn_tc(const void* proj, int64_t stride, int q_off, const void* k_cache, const void* v_cache,
                                  const void* block_table, const void* row_req, const void* positions, const void* run_start, const void* run_len,
                                  void* out, int64_t out_stride, void* raw, int runs, int tiles, int hq, int hkv, int maps, int D, int DV, int page,
                                  int max_blocks, int num_blocks, int window, int chunked, int gate_off, float scale, float out_scale,
-                                 cudaStream_t st) {
-  DGPP_REQUIRE(maps == 1 || (maps == 2 && raw), "window_attn_tc: %d maps", maps);
+                                 const void* sink, const void* turn, int keep_first, float softcap, cudaStream_t st) {
+  DGPP_REQUIRE(maps == 1 || (maps == 2 && raw && !sink), "window_attn_tc: %d maps", maps);
+  DGPP_REQUIRE(!turn || !raw, "window_attn_tc: fp32 outputs are not turned back");
+  DGPP_REQUIRE(keep_first >= 0 && (!chunked || keep_first == 0) && softcap >= 0.f, "window_attn_tc: %d kept tokens, cap %f", keep_first, static_cast<double>(softcap));
   if (wt_check(proj, stride, q_off, out, out_stride, runs, hq, hkv * maps, D, DV, page, window)) return -1;
   if (tiles == 0) return 0;
   WindowTcParams p;
@@ -385,13 +427,14 @@ DGPP_API int dgpp_window_attn_tc(const void* proj, int64_t stride, int q_off, co
   p.status = device_status_ptr();
   p.runs = runs; p.hq = hq; p.hkv = hkv * maps; p.maps = maps; p.chunked = chunked; p.D = D; p.DV = DV; p.max_blocks = max_blocks; p.window = window;
   p.scale = scale; p.out_scale = out_scale;
+  p.sink = static_cast<const float*>(sink); p.turn = static_cast<const float2*>(turn); p.keep_first = keep_first; p.softcap = softcap;
   const uint64_t rows = static_cast<uint64_t>(num_blocks) * hkv * page;
   CUtensorMap tK, tV;
   if (make_tmap_2d(&tK, k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, rows * maps, static_cast<uint64_t>(D) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
   if (make_tmap_2d(&tV, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, DV, rows, static_cast<uint64_t>(DV) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
-  return launch_wt<false>(tK, tV, p, tiles, st);
+  return p.softcap > 0.f ? launch_wt<false, true>(tK, tV, p, tiles, st) : launch_wt<false, false>(tK, tV, p, tiles, st);
 }
 
 // The same over keys and values expanded from a latent cache: `flat` [flat_rows, heads * (dn + dv)] bf16, `lat` [flat_rows, lat_cols]
@@ -425,5 +468,5 @@ DGPP_API int dgpp_latent_prefill_tc(const void* proj, int64_t stride, int q_off,
   CUtensorMap tK, tV;
   if (make_tmap_2d(&tK, flat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cols, flat_rows, cols * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
   if (make_tmap_2d(&tV, lat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, lat_cols, flat_rows, static_cast<uint64_t>(lat_cols) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
-  return launch_wt<true>(tK, tV, p, tiles, st);
+  return launch_wt<true, false>(tK, tV, p, tiles, st);
 }

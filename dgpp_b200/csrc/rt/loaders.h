@@ -288,7 +288,7 @@ inline std::string resolve_model(const std::string& spec, const std::string& cac
 }
 
 // ------------------------------------------------------------------------------------------- architecture detect
-enum class Family { Unknown, QwenHybrid, QwenFlashNext, Glm4, GlmFlash, GlmDsa, DeepSeekV4, DeepSeekV41, MiMo, MiniMax, Flint, Dory, Sitirax, Potivik, Vevapel, DenseGqa };
+enum class Family { Unknown, QwenHybrid, QwenFlashNext, Glm4, GlmFlash, GlmDsa, DeepSeekV4, DeepSeekV41, MiMo, MiniMax, Flint, Dory, Sitirax, Potivik, Vevapel, Tefudra, DenseGqa };
 
 inline const char* family_name(Family f) {
   switch (f) {
@@ -306,6 +306,7 @@ inline const char* family_name(Family f) {
     case Family::Sitirax: return "sitirax";
     case Family::Potivik: return "potivik";
     case Family::Vevapel: return "vevapel";
+    case Family::Tefudra: return "tefudra";
     case Family::DenseGqa: return "dense_gqa";
     default: return "unknown";
   }
@@ -339,6 +340,7 @@ inline Family detect_family(const json::Value& config) {
   if (has("sitirax")) return Family::Sitirax;
   if (has("potivik")) return Family::Potivik;
   if (has("vevapel")) return Family::Vevapel;
+  if (has("tefudra")) return Family::Tefudra;
   if (has("qwen3") || has("qwen2") || has("llama") || has("mistral")) return Family::DenseGqa;
   throw std::runtime_error("detect_family: unsupported architecture '" + arch + "' / model_type '" + type + "'");
 }

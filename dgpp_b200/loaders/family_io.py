@@ -3,8 +3,8 @@ under its path in the model object (`layers.3.qkv.payload`, `layers.3.moe.expert
 `config.json` that names the family (`model_type` = "dgpp-<family>") and carries the configuration and the format of
 every quantised matrix.  `save_family` writes one; `load_family` rebuilds the model on a device.  Quantised payloads
 and scales travel byte for byte.  The fixture writer of the per-family load / bind / forward checks, and the hand-off
-format between a conversion script and the server for these families.  The Sitirax, Potivik and Vevapel families have published layouts
-of their own (`"architecture": "Sitirax"` in config.json, bf16 tensors named layer by layer); they are read and written as
+format between a conversion script and the server for these families.  The Sitirax, Potivik, Vevapel and Tefudra families have
+published layouts of their own (`"architecture": "Sitirax"` in config.json, bf16 tensors named layer by layer); they are read and written as
 published, and run in bf16 or in true fp32.
 (reference counterparts: src/models/*/loader.cpp + binding.cpp per family, tools' fixture writers; there every family
  binds its publisher's tensor names, which this build does for the dense family only.)
@@ -84,6 +84,9 @@ def published(family: str):
     if family == "vevapel":
         from ..models import vevapel as m
         return m.VevapelConfig, m.VevapelModel, m.VevapelRunner, m.tensor_shapes, m.random_tensors
+    if family == "tefudra":
+        from ..models import tefudra as m
+        return m.TefudraConfig, m.TefudraModel, m.TefudraRunner, m.tensor_shapes, m.random_tensors
     return None
 
 
@@ -254,13 +257,21 @@ def _tiny_vevapel(vocab: int):
                                embed_scale=4.0, residual=0.8)
 
 
+def _tiny_tefudra(vocab: int):
+    from ..models.tefudra import DenseSpec, ExpertsSpec, MatrixSpec, ParallelSpec, TefudraConfig, WindowSpec
+
+    mixers = (WindowSpec(8, 2, 64, 64, 0.125, 256, 1e5, 32, 4),
+              ParallelSpec(WindowSpec(8, 2, 64, 128, 0.125, 128, 1e5, 64, softcap=30.0, taps=4), MatrixSpec(4, 64, 128, 12.0)))
+    return TefudraConfig.cycle(4, 512, vocab, mixers, (DenseSpec(1024), ExpertsSpec(14, 2, 2, 256, 384)), 2, shared=((2, 0),))
+
+
 def tiny_model(family: str, device="cpu", seed: int = 0, vocab: int = 4096) -> Any:
     """A small random-init model of `family` (the shapes the server's `--model <family>-tiny` choices use)."""
     from ..models.moe import MoEConfig
 
     if family in PUBLISHED:
         _, model, _, _, random_tensors = published(family)
-        cfg = {"sitirax": _tiny_sitirax, "potivik": _tiny_potivik, "vevapel": _tiny_vevapel}[family](vocab)
+        cfg = {"sitirax": _tiny_sitirax, "potivik": _tiny_potivik, "vevapel": _tiny_vevapel, "tefudra": _tiny_tefudra}[family](vocab)
         return model.from_tensors(cfg, random_tensors(cfg, seed).__getitem__, device)
     cfg_cls, model_cls = _registry()[family]
     moe = MoEConfig(hidden=512, experts=16, top_k=2, moe_ffn=512, shared_ffn=512)

@@ -34,11 +34,11 @@ from ..ops import mixers as mx
 from ..quant.formats import QuantLinear
 from .packing import only_keys, pad_cols, pad_rows, pad_vec, up8
 from .row_moe import RowExperts, RowExpertsScratch, run_experts
-from .rows import RowRunner, RowRuns
+from .rows import RowRuns
+from .window_rows import WindowRowRunner
 
 BF = torch.bfloat16
 UNIT_EPS = 1e-6                 # inside the root of the delta rule's unit vectors
-SINGLE_RUN = 8                  # runs of a mixed pass up to this length attend row by row, longer ones on the prompt kernel
 
 
 # ---------------------------------------------------------------------------------------------- configuration
@@ -501,7 +501,7 @@ class VevapelModel:
 
 
 # ---------------------------------------------------------------------------------------------- kernel runner
-class VevapelRunner(RowRunner):
+class VevapelRunner(WindowRowRunner):
     """Executes the model on the sm_100a kernels.  A request holds pages of the shared key / value pool (one table for every run of an
     attention layer, each with planes of its own) and one slot of the fp32 state of every run of a delta layer; both are reused without
     clearing (a request's first token starts from zero states)."""
@@ -531,13 +531,7 @@ class VevapelRunner(RowRunner):
         self.o = e(R * big(s.hv * s.DV for s in states), torch.float32)
         self.prep = e(big(s.prep_floats(R, slots) for s in states), torch.float32)
         self.moe = RowExpertsScratch([P.moe for P in model.layers if P.moe is not None], R, T, device)
-        # attention: partial results of single rows; a differential layer's outputs of all rows
-        self.tc_prefill = True
-        self.max_span = self.kv.max_blocks * c.page
-        self.max_splits = 32
-        self.parts = slots * self.max_splits
-        cap = lambda g: max(self.parts, R) if g.maps == 2 else self.parts
-        self.scratch = (e(big(cap(g) * g.hq * 2 for g in heads), torch.float32), e(big(cap(g) * g.hq * g.DV for g in heads), torch.float32))
+        self._init_attention(heads, R, slots, c.page, T, device)
         self.capture: Optional[list] = None        # a list: receives the residual stream after every layer run (tests, debugging)
 
     def _state_tensors(self):
@@ -548,42 +542,9 @@ class VevapelRunner(RowRunner):
             return ops.gemm_tc(x, w, out32=out)
         return ops.linear(x, w, out=out)
 
-    def _plan(self, runs: RowRuns):
-        """(single rows, (first rows, lengths, lengths on the host) of the longer runs, rows of the longer runs) on the device; None for
-        an empty part, and for a list that would name every row."""
-        short, long, start = runs.split(SINGLE_RUN)
-        lens = [runs.lens[r] for r in long]
-        if not short:
-            return None, (runs.start, None, lens), None
-        rows = [start[r] + k for r in long for k in range(runs.lens[r])]
-        dev = torch.tensor(short + [start[r] for r in long] + lens + rows, dtype=torch.int32).to(self.dev)
-        n, k = len(short), len(long)
-        return dev[:n], ((dev[n:n + k], dev[n + k:n + 2 * k], lens) if long else None), dev[n + 2 * k:]
-
-    def _attend_rows(self, P: Packed, proj, mixed, positions, row_req, cache, splits: int, fused: bool, row_list=None) -> None:
-        g = P.heads
-        mx.window_attn(g, proj, P.q_norm, P.k_norm, cache, self.kv.block_table, row_req, positions, mixed, fused=fused, splits=splits,
-                       scratch=self.scratch, row_list=row_list)
-        if g.maps == 2:
-            mx.diff_combine(g, self.scratch, proj, P.gate_off, mixed, P.lam, P.factor, splits, row_list)
-
     def _attention(self, r: int, P: Packed, proj, mixed, positions, row_req, runs: Optional[RowRuns], plan) -> None:
-        g, cache, bt, rows = P.heads, self.kv.layers[self.kv_index[r]], self.kv.block_table, proj.shape[0]
-        if runs is None:
-            return self._attend_rows(P, proj, mixed, positions, row_req, cache, g.splits(rows, self.max_span, self.max_splits), True)
-        mx.qk_norm_append(g, proj, P.q_norm, P.k_norm, cache, bt, row_req, positions)
-        if not (self.tc_prefill and mx.window_prefill_usable(g, proj, cache.page)):
-            return self._attend_rows(P, proj, mixed, positions, row_req, cache, 1, False)
-        short, long, long_rows = plan
-        if long is not None:
-            raw = self.scratch[1] if g.maps == 2 else None
-            mx.window_prefill(g, proj, cache, bt, row_req, positions, runs, mixed, raw=raw, some=long)
-            if raw is not None:
-                mx.diff_combine(g, raw, proj, P.gate_off, mixed, P.lam, P.factor, row_list=long_rows, finished=True)
-        if short is not None:
-            n = short.numel()
-            splits = min(g.splits(n, self.max_span, self.max_splits), max(1, self.parts // n))
-            self._attend_rows(P, proj, mixed, positions, row_req, cache, splits, False, short)
+        diff = (proj, P.gate_off, P.lam, P.factor) if P.heads.maps == 2 else None
+        self._attend(P.heads, (P.q_norm, P.k_norm), self.kv.layers[self.kv_index[r]], proj, mixed, positions, row_req, runs, plan, diff)
 
     def _delta(self, r: int, P: Packed, proj, mixed, positions, row_req, runs: Optional[RowRuns]) -> None:
         s, rows = P.state, proj.shape[0]

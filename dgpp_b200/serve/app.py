@@ -540,7 +540,7 @@ def main(argv=None) -> int:
     ap.add_argument("--host", default="127.0.0.1")
     ap.add_argument("--port", type=int, default=8000)
     ap.add_argument("--model", default="tiny", choices=["tiny", "fake", "hybrid-tiny", "hybrid", "glm-flash-tiny", "dory-tiny", "flash-next-tiny",
-                                                           "minimax-tiny", "mimo-tiny", "sitirax-tiny", "potivik-tiny", "vevapel-tiny"])
+                                                           "minimax-tiny", "mimo-tiny", "sitirax-tiny", "potivik-tiny", "vevapel-tiny", "tefudra-tiny"])
     ap.add_argument("--family-dir", default="",
                     help="a native family checkpoint (dgpp_b200.loaders.family_io.save_family) served through the runner adapter")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
@@ -604,7 +604,7 @@ def main(argv=None) -> int:
         tok = rt.Tokenizer.byte_level([], [("<|im_start|>", 256, True), ("<|im_end|>", 257, True)] +
                                       [(f"<{i}>", i, False) for i in range(258, hc.vocab)], rt.SplitPattern.Qwen2)
     elif args.family_dir or args.model in ("glm-flash-tiny", "dory-tiny", "flash-next-tiny", "minimax-tiny", "mimo-tiny", "sitirax-tiny",
-                                            "potivik-tiny", "vevapel-tiny"):
+                                            "potivik-tiny", "vevapel-tiny", "tefudra-tiny"):
         # the smaller families behind the generic runner adapter (a native family checkpoint, or random-init smoke
         # models; needs a GPU)
         from ..engine.adapters import RunnerEngine
@@ -615,7 +615,7 @@ def main(argv=None) -> int:
             import torch
             model = load_family(args.family_dir, "cuda", getattr(torch, args.dtype))
             runner = runner_for(model, 256, args.slots, args.max_context, "cuda", args.pool_tokens)
-        elif args.model in ("sitirax-tiny", "potivik-tiny", "vevapel-tiny"):
+        elif args.model in ("sitirax-tiny", "potivik-tiny", "vevapel-tiny", "tefudra-tiny"):
             from ..loaders.family_io import runner_for, tiny_model
             runner = runner_for(tiny_model(args.model[:-5], "cuda"), 256, args.slots, args.max_context, "cuda", args.pool_tokens)
         elif args.model == "glm-flash-tiny":
