@@ -15,6 +15,7 @@ def test_arguments_are_judged_before_anything_is_built(tmp_path):
             "from dgpp_b200.tools.trace_run import main\n"
             "sys.exit(main(sys.argv[2:]))\n")
     for cfg, dtype, code_want in (({"architecture": "Potivik"}, "float32", 7), ({"architecture": "Vevapel"}, "float32", 7),
+                                  ({"architecture": "Tefudra"}, "float32", 7),
                                   ({"architecture": "Sitirax"}, "bfloat16", 7),
                                   ({"architectures": ["Qwen3ForCausalLM"], "model_type": "qwen3"}, "float32", 3)):
         (tmp_path / "config.json").write_text(json.dumps(cfg))
