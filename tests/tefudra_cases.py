@@ -64,7 +64,8 @@ CONFIGS = {
 
 def tensors(cfg, seed=0, alike=False):
     """bf16 tensors; norms, biases, sinks and corrections away from their neutral values, gates that remember and gates that forget.  alike:
-    a layer's experts are variations of one another, so a routing decision that 16-bit rounding tips over moves the result little."""
+    a layer's experts are variations of one another, and which identity experts are chosen is beyond doubt, so a routing decision that
+    16-bit rounding tips over moves the result little."""
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, s in tensor_shapes(TefudraConfig.from_dict(cfg)).items():
@@ -84,7 +85,7 @@ def tensors(cfg, seed=0, alike=False):
         elif last == "conv":
             t = 0.7 * r
         elif name == "embed":
-            t = r
+            t = 0.1 * r
         elif last == "router":
             t = r * s[1] ** -0.5 * 2
         else:
@@ -95,6 +96,11 @@ def tensors(cfg, seed=0, alike=False):
         if rest:
             first = out[f"{layer_}.mlp.e0.{rest.partition('.')[2]}"]
             out[name] = (first.float() + 0.1 * (t.float() - first.float())).to(torch.bfloat16)
+        elif name.endswith("correction"):
+            f = cfg["layers"][int(layer_.split(".")[0][1:])]["mlp"]["router"]
+            t[f["experts"]:] = -2
+            if f["top"] > 1:
+                t[f["experts"]:f["experts"] + 1] = 2
     return out
 
 
