@@ -172,7 +172,7 @@ def main() -> int:
     ap.add_argument("--config", type=int, default=1,
                     help="1: the dense 27B-class headline (default); 2 / 3 / 4: end-to-end timings of the MLA + MoE, the "
                          "sparse-index MLA + MoE and the hybrid GDN + MoE families at their named shapes (one GPU)")
-    ap.add_argument("--family", default="", choices=["", "sitirax", "potivik", "vevapel"],
+    ap.add_argument("--family", default="", choices=["", "sitirax", "potivik", "vevapel", "tefudra"],
                     help="kernel and model throughput of one family beside its closest relatives, instead of the headline run")
     ap.add_argument("--sizes", default="2048,4096", help="--family: model widths ('' = kernels only)")
     ap.add_argument("--bf12-head", action="store_true",
