@@ -42,8 +42,8 @@ KERNEL_SETS = {
                 "state_space", "graph_exec"],
     "vevapel": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "moe", "moe_prefill", "moe_rows", "window_attn", "window_attn_tc",
                 "gated_delta", "graph_exec"],
-    "tefudra": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "moe", "moe_prefill", "moe_rows", "short_conv", "window_attn",
-                "window_attn_tc", "matrix_memory", "graph_exec"],
+    "tefudra": ["status", "misc_ops", "gemm_tc", "gemm_f32", "stream_ops", "moe", "moe_prefill", "moe_rows", "short_conv",
+                "window_attn_ext", "window_attn_tc", "matrix_memory", "graph_exec"],
 }
 # Translation units that must not contract a*b+c into fma (sampler parity with the host oracle).
 NO_FMA = {"sample.cu"}

@@ -251,7 +251,7 @@ struct StreamNorm {
   int cols, n, parts;        // parts: of the norms over parts
 };
 
-// PARTS: post and pre are norms over parts.  PAIR: the delta is the sum of two rows.
+// PARTS: post and pre are norms over parts, and expert rows may be the input itself.  PAIR: the delta is the sum of two rows.
 template <typename T, int NT, int NV, bool PARTS, bool PAIR>
 __global__ void __launch_bounds__(NT)
 stream_norm_kernel(StreamNorm p, MoeRows<T> moe, SecondRow pair, T* __restrict__ out) {
@@ -280,7 +280,7 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, SecondRow pair, T* __restrict__
       for (int k = 0; k < moe.top; ++k) {
         const int pr = moe.pair_row[row * moe.top + k];
         if (pr < 0) {                                      // the input itself
-          if (moe.self == nullptr) continue;
+          if (!PARTS || moe.self == nullptr) continue;
           const float4 a = ld_elem4(moe.self + base + i);
           const float f = moe.wts[row * moe.top + k];
           v[j].x = fmaf(f, a.x, v[j].x); v[j].y = fmaf(f, a.y, v[j].y); v[j].z = fmaf(f, a.z, v[j].z); v[j].w = fmaf(f, a.w, v[j].w);
@@ -433,6 +433,17 @@ clamped_glu_kernel(const TI* __restrict__ gate_up, int64_t stride, const float* 
 
 enum RowAct { kRelu2 = 0, kGeluErf = 1 };
 
+// erf for rows that are rounded to 16 bits (absolute error 1.5e-7): formula 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical
+// Functions.
+__device__ __forceinline__ float erf_rows(float x) {
+  const float a = fabsf(x), t = __fdividef(1.f, fmaf(0.3275911f, a, 1.f));
+  float p = fmaf(1.061405429f, t, -1.453152027f);
+  p = fmaf(p, t, 1.421413741f);
+  p = fmaf(p, t, -0.284496736f);
+  p = fmaf(p, t, 0.254829592f);
+  return copysignf(fmaf(-p * t, __expf(-a * a), 1.f), x);
+}
+
 // x [rows, stride] (TI) -> out [rows, inter]; tiles: rows come in tiles of `bn`, and those whose entry is negative are skipped.
 template <typename TI, typename T, int ACT>
 __global__ void __launch_bounds__(kStreamThreads)
@@ -449,7 +460,8 @@ act_rows_kernel(const TI* __restrict__ x, int64_t stride, const float* __restric
 #pragma unroll
   for (int e = 0; e < 8; ++e) {
     const float z = ACT == kRelu2 ? fmaxf(v[e], 0.f) : v[e];
-    v[e] = r * (ACT == kRelu2 ? z * z : 0.5f * z * (1.f + erff(z * 0.70710678118654752f)));
+    const float s = z * 0.70710678118654752f;
+    v[e] = r * (ACT == kRelu2 ? z * z : 0.5f * z * (1.f + (sizeof(T) == 4 ? erff(s) : erf_rows(s))));
   }
   st_elem8(out + row * inter + i, v);
 }
@@ -551,6 +563,7 @@ DGPP_API int dgpp_stream_norm(void* x, const void* delta, const void* y, const v
   const bool in_parts = post == kNormParts || pre == kNormParts;
   DGPP_REQUIRE(!in_parts || ((post == kNormParts || !(delta || y)) && pre == kNormParts && parts >= 1 && n % parts == 0),
                "stream_norm: norms %d / %d over %d parts of %d columns", post, pre, parts, n);
+  DGPP_REQUIRE(!self || in_parts, "stream_norm: identity experts come with norms over parts (perhaps one)");
   if (rows == 0) return 0;
   auto f = [](const void* q) { return static_cast<const float*>(q); };
   const StreamNorm p = {static_cast<float*>(x), f(delta), f(delta_b), f(vec), mult, eps, {post, f(post_w), f(post_b)}, {pre, f(pre_w), f(pre_b)},

@@ -14,8 +14,8 @@
 // softmax either way.
 // Warps: 0 = TMA producer (one page of keys and values per stage), 1 = MMA issuer / TMEM owner, 2..5 = softmax.
 //
-// Kept first tokens: their pages come before those of the window.  CAP: scores pass cap * tanh(s / cap).  A sink joins the sum of the weights
-// at the end; rotated values are turned back there too, columns m and m + DV / 2 of a row together.
+// EXT: kept first tokens, whose pages come before those of the window; a sink, which joins the sum of the weights at the end; rotated values,
+// turned back there too, columns m and m + DV / 2 of a row together.  CAP: scores pass cap * tanh(s / cap) as well.
 //
 // FLAT is the form for latent attention, whose keys and values are expanded from the cached latents before the launch: every head
 // is its own kv head; key columns 0 .. DN - 1 and the values come from the expanded rows [flat rows, hq * DN + hq * DV], the other
@@ -68,7 +68,7 @@ __device__ __forceinline__ uint32_t wt_sw128(uint32_t row, uint32_t byte_in_row)
 __device__ __forceinline__ int wt_first_key(const WindowTcParams& p, int i) { return p.chunked ? i - i % p.window : max(0, i + 1 - p.window); }
 
 // Largest masked score of 64 keys (row of this thread); keys below `keep` are seen although they lie before lo
-template <bool kMask>
+template <bool kMask, bool EXT>
 __device__ __forceinline__ float wt_row_max(uint32_t taddr, int t0, int lo, int hi, int keep) {
   float mt = -INFINITY;
 #pragma unroll
@@ -78,7 +78,7 @@ __device__ __forceinline__ float wt_row_max(uint32_t taddr, int t0, int lo, int 
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
       const int t = t0 + c0 + j;
-      mt = fmaxf(mt, (!kMask || (t <= hi && (t >= lo || t < keep))) ? __uint_as_float(raw[j]) : -INFINITY);
+      mt = fmaxf(mt, (!kMask || (t <= hi && (t >= lo || (EXT && t < keep)))) ? __uint_as_float(raw[j]) : -INFINITY);
     }
   }
   return mt;
@@ -88,7 +88,7 @@ __device__ __forceinline__ float wt_row_max(uint32_t taddr, int t0, int lo, int 
 __device__ __forceinline__ float wt_cap(float s, float in, float top) { return top - __fdividef(2.f * top, 1.f + fast_exp2(s * in)); }
 
 // p = 2^(s * sm - m) (CAP: 2^(wt_cap(s, sm, top) - m)) as two bf16 terms into row r of the A operand; returns the row's sum
-template <bool kMask, bool CAP>
+template <bool kMask, bool EXT, bool CAP>
 __device__ __forceinline__ float wt_probs(uint32_t taddr, unsigned char* sP, int r, float sm, float top, float neg_m, int t0, int lo, int hi, int keep) {
   float sum = 0.f;
 #pragma unroll
@@ -100,7 +100,7 @@ __device__ __forceinline__ float wt_probs(uint32_t taddr, unsigned char* sP, int
     for (int j = 0; j < 16; ++j) {
       const int t = t0 + c0 + j;
       const float s = __uint_as_float(raw[j]);
-      const float p = (!kMask || (t <= hi && (t >= lo || t < keep))) ? fast_exp2(CAP ? wt_cap(s, sm, top) + neg_m : fmaf(s, sm, neg_m)) : 0.f;
+      const float p = (!kMask || (t <= hi && (t >= lo || (EXT && t < keep)))) ? fast_exp2(CAP ? wt_cap(s, sm, top) + neg_m : fmaf(s, sm, neg_m)) : 0.f;
       sum += p;
       const bf16 h = f32_to_bf16(p);
       a[j >> 3].h[j & 7] = h;
@@ -116,7 +116,7 @@ __device__ __forceinline__ float wt_probs(uint32_t taddr, unsigned char* sP, int
 }
 
 // grid (tiles of all runs, hkv)
-template <bool FLAT, bool CAP>
+template <bool FLAT, bool EXT, bool CAP>
 __global__ void __launch_bounds__(kWtThreads, 1)
 window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, WindowTcParams p) {
   extern __shared__ __align__(1024) unsigned char smem_dyn[];
@@ -169,9 +169,9 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   const int first_pos = p.positions[row0], last_pos = first_pos + ntok - 1;
   const int32_t* bt = p.block_table + static_cast<size_t>(p.row_req[row0]) * p.max_blocks;
   // pages in order: those of the kept first tokens, then from the first one that the window of the tile's first token reaches
-  const int page0 = wt_first_key(p, first_pos) / kWtKeys, nkeep = min((p.keep_first + kWtKeys - 1) / kWtKeys, page0);
+  const int page0 = wt_first_key(p, first_pos) / kWtKeys, nkeep = EXT ? min((p.keep_first + kWtKeys - 1) / kWtKeys, page0) : 0;
   const int ntiles = ntok > 0 ? last_pos / kWtKeys - page0 + 1 + nkeep : 0;
-  auto page_of = [&](int i) { return i < nkeep ? i : page0 - nkeep + i; };
+  auto page_of = [&](int i) { return EXT && i < nkeep ? i : page0 - nkeep + i; };
   if (warp >= 2) {
     // ---- this thread's query row into the swizzled A operand
     const int r = (warp & 3) * 32 + lane, tok = r / group;
@@ -265,7 +265,7 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     const int hi = first_pos + (live ? tok : 0), lo = wt_first_key(p, hi);
     const float log2e = 1.4426950408889634f, top = CAP ? p.softcap * log2e : 0.f;
     const float sm = CAP ? 2.f * p.scale * log2e / p.softcap : p.scale * log2e;
-    const int keep = p.keep_first;
+    const int keep = EXT ? p.keep_first : 0;
     float m_used = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int i = 0; i < ntiles; ++i) {
@@ -274,9 +274,9 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       if (!ok) { report(p.status, kTimeoutAccum, 75); *abort_flag = 1; break; }
       tc_fence_after();
       // warp-uniform choices: the TMEM accesses are .sync.aligned
-      const bool full = __all_sync(0xffffffffu, t0 + kWtKeys - 1 <= hi && (t0 >= lo || t0 + kWtKeys <= keep)) != 0;
-      const float mt = full ? wt_row_max<false>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep)
-                            : wt_row_max<true>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep);
+      const bool full = __all_sync(0xffffffffu, t0 + kWtKeys - 1 <= hi && (t0 >= lo || (EXT && t0 + kWtKeys <= keep))) != 0;
+      const float mt = full ? wt_row_max<false, EXT>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep)
+                            : wt_row_max<true, EXT>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep);
       const float mn = fmaxf(m_used, mt == -INFINITY ? -INFINITY : (CAP ? wt_cap(mt, sm, top) : mt * sm));
       const bool grow = mn > m_used + 8.f || (m_used == -INFINITY && mn != -INFINITY);
       if (i > 0) {
@@ -300,8 +300,8 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         }
       }
       const float neg_m = m_used == -INFINITY ? 0.f : -m_used;
-      l_run += full ? wt_probs<false, CAP>(tmem_s + b * kWtKeys + lane_addr, sP, r, sm, top, neg_m, t0, lo, hi, keep)
-                    : wt_probs<true, CAP>(tmem_s + b * kWtKeys + lane_addr, sP, r, sm, top, neg_m, t0, lo, hi, keep);
+      l_run += full ? wt_probs<false, EXT, CAP>(tmem_s + b * kWtKeys + lane_addr, sP, r, sm, top, neg_m, t0, lo, hi, keep)
+                    : wt_probs<true, EXT, CAP>(tmem_s + b * kWtKeys + lane_addr, sP, r, sm, top, neg_m, t0, lo, hi, keep);
       fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
@@ -314,16 +314,16 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         *abort_flag = 1;
       } else {
         tc_fence_after();
-        if (p.sink != nullptr && l_run > 0.f) l_run += fast_exp2(fmaf(p.sink[kvh * group + r % group], log2e, -m_used));
+        if (EXT && p.sink != nullptr && l_run > 0.f) l_run += fast_exp2(fmaf(p.sink[kvh * group + r % group], log2e, -m_used));
         float f = l_run > 0.f ? p.out_scale / l_run : 0.f;
         if (p.gate != nullptr && live) f *= sigmoid_f32(bf16_to_f32(p.gate[static_cast<size_t>(row0 + tok) * p.stride + kvh * group + r % group]));
         float* dst32 = p.raw != nullptr ? p.raw + (static_cast<size_t>(row0 + (live ? tok : 0)) * p.hq + kvh * group + r % group) * p.DV : nullptr;
         bf16* dst = p.out + static_cast<size_t>(row0 + (live ? tok : 0)) * p.out_stride + static_cast<size_t>(kvh * group + r % group) * p.DV;
         const int half = p.DV / 2;
-        const float2* turn = p.turn != nullptr ? p.turn + static_cast<size_t>(row0 + (live ? tok : 0)) * half : nullptr;
+        const float2* turn = EXT && p.turn != nullptr ? p.turn + static_cast<size_t>(row0 + (live ? tok : 0)) * half : nullptr;
         for (int c0 = 0; c0 < p.DV; c0 += 16) {
           uint32_t raw[16];
-          if (turn != nullptr) {                                 // 16 columns of both halves (DV / 2 is a multiple of 32)
+          if (EXT && turn != nullptr) {                                 // 16 columns of both halves (DV / 2 is a multiple of 32)
             if (c0 >= half) break;
             uint32_t other[16];
             tmem_ld_x16(tmem_o + lane_addr + c0, raw);
@@ -381,7 +381,7 @@ static int wt_check(const void* proj, int64_t stride, int q_off, const void* out
   return 0;
 }
 
-template <bool FLAT, bool CAP>
+template <bool FLAT, bool EXT, bool CAP>
 static int launch_wt(const CUtensorMap& tK, const CUtensorMap& tV, WindowTcParams& p, int tiles, cudaStream_t st) {
   const size_t fixed = 1024 + static_cast<size_t>(p.D / 64 + 2) * kWtRows * 128 + 192, stage = static_cast<size_t>(p.D + p.DV) * 128;
   const size_t limit = 227 * 1024;
@@ -390,10 +390,10 @@ static int launch_wt(const CUtensorMap& tK, const CUtensorMap& tV, WindowTcParam
   DGPP_REQUIRE(p.stages >= 2, "window_attn_tc: head widths %d / %d do not fit shared memory", p.D, p.DV);
   static bool attr = false;
   if (!attr) {
-    DGPP_CUDA_OK(cudaFuncSetAttribute(window_attn_tc_kernel<FLAT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(limit)));
+    DGPP_CUDA_OK(cudaFuncSetAttribute(window_attn_tc_kernel<FLAT, EXT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(limit)));
     attr = true;
   }
-  window_attn_tc_kernel<FLAT, CAP><<<dim3(tiles, p.hkv), kWtThreads, fixed + p.stages * stage, st>>>(tK, tV, p);
+  window_attn_tc_kernel<FLAT, EXT, CAP><<<dim3(tiles, p.hkv), kWtThreads, fixed + p.stages * stage, st>>>(tK, tV, p);
   DGPP_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -434,7 +434,9 @@ DGPP_API int dgpp_window_attn_tc(const void* proj, int64_t stride, int q_off, co
     return -1;
   if (make_tmap_2d(&tV, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, DV, rows, static_cast<uint64_t>(DV) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
-  return p.softcap > 0.f ? launch_wt<false, true>(tK, tV, p, tiles, st) : launch_wt<false, false>(tK, tV, p, tiles, st);
+  if (p.softcap > 0.f) return launch_wt<false, true, true>(tK, tV, p, tiles, st);
+  const bool ext = p.sink != nullptr || p.turn != nullptr || p.keep_first > 0;
+  return ext ? launch_wt<false, true, false>(tK, tV, p, tiles, st) : launch_wt<false, false, false>(tK, tV, p, tiles, st);
 }
 
 // The same over keys and values expanded from a latent cache: `flat` [flat_rows, heads * (dn + dv)] bf16, `lat` [flat_rows, lat_cols]
@@ -468,5 +470,5 @@ DGPP_API int dgpp_latent_prefill_tc(const void* proj, int64_t stride, int q_off,
   CUtensorMap tK, tV;
   if (make_tmap_2d(&tK, flat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cols, flat_rows, cols * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
   if (make_tmap_2d(&tV, lat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, lat_cols, flat_rows, static_cast<uint64_t>(lat_cols) * 2, 64, kWtKeys, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
-  return launch_wt<true, false>(tK, tV, p, tiles, st);
+  return launch_wt<true, false, false>(tK, tV, p, tiles, st);
 }

@@ -588,12 +588,11 @@ class TefudraRunner(WindowRowRunner):
         x, xn, xf, dx, dx2 = (t[:rows] for t in (self.x, self.xn, self.xf, self.dx, self.dx2))
         view = lambda buf, n: buf[:rows * n].view(rows, n)
         plan = self._plan(runs) if runs is not None else None
-        kind = "rms" if c.groups == 1 else "parts"
         mx.embed_rows(tokens, m.embed, x)
         last = (None, (None, None))                                 # what the stream has still to take in: delta and its norm
 
         def take(out, w):
-            mx.stream_norm(x, c.width, c.eps, out, *last, (kind, w), parts=c.groups)
+            mx.stream_norm(x, c.width, c.eps, out, *last, ("parts", w), parts=c.groups)
 
         for i, P in enumerate(m.layers):
             take(xn, P.norm1)
@@ -606,7 +605,7 @@ class TefudraRunner(WindowRowRunner):
                 mixed2 = view(self.mixed2, P.right_out.k)
                 self._memory(i, P.memory, proj, mixed2, positions, row_req, runs)
                 delta = mx.PairDelta(delta, P.mix[0], self._lin(mixed2, P.right_out, dx2), P.mix[1], 0.5, P.out_b)
-            last = delta, (kind, P.norm1b)
+            last = delta, ("parts", P.norm1b)
             if P.norm2 is None:
                 continue
             take(xf, P.norm2)
@@ -615,7 +614,7 @@ class TefudraRunner(WindowRowRunner):
             else:
                 up = self._lin(xf, P.up, view(self.up, P.up.n))
                 delta = self._lin(mx.act_rows(up, view(self.act, P.up.n), DENSE_ACT), P.down, dx)
-            last = delta, (kind, P.norm2b)
+            last = delta, ("parts", P.norm2b)
         take(xn, m.final_norm)
         if self.capture is not None:
             self.capture.append(x[:, :c.width].clone())

@@ -1,6 +1,6 @@
 """Front ends of the kernels behind models with an fp32 residual stream, sliding-window attention (grouped heads, or a
 shared latent), fp32 linear-attention, state-space and matrix memories, and experts of plain rows (``csrc/kernels/stream_ops.cu``,
-``short_conv.cu``, ``window_attn.cu``, ``window_attn_tc.cu``, ``latent_attn.cu``, ``mla_tc.cu``, ``linear_state.cu``, ``gated_delta.cu``,
+``short_conv.cu``, ``window_attn.cuh``, ``window_attn_tc.cu``, ``latent_attn.cu``, ``mla_tc.cu``, ``linear_state.cu``, ``gated_delta.cu``,
 ``state_space.cu``, ``matrix_memory.cu``, ``moe_rows.cu``).  Every operator exists for bf16 and for true fp32 activations; the dtype of the tensors decides."""
 from __future__ import annotations
 
@@ -19,8 +19,9 @@ _lib.declare("dgpp_resid_norm", [P, P, P, P, I, I, I, F, I, P])
 _lib.declare("dgpp_gated_group_norm", [P, P, P, L, P, I, P, L, I, I, I, I, F, F, I, I, I, P])
 _lib.declare("dgpp_geglu", [P, P, I, I, I, P])
 _WINDOW = [P, L, I, I, I] + [P] * 11 + [I] * 12 + [F, F, P]
-_lib.declare("dgpp_qk_norm_append", _WINDOW + [I, P])
-_lib.declare("dgpp_window_attn", _WINDOW + [P, P, P, P, L, I, I, I, I, I, F, F, I, P])
+for _form in ("", "_ext"):
+    _lib.declare("dgpp_qk_norm_append" + _form, _WINDOW + [I, P])
+    _lib.declare("dgpp_window_attn" + _form, _WINDOW + [P, P, P, P, L, I, I, I, I, I, F, F, I, P])
 _lib.declare("dgpp_diff_combine", [P, P, P, L, P, P, L, I, I, I, I, I, I, F, F, F, I, P])
 _lib.declare("dgpp_state_space", [P, L, I, I, P, P, P, I, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, P])
 _lib.declare("dgpp_gated_delta", [P, L, I, I, I, I, P, P, I, P, P, P, P, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, F, F, I, I, P])
@@ -247,6 +248,11 @@ class WindowHeads:
     def taps(self) -> int:
         return 0 if self.conv_w is None else self.conv_w.shape[0]
 
+    @property
+    def ext(self) -> bool:
+        """Whether these heads take the kernels' form with extras."""
+        return bool(self.keep_first or self.softcap or self.sink is not None or self.conv_w is not None or self.vnorm or self.vfreq is not None)
+
     def new_ring(self, slots: int, device) -> Optional[torch.Tensor]:
         """History of the convolution [slots, taps, channels] fp32.  Needs no clearing between requests."""
         return torch.zeros(slots, self.taps, self.channels, dtype=torch.float32, device=device) if self.taps else None
@@ -282,7 +288,7 @@ def value_freqs(base: float, vdim: int, width: int, device) -> torch.Tensor:
 
 
 class _WindowExtras(ctypes.Structure):
-    """``WindowExtras`` of csrc/kernels/window_attn.cu."""
+    """``WindowExtras`` of csrc/kernels/window_attn.cuh."""
     _fields_ = [(n, ctypes.c_void_p) for n in ("vfreq", "turn", "conv_w", "ring", "sink")] + \
                [(n, ctypes.c_int) for n in ("vdim", "vnorm", "taps", "keep_first")] + [("softcap", ctypes.c_float)]
 
@@ -290,11 +296,14 @@ class _WindowExtras(ctypes.Structure):
 def _wa_common(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, positions, rows: int, ring=None, turn=None):
     coef, every = g.temp
     norm = {None: 0, "head": 1, "row": 2}[g.norm]
-    x = _WindowExtras(ptr(g.vfreq), ptr(turn), ptr(g.conv_w) if ring is not None else None, ptr(ring), ptr(g.sink), g.vdim, int(g.vnorm), g.taps,
-                      g.keep_first, float(g.softcap))
+    x = None
+    if g.ext:
+        x = _WindowExtras(ptr(g.vfreq), ptr(turn), ptr(g.conv_w) if ring is not None else None, ptr(ring), ptr(g.sink), g.vdim, int(g.vnorm), g.taps,
+                          g.keep_first, float(g.softcap))
+        x = ctypes.cast(ctypes.pointer(x), ctypes.c_void_p)
     return (ptr(proj), proj.stride(0), g.q_off, g.k_off, g.v_off, ptr(wq), ptr(wk), *(ptr(b) for b in g.bias), ptr(g.freq), ptr(cache.k), ptr(cache.v),
             ptr(block_table), ptr(row_req), ptr(positions), rows, g.hq, g.hkv, g.maps, g.D, g.DV, g.dim, cache.page, block_table.shape[1], norm,
-            g.rot, int(every), float(coef), float(g.eps), ctypes.cast(ctypes.pointer(x), ctypes.c_void_p))
+            g.rot, int(every), float(coef), float(g.eps), x)
 
 
 def qk_norm_append(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, positions, turn=None) -> None:
@@ -302,7 +311,7 @@ def qk_norm_append(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, po
     paged cache.  A convolution comes before (``short_conv``; then g is ``WindowHeads.after_conv``).  turn: fp32 [rows, DV] takes the
     angles that ``window_prefill`` needs where values are rotated."""
     assert cache.k.dtype == proj.dtype and g.conv_w is None and (turn is None or turn.numel() >= proj.shape[0] * g.DV)
-    call("dgpp_qk_norm_append", *_wa_common(g, proj, wq, wk, cache, block_table, row_req, positions, proj.shape[0], turn=turn), _f32(proj), stream_ptr())
+    call("dgpp_qk_norm_append" + ("_ext" if g.ext else ""), *_wa_common(g, proj, wq, wk, cache, block_table, row_req, positions, proj.shape[0], turn=turn), _f32(proj), stream_ptr())
 
 
 def window_attn(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, positions, out, out_scale: float = 1.0,
@@ -318,7 +327,7 @@ def window_attn(g: WindowHeads, proj, wq, wk, cache, block_table, row_req, posit
     ml, acc = scratch if splits > 1 or g.maps == 2 else (None, None)
     assert ml is None or (ml.numel() >= rows * g.hq * splits * 2 and acc.numel() >= rows * g.hq * splits * g.DV)
     out = None if g.maps == 2 else out
-    call("dgpp_window_attn", *_wa_common(g, proj, wq, wk, cache, block_table, row_req, positions, rows, ring), ptr(row_list), ptr(ml), ptr(acc),
+    call("dgpp_window_attn" + ("_ext" if g.ext else ""), *_wa_common(g, proj, wq, wk, cache, block_table, row_req, positions, rows, ring), ptr(row_list), ptr(ml), ptr(acc),
          ptr(out), 0 if out is None else out.stride(0), splits, g.window, int(g.chunked), int(fused), g.gate_off, float(g.scale), float(out_scale),
          _f32(proj), stream_ptr())
     return out
