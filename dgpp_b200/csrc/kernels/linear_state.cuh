@@ -26,8 +26,8 @@
 //   lin_block    16-token blocks in parallel: the block's decay products and token-pair matrices (ssd_block, gated_block:
 //                the same for scalar decays, which leave q and k as they are, shared by a group of heads)
 //   lin_scan     block-sequential part: one CTA per (32 state columns, head, run), S in registers, the next block's operands
-//                streaming in with cp.async while the current one is consumed.  Matrix memory: one more CTA per head carries n as the
-//                state's column for a value that is always one, and finishes the denominators
+//                streaming in with cp.async while the current one is consumed.  Matrix memory: one more warp of a head's first CTA
+//                carries n as the state's column for a value that is always one, and finishes the denominators
 //   lin_tail     the newest inputs of the convolution go to the request's ring after every reader is done
 //
 // The decode kernel takes o_t as (g S)^T q + (k . q) u, the read-out after the write, so both reductions over the key channels
@@ -599,43 +599,58 @@ __global__ void __launch_bounds__(256) matrix_prep_kernel(LinearArgs a) {
   *reinterpret_cast<float4*>(dst) = x;
 }
 
-// The running maximum of a run and head, 32 tokens at a time: (F, M) of consecutive tokens combine to (F1 + F2, max(M1 + F2, M2)), and
-// m_t = max(m + F, M).  grid (ceil(hv / 4), runs), one warp per head; the next tokens' gates are loaded while these are scanned.
+constexpr int kGateThreads = 512;
+
+// (F, M) of consecutive tokens combine to (F1 + F2, max(M1 + F2, M2)): inclusive scan over the lanes.
+__device__ __forceinline__ void gate_scan(float& F, float& M, int lane) {
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
+    if (lane >= o) {
+      M = fmaxf(Mp + F, M);
+      F += Fp;
+    }
+  }
+}
+
+// The running maximum of a run and head, 512 tokens at a time: m_t = max(m + F_t, M_t).  grid (hv, runs)
 template <typename T, int DK, int DV>
-__global__ void __launch_bounds__(128) matrix_gates_kernel(LinearArgs a) {
+__global__ void __launch_bounds__(kGateThreads) matrix_gates_kernel(LinearArgs a) {
+  constexpr int NW = kGateThreads / 32;
+  __shared__ float Fw[NW], Mw[NW], ends[NW + 1];
   pdl_wait();
-  const int h = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (h >= a.hv) return;
+  const int h = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int first = a.run_start[blockIdx.y], last = a.run_start[blockIdx.y + 1];
   const PrepView pv = prep_view<DK, DV, kMatrix>(a);
   float* ns = a.nstate + (static_cast<size_t>(a.row_slot[first]) * a.hv + h) * (DK + 4) + DK;
   float m = a.positions[first] == 0 ? 0.f : *ns;
-  const float2 none = make_float2(-INFINITY, 0.f);
-  float2 next = first + lane < last ? matrix_gates<T>(a, first + lane, h) : none;
-  for (int t0 = first; t0 < last; t0 += 32) {
-    const float2 g = next;
-    next = t0 + 32 + lane < last ? matrix_gates<T>(a, t0 + 32 + lane, h) : none;
+  for (int t0 = first; t0 < last; t0 += kGateThreads) {
+    const bool live = t0 + tid < last;
+    const float2 g = live ? matrix_gates<T>(a, t0 + tid, h) : make_float2(-INFINITY, 0.f);
     float F = g.y, M = g.x;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
-      if (lane >= o) {
-        M = fmaxf(Mp + F, M);
-        F += Fp;
-      }
+    gate_scan(F, M, lane);
+    if (lane == 31) { Fw[warp] = F; Mw[warp] = M; }
+    __syncthreads();
+    if (warp == 0) {                                       // maximum in front of every warp's tokens, and behind all
+      float Fs = lane < NW ? Fw[lane] : 0.f, Ms = lane < NW ? Mw[lane] : -INFINITY;
+      gate_scan(Fs, Ms, lane);
+      if (lane < NW) ends[lane + 1] = fmaxf(m + Fs, Ms);
+      if (lane == 0) ends[0] = m;
     }
-    const float mt = fmaxf(m + F, M);
+    __syncthreads();
+    const float mw = ends[warp], mt = fmaxf(mw + F, M);
     float before = __shfl_up_sync(0xffffffffu, mt, 1);
-    if (lane == 0) before = m;
-    if (t0 + lane < last) {
-      const size_t o = static_cast<size_t>(t0 + lane) * a.hv + h;
+    if (lane == 0) before = mw;
+    if (live) {
+      const size_t o = static_cast<size_t>(t0 + tid) * a.hv + h;
       pv.g[o] = expf(fminf(g.y + before - mt, 0.f));
       pv.b[o] = expf(g.x - mt);
       pv.fl[o] = expf(-mt);
     }
-    m = __shfl_sync(0xffffffffu, mt, 31);
+    m = ends[NW];
+    __syncthreads();
   }
-  if (lane == 0) *ns = m;
+  if (tid == 0) *ns = m;
 }
 
 constexpr int kSsdHeads = 8;
@@ -783,7 +798,7 @@ constexpr int kScanCols = 32;
 template <int DK, int RULE>
 struct ScanGeom {
   static constexpr int kParts = DK >= 128 ? 32 : DK / 4;    // threads that share a column
-  static constexpr int kThreads = kParts * (kScanCols / 4);
+  static constexpr int kThreads = kParts * (kScanCols / 4) + (RULE == kMatrix ? 32 : 0);
   static constexpr int kNI = DK / (4 * kParts);
   // floats of one staging buffer
   static constexpr int kQ = 0, kH = kBlk * DK, kK = 2 * kBlk * DK;
@@ -797,7 +812,7 @@ struct ScanGeom {
 // Block-sequential pass.  A CTA owns 32 columns of one head's state in registers: a thread 4 columns and the rows
 // 4 part + 4 PARTS i + e; the PARTS lanes of a column group sit in one warp, so a group works through a block on its own and
 // the CTA only meets at the staging buffers (the next block streams in with cp.async meanwhile).
-// grid (DV / 32, hv, runs); matrix memory: one more column of CTAs for n
+// Matrix memory: the last warp's first group holds n (in the first CTA of a head).  grid (DV / 32, hv, runs)
 template <int DK, int DV, int RULE>
 __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(LinearArgs a) {
   constexpr bool DELTA = is_delta(RULE), CH = RULE == kDelta, SCALAR = scalar_decay(RULE);
@@ -817,7 +832,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
   float* us = ws + NV;                                      // [16][4] U
   float* sp = a.state + (static_cast<size_t>(slot) * a.hv + h) * DK * DV + j0;
   const bool fresh = a.positions[first] == 0;
-  const bool ones = RULE == kMatrix && jb >= DV;            // this CTA carries n, in its first column
+  const bool ones = RULE == kMatrix && cg >= kScanCols / 4;  // the warp for n: column 0 of its first group
   float* ns = ones ? a.nstate + (static_cast<size_t>(slot) * a.hv + h) * (DK + 4) : nullptr;
   float s[NI][4][4];                                        // [i][row e][column]
 #pragma unroll
@@ -825,7 +840,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       if (ones) {
-        s[i][e][0] = cg == 0 && !fresh ? ns[4 * PARTS * i + 4 * part + e] : 0.f;
+        s[i][e][0] = cg == kScanCols / 4 && !fresh ? ns[4 * PARTS * i + 4 * part + e] : 0.f;
         s[i][e][1] = s[i][e][2] = s[i][e][3] = 0.f;
         continue;
       }
@@ -852,8 +867,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
     }
     for (int i = tid; i < kBlk * (kScanCols / 4); i += NT) {
       const int t = i / (kScanCols / 4), c = (i % (kScanCols / 4)) * 4;
-      if (ones) *reinterpret_cast<float4*>(d + G::kV + t * kScanCols + c) = make_float4(c == 0 && t < n ? 1.f : 0.f, 0.f, 0.f, 0.f);
-      else if (t < n) cp_async_16(d + G::kV + t * kScanCols + c, pv.v + (static_cast<size_t>(t0 + t) * a.hv + h) * DV + jb + c);
+      if (t < n) cp_async_16(d + G::kV + t * kScanCols + c, pv.v + (static_cast<size_t>(t0 + t) * a.hv + h) * DV + jb + c);
       else *reinterpret_cast<float4*>(d + G::kV + t * kScanCols + c) = zero;
     }
     const size_t bh = static_cast<size_t>(b) * a.hv + h;
@@ -899,6 +913,9 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
       out[i] = acc;
     }
   };
+  float* one_v = sc_smem + 2 * G::kTotal;                   // matrix memory: [16] rows of 32 columns, ones in the first (no W and U there)
+  if (RULE == kMatrix)
+    for (int i = tid; i < kBlk * kScanCols; i += NT) one_v[i] = i % kScanCols == 0 ? 1.f : 0.f;
   stage(0, first, blk);
   int buf = 0;
   for (int t0 = first; t0 < last; t0 += kBlk, buf ^= 1, ++blk) {
@@ -910,9 +927,9 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
     }
     __syncthreads();
     const float* d = sc_smem + buf * G::kTotal;
-    const float* vb = d + G::kV + 4 * cg;                   // [16] rows of 32 columns, this group's 4
+    const float* vb = ones ? one_v : d + G::kV + 4 * cg;                   // [16] rows of 32 columns, this group's 4
     const int n = min(kBlk, last - t0);
-    if (ones && tid >= 32) {                                // columns of zeros
+    if (ones && blockIdx.x > 0) {                           // n has its place in the first CTA
       __syncthreads();
       continue;
     }
@@ -940,7 +957,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
       const float w = SCALAR ? d[G::kG + idx / 4] : 1.f;
       if (ones) {
         const size_t rh = static_cast<size_t>(t0 + idx / 4) * a.hv + h;
-        if (idx / 4 < n && cg == 0 && idx % 4 == 0) a.den[rh] = matrix_den(fmaf(w, val[i], x[i]), pv.fl[rh]);
+        if (idx / 4 < n && cg == kScanCols / 4 && idx % 4 == 0) a.den[rh] = matrix_den(fmaf(w, val[i], x[i]), pv.fl[rh]);
       } else if (idx / 4 < n && j0 + idx % 4 < a.ow) a.o[(static_cast<size_t>(t0 + idx / 4) * a.hv + h) * a.ow + j0 + idx % 4] = fmaf(w, val[i], x[i]);
     }
 #pragma unroll
@@ -976,7 +993,7 @@ __global__ void __launch_bounds__(ScanGeom<DK, RULE>::kThreads) lin_scan_kernel(
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       if (ones) {
-        if (cg == 0) ns[4 * PARTS * i + 4 * part + e] = s[i][e][0];
+        if (cg == kScanCols / 4 && blockIdx.x == 0) ns[4 * PARTS * i + 4 * part + e] = s[i][e][0];
       } else {
         *reinterpret_cast<float4*>(sp + static_cast<size_t>(4 * PARTS * i + 4 * part + e) * DV) =
             make_float4(s[i][e][0], s[i][e][1], s[i][e][2], s[i][e][3]);
@@ -1008,7 +1025,7 @@ static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
   if constexpr (RULE == kMatrix) {
     matrix_prep_kernel<T, DK, DV><<<dim3(dgpp_ceil_div(2 * a.hk * DK + a.hv * DV, 1024), a.rows), 256, 0, st>>>(a);
     DGPP_CUDA_OK(cudaGetLastError());
-    matrix_gates_kernel<T, DK, DV><<<dim3(dgpp_ceil_div(a.hv, 4), a.runs), 128, 0, st>>>(a);
+    matrix_gates_kernel<T, DK, DV><<<dim3(a.hv, a.runs), kGateThreads, 0, st>>>(a);
     prepared = true;
   } else if constexpr (scalar_decay(RULE)) {
     const dim3 grid(dgpp_ceil_div(2 * a.hk * DK + a.hv * DV, 512) + 1, a.blocks);
@@ -1027,7 +1044,7 @@ static int launch_lin(const LinearArgs& a, int decode, cudaStream_t st) {
   else if constexpr (RULE == kScalarDelta) gated_block_kernel<DK, DV><<<groups, 256, 0, st>>>(a);
   else lin_block_kernel<DK, DV, RULE><<<dim3(a.hv, a.blocks), 256, bsmem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
-  lin_scan_kernel<DK, DV, RULE><<<dim3(DV / kScanCols + (RULE == kMatrix ? 1 : 0), a.hv, a.runs), ScanGeom<DK, RULE>::kThreads, smem, st>>>(a);
+  lin_scan_kernel<DK, DV, RULE><<<dim3(DV / kScanCols, a.hv, a.runs), ScanGeom<DK, RULE>::kThreads, smem, st>>>(a);
   DGPP_CUDA_OK(cudaGetLastError());
   if (a.conv_w != nullptr) {
     const int C = 2 * a.hk * DK + a.hv * DV;

@@ -267,8 +267,8 @@ stream_norm_kernel(StreamNorm p, MoeRows<T> moe, SecondRow pair, T* __restrict__
   const bool add = delta != nullptr || moe.y != nullptr;
   const float sg = moe.gate != nullptr ? sigmoid_f32(moe.gate[row * moe.gate_stride]) : 1.f;
   auto norm = [&](float4 (&u)[NV], const RowNorm& w) {
-    if (PARTS) norm_parts<NT, NV>(u, w, cols, n, p.parts, p.eps, sn_smem);
-    else norm_row<NT, NV>(u, w, cols, n, p.eps, scratch);
+    if (PARTS && w.kind == kNormParts) norm_parts<NT, NV>(u, w, cols, n, p.parts, p.eps, sn_smem);
+    else if (!PARTS) norm_row<NT, NV>(u, w, cols, n, p.eps, scratch);
   };
   if (add) {
 #pragma unroll
@@ -545,7 +545,7 @@ DGPP_API int dgpp_geglu(const void* gate_up, void* out, int rows, int inter, int
   return 0;
 }
 
-// post / pre: 0 nothing, 1 RMS norm, 2 layer norm, 3 RMS norm over each of `parts` equal parts (both of them then), each with its weights
+// post / pre: 0 nothing, 1 RMS norm, 2 layer norm, 3 RMS norm over each of `parts` equal parts (then the other one too, or nothing), each with its weights
 // and perhaps a bias.  The delta is `delta` (fp32 [rows, cols]), or the expert rows y[pair_row[r * top + j]] (negative: wts[r * top + j]
 // times `self`, or nothing) plus sigmoid(gate) * shared (no gate: shared; y, shared, self: activations), or absent; delta_b [cols] is
 // added to it.  delta2: the delta is pair_factor * (rms(delta + delta_b) * pair_w1 + rms(delta2 + delta2_b) * pair_w2).  vec [cols]: added to every
@@ -561,7 +561,7 @@ DGPP_API int dgpp_stream_norm(void* x, const void* delta, const void* y, const v
   DGPP_REQUIRE(!delta2 || (delta && pair_w1 && pair_w2), "stream_norm: the second row needs a first one, and weights");
   DGPP_REQUIRE(out_stride % 8 == 0 && out_stride >= cols && (!delta_b || delta || y), "stream_norm: output rows of %lld", static_cast<long long>(out_stride));
   const bool in_parts = post == kNormParts || pre == kNormParts;
-  DGPP_REQUIRE(!in_parts || ((post == kNormParts || !(delta || y)) && pre == kNormParts && parts >= 1 && n % parts == 0),
+  DGPP_REQUIRE(!in_parts || (post % kNormParts == 0 && pre % kNormParts == 0 && parts >= 1 && n % parts == 0),
                "stream_norm: norms %d / %d over %d parts of %d columns", post, pre, parts, n);
   DGPP_REQUIRE(!self || in_parts, "stream_norm: identity experts come with norms over parts (perhaps one)");
   if (rows == 0) return 0;

@@ -287,7 +287,7 @@ __device__ __forceinline__ float wa_gate(const WindowAttnParams& p, int row, int
 // grid (hkv * head_chunks, splits, rows).  NG query heads of one kv head per CTA, NG / MAPS of every map; a warp scores 32 keys at a
 // time (lane = key), then the lanes take value columns 2 * lane + 64 * j.
 template <typename T, int NV, int NG, int MAPS, bool EXT>
-__global__ void __launch_bounds__(kWaWarps * 32) window_attn_kernel(const __grid_constant__ WindowAttnParams p) {
+__global__ void __launch_bounds__(kWaWarps * 32, EXT && NG == 4 ? 5 : 0) window_attn_kernel(const __grid_constant__ WindowAttnParams p) {
   constexpr int DV = NV * 64, VN = Vec16<T>::N, NGM = NG / MAPS, VU = NV <= 2 ? 8 : 4;
   extern __shared__ __align__(16) float wa_smem[];
   float* q_s = wa_smem;                                   // [NG][D]

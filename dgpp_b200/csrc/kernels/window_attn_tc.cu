@@ -15,7 +15,8 @@
 // Warps: 0 = TMA producer (one page of keys and values per stage), 1 = MMA issuer / TMEM owner, 2..5 = softmax.
 //
 // EXT: kept first tokens, whose pages come before those of the window; a sink, which joins the sum of the weights at the end; rotated values,
-// turned back there too, columns m and m + DV / 2 of a row together.  CAP: scores pass cap * tanh(s / cap) as well.
+// turned back there too, columns m and m + DV / 2 of a row together.  CAP: scores pass cap * tanh(s / cap) as well; caps of up to 38
+// bound the exponents by 110 binary orders, so the cap itself stands for the maximum and nothing is ever rescaled.
 //
 // FLAT is the form for latent attention, whose keys and values are expanded from the cached latents before the launch: every head
 // is its own kv head; key columns 0 .. DN - 1 and the values come from the expanded rows [flat rows, hq * DN + hq * DV], the other
@@ -266,7 +267,8 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     const float log2e = 1.4426950408889634f, top = CAP ? p.softcap * log2e : 0.f;
     const float sm = CAP ? 2.f * p.scale * log2e / p.softcap : p.scale * log2e;
     const int keep = EXT ? p.keep_first : 0;
-    float m_used = -INFINITY, l_run = 0.f;
+    const bool bounded = CAP && top <= 55.f;
+    float m_used = bounded ? top : -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int i = 0; i < ntiles; ++i) {
       const int b = i & 1, t0 = page_of(i) * kWtKeys;
@@ -275,7 +277,7 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       tc_fence_after();
       // warp-uniform choices: the TMEM accesses are .sync.aligned
       const bool full = __all_sync(0xffffffffu, t0 + kWtKeys - 1 <= hi && (t0 >= lo || (EXT && t0 + kWtKeys <= keep))) != 0;
-      const float mt = full ? wt_row_max<false, EXT>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep)
+      const float mt = bounded ? -INFINITY : full ? wt_row_max<false, EXT>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep)
                             : wt_row_max<true, EXT>(tmem_s + b * kWtKeys + lane_addr, t0, lo, hi, keep);
       const float mn = fmaxf(m_used, mt == -INFINITY ? -INFINITY : (CAP ? wt_cap(mt, sm, top) : mt * sm));
       const bool grow = mn > m_used + 8.f || (m_used == -INFINITY && mn != -INFINITY);

@@ -276,9 +276,10 @@ class WindowHeads:
         return self.hkv * self.maps, self.D, self.DV, self.hkv
 
     def splits(self, rows: int, max_span: int, most: int) -> int:
-        """Splits of single rows' keys: at most one wave of CTAs (four per SM, three with two maps), at least 128 keys each."""
+        """Splits of single rows' keys: at most one wave of CTAs (four per SM, three with two maps), at least 128 keys each (one more
+        split for kept tokens, which lie in front of a window of whole rounds)."""
         chunks = -(-self.group // (8 // self.maps))
-        return max(1, min(most, 148 * (5 - self.maps) // (self.hkv * chunks * rows), min(self.window + self.keep_first, max_span) // 128))
+        return max(1, min(most, 148 * (5 - self.maps) // (self.hkv * chunks * rows), min(self.window, max_span) // 128 + (self.keep_first > 0)))
 
 
 def value_freqs(base: float, vdim: int, width: int, device) -> torch.Tensor:

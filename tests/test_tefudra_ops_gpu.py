@@ -182,7 +182,8 @@ def test_expert_block(dev, dtype, rows, identity, shared):
                    identity=identity, act="gelu", shared_gated=False)
     h = torch.randn(rows, H, generator=g).to(dtype)
     x, out = torch.zeros(rows, H, device=dev), torch.empty(rows, H, dtype=dtype, device=dev)
-    mx.stream_norm(x, H, 1e-5, out, run_experts(b, RowExpertsScratch([b], 64, dtype, dev), h.to(dev)))
+    ones = torch.ones(H, device=dev)
+    mx.stream_norm(x, H, 1e-5, out, run_experts(b, RowExpertsScratch([b], 64, dtype, dev), h.to(dev)), (None, None), ("parts", ones))
     cfg = {"router": {"experts": E, "top": top}, "shared": {"ff": shared} if shared else None}
     _close(x, plain.experts(h.double(), "", cfg, {k: v.double() for k, v in w.items()}), dtype, 5e-6, 1.5e-2)
 
