@@ -6,7 +6,7 @@
 //                rows); inputs before the run's first row come from the request's ring
 //   conv_tail    the newest inputs of every run go to the ring, once every reader is done
 //
-// The ring holds `taps` inputs per channel and request (fp32, bias included), entry p % taps for position p: see window_attn.cu, whose
+// The ring holds `taps` inputs per channel and request (fp32, bias included), entry p % taps for position p: see window_attn.cuh, whose
 // decode form convolves single tokens itself.
 #include "common/common.h"
 #include "common/dtypes.cuh"

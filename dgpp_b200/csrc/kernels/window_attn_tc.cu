@@ -1,4 +1,4 @@
-// GQA for prompt rows on the 5th-generation tensor cores (bf16 queries, keys and values; see window_attn.cu for the layer, its windows,
+// GQA for prompt rows on the 5th-generation tensor cores (bf16 queries, keys and values; see window_attn.cuh for the layer, its windows,
 // chunks and maps, and for the cache, whose new positions and prepared queries `qk_norm_append` has written).
 //
 // One CTA = 128 query rows of one key head: 128 / G consecutive tokens of one run with their G = hq / hkv query heads, row
